@@ -51,12 +51,14 @@ def parse_args():
     ap.add_argument("--layered", default="", help="instead of the headline benchmark: prefill and decode throughput of the "
                     "layer-list design (Ribivik: Mamba-2 + latent attention, bf16) beside a Q40 Llama of equal width, "
                     "feed-forward size and depth, at these sizes (comma separated: w2048, w4096); prints one JSON line")
-    ap.add_argument("--layered-design", default="ribivik", choices=("ribivik", "sunesun", "venadra", "darusun"),
+    ap.add_argument("--layered-design", default="ribivik", choices=("ribivik", "sunesun", "venadra", "darusun", "vopedra"),
                     help="--layered: which layer-list design runs beside the Llama arm (ribivik: Mamba-2 + latent attention; "
                          "sunesun: windowed attention whose values are its keys + routed experts on hyper-connected streams; "
                          "venadra: lightning and chunked sink attention, PolyNorm and gated experts; darusun: post-norm layers, "
                          "head-mixed attention, windowed latent attention, xIELU and experts with a shared one -- beside these two "
-                         "also Sunesun, the closest layer-list design, at equal width, depth and experts)")
+                         "also Sunesun, the closest layer-list design, at equal width, depth and experts; vopedra: matrix memory, "
+                         "selective scan, attention with mixed softmax weights beside HGRN2, gated feed-forwards -- beside it Venadra "
+                         "(linear attention) and Darusun (head-mixed attention))")
     ap.add_argument("--layered-layers", type=int, default=4, help="--layered: layers of both models")
     ap.add_argument("--layered-prompt", type=int, default=2048, help="--layered: prompt length (one batch)")
     return ap.parse_args()
@@ -486,6 +488,21 @@ def darusun_config(name: str, n_layers: int, vocab: int, window: int = 1024) -> 
     return {"architecture": "Darusun", "width": sz["width"], "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "layers": layers}
 
 
+def vopedra_config(name: str, n_layers: int, vocab: int) -> dict:
+    """Width, heads and feed-forward of the Llama arm.  Layers in turn: matrix memory, selective scan, attention (four key/value
+    heads, 64 rotated dimensions) beside HGRN2, matrix memory; every layer with a gated feed-forward, no loop."""
+    import math
+    sz, ss = LAYERED_SIZES[name], SUNESUN_SIZES[name]
+    W = sz["width"]
+    mlstm = {"heads": W // 256, "dim": 128, "vdim": 256, "gate_cap": 15.0}
+    mamba = {"inner": 2 * W, "state": 16, "conv": 4, "dt_rank": W // 16}
+    left = {"heads": ss["heads"], "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 1.0 / math.sqrt(128.0), "rot": {"base": 500000.0, "dims": 64}}
+    right = {"heads": W // 128, "dim": 128, "vdim": 128}
+    kinds = [("mlstm", mlstm), ("mamba1", mamba), ("parallel", {"left": left, "right": right}), ("mlstm", mlstm)]
+    layers = [{"type": kinds[i % 4][0], "mixer": dict(kinds[i % 4][1]), "mlp": {"kind": "dense", "ff": sz["ff"]}} for i in range(n_layers)]
+    return {"architecture": "Vopedra", "width": W, "vocab": vocab, "norm": {"eps": 1e-5}, "layers": layers}
+
+
 def _time_ms(fn, warmup: int, steps: int):
     import torch
     for _ in range(warmup):
@@ -554,7 +571,8 @@ def run_layered(args):
         sz = LAYERED_SIZES[name]
         design = args.layered_design
         configs = {"ribivik": lambda: layered_config(sz, nl, vocab), "sunesun": lambda: sunesun_config(name, nl, vocab),
-                   "venadra": lambda: venadra_config(name, nl, vocab), "darusun": lambda: darusun_config(name, nl, vocab)}
+                   "venadra": lambda: venadra_config(name, nl, vocab), "darusun": lambda: darusun_config(name, nl, vocab),
+                   "vopedra": lambda: vopedra_config(name, nl, vocab)}
 
         def layer_list_arm(dsg):
             d = os.path.join(args.model_dir, f"dllama_b200_{'layered' if dsg == 'ribivik' else dsg}_{name}_l{nl}")
@@ -569,7 +587,8 @@ def run_layered(args):
             return r
 
         r = layer_list_arm(design)
-        beside = {"sunesun_bf16": layer_list_arm("sunesun")} if design in ("venadra", "darusun") else {}
+        beside = {"sunesun_bf16": layer_list_arm("sunesun")} if design in ("venadra", "darusun") else \
+            {d + "_bf16": layer_list_arm(d) for d in ("venadra", "darusun")} if design == "vopedra" else {}
         shape = dict(dim=sz["width"], hidden_dim=sz["ff"], n_layers=nl, n_heads=sz["heads"], n_kv_heads=8, vocab_size=vocab,
                      max_seq_len=8192, rope_theta=10000, rope=None)
         path = os.path.join(args.model_dir, f"dllama_b200_llama_{name}_l{nl}_q40.m")

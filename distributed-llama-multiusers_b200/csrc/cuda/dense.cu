@@ -35,6 +35,11 @@ __device__ __forceinline__ void dense_store(const DlDenseArgs& a, int b, int m, 
     *y = dense_epi(acc, a.epi, aux, a.param, a.param2);
 }
 
+// paired output columns (weight rows gate_0, up_0, gate_1, up_1, ...): value j of row m from its two products
+__device__ __forceinline__ void dense_store_pair(const DlDenseArgs& a, int b, int m, int j, float gate, float up) {
+    a.Y[(size_t)b * a.y_bs + (size_t)m * a.ldy + j] = gelu_tanh_f(gate) * up;
+}
+
 // ------------------------------------------------------------------------------------------------
 // embedding gather: x[m][c] = scale * table[tokens[m]] for each of `copies` copies of the row (row layout [copies][dim])
 // ------------------------------------------------------------------------------------------------
@@ -150,6 +155,62 @@ __global__ void __launch_bounds__(GV_WARPS * 32) dense_gemv_vec_kernel(DlDenseAr
     }
 }
 
+// paired columns (GLU): one warp per value, its gate row and its up row side by side
+template <typename WT, int MT, bool RX>
+__global__ void __launch_bounds__(GV_WARPS * 32) dense_gemv_pair_kernel(DlDenseArgs a, int vec) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int j = blockIdx.x * GV_WARPS + warp;
+    const int b = blockIdx.z;
+    if (2 * j + 1 >= a.N) return;
+    const WT* w0 = (const WT*)a.W + (size_t)b * a.w_bs + (size_t)(2 * j) * a.ldw;
+    const WT* w1 = w0 + a.ldw;
+    const float* x = a.X + (size_t)b * a.x_bs;
+    float g[MT], u[MT];
+#pragma unroll
+    for (int m = 0; m < MT; ++m) g[m] = u[m] = 0.f;
+    if (vec) {
+#pragma unroll 2
+        for (int k = lane * 8; k < a.K; k += 256) {
+            float wg[8], wu[8];
+            WVec<WT>::load8(w0 + k, wg);
+            WVec<WT>::load8(w1 + k, wu);
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+                if (m < a.M) {
+                    float xv[8];
+                    WVec<float>::load8(x + (size_t)m * a.ldx + k, xv);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        const float v = RX ? round_bf16(xv[i]) : xv[i];
+                        g[m] = fmaf(v, wg[i], g[m]);
+                        u[m] = fmaf(v, wu[i], u[m]);
+                    }
+                }
+            }
+        }
+    } else {
+        for (int k = lane; k < a.K; k += 32) {
+            const float wg = ld_f(w0 + k), wu = ld_f(w1 + k);
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+                if (m < a.M) {
+                    float v = x[(size_t)m * a.ldx + k];
+                    if (RX) v = round_bf16(v);
+                    g[m] = fmaf(v, wg, g[m]);
+                    u[m] = fmaf(v, wu, u[m]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m) { g[m] = warp_sum(g[m]); u[m] = warp_sum(u[m]); }
+    if (lane == 0) {
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+            if (m < a.M) dense_store_pair(a, b, m, j, g[m], u[m]);
+    }
+}
+
 // ------------------------------------------------------------------------------------------------
 // more rows: 64 x 64 output tile per CTA, 16-wide K steps through shared memory, 4 x 4 outputs per thread
 // ------------------------------------------------------------------------------------------------
@@ -201,6 +262,14 @@ __global__ void __launch_bounds__(256) dense_tile_kernel(DlDenseArgs a) {
     for (int i = 0; i < 4; ++i) {
         const int m = m0 + ty * 4 + i;
         if (m >= a.M) continue;
+        if (a.epi == DL_DENSE_GLU_GELU) {          // this thread's columns are two (gate, up) pairs
+#pragma unroll
+            for (int j = 0; j < 4; j += 2) {
+                const int n = n0 + tx * 4 + j;
+                if (n + 1 < a.N) dense_store_pair(a, b, m, n >> 1, acc[i][j], acc[i][j + 1]);
+            }
+            continue;
+        }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
@@ -215,11 +284,13 @@ static void launch_dense(const DlDenseArgs& a, cudaStream_t st) {
     if (a.M <= 8) {
         const bool vec = a.K % 8 == 0 && a.ldw % 8 == 0 && a.w_bs % 8 == 0 && a.ldx % 4 == 0 && a.x_bs % 4 == 0 &&
                          ((uintptr_t)a.W & 15) == 0 && ((uintptr_t)a.X & 15) == 0;
-        dim3 grid((a.N + GV_WARPS - 1) / GV_WARPS, 1, a.batch);
+        const bool pair = a.epi == DL_DENSE_GLU_GELU;
+        dim3 grid(((pair ? a.N / 2 : a.N) + GV_WARPS - 1) / GV_WARPS, 1, a.batch);
         const int mt = a.M <= 1 ? 1 : a.M <= 2 ? 2 : a.M <= 4 ? 4 : 8;
 #define GV_CASE(MT_)                                                                                   \
     case MT_:                                                                                          \
-        if (vec) dense_gemv_vec_kernel<WT, MT_, RX><<<grid, GV_WARPS * 32, 0, st>>>(a);                \
+        if (pair) dense_gemv_pair_kernel<WT, MT_, RX><<<grid, GV_WARPS * 32, 0, st>>>(a, vec ? 1 : 0);  \
+        else if (vec) dense_gemv_vec_kernel<WT, MT_, RX><<<grid, GV_WARPS * 32, 0, st>>>(a);                \
         else dense_gemv_kernel<WT, MT_, RX><<<grid, GV_WARPS * 32, 0, st>>>(a);                        \
         break;
         switch (mt) { GV_CASE(1) GV_CASE(2) GV_CASE(4) GV_CASE(8) }
@@ -235,6 +306,7 @@ extern "C" int dl_dense(const DlDenseArgs* args, void* stream) {
     if (a.M < 1 || a.N < 1 || a.K < 1 || a.batch < 1) { dl_set_error("dl_dense: empty problem"); return -1; }
     if ((a.epi == DL_DENSE_SIGMOID_MUL || a.epi == DL_DENSE_MUL || a.epi == DL_DENSE_ROWGATE_ADD) && a.aux == nullptr) { dl_set_error("dl_dense: the gate epilogue needs aux"); return -1; }
     if (a.epi == DL_DENSE_GLU_CLAMP || a.epi == DL_DENSE_GLU_SILU) { dl_set_error("dl_dense: the paired-column epilogue belongs to the tensor-core GEMM"); return -1; }
+    if (a.epi == DL_DENSE_GLU_GELU && (a.N & 1)) { dl_set_error("dl_dense: paired columns need an even number of weight rows"); return -1; }
     cudaStream_t st = (cudaStream_t)stream;
     if (a.wtype == DL_T_BF16) {
         if (a.round_x) launch_dense<__nv_bfloat16, true>(a, st);

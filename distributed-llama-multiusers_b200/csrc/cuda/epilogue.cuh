@@ -175,7 +175,7 @@ DL_DEVINL void epilogue_rows(const DlEpilogue& e, const float* out_s, int out_ld
         }
     } else if (e.kind == DL_EPI_DENSE) {
         // dense-weight models: an element-wise op on the f32 result, then a plain store (one destination)
-        if (e.dense_op == DL_DENSE_GLU_CLAMP || e.dense_op == DL_DENSE_GLU_SILU) {
+        if (e.dense_op == DL_DENSE_GLU_CLAMP || e.dense_op == DL_DENSE_GLU_SILU || e.dense_op == DL_DENSE_GLU_GELU) {
             // output rows interleaved (gate_j, up_j): thread j < rows/2 owns value j of the tile and stores column
             // grow0 / 2 + j:  a = min(gate, limit), b = clamp(up, +-limit), hidden = a * sigma(1.702 a) * (1 + b)
             const int col = (grow0 >> 1) + tid;
@@ -184,11 +184,13 @@ DL_DEVINL void epilogue_rows(const DlEpilogue& e, const float* out_s, int out_ld
                 float* d0 = e.dst[0] + (size_t)e.dst_off + (size_t)m0 * ld + col;
                 const float lim = e.dense_param;
                 const bool silu = e.dense_op == DL_DENSE_GLU_SILU;      // silu(gate) * up, no clamps
+                const bool gelu = e.dense_op == DL_DENSE_GLU_GELU;      // gelu_tanh(gate) * up
 #pragma unroll 4
                 for (int m = m_first; m < M; m += m_step) {
                     const float2 gu = *reinterpret_cast<const float2*>(out_s + m * out_ld + 2 * tid);
                     float g = gu.x, u = gu.y;
                     if (silu) { d0[m * ld] = g / (1.0f + expf(-g)) * u; continue; }
+                    if (gelu) { d0[m * ld] = act_gelu(g) * u; continue; }
                     if (lim > 0.0f) { g = fminf(g, lim); u = fminf(fmaxf(u, -lim), lim); }
                     d0[m * ld] = g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
                 }

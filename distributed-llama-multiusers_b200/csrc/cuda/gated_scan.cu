@@ -1,0 +1,713 @@
+// Linear attention whose decay depends on the data.  Per head, state S [dim][vdim] f32, one per sequence slot:
+//   channel form:  S <- diag(f_t) S + (1 - f_t) v_t^T                    f = lower + (1 - lower) sigmoid(z + bias), per channel of q
+//   head form:     S <- e^l_t S + p_t k_t v_t^T,  n <- e^l_t n + p_t k_t   one log decay l and one weight p per head and token
+//   both:          y_t = S_t^T q_t  (and den_t = n_t . q_t in the head form)
+// Everything is f32.  A batch is any mix of sequences with one or more consecutive rows each (DlMambaBatch); a sequence
+// whose first row is position 0 starts from zeros whatever its slot held.
+//
+// Two forms of each.  Token by token (decoding, short portions): the state in registers.  Chunked (long portions): a
+// sequence's rows in chunks of GC = 64, counted from the portion's first row:
+//     y_i = sum_{j <= i in chunk} ( sum_d q_i[d] D_ij[d] k_j[d] ) v_j + P^T (D_i0 q_i)       D_ij: the decay from j to i
+//     P   = the state before the chunk;  state after it = D_end,0 P + sum_j (D_end,j k_j) v_j^T
+// in three launches: every chunk's own sum, the prefix over a sequence's chunks (which also leaves the slot's new state),
+// the outputs.  Per channel no quotient of decays is ever formed (a decay may be as small as it likes): rows are taken in
+// sub-blocks of 16; between two sub-blocks the decay splits into three factors <= 1 (from the column's row to the end of its
+// block, over the blocks between, from the start of the row's block to the row), inside a sub-block it is the running
+// product itself.  Per head the log decays of a chunk are summed in f64.
+#include "layer_common.cuh"
+#include "../../../include/dllama_b200.h"
+
+#define GT_TB 8                   // tokens staged per barrier pair of the token-by-token kernel
+#define GT_COLS 32                // columns of S per CTA of the token-by-token kernel
+#define GC DL_GATED_CHUNK
+#define GC_THREADS 256
+#define GC_AS 68                  // row stride of the score matrix
+
+__device__ __forceinline__ float gated_q(const DlGatedArgs& a, size_t row, int i) {
+    const float v = a.q[row * a.ldq + i];
+    if (!a.q_silu) return v * a.q_scale;
+    float s, c;
+    sigmoid_pair_f(v, s, c);
+    return v * s;
+}
+// channel form: f and 1 - f of channel i (over all heads)
+__device__ __forceinline__ void gated_f(const DlGatedArgs& a, size_t row, int i, float& f, float& k) {
+    float s, c;
+    sigmoid_pair_f(a.f[row * a.ldf + i] + a.f_bias[i], s, c);
+    const float l = a.lower[i];
+    f = fmaf(1.f - l, s, l);
+    k = (1.f - l) * c;
+}
+
+// ------------------------------------------------------------------------------------------------
+// token by token: a CTA owns GT_COLS columns of one head's S; thread (column, dq) keeps the rows d with (d / 4) % 4 == dq of its
+// column (NR registers; rows in groups of four so that q, k and f leave shared memory as 16-byte words), the four threads
+// of a column are neighbouring lanes and sum their shares of y by two shuffles.  In the head form column `vdim` is n: its
+// value is 1 for every token and its output is den.
+// ------------------------------------------------------------------------------------------------
+template <int NR, bool CH>
+__global__ void __launch_bounds__(GT_COLS * 4) gated_scan_kernel(DlMambaBatch b, DlGatedArgs a) {
+    constexpr int DP = NR * 4;
+    extern __shared__ __align__(16) float sm[];
+    const int n = blockIdx.x, h = blockIdx.y, dq = threadIdx.x & 3, c = blockIdx.z * GT_COLS + (threadIdx.x >> 2);
+    const int D = a.dim, V = a.vdim, H = a.n_heads;
+    float* qs = sm;                             // [GT_TB][DP]
+    float* ks = qs + GT_TB * DP;                // [GT_TB][DP]
+    float* fs = ks + GT_TB * DP;                // channel form: [GT_TB][DP]; head form: [GT_TB] decays
+    const size_t sh = (size_t)b.seq_slot[n] * H + h;
+    const bool fresh = b.seq_pos0[n] == 0, is_n = !CH && c == V, live = c < V || is_n;
+    float* Sg = is_n ? a.n_state + sh * D : a.state + sh * D * V + c;       // row d at Sg[d * step]
+    const size_t step = is_n ? 1 : V;
+    float s[NR];
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        const int d = (i >> 2) * 16 + dq * 4 + (i & 3);
+        s[i] = (live && !fresh && d < D) ? Sg[d * step] : 0.f;
+    }
+    const int r0 = b.seq_start[n], r1 = b.seq_start[n + 1];
+    for (int rb = r0; rb < r1; rb += GT_TB) {
+        const int nt = min(GT_TB, r1 - rb);
+        __syncthreads();
+        for (int t = threadIdx.x / 32; t < nt; t += GT_COLS * 4 / 32) {
+            const size_t row = b.seq_rows[rb + t];
+            const float put = CH ? 0.f : a.put[row * H + h];
+            for (int d = threadIdx.x & 31; d < DP; d += 32) {
+                float q = 0.f, k = 0.f, f = 0.f;
+                if (d < D) {
+                    q = gated_q(a, row, h * D + d);
+                    if (CH) gated_f(a, row, h * D + d, f, k);
+                    else k = put * a.k[row * a.ldk + h * D + d];
+                }
+                qs[t * DP + d] = q;
+                ks[t * DP + d] = k;
+                if (CH) fs[t * DP + d] = f;
+            }
+            if (!CH && (threadIdx.x & 31) == 0) fs[t] = expf(a.log_keep[row * H + h]);
+        }
+        __syncthreads();
+        for (int t = 0; t < nt; ++t) {
+            const size_t row = b.seq_rows[rb + t];
+            const float v = c < V ? a.v[row * a.ldv + h * V + c] : 1.f;
+            const float keep = CH ? 0.f : fs[t];
+            float y0 = 0.f, y1 = 0.f;
+#pragma unroll
+            for (int i = 0; i < NR; i += 4) {
+                const int at = t * DP + i * 4 + dq * 4;
+                const float4 q = *reinterpret_cast<const float4*>(qs + at), k = *reinterpret_cast<const float4*>(ks + at);
+                float4 f = make_float4(keep, keep, keep, keep);
+                if (CH) f = *reinterpret_cast<const float4*>(fs + at);
+                s[i] = fmaf(f.x, s[i], k.x * v);             y0 = fmaf(s[i], q.x, y0);
+                s[i + 1] = fmaf(f.y, s[i + 1], k.y * v);     y1 = fmaf(s[i + 1], q.y, y1);
+                s[i + 2] = fmaf(f.z, s[i + 2], k.z * v);     y0 = fmaf(s[i + 2], q.z, y0);
+                s[i + 3] = fmaf(f.w, s[i + 3], k.w * v);     y1 = fmaf(s[i + 3], q.w, y1);
+            }
+            float y = y0 + y1;
+            y += __shfl_xor_sync(0xffffffffu, y, 1);
+            y += __shfl_xor_sync(0xffffffffu, y, 2);
+            if (live && dq == 0) {
+                if (is_n) a.den[row * H + h] = y;
+                else a.y[row * a.ld_y + h * V + c] = y;
+            }
+        }
+    }
+    if (live) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int d = (i >> 2) * 16 + dq * 4 + (i & 3);
+            if (d < D) Sg[d * step] = s[i];
+        }
+    }
+}
+
+static int gated_args_ok(const DlGatedArgs& a, const char* who) {
+    const bool ch = a.f != nullptr;
+    if (a.n_heads < 1 || a.dim < 1 || a.vdim < 1 || a.dim > 512) { dl_set_error("%s: bad shape (heads %d, dim %d, vdim %d)", who, a.n_heads, a.dim, a.vdim); return -1; }
+    if (ch ? (!a.f_bias || !a.lower) : (!a.k || !a.log_keep || !a.put || !a.den || !a.n_state)) { dl_set_error("%s: the gates are incomplete", who); return -1; }
+    return 0;
+}
+
+extern "C" int dl_gated_scan_supported(int dim, int vdim) { return dim >= 1 && dim <= 512 && vdim >= 1 ? 0 : -1; }
+
+template <int NR>
+static void launch_gated(const DlMambaBatch& b, int n_seq, const DlGatedArgs& a, cudaStream_t st) {
+    const bool ch = a.f != nullptr;
+    const size_t smem = ((size_t)(ch ? 3 : 2) * GT_TB * NR * 4 + GT_TB) * sizeof(float);
+    const dim3 grid(n_seq, a.n_heads, (a.vdim + (ch ? 0 : 1) + GT_COLS - 1) / GT_COLS);
+    if (ch) gated_scan_kernel<NR, true><<<grid, GT_COLS * 4, smem, st>>>(b, a);
+    else gated_scan_kernel<NR, false><<<grid, GT_COLS * 4, smem, st>>>(b, a);
+}
+
+extern "C" int dl_gated_scan(const DlMambaBatch* batch, int n_seq, const DlGatedArgs* args, void* stream) {
+    const DlGatedArgs& a = *args;
+    if (gated_args_ok(a, "dl_gated_scan")) return -1;
+    if (n_seq < 1) return 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (a.dim <= 32) launch_gated<8>(*batch, n_seq, a, st);
+    else if (a.dim <= 64) launch_gated<16>(*batch, n_seq, a, st);
+    else if (a.dim <= 128) launch_gated<32>(*batch, n_seq, a, st);
+    else if (a.dim <= 256) launch_gated<64>(*batch, n_seq, a, st);
+    else {                                      // 48 KB + 32 B of staged tokens at most in the channel form
+        const size_t smem = ((size_t)3 * GT_TB * 512 + GT_TB) * sizeof(float);
+        cudaError_t e = cudaFuncSetAttribute(gated_scan_kernel<128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) { dl_set_error("dl_gated_scan: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
+        launch_gated<128>(*batch, n_seq, a, st);
+    }
+    LAYER_CHECK_LAUNCH("dl_gated_scan");
+    return 0;
+}
+
+// ------------------------------------------------------------------------------------------------
+// chunked.  Chunk c of sequence n covers rows seq_start[n] + c GC ..; its scratch slot is seq_start[n] / GC + n + c.
+// Scratch: states [slots][H][D][V] | decay of the whole chunk [slots][H][D] (head form: entry 0 of D) | n sums [slots][H][D].
+// ------------------------------------------------------------------------------------------------
+struct GatedScratch { float* S; float* dec; float* ns; };
+
+__device__ __forceinline__ bool gated_chunk_of(const DlMambaBatch& b, int n, int c, int& row0, int& len, int& ci) {
+    const int s0 = b.seq_start[n], total = b.seq_start[n + 1] - s0;
+    if (c * GC >= total) return false;
+    row0 = s0 + c * GC;
+    len = min(GC, total - c * GC);
+    ci = s0 / GC + n + c;
+    return true;
+}
+
+// V columns c0 .. c0 + 127 of the chunk's values into [GC][128] (zeros beyond the chunk or the head's width)
+__device__ __forceinline__ void gated_stage_v(const DlGatedArgs& a, const int* rows, int len, int h, int c0, float* vt) {
+    const int lane = threadIdx.x & 31;
+    for (int j = threadIdx.x >> 5; j < GC; j += GC_THREADS / 32) {
+        const float* src = j < len ? a.v + (size_t)rows[j] * a.ldv + (size_t)h * a.vdim + c0 : nullptr;
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int cc = lane + 32 * u;
+            vt[j * 128 + cc] = (src && c0 + cc < a.vdim) ? src[cc] : 0.f;
+        }
+    }
+}
+
+// pass 1: a chunk's own sum of (decay to the chunk's end * k_j) v_j^T, and the decay of the whole chunk
+template <bool CH>
+__global__ void __launch_bounds__(GC_THREADS) gated_chunk_state_kernel(DlMambaBatch b, DlGatedArgs a, GatedScratch sc) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ int rows[GC];
+    __shared__ float w_s[GC];
+    __shared__ double l_s[GC];
+    const int n = blockIdx.x, c = blockIdx.y, h = blockIdx.z;
+    int row0, len, ci;
+    if (!gated_chunk_of(b, n, c, row0, len, ci)) return;
+    const int D = a.dim, V = a.vdim, H = a.n_heads, D8 = (D + 7) & ~7;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* ks = sm;                             // [GC][D8]
+    float* vt = ks + (size_t)GC * D8;           // channel form: the decays [GC][D8] first; then value tiles [GC][128]
+    if (threadIdx.x < GC) rows[threadIdx.x] = threadIdx.x < len ? b.seq_rows[row0 + threadIdx.x] : 0;
+    if (!CH && threadIdx.x < GC) l_s[threadIdx.x] = threadIdx.x < len ? (double)a.log_keep[(size_t)b.seq_rows[row0 + threadIdx.x] * H + h] : 0.0;
+    __syncthreads();
+    if (!CH && threadIdx.x < GC) {              // p_j e^(l_(j+1) + ... + l_end)
+        double g = 0.0;
+        for (int j = threadIdx.x + 1; j < len; ++j) g += l_s[j];
+        w_s[threadIdx.x] = threadIdx.x < len ? a.put[(size_t)rows[threadIdx.x] * H + h] * expf((float)g) : 0.f;
+        if (threadIdx.x == 0) sc.dec[((size_t)ci * H + h) * D] = expf((float)(g + l_s[0]));
+    }
+    if (!CH) __syncthreads();
+    for (int j = warp; j < GC; j += GC_THREADS / 32) {
+        const size_t row = rows[j];
+#pragma unroll 4
+        for (int d = lane; d < D8; d += 32) {
+            float k = 0.f, f = 1.f;
+            if (j < len && d < D) {
+                if (CH) gated_f(a, row, h * D + d, f, k);
+                else k = w_s[j] * a.k[row * a.ldk + h * D + d];
+            }
+            ks[j * D8 + d] = k;
+            if (CH) vt[j * D8 + d] = f;
+        }
+    }
+    __syncthreads();
+    if (CH) {
+        for (int d = threadIdx.x; d < D; d += GC_THREADS) {
+            float p = 1.f;
+#pragma unroll 8
+            for (int j = GC - 1; j >= 0; --j) {
+                ks[j * D8 + d] *= p;
+                p *= vt[j * D8 + d];
+            }
+            sc.dec[((size_t)ci * H + h) * D + d] = p;
+        }
+    } else {
+        for (int d = threadIdx.x; d < D; d += GC_THREADS) {
+            float s = 0.f;
+#pragma unroll 8
+            for (int j = 0; j < GC; ++j) s += ks[j * D8 + d];
+            sc.ns[((size_t)ci * H + h) * D + d] = s;
+        }
+    }
+    float* out = sc.S + ((size_t)ci * H + h) * D * V;
+    const int tb = threadIdx.x >> 4, cb = threadIdx.x & 15;
+    for (int c0 = 0; c0 < V; c0 += 128) {
+        __syncthreads();
+        gated_stage_v(a, rows, len, h, c0, vt);
+        __syncthreads();
+        for (int d0 = 0; d0 < D; d0 += 128) {
+            const int dt = d0 + tb * 8;          // this thread: 8 rows of S, columns cb * 4 .. + 3 and 64 + cb * 4 .. + 3 of the tile
+            if (dt >= D8) continue;
+            float acc[8][8];
+#pragma unroll
+            for (int r = 0; r < 8; ++r)
+#pragma unroll
+                for (int u = 0; u < 8; ++u) acc[r][u] = 0.f;
+            for (int j = 0; j < len; ++j) {
+                const float4 k0 = *reinterpret_cast<const float4*>(ks + j * D8 + dt), k1 = *reinterpret_cast<const float4*>(ks + j * D8 + dt + 4);
+                const float4 v0 = *reinterpret_cast<const float4*>(vt + j * 128 + cb * 4), v1 = *reinterpret_cast<const float4*>(vt + j * 128 + 64 + cb * 4);
+                const float kk[8] = {k0.x, k0.y, k0.z, k0.w, k1.x, k1.y, k1.z, k1.w};
+                const float vv[8] = {v0.x, v0.y, v0.z, v0.w, v1.x, v1.y, v1.z, v1.w};
+#pragma unroll
+                for (int r = 0; r < 8; ++r)
+#pragma unroll
+                    for (int u = 0; u < 8; ++u) acc[r][u] = fmaf(kk[r], vv[u], acc[r][u]);
+            }
+#pragma unroll
+            for (int r = 0; r < 8; ++r)
+#pragma unroll
+                for (int u = 0; u < 8; ++u) {
+                    const int d = dt + r, cc = c0 + (u >> 2) * 64 + cb * 4 + (u & 3);
+                    if (d < D && cc < V) out[(size_t)d * V + cc] = acc[r][u];
+                }
+        }
+    }
+}
+
+// pass 2: over a sequence's chunks in order, scratch <- the state BEFORE the chunk; the slot gets the state after the last
+// one.  One thread per state element (head form: and per element of n).
+template <bool CH>
+__global__ void __launch_bounds__(256) gated_chunk_prefix_kernel(DlMambaBatch b, DlGatedArgs a, GatedScratch sc) {
+    const int n = blockIdx.x, h = blockIdx.y;
+    const int D = a.dim, V = a.vdim, H = a.n_heads, DV = D * V;
+    const int e = blockIdx.z * blockDim.x + threadIdx.x;
+    if (e >= DV + (CH ? 0 : D)) return;
+    const bool is_n = e >= DV;
+    const int s0 = b.seq_start[n], nc = (b.seq_start[n + 1] - s0 + GC - 1) / GC;
+    const size_t sh = (size_t)b.seq_slot[n] * H + h, ch0 = (size_t)(s0 / GC + n) * H + h;
+    float* Sg = is_n ? a.n_state + sh * D + (e - DV) : a.state + sh * DV + e;
+    float R = b.seq_pos0[n] == 0 ? 0.f : *Sg;
+    float* p0 = is_n ? sc.ns + ch0 * D + (e - DV) : sc.S + ch0 * DV + e;
+    const size_t step = is_n ? (size_t)H * D : (size_t)H * DV, dstep = (size_t)H * D;
+    const float* t0 = sc.dec + ch0 * D + (CH ? e / V : 0);
+    for (int c0 = 0; c0 < nc; c0 += 8) {          // eight chunks' sums are loaded together, then chained
+        float own[8], dec[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            own[i] = c0 + i < nc ? p0[(size_t)(c0 + i) * step] : 0.f;
+            dec[i] = c0 + i < nc ? t0[(size_t)(c0 + i) * dstep] : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+            if (c0 + i < nc) {
+                p0[(size_t)(c0 + i) * step] = R;
+                R = fmaf(dec[i], R, own[i]);
+            }
+    }
+    *Sg = R;
+}
+
+__device__ __forceinline__ float dot4(float4 x, float4 y, float acc) { return fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, acc)))); }
+__device__ __forceinline__ float4 mul4(float4 x, float4 y) { return make_float4(x.x * y.x, x.y * y.y, x.z * y.z, x.w * y.w); }
+
+// pass 3: the outputs of a chunk.  Shared memory: Q [GC][DP] | K [GC][DP], later tiles of V and of the carried state
+// [GC][128] | F [GC][DP] (channel form), later the scores A [GC][GC_AS] | block decays [4][DP].
+template <bool CH>
+__global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaBatch b, DlGatedArgs a, GatedScratch sc) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ int rows[GC];
+    __shared__ float put_s[GC], carry_s[GC];
+    __shared__ double g_s[GC];
+    const int n = blockIdx.x, c = blockIdx.y, h = blockIdx.z;
+    int row0, len, ci;
+    if (!gated_chunk_of(b, n, c, row0, len, ci)) return;
+    const int D = a.dim, V = a.vdim, H = a.n_heads, D4 = (D + 3) & ~3, DP = D4 + 4;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tb = threadIdx.x >> 4, cb = threadIdx.x & 15;
+    float* Q = sm;
+    float* K = Q + (size_t)GC * DP;
+    float* F = K + max((size_t)GC * DP, (size_t)GC * 128);
+    float* A = F;
+    float* T = F + max(CH ? (size_t)GC * DP : 0, (size_t)GC * GC_AS);      // channel form: [4][DP]
+    if (threadIdx.x < GC) {
+        const int i = threadIdx.x;
+        const int row = i < len ? b.seq_rows[row0 + i] : 0;
+        rows[i] = row;
+        if (!CH) {
+            g_s[i] = i < len ? (double)a.log_keep[(size_t)row * H + h] : 0.0;
+            put_s[i] = i < len ? a.put[(size_t)row * H + h] : 0.f;
+        }
+    }
+    __syncthreads();
+    for (int j = warp; j < GC; j += GC_THREADS / 32) {
+        const size_t row = rows[j];
+#pragma unroll 4
+        for (int d = lane; d < D4; d += 32) {
+            float q = 0.f, k = 0.f, f = 1.f;
+            if (j < len && d < D) {
+                q = gated_q(a, row, h * D + d);
+                if (CH) gated_f(a, row, h * D + d, f, k);
+                else k = a.k[row * a.ldk + h * D + d];
+            }
+            Q[j * DP + d] = q;
+            K[j * DP + d] = k;
+            if (CH) F[j * DP + d] = f;
+        }
+    }
+    double gsum = 0.0;
+    if (!CH && threadIdx.x < GC)
+        for (int j = 0; j <= threadIdx.x; ++j) gsum += g_s[j];
+    __syncthreads();
+    if (!CH && threadIdx.x < GC) { g_s[threadIdx.x] = gsum; carry_s[threadIdx.x] = expf((float)gsum); }
+    if (CH) {
+        // inside a sub-block: for column j the running product k_j f_(j+1) .. f_i, lanes along d.  Two warps per sub-block
+        // take its columns in turn; a lane's shares for all rows i are reduced together (16 values over 32 lanes).
+        const int blk = warp >> 1;
+        const float* Qb = Q + (size_t)blk * 16 * DP;
+        const float* Kb = K + (size_t)blk * 16 * DP;
+        const float* Fb = F + (size_t)blk * 16 * DP;
+        float diag[8];
+#pragma unroll 1
+        for (int jj = 0; jj < 8; ++jj) {
+            const int j = jj * 2 + (warp & 1);
+            float acc[16];
+#pragma unroll
+            for (int i = 0; i < 16; ++i) acc[i] = 0.f;
+            for (int d = lane; d < D4; d += 32) {
+                float p = Kb[j * DP + d];
+#pragma unroll
+                for (int i = 0; i < 16; ++i)
+                    if (i >= j) {
+                        if (i > j) p *= Fb[i * DP + d];
+                        acc[i] = fmaf(Qb[i * DP + d], p, acc[i]);
+                    }
+            }
+#pragma unroll
+            for (int o = 16, m = 8; o >= 2; o >>= 1, m >>= 1) {
+                const bool hi = lane & o;
+#pragma unroll
+                for (int t = 0; t < m; ++t) {
+                    const float keep = hi ? acc[t + m] : acc[t], send = hi ? acc[t] : acc[t + m];
+                    acc[t] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+            }
+            acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1);
+            // this lane now holds row i = lane / 2 of column j
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+                if (u == jj) diag[u] = acc[0];
+        }
+        __syncthreads();
+        // rows scaled by the decay from their block's start (Q) / to their block's end (K); T: a block's whole decay
+        for (int t = threadIdx.x; t < 4 * D4; t += GC_THREADS) {
+            const int bk = t / D4, d = t - bk * D4;
+            float p = 1.f;
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+                p *= F[(bk * 16 + i) * DP + d];
+                Q[(bk * 16 + i) * DP + d] *= p;
+            }
+            T[bk * DP + d] = p;
+            p = 1.f;
+#pragma unroll
+            for (int i = 15; i >= 0; --i) {
+                K[(bk * 16 + i) * DP + d] *= p;
+                p *= F[(bk * 16 + i) * DP + d];
+            }
+        }
+        __syncthreads();
+        // between sub-blocks: thread (i, j) = (tb, cb) of the six block pairs
+        float a10 = 0.f, a20 = 0.f, a21 = 0.f, a30 = 0.f, a31 = 0.f, a32 = 0.f;
+        for (int d = 0; d < D4; d += 4) {
+            const float4 q1 = *reinterpret_cast<const float4*>(Q + (16 + tb) * DP + d), q2 = *reinterpret_cast<const float4*>(Q + (32 + tb) * DP + d);
+            const float4 q3 = *reinterpret_cast<const float4*>(Q + (48 + tb) * DP + d);
+            const float4 k0 = *reinterpret_cast<const float4*>(K + cb * DP + d), k1 = *reinterpret_cast<const float4*>(K + (16 + cb) * DP + d);
+            const float4 k2 = *reinterpret_cast<const float4*>(K + (32 + cb) * DP + d);
+            const float4 t1 = *reinterpret_cast<const float4*>(T + DP + d), t2 = *reinterpret_cast<const float4*>(T + 2 * DP + d);
+            const float4 k0t = mul4(k0, t1), k1t = mul4(k1, t2);
+            a10 = dot4(q1, k0, a10);
+            a21 = dot4(q2, k1, a21);
+            a32 = dot4(q3, k2, a32);
+            a20 = dot4(q2, k0t, a20);
+            a31 = dot4(q3, k1t, a31);
+            a30 = dot4(q3, mul4(k0t, t2), a30);
+        }
+        __syncthreads();                          // F is done with: A takes its place
+        A[(16 + tb) * GC_AS + cb] = a10;
+        A[(32 + tb) * GC_AS + cb] = a20;
+        A[(32 + tb) * GC_AS + 16 + cb] = a21;
+        A[(48 + tb) * GC_AS + cb] = a30;
+        A[(48 + tb) * GC_AS + 16 + cb] = a31;
+        A[(48 + tb) * GC_AS + 32 + cb] = a32;
+#pragma unroll
+        for (int jj = 0; jj < 8; ++jj) {
+            const int j = jj * 2 + (warp & 1), i = lane >> 1;
+            if ((lane & 1) == 0) A[(blk * 16 + i) * GC_AS + blk * 16 + j] = i >= j ? diag[jj] : 0.f;
+        }
+        // Q: the decay from the chunk's start
+        for (int t = threadIdx.x; t < 3 * D4; t += GC_THREADS) {
+            const int bk = t / D4 + 1, d = t - (bk - 1) * D4;
+            float p = T[d];
+            for (int u = 1; u < bk; ++u) p *= T[u * DP + d];
+#pragma unroll
+            for (int i = 0; i < 16; ++i) Q[(bk * 16 + i) * DP + d] *= p;
+        }
+    } else {
+        __syncthreads();
+        // A[i][j] = e^(G_i - G_j) p_j q_i . k_j, rows tb * 4 + r, columns cb + 16 u
+        float acc[4][4];
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+#pragma unroll
+            for (int u = 0; u < 4; ++u) acc[r][u] = 0.f;
+        for (int d = 0; d < D4; d += 4) {
+            float4 qv[4], kv[4];
+#pragma unroll
+            for (int r = 0; r < 4; ++r) qv[r] = *reinterpret_cast<const float4*>(Q + (tb * 4 + r) * DP + d);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) kv[u] = *reinterpret_cast<const float4*>(K + (cb + 16 * u) * DP + d);
+#pragma unroll
+            for (int r = 0; r < 4; ++r)
+#pragma unroll
+                for (int u = 0; u < 4; ++u) acc[r][u] = dot4(qv[r], kv[u], acc[r][u]);
+        }
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int i = tb * 4 + r, j = cb + 16 * u;
+                A[i * GC_AS + j] = j <= i ? acc[r][u] * put_s[j] * expf((float)(g_s[i] - g_s[j])) : 0.f;
+            }
+        __syncthreads();
+        // den_i = sum_j A[i][j] + e^G_i n . q_i; Q leaves scaled by e^G_i
+        const float* nP = sc.ns + ((size_t)ci * H + h) * D;
+        for (int i = warp; i < GC; i += GC_THREADS / 32) {
+            const float cy = carry_s[i];
+            float s = A[i * GC_AS + lane] + A[i * GC_AS + 32 + lane];      // zeros above the diagonal
+            for (int d = lane; d < D; d += 32) {
+                const float q = Q[i * DP + d] * cy;
+                Q[i * DP + d] = q;
+                s = fmaf(q, nP[d], s);
+            }
+            s = warp_sum(s);
+            if (lane == 0 && i < len) a.den[(size_t)rows[i] * H + h] = s;
+        }
+    }
+    // y = A V + Q P, V and P in tiles of 128 columns (P also 64 rows at a time) in the keys' place
+    const float* P = sc.S + ((size_t)ci * H + h) * D * V;
+    float* W = K;
+    for (int c0 = 0; c0 < V; c0 += 128) {
+        const int cw = min(128, V - c0);
+        float acc[4][8];
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+#pragma unroll
+            for (int u = 0; u < 8; ++u) acc[r][u] = 0.f;
+        __syncthreads();
+        gated_stage_v(a, rows, len, h, c0, W);
+        __syncthreads();
+        auto tile_mac = [&](const float* X, int ldx, int kn) {           // acc += X[rows][0 .. kn) . W[0 .. kn)[columns], kn a multiple of 4
+            for (int k = 0; k < kn; k += 4) {
+                float4 x[4];
+#pragma unroll
+                for (int r = 0; r < 4; ++r) x[r] = *reinterpret_cast<const float4*>(X + (tb * 4 + r) * ldx + k);
+#pragma unroll
+                for (int kk = 0; kk < 4; ++kk) {
+                    const float4 w0 = *reinterpret_cast<const float4*>(W + (k + kk) * 128 + cb * 4), w1 = *reinterpret_cast<const float4*>(W + (k + kk) * 128 + 64 + cb * 4);
+                    const float wv[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+                    for (int r = 0; r < 4; ++r) {
+                        const float xv = kk == 0 ? x[r].x : kk == 1 ? x[r].y : kk == 2 ? x[r].z : x[r].w;
+#pragma unroll
+                        for (int u = 0; u < 8; ++u) acc[r][u] = fmaf(xv, wv[u], acc[r][u]);
+                    }
+                }
+            }
+        };
+        if (tb * 4 < len) tile_mac(A, GC_AS, tb * 4 + 4);
+        for (int d0 = 0; d0 < D; d0 += GC) {
+            const int dn = min(GC, D - d0), dn4 = (dn + 3) & ~3;
+            __syncthreads();
+            for (int d = warp; d < dn4; d += GC_THREADS / 32) {
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    const int cc = lane + 32 * u;
+                    W[d * 128 + cc] = (d < dn && cc < cw) ? P[(size_t)(d0 + d) * V + c0 + cc] : 0.f;
+                }
+            }
+            __syncthreads();
+            if (tb * 4 < len) tile_mac(Q + d0, DP, dn4);
+        }
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+            const int i = tb * 4 + r;
+            if (i >= len) continue;
+            float* y = a.y + (size_t)rows[i] * a.ld_y + (size_t)h * V + c0;
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const int cc = (u >> 2) * 64 + cb * 4 + (u & 3);
+                if (cc < cw) y[cc] = acc[r][u];
+            }
+        }
+    }
+}
+
+static size_t gated_state_smem(int dim, bool ch) {
+    const size_t D8 = (dim + 7) & ~7, vt = (ch && D8 > 128) ? D8 : 128;
+    return (size_t)GC * (D8 + vt) * sizeof(float);
+}
+static size_t gated_out_smem(int dim, bool ch) {
+    const size_t DP = ((dim + 3) & ~3) + 4, k = DP > 128 ? DP : 128, f = (ch && DP > GC_AS) ? DP : GC_AS;
+    return ((size_t)GC * (DP + k + f) + (ch ? 4 * DP : 0)) * sizeof(float);
+}
+
+// 0 if the chunked kernels take these sizes
+extern "C" int dl_gated_scan_chunked_supported(int dim, int vdim, int channel) {
+    return dim >= 1 && vdim >= 1 && gated_out_smem(dim, channel) <= 225 * 1024 && gated_state_smem(dim, channel) <= 225 * 1024 ? 0 : -1;
+}
+
+// f32 of scratch for a batch of M rows in n_seq sequences
+extern "C" long long dl_gated_chunk_floats(int M, int n_seq, int n_heads, int dim, int vdim) {
+    return (long long)(M / GC + n_seq) * n_heads * dim * ((long long)vdim + 2);
+}
+
+template <bool CH>
+static int launch_gated_chunked(const DlMambaBatch& b, int n_seq, int max_chunks, const DlGatedArgs& a, const GatedScratch& sc, cudaStream_t st) {
+    const size_t smem1 = gated_state_smem(a.dim, CH), smem3 = gated_out_smem(a.dim, CH);
+    cudaError_t e = cudaFuncSetAttribute(gated_chunk_state_kernel<CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gated_chunk_out_kernel<CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
+    if (e != cudaSuccess) { dl_set_error("dl_gated_scan_chunked: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
+    const dim3 grid(n_seq, max_chunks, a.n_heads);
+    gated_chunk_state_kernel<CH><<<grid, GC_THREADS, smem1, st>>>(b, a, sc);
+    gated_chunk_prefix_kernel<CH><<<dim3(n_seq, a.n_heads, (a.dim * (a.vdim + (CH ? 0 : 1)) + 255) / 256), 256, 0, st>>>(b, a, sc);
+    gated_chunk_out_kernel<CH><<<grid, GC_THREADS, smem3, st>>>(b, a, sc);
+    return 0;
+}
+
+// max_chunks: the most chunks any sequence of the batch has; chunk_slots: M / GC + n_seq of the largest batch the scratch is for
+extern "C" int dl_gated_scan_chunked(const DlMambaBatch* batch, int n_seq, int max_chunks, const DlGatedArgs* args, float* scratch,
+                                     int chunk_slots, void* stream) {
+    const DlGatedArgs& a = *args;
+    const bool ch = a.f != nullptr;
+    if (gated_args_ok(a, "dl_gated_scan_chunked")) return -1;
+    if (dl_gated_scan_chunked_supported(a.dim, a.vdim, ch) != 0 || scratch == nullptr) { dl_set_error("dl_gated_scan_chunked: sizes not supported (dim %d, vdim %d)", a.dim, a.vdim); return -1; }
+    if (n_seq < 1 || max_chunks < 1) return 0;
+    GatedScratch sc;
+    const size_t slots = (size_t)chunk_slots;
+    sc.S = scratch;
+    sc.dec = sc.S + slots * a.n_heads * a.dim * a.vdim;
+    sc.ns = sc.dec + slots * a.n_heads * a.dim;
+    const int rc = ch ? launch_gated_chunked<true>(*batch, n_seq, max_chunks, a, sc, (cudaStream_t)stream)
+                      : launch_gated_chunked<false>(*batch, n_seq, max_chunks, a, sc, (cudaStream_t)stream);
+    if (rc != 0) return rc;
+    LAYER_CHECK_LAUNCH("dl_gated_scan_chunked");
+    return 0;
+}
+
+// ------------------------------------------------------------------------------------------------
+// gates of the matrix memory: one warp per (sequence, head).  A token maps the running maximum u to max(b + u, a); such maps
+// compose (F, A) o (F', A') = (F + F', max(F' + A, A')), so 32 tokens are scanned by shuffles; four blocks of 32 tokens are
+// loaded together.
+// ------------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(32) mlstm_gates_kernel(DlMambaBatch b, DlMlstmGatesArgs a) {
+    const int n = blockIdx.x, h = blockIdx.y, lane = threadIdx.x, H = a.n_heads;
+    float* ug = a.u_state + (size_t)b.seq_slot[n] * H + h;
+    float u = b.seq_pos0[n] == 0 ? 0.f : *ug;
+    const float bi = a.bi[h], bf = a.bf[h], cap = a.cap;
+    const int r0 = b.seq_start[n], r1 = b.seq_start[n + 1];
+    for (int rb = r0; rb < r1; rb += 128) {
+        int row[4];
+        float zi[4], zf[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) { const int r = rb + k * 32 + lane; row[k] = r < r1 ? b.seq_rows[r] : -1; }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            zi[k] = row[k] >= 0 ? a.zi[(size_t)row[k] * a.ld + h] : 0.f;
+            zf[k] = row[k] >= 0 ? a.zf[(size_t)row[k] * a.ld + h] : 0.f;
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            if (rb + k * 32 >= r1) break;
+            const bool live = row[k] >= 0;
+            const float ai = cap * tanhf((zi[k] + bi) / cap);
+            const float lb = -softplus_f(-cap * tanhf((zf[k] + bf) / cap));
+            float F = live ? lb : 0.f, A = live ? ai : -INFINITY;      // a lane without a token: the identity
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float Fp = __shfl_up_sync(0xffffffffu, F, o), Ap = __shfl_up_sync(0xffffffffu, A, o);
+                if (lane >= o) { A = fmaxf(F + Ap, A); F += Fp; }
+            }
+            const float un = fmaxf(F + u, A);
+            float up = __shfl_up_sync(0xffffffffu, un, 1);
+            if (lane == 0) up = u;
+            if (live) {
+                const size_t at = (size_t)row[k] * H + h;
+                a.log_keep[at] = lb + up - un;
+                a.put[at] = expf(ai - un);
+                a.floor_[at] = expf(-un);
+            }
+            u = __shfl_sync(0xffffffffu, un, 31);
+        }
+    }
+    if (lane == 0) *ug = u;
+}
+
+extern "C" int dl_mlstm_gates(const DlMambaBatch* batch, int n_seq, const DlMlstmGatesArgs* args, void* stream) {
+    if (args->n_heads < 1 || !(args->cap > 0.f)) { dl_set_error("dl_mlstm_gates: bad shape"); return -1; }
+    if (n_seq < 1) return 0;
+    mlstm_gates_kernel<<<dim3(n_seq, args->n_heads), 32, 0, (cudaStream_t)stream>>>(*batch, *args);
+    LAYER_CHECK_LAUNCH("dl_mlstm_gates");
+    return 0;
+}
+
+// ------------------------------------------------------------------------------------------------
+// normalised heads: one warp per (row, head), up to 512 columns kept in registers between the sum and the scaling
+// ------------------------------------------------------------------------------------------------
+#define HN_WARPS 8
+#define HN_CACHE 16
+__global__ void __launch_bounds__(HN_WARPS * 32) head_norm_kernel(DlHeadNormArgs a) {
+    const int m = blockIdx.x, lane = threadIdx.x & 31, V = a.vdim;
+    const int h = blockIdx.y * HN_WARPS + (threadIdx.x >> 5);
+    if (a.xh && blockIdx.y == 0) xh_zero_tail(a.xh, a.ncap, m, a.n_heads * V, threadIdx.x, HN_WARPS * 32);
+    if (h >= a.n_heads) return;
+    const float* y = a.y + (size_t)m * a.ld_y + (size_t)h * V;
+    float scale = 1.f;
+    if (a.den) scale = 1.f / (fmaxf(fabsf(a.den[(size_t)m * a.n_heads + h]), a.floor_[(size_t)m * a.n_heads + h]) + 1e-6f);
+    const bool cached = V <= 32 * HN_CACHE;
+    float v[HN_CACHE];
+    float ss = 0.f;
+    if (cached) {
+#pragma unroll
+        for (int k = 0; k < HN_CACHE; ++k) {
+            const int i = lane + 32 * k;
+            v[k] = i < V ? y[i] * scale : 0.f;
+            ss = fmaf(v[k], v[k], ss);
+        }
+    } else {
+        for (int i = lane; i < V; i += 32) { const float t = y[i] * scale; ss = fmaf(t, t, ss); }
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)V + a.eps);
+    const float* w = a.w + (a.w_full ? (size_t)h * V : 0);
+    const float* g = a.gate ? a.gate + (size_t)m * a.ld_gate + (size_t)h * V : nullptr;
+    auto put = [&](int i, float t) {
+        t = t * inv * w[i];
+        if (g) t *= sigmoid_f(g[i]);
+        if (a.xh) xh_store(a.xh, a.ncap, m, h * V + i, t);
+        else a.out[(size_t)m * a.ld_out + (size_t)h * V + i] = t;
+    };
+    if (cached) {
+#pragma unroll
+        for (int k = 0; k < HN_CACHE; ++k)
+            if (lane + 32 * k < V) put(lane + 32 * k, v[k]);
+    } else {
+        for (int i = lane; i < V; i += 32) put(i, y[i] * scale);
+    }
+}
+
+extern "C" int dl_head_norm(const DlHeadNormArgs* args, void* stream) {
+    const DlHeadNormArgs& a = *args;
+    if (a.M < 1 || a.n_heads < 1 || a.vdim < 1 || !a.w || (!a.out && !a.xh) || (a.den && !a.floor_)) { dl_set_error("dl_head_norm: bad arguments"); return -1; }
+    head_norm_kernel<<<dim3(a.M, (a.n_heads + HN_WARPS - 1) / HN_WARPS), HN_WARPS * 32, 0, (cudaStream_t)stream>>>(a);
+    LAYER_CHECK_LAUNCH("dl_head_norm");
+    return 0;
+}

@@ -59,3 +59,27 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log1pf(expf(v)); }
+
+// sigma(v) and 1 - sigma(v), both without cancellation.  The divisor lies in [1, 2], where the fast division is good to 2 ulp (and
+// brings no slow-path call into kernels that hold much in registers)
+__device__ __forceinline__ void sigmoid_pair_f(float v, float& s, float& c) {
+    const float e = expf(-fabsf(v)), r = __fdividef(1.f, 1.f + e);
+    s = v >= 0.f ? r : e * r;
+    c = v >= 0.f ? e * r : r;
+}
+__device__ __forceinline__ float gelu_tanh_f(float v) {
+    return 0.5f * v * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * v * v, v, v)));
+}
+
+// Activation image of the tcgen05 GEMM (see dense.cu): bytes from the image's start to element (row m, column k).  Eight
+// neighbouring columns k .. k + 7 (k % 8 == 0) of a row are 16 consecutive bytes.
+__device__ __forceinline__ size_t xh_offset(int ncap, int m, int k) {
+    return ((size_t)(k >> 7) * (ncap >> 3) + (m >> 3)) * 2048 + (size_t)((k & 127) >> 3) * 128 + (m & 7) * 16 + (k & 7) * 2;
+}
+__device__ __forceinline__ void xh_store(uint8_t* xh, int ncap, int m, int k, float v) {
+    *reinterpret_cast<__nv_bfloat16*>(xh + xh_offset(ncap, m, k)) = __float2bfloat16_rn(v);
+}
+// zeros in columns [K, round_up(K, 128)) of row m, by the threads of one CTA or warp (thread t of n)
+__device__ __forceinline__ void xh_zero_tail(uint8_t* xh, int ncap, int m, int K, int t, int n) {
+    for (int k = K + t; k < ((K + 127) & ~127); k += n) xh_store(xh, ncap, m, k, 0.f);
+}

@@ -127,3 +127,88 @@ extern "C" int dl_poly_norm(const float* x, long long ldx, float* y, long long l
     LAYER_CHECK_LAUNCH("dl_poly_norm");
     return 0;
 }
+
+// ------------------------------------------------------------------------------------------------
+// One step of a residual stream: a row's sum (the stream, plain terms, terms normalised first, a vector for every row), then up
+// to two normed copies of it, as f32 rows or straight into the bf16 activation image of the products that read them.  One
+// CTA per row; the row stays in shared memory between the sums.  Three dependent passes at most: the roots of the normalised
+// terms, the sum and its root, the copies.
+// ------------------------------------------------------------------------------------------------
+#define RS_THREADS 256
+__global__ void __launch_bounds__(RS_THREADS) residual_step_kernel(DlResidualArgs a) {
+    extern __shared__ __align__(16) float row_s[];           // [dim], then a and b's rows when they are there
+    __shared__ float red[32];
+    const int m = blockIdx.x, dim = a.dim, tid = threadIdx.x;
+    const size_t src = a.rows ? a.rows[m] : m;
+    const float* xi = a.x_in ? a.x_in + src * a.ld_in : nullptr;
+    float inv_a = 0.f, inv_b = 0.f;
+    float* ra = row_s + dim;
+    float* rb = ra + dim;
+    if (a.norm_a) {
+        const float* pa = a.norm_a + src * a.ld_a;
+        const float* pb = a.norm_b ? a.norm_b + src * a.ld_b : nullptr;
+        float sa = 0.f, sb = 0.f;
+#pragma unroll 4
+        for (int i = tid; i < dim; i += RS_THREADS) {
+            const float u = pa[i], v = pb ? pb[i] : 0.f;
+            ra[i] = u;
+            if (pb) rb[i] = v;
+            sa = fmaf(u, u, sa);
+            sb = fmaf(v, v, sb);
+        }
+        inv_a = 1.f / sqrtf(block_sum(sa, red) / (float)dim + a.eps);
+        if (pb) inv_b = 1.f / sqrtf(block_sum(sb, red) / (float)dim + a.eps);
+    }
+    const float* p1 = a.add1 ? a.add1 + src * a.ld_add1 : nullptr;
+    const float* p2 = a.add2 ? a.add2 + src * a.ld_add2 : nullptr;
+    const float* p3 = a.add3 ? a.add3 + src * a.ld_add3 : nullptr;
+    float ss = 0.f;
+#pragma unroll 4
+    for (int i = tid; i < dim; i += RS_THREADS) {            // a thread meets only its own columns again: no barrier for row_s, ra, rb
+        float t = 0.f;
+        if (a.norm_a) {
+            t = a.w_a[i] * (ra[i] * inv_a);
+            if (a.norm_b) t = fmaf(a.w_b[i], rb[i] * inv_b, t);
+        }
+        if (p1) t += p1[i];
+        if (p2) t += p2[i];
+        if (p3) t += p3[i];
+        if (xi) t += xi[i];
+        if (a.vec) t += a.vec[i];
+        row_s[i] = t;
+        if (a.x) a.x[(size_t)m * a.ldx + i] = t;
+        ss = fmaf(t, t, ss);
+    }
+    if (!a.w1) return;
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)dim + a.eps);
+#pragma unroll 4
+    for (int i = tid; i < dim; i += RS_THREADS) {
+        const float t = row_s[i] * inv;
+        const float u = t * a.w1[i];
+        if (a.xh1) xh_store(a.xh1, a.ncap, m, i, u); else a.h1[(size_t)m * a.ldh + i] = u;
+        if (a.w2) {
+            const float v = t * a.w2[i];
+            if (a.xh2) xh_store(a.xh2, a.ncap, m, i, v); else a.h2[(size_t)m * a.ldh + i] = v;
+        }
+    }
+    if (a.xh1) xh_zero_tail(a.xh1, a.ncap, m, dim, tid, RS_THREADS);
+    if (a.xh2) xh_zero_tail(a.xh2, a.ncap, m, dim, tid, RS_THREADS);
+}
+
+extern "C" int dl_residual_step(const DlResidualArgs* args, void* stream) {
+    const DlResidualArgs& a = *args;
+    if (a.M < 1 || a.dim < 1) { dl_set_error("dl_residual_step: bad shape"); return -1; }
+    if ((a.norm_b && !a.norm_a) || (a.norm_a && !a.w_a) || (a.norm_b && !a.w_b) || (a.w2 && !a.w1) || (a.w1 && !a.h1 && !a.xh1) || (a.w2 && !a.h2 && !a.xh2)) {
+        dl_set_error("dl_residual_step: terms do not fit together");
+        return -1;
+    }
+    const size_t smem = (size_t)a.dim * (1 + (a.norm_a ? 1 : 0) + (a.norm_b ? 1 : 0)) * sizeof(float);
+    if (smem > 200 * 1024) { dl_set_error("dl_residual_step: rows of %d do not fit shared memory", a.dim); return -1; }
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(residual_step_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) { dl_set_error("dl_residual_step: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
+    }
+    residual_step_kernel<<<a.M, RS_THREADS, smem, (cudaStream_t)stream>>>(a);
+    LAYER_CHECK_LAUNCH("dl_residual_step");
+    return 0;
+}

@@ -8,6 +8,10 @@
 // -- head h carries ONE query of key_heads * dim numbers that meets the keys of ALL key/value heads side by side, and
 // the kernel is an ordinary attention tile kernel whose K dimension is key_heads * dim: nothing is exchanged between
 // heads here.  key_heads <= 1 is plain grouped-query attention (the query meets its own group's key only).
+// The mirror image, weights mixed AFTER the softmax (value_heads = kv_heads):
+//     out_h(i) = sum_j ( sum_g talk[h][g] p_g(i, j) ) v_c(h),j = sum_g talk[h][g] ( sum_j p_g(i, j) v_c(h),j )
+// head g's weights meet the values of EVERY key/value head side by side (WIDE: a CTA's warps accumulate `vs` value heads,
+// 8 NV columns, of one group of query heads; ceil(kv_heads / vs) CTAs share a group), and dl_talk_mix sums the heads.
 //
 // Cache [page][kv_head][32][dim + vdim] bf16, one line = key | value.  A CTA owns a tile of up to `rq` consecutive
 // positions of one sequence and the query heads of ONE key/value head g: (position, head-of-the-group) pairs stack on the
@@ -42,30 +46,34 @@ __host__ __device__ __forceinline__ int ta_stride(int n) {      // bf16 elements
     return s;
 }
 
-template <int DK, int NV, int NR, bool ALLG>
+template <int DK, int NV, int NR, bool ALLG, bool WIDE>
 __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_mma_kernel(DlWindowAttnArgs a, const int* __restrict__ tile_rows, int rq, int n_splits,
-                                                                float* __restrict__ partial) {
+                                                                float* __restrict__ partial, int vs) {
     constexpr int DP = 16 * DK, DVP = 8 * NV, TA_ROWS = 16 * NR;
+    const int DVH = WIDE ? DVP / vs : DVP;                                          // a value head's columns, padding included
+    const int nvb = WIDE ? (a.kv_heads + vs - 1) / vs : 1;                          // blocks of `vs` value heads
     const int THREADS = blockDim.x;
     extern __shared__ __align__(16) uint8_t smraw[];
     __shared__ int s_row[TA_ROWS];
     const int D = a.dim, DV = a.vdim, LD = D + DV;
     const int KH = a.key_heads > 1 ? a.key_heads : 1, QD = KH * D, QDP = KH * DP;
     // staged line: [ keys of KS heads | values of VS heads ]; ALLG: every head's, else all (or this group's) keys and this group's values
-    const int KS = ALLG ? a.kv_heads : KH, VS = ALLG ? a.kv_heads : 1, VOFF = KS * DP;
-    const int LDS = ta_stride(VOFF + VS * DVP), QS = ta_stride(QDP);
+    const int KS = ALLG ? a.kv_heads : KH, VS = WIDE ? (ALLG ? nvb * vs : vs) : ALLG ? a.kv_heads : 1, VOFF = KS * DP;
+    const int LDS = ta_stride(VOFF + VS * DVH), QS = ta_stride(QDP);
     __nv_bfloat16* kv_s = reinterpret_cast<__nv_bfloat16*>(smraw);                  // [2][TA_PAGE][LDS]
     __nv_bfloat16* q_s = kv_s + (size_t)2 * TA_PAGE * LDS;                          // [TA_ROWS (ALLG: per key/value head)][QS]: the stacked queries
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
     // grid (key/value heads, tiles, page shares).  A sequence's later tiles walk more pages: they start first, so that the
     // short ones fill the SMs at the end
     const int tile = (int)gridDim.y - 1 - (int)blockIdx.y, rep = a.heads / a.kv_heads;
-    const int g = ALLG ? min(warp, a.kv_heads - 1) : (int)blockIdx.x;              // ALLG: warp g multiplies key/value head g
+    // ALLG: warp g multiplies key/value head g (WIDE: warp g * nvb + vb its value block vb); else the same by CTA
+    const int gv = ALLG ? min(warp, a.kv_heads * nvb - 1) : (int)blockIdx.x;
+    const int g = WIDE ? gv / nvb : gv, vb = WIDE ? gv - g * nvb : 0, v0 = WIDE ? vb * vs : g;      // v0: first value head
     const int wrow = ALLG ? 0 : warp;                                               // this warp's block of 16 stacked rows among its group's
     const int qrow0 = ALLG ? g * 16 : warp * 16;                                    // ... and where that block's queries sit in q_s
     if (threadIdx.x < rq) s_row[threadIdx.x] = tile_rows[(size_t)tile * rq + threadIdx.x];
     // the padding of keys and values stays zero: the copies below never touch it
-    if (D != DP || DV != DVP)
+    if (D != DP || DV != DVH || (WIDE && nvb * vs != a.kv_heads))
         for (int i = threadIdx.x; i < 2 * TA_PAGE * LDS / 8; i += THREADS) reinterpret_cast<uint4*>(kv_s)[i] = make_uint4(0u, 0u, 0u, 0u);
     __syncthreads();
     int n_rows = 0;
@@ -80,7 +88,7 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
         pg_lo += (int)blockIdx.z * per;
         pg_hi = min(pg_hi, pg_lo + per - 1);
     }
-    const bool active = ALLG ? warp < a.kv_heads : (warp < NR && warp * 16 < n_rows * rep);
+    const bool active = ALLG ? warp < a.kv_heads * nvb : (warp < NR && warp * 16 < n_rows * rep);
     const float c1 = a.scale * TA_LOG2E;
 
     // this thread's two stacked rows: s = position-in-tile * rep + head-in-group
@@ -119,8 +127,10 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
             for (int p = sl; p < kch; p += TPL) cp_async16(dst + c * DP + p * 8, sk + p * 8);
         }
         for (int c = 0; c < VS; ++c) {
-            const __nv_bfloat16* sv = src0 + (size_t)(ALLG ? c : g) * TA_PAGE * LD + D;
-            for (int p = sl; p < vch; p += TPL) cp_async16(dst + VOFF + c * DVP + p * 8, sv + p * 8);
+            const int vh = ALLG ? c : v0 + c;
+            if (WIDE && vh >= a.kv_heads) break;
+            const __nv_bfloat16* sv = src0 + (size_t)vh * TA_PAGE * LD + D;
+            for (int p = sl; p < vch; p += TPL) cp_async16(dst + VOFF + c * DVH + p * 8, sv + p * 8);
         }
     };
     if (pg_lo <= pg_hi) issue(pg_lo, 0);
@@ -198,7 +208,7 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
             for (int vp = 0; vp < NV / 2; ++vp) {
                 const int vt = 2 * vp + (mat >> 1);
                 uint32_t b[4];
-                ldmatrix_x4_trans(b, kv + (size_t)(ks * 16 + (mat & 1) * 8 + rr) * LDS + VOFF + (ALLG ? g * DVP : 0) + vt * 8);
+                ldmatrix_x4_trans(b, kv + (size_t)(ks * 16 + (mat & 1) * 8 + rr) * LDS + VOFF + (ALLG ? v0 * DVH : 0) + vt * 8);
                 mma_bf16(o[2 * vp], pa, b[0], b[1]);
                 mma_bf16(o[2 * vp + 1], pa, b[2], b[3]);
             }
@@ -208,7 +218,7 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     if (n_splits > 1) {                  // unnormalised sums, running maximum and sum per stacked row, for the merge kernel
-        float* base = partial + (((size_t)tile * a.kv_heads + g) * n_splits + blockIdx.z) * TA_ROWS * (DVP + 2);
+        float* base = partial + (((size_t)tile * a.kv_heads * nvb + gv) * n_splits + blockIdx.z) * TA_ROWS * (DVP + 2);
         if (ok0) {
             float* dst = base + (size_t)s0 * (DVP + 2);
 #pragma unroll
@@ -228,18 +238,34 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
         if (ok1) l1 += ta_ex2(a.sink[g * rep + s1 % rep] * TA_LOG2E - m1);
     }
     if (ok0) {
-        float* dst = a.out + (size_t)s_row[r0] * a.ldo + (size_t)(g * rep + s0 % rep) * DV;
+        float* dst = a.out + (size_t)s_row[r0] * a.ldo + (size_t)(g * rep + s0 % rep) * (WIDE ? a.kv_heads * DV : DV);
         const float inv = 1.f / l0;
+        if (WIDE) {
+#pragma unroll
+            for (int v = 0; v < NV; ++v) {
+                const int vh = v * 8 / DVH, i = v * 8 - vh * DVH;
+                if (i < DV && v0 + vh < a.kv_heads)
+                    *reinterpret_cast<float2*>(dst + (size_t)(v0 + vh) * DV + i + tig * 2) = make_float2(o[v][0] * inv, o[v][1] * inv);
+            }
+        }
 #pragma unroll
         for (int v = 0; v < NV; ++v)
-            if (v * 8 < DV) *reinterpret_cast<float2*>(dst + v * 8 + tig * 2) = make_float2(o[v][0] * inv, o[v][1] * inv);
+            if (!WIDE && v * 8 < DV) *reinterpret_cast<float2*>(dst + v * 8 + tig * 2) = make_float2(o[v][0] * inv, o[v][1] * inv);
     }
     if (ok1) {
-        float* dst = a.out + (size_t)s_row[r1] * a.ldo + (size_t)(g * rep + s1 % rep) * DV;
+        float* dst = a.out + (size_t)s_row[r1] * a.ldo + (size_t)(g * rep + s1 % rep) * (WIDE ? a.kv_heads * DV : DV);
         const float inv = 1.f / l1;
+        if (WIDE) {
+#pragma unroll
+            for (int v = 0; v < NV; ++v) {
+                const int vh = v * 8 / DVH, i = v * 8 - vh * DVH;
+                if (i < DV && v0 + vh < a.kv_heads)
+                    *reinterpret_cast<float2*>(dst + (size_t)(v0 + vh) * DV + i + tig * 2) = make_float2(o[v][2] * inv, o[v][3] * inv);
+            }
+        }
 #pragma unroll
         for (int v = 0; v < NV; ++v)
-            if (v * 8 < DV) *reinterpret_cast<float2*>(dst + v * 8 + tig * 2) = make_float2(o[v][2] * inv, o[v][3] * inv);
+            if (!WIDE && v * 8 < DV) *reinterpret_cast<float2*>(dst + v * 8 + tig * 2) = make_float2(o[v][2] * inv, o[v][3] * inv);
     }
 }
 
@@ -247,12 +273,14 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
 // gathered into shared memory, every (head, share) weight e^(m_k - m) / l is formed once, then a thread per (head,
 // column) sums the shares.
 __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, const int* __restrict__ tile_rows, int rq, int n_splits,
-                                                         const float* __restrict__ partial, int DVP, int TA_ROWS) {
+                                                         const float* __restrict__ partial, int DVP, int TA_ROWS, int vs) {
     __shared__ float w_s[64 * TA_MAX_SPLITS], l_s[64 * TA_MAX_SPLITS];      // heads of one group x shares
-    const int tile = blockIdx.x, g = blockIdx.y, r = blockIdx.z, DV = a.vdim, rep = a.heads / a.kv_heads;
+    const bool wide = a.value_heads > 1;                      // blockIdx.y: (key/value head of the scores, block of vs value heads)
+    const int nvb = wide ? (a.kv_heads + vs - 1) / vs : 1, DVH = wide ? DVP / vs : DVP;
+    const int tile = blockIdx.x, g = blockIdx.y / nvb, v0 = ((int)blockIdx.y - g * nvb) * vs, r = blockIdx.z, DV = a.vdim, rep = a.heads / a.kv_heads;
     const int m = tile_rows[(size_t)tile * rq + r];
     if (m < 0) return;
-    const float* base = partial + ((size_t)tile * a.kv_heads + g) * n_splits * TA_ROWS * (DVP + 2);
+    const float* base = partial + ((size_t)tile * a.kv_heads * nvb + blockIdx.y) * n_splits * TA_ROWS * (DVP + 2);
     for (int idx = threadIdx.x; idx < rep * n_splits; idx += blockDim.x) {
         const int hg = idx / n_splits, k = idx - hg * n_splits;
         const float* p = base + ((size_t)k * TA_ROWS + r * rep + hg) * (DVP + 2);
@@ -274,83 +302,136 @@ __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, con
         for (int k = 0; k < n_splits; ++k) w_s[hg * n_splits + k] *= inv;
     }
     __syncthreads();
-    for (int idx = threadIdx.x; idx < rep * DV; idx += blockDim.x) {
-        const int hg = idx / DV, c = idx - hg * DV;
-        const float* p = base + (size_t)(r * rep + hg) * (DVP + 2) + c;
+    const int nv = wide ? min(vs, a.kv_heads - v0) : 1, W = nv * DV;
+    for (int idx = threadIdx.x; idx < rep * W; idx += blockDim.x) {
+        const int hg = idx / W, c = idx - hg * W, vh = c / DV;
+        const float* p = base + (size_t)(r * rep + hg) * (DVP + 2) + vh * DVH + (c - vh * DV);
         float acc = 0.f;                      // a share without pages left zeros and weighs 0: every load can go out at once
 #pragma unroll 8
         for (int k = 0; k < n_splits; ++k) acc = fmaf(w_s[hg * n_splits + k], p[(size_t)k * TA_ROWS * (DVP + 2)], acc);
-        a.out[(size_t)m * a.ldo + (size_t)(g * rep + hg) * DV + c] = acc;
+        a.out[(size_t)m * a.ldo + (wide ? (size_t)((g * rep + hg) * a.kv_heads + v0) * DV : (size_t)(g * rep + hg) * DV) + c] = acc;
     }
 }
 
+// out_h = sum_g talk[h][g] wide_g[c(h)]: one CTA per (row, key/value head c); the columns of head c of every head's wide row are
+// read once, each thread forms its column of all heads of group c
+template <int REP>
+__global__ void __launch_bounds__(128) talk_mix_kernel(const float* __restrict__ wide, const float* __restrict__ talk, int heads, int kv_heads,
+                                                       int vdim, float* __restrict__ out, long long ld_out, uint8_t* __restrict__ xh, int ncap) {
+    const int m = blockIdx.x, c = blockIdx.y, rep = heads / kv_heads;
+    const size_t row = (size_t)m * heads * kv_heads * vdim + (size_t)c * vdim;
+    if (xh && c == 0) xh_zero_tail(xh, ncap, m, heads * vdim, threadIdx.x, blockDim.x);
+    for (int i = threadIdx.x; i < vdim; i += blockDim.x)
+        for (int h0 = 0; h0 < rep; h0 += REP) {
+            float acc[REP];
+#pragma unroll
+            for (int r = 0; r < REP; ++r) acc[r] = 0.f;
+#pragma unroll 8
+            for (int g = 0; g < heads; ++g) {
+                const float v = wide[row + (size_t)g * kv_heads * vdim + i];
+#pragma unroll
+                for (int r = 0; r < REP; ++r)
+                    if (h0 + r < rep) acc[r] = fmaf(talk[(size_t)(c * rep + h0 + r) * heads + g], v, acc[r]);
+            }
+#pragma unroll
+            for (int r = 0; r < REP; ++r)
+                if (h0 + r < rep) {
+                    const int k = (c * rep + h0 + r) * vdim + i;
+                    if (xh) xh_store(xh, ncap, m, k, acc[r]);
+                    else out[(size_t)m * ld_out + k] = acc[r];
+                }
+        }
+}
+
+extern "C" int dl_talk_mix(const float* wide, const float* talk, int M, int heads, int kv_heads, int vdim, float* out, long long ld_out,
+                           uint8_t* xh, int ncap, void* stream) {
+    if (M < 1 || kv_heads < 1 || heads % kv_heads || vdim < 1 || (!out && !xh)) { dl_set_error("dl_talk_mix: bad shape"); return -1; }
+    const dim3 grid(M, kv_heads);
+    const int threads = vdim <= 32 ? 32 : vdim <= 64 ? 64 : 128, rep = heads / kv_heads;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (rep <= 2) talk_mix_kernel<2><<<grid, threads, 0, st>>>(wide, talk, heads, kv_heads, vdim, out, ld_out, xh, ncap);
+    else if (rep <= 4) talk_mix_kernel<4><<<grid, threads, 0, st>>>(wide, talk, heads, kv_heads, vdim, out, ld_out, xh, ncap);
+    else talk_mix_kernel<8><<<grid, threads, 0, st>>>(wide, talk, heads, kv_heads, vdim, out, ld_out, xh, ncap);
+    LAYER_CHECK_LAUNCH("dl_talk_mix");
+    return 0;
+}
+
 static int ta_dk(int dim) { return dim <= 32 ? 2 : dim <= 64 ? 4 : 8; }
-static int ta_nv(int vdim) { return vdim <= 64 ? 8 : vdim <= 96 ? 12 : 16; }
-static size_t ta_smem(int dim, int vdim, int key_heads, int rows) {
+// column tiles (of 8) a warp accumulates, and value heads they hold: one head of 64, 96 or 128 columns; WIDE: 2 or 4 heads of 64
+// or 2 of 128
+static int ta_vs(int vdim, int value_heads) { return value_heads <= 1 ? 1 : (vdim <= 64 && value_heads > 2) ? 4 : 2; }
+static int ta_nv(int vdim, int value_heads) {
+    if (value_heads > 1) return ta_vs(vdim, value_heads) * (vdim <= 64 ? 8 : 16);
+    return vdim <= 64 ? 8 : vdim <= 96 ? 12 : 16;
+}
+static int ta_nvb(int vdim, int value_heads) { const int vs = ta_vs(vdim, value_heads); return value_heads <= 1 ? 1 : (value_heads + vs - 1) / vs; }
+static size_t ta_smem(int dim, int vdim, int key_heads, int value_heads, int rows) {
     const int KH = key_heads > 1 ? key_heads : 1, QDP = KH * 16 * ta_dk(dim);
-    return ((size_t)2 * TA_PAGE * ta_stride(QDP + 8 * ta_nv(vdim)) + (size_t)rows * ta_stride(QDP)) * sizeof(__nv_bfloat16);
+    return ((size_t)2 * TA_PAGE * ta_stride(QDP + 8 * ta_nv(vdim, value_heads)) + (size_t)rows * ta_stride(QDP)) * sizeof(__nv_bfloat16);
 }
 // the ALLG form: every head's keys and values in a staged line, 16 stacked rows of queries per key/value head
-static size_t ta_smem_allg(int dim, int vdim, int key_heads, int kv_heads) {
+static size_t ta_smem_allg(int dim, int vdim, int key_heads, int value_heads, int kv_heads) {
     const int KH = key_heads > 1 ? key_heads : 1, DP = 16 * ta_dk(dim);
-    return ((size_t)2 * TA_PAGE * ta_stride(kv_heads * (DP + 8 * ta_nv(vdim))) + (size_t)kv_heads * 16 * ta_stride(KH * DP)) * sizeof(__nv_bfloat16);
+    const int values = value_heads > 1 ? ta_nvb(vdim, value_heads) * 8 * ta_nv(vdim, value_heads) : kv_heads * 8 * ta_nv(vdim, 1);
+    return ((size_t)2 * TA_PAGE * ta_stride(kv_heads * DP + values) + (size_t)kv_heads * 16 * ta_stride(KH * DP)) * sizeof(__nv_bfloat16);
 }
 #define TA_SMEM_MAX (220 * 1024)
-static bool ta_allg(int kv_heads, int dim, int vdim, int key_heads) {
-    return kv_heads >= 2 && kv_heads <= 8 && ta_smem_allg(dim, vdim, key_heads, kv_heads) <= TA_SMEM_MAX;
+static bool ta_allg(int kv_heads, int dim, int vdim, int key_heads, int value_heads) {
+    return kv_heads >= 2 && kv_heads * ta_nvb(vdim, value_heads) <= 8 && ta_smem_allg(dim, vdim, key_heads, value_heads, kv_heads) <= TA_SMEM_MAX;
 }
 
 // Stacked rows of a tile for portions of `longest` rows of a sequence: 128 where long portions fit the shared memory, 16
 // for decoding (at most 16 query heads per key/value head), else 64; 0: the sizes do not fit at all.
-extern "C" int dl_talk_tc_tile_rows(int heads, int kv_heads, int dim, int vdim, int key_heads, int longest) {
+extern "C" int dl_talk_tc_tile_rows(int heads, int kv_heads, int dim, int vdim, int key_heads, int value_heads, int longest) {
     if (heads < 1 || kv_heads < 1 || heads % kv_heads) return 0;
     const int rep = heads / kv_heads;
-    if (rep <= 16 && longest <= 16 / rep && ta_smem(dim, vdim, key_heads, 16) <= TA_SMEM_MAX) return 16;
-    if (rep <= 128 && longest > 64 / rep && ta_smem(dim, vdim, key_heads, 128) <= TA_SMEM_MAX) return 128;
-    if (rep <= 64 && ta_smem(dim, vdim, key_heads, 64) <= TA_SMEM_MAX) return 64;
+    if (rep <= 16 && longest <= 16 / rep && ta_smem(dim, vdim, key_heads, value_heads, 16) <= TA_SMEM_MAX) return 16;
+    if (rep <= 128 && longest > 64 / rep && ta_smem(dim, vdim, key_heads, value_heads, 128) <= TA_SMEM_MAX) return 128;
+    if (rep <= 64 && ta_smem(dim, vdim, key_heads, value_heads, 64) <= TA_SMEM_MAX) return 64;
     return 0;
 }
 
 // 0 if the kernel takes these sizes: a bf16 cache, dim and vdim multiples of 8 up to 128, at most 64 query heads per
 // key/value head, and a tile's queries plus two pages of all key heads within the shared memory of an SM
-extern "C" int dl_talk_attention_tc_supported(int heads, int kv_heads, int dim, int vdim, int key_heads, int ctype) {
+extern "C" int dl_talk_attention_tc_supported(int heads, int kv_heads, int dim, int vdim, int key_heads, int value_heads, int ctype) {
     if (ctype != DL_T_BF16 || heads < 1 || kv_heads < 1 || heads % kv_heads || heads / kv_heads > 64) return -1;
     if (dim < 8 || dim % 8 || dim > 128 || vdim < 8 || vdim % 8 || vdim > 128) return -1;
-    if (key_heads > 1 && key_heads != kv_heads) return -1;
-    if (ta_smem(dim, vdim, key_heads, 64) > TA_SMEM_MAX) return -1;
+    if ((key_heads > 1 && key_heads != kv_heads) || (value_heads > 1 && (value_heads != kv_heads || key_heads > 1))) return -1;
+    if (ta_smem(dim, vdim, key_heads, value_heads, 64) > TA_SMEM_MAX) return -1;
     return 0;
 }
 
-// partial sums of the page shares: tiles x key/value heads x shares x stacked rows (rq rows x heads of a group, rounded up
-// to the kernel's 16, 64 or 128)
+// partial sums of the page shares: tiles x key/value heads (x blocks of value heads) x shares x stacked rows (rq rows x heads of
+// a group, rounded up to the kernel's 16, 64 or 128)
 static int ta_rows_of(int rq, int rep) { return rq * rep <= 16 ? 16 : rq * rep <= 64 ? 64 : 128; }
-extern "C" long long dl_talk_tc_partial_floats(int n_tiles, int kv_heads, int n_splits, int vdim, int rows) {
-    return (long long)n_tiles * kv_heads * n_splits * rows * (8 * ta_nv(vdim) + 2);
+extern "C" long long dl_talk_tc_partial_floats(int n_tiles, int kv_heads, int n_splits, int vdim, int value_heads, int rows) {
+    return (long long)n_tiles * kv_heads * ta_nvb(vdim, value_heads) * n_splits * rows * (8 * ta_nv(vdim, value_heads) + 2);
 }
 
-template <int DK, int NV, int NR, bool ALLG>
+template <int DK, int NV, int NR, bool ALLG, bool WIDE>
 static int launch_talk_nr(const DlWindowAttnArgs& a, const int* tile_rows, int n_tiles, int rq, int n_splits, float* partial, cudaStream_t st) {
-    const size_t smem = ALLG ? ta_smem_allg(a.dim, a.vdim, a.key_heads, a.kv_heads) : ta_smem(a.dim, a.vdim, a.key_heads, 16 * NR);
+    const size_t smem = ALLG ? ta_smem_allg(a.dim, a.vdim, a.key_heads, a.value_heads, a.kv_heads) : ta_smem(a.dim, a.vdim, a.key_heads, a.value_heads, 16 * NR);
     if (smem > TA_SMEM_MAX) { dl_set_error("dl_talk_attention_tc: %zu bytes of shared memory", smem); return -1; }
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(talk_attention_mma_kernel<DK, NV, NR, ALLG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(talk_attention_mma_kernel<DK, NV, NR, ALLG, WIDE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) { dl_set_error("dl_talk_attention_tc: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
     }
-    const dim3 grid(ALLG ? 1 : a.kv_heads, n_tiles, n_splits);
-    const int threads = ALLG ? (a.kv_heads > 4 ? 256 : 128) : (NR == 8 ? 256 : 128);
-    talk_attention_mma_kernel<DK, NV, NR, ALLG><<<grid, threads, smem, st>>>(a, tile_rows, rq, n_splits, partial);
+    const int warps = a.kv_heads * ta_nvb(a.vdim, a.value_heads);
+    const dim3 grid(ALLG ? 1 : warps, n_tiles, n_splits);
+    const int threads = ALLG ? (warps > 4 ? 256 : 128) : (NR == 8 ? 256 : 128);
+    talk_attention_mma_kernel<DK, NV, NR, ALLG, WIDE><<<grid, threads, smem, st>>>(a, tile_rows, rq, n_splits, partial, ta_vs(a.vdim, a.value_heads));
     return 0;
 }
 
-template <int DK, int NV>
+template <int DK, int NV, bool WIDE>
 static int launch_talk(const DlWindowAttnArgs& a, const int* tile_rows, int n_tiles, int rq, int n_splits, float* partial, cudaStream_t st) {
     const int rows = ta_rows_of(rq, a.heads / a.kv_heads);
     // many small tiles (batched decoding): one CTA per tile stages every head's keys and values once; few (one stream): a CTA
     // per key/value head, so that more SMs share the pages
-    if (rows == 16 && n_tiles * a.kv_heads * n_splits >= 512 && ta_allg(a.kv_heads, a.dim, a.vdim, a.key_heads)) return launch_talk_nr<DK, NV, 1, true>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
-    if (rows == 16) return launch_talk_nr<DK, NV, 1, false>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
-    if (rows == 64) return launch_talk_nr<DK, NV, 4, false>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
-    return launch_talk_nr<DK, NV, 8, false>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
+    if (rows == 16 && n_tiles * a.kv_heads * n_splits >= 512 && ta_allg(a.kv_heads, a.dim, a.vdim, a.key_heads, a.value_heads)) return launch_talk_nr<DK, NV, 1, true, WIDE>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
+    if (rows == 16) return launch_talk_nr<DK, NV, 1, false, WIDE>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
+    if (rows == 64) return launch_talk_nr<DK, NV, 4, false, WIDE>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
+    return launch_talk_nr<DK, NV, 8, false, WIDE>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
 }
 
 // tile_rows[n_tiles][rq] (device; -1 where a tile has fewer rows): up to rq consecutive rows of one sequence per tile,
@@ -361,25 +442,29 @@ extern "C" int dl_talk_attention_tc(const DlWindowAttnArgs* args, const int* til
                                     float* partial, void* stream) {
     const DlWindowAttnArgs& a = *args;
     if (a.page_size != TA_PAGE || a.softcap != 0.f || a.rope_dims != 0 || a.window < 0 || a.chunk < 0 ||
-        dl_talk_attention_tc_supported(a.heads, a.kv_heads, a.dim, a.vdim, a.key_heads, a.ctype) != 0 || rq < 1 ||
+        dl_talk_attention_tc_supported(a.heads, a.kv_heads, a.dim, a.vdim, a.key_heads, a.value_heads, a.ctype) != 0 || rq < 1 ||
         rq * (a.heads / a.kv_heads) > TA_MAX_ROWS || (a.ldq & 3) || (a.ldo & 1) || ((uintptr_t)a.q & 15) || ((uintptr_t)a.out & 7)) {
-        dl_set_error("dl_talk_attention_tc: sizes not supported (heads %d / %d, dim %d, vdim %d, key heads %d, rq %d)", a.heads, a.kv_heads, a.dim, a.vdim, a.key_heads, rq);
+        dl_set_error("dl_talk_attention_tc: sizes not supported (heads %d / %d, dim %d, vdim %d, key heads %d, value heads %d, rq %d)", a.heads, a.kv_heads, a.dim, a.vdim, a.key_heads, a.value_heads, rq);
         return -1;
     }
     if (n_tiles < 1) return 0;
     if (n_tiles > 65535) { dl_set_error("dl_talk_attention_tc: %d tiles in one launch", n_tiles); return -1; }
     if (n_splits < 1 || n_splits > TA_MAX_SPLITS || (n_splits > 1 && partial == nullptr)) { dl_set_error("dl_talk_attention_tc: n_splits %d without scratch", n_splits); return -1; }
     cudaStream_t st = (cudaStream_t)stream;
-    const int dk = ta_dk(a.dim), nv = ta_nv(a.vdim);
+    const int dk = ta_dk(a.dim), nv = ta_nv(a.vdim, a.value_heads);
     int rc = -1;
-#define TA_CASE(DK_, NV_) if (dk == DK_ && nv == NV_) rc = launch_talk<DK_, NV_>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
-    TA_CASE(2, 8) TA_CASE(2, 12) TA_CASE(2, 16)
-    TA_CASE(4, 8) TA_CASE(4, 12) TA_CASE(4, 16)
-    TA_CASE(8, 8) TA_CASE(8, 12) TA_CASE(8, 16)
+#define TA_CASE(DK_, NV_, WIDE_) if (dk == DK_ && nv == NV_ && (a.value_heads > 1) == WIDE_) rc = launch_talk<DK_, NV_, WIDE_>(a, tile_rows, n_tiles, rq, n_splits, partial, st);
+    TA_CASE(2, 8, false) TA_CASE(2, 12, false) TA_CASE(2, 16, false)
+    TA_CASE(4, 8, false) TA_CASE(4, 12, false) TA_CASE(4, 16, false)
+    TA_CASE(8, 8, false) TA_CASE(8, 12, false) TA_CASE(8, 16, false)
+    TA_CASE(2, 16, true) TA_CASE(2, 32, true)
+    TA_CASE(4, 16, true) TA_CASE(4, 32, true)
+    TA_CASE(8, 16, true) TA_CASE(8, 32, true)
 #undef TA_CASE
     if (rc != 0) return rc;
     if (n_splits > 1)
-        talk_merge_kernel<<<dim3(n_tiles, a.kv_heads, rq), 128, 0, st>>>(a, tile_rows, rq, n_splits, partial, 8 * nv, ta_rows_of(rq, a.heads / a.kv_heads));
+        talk_merge_kernel<<<dim3(n_tiles, a.kv_heads * ta_nvb(a.vdim, a.value_heads), rq), 128, 0, st>>>(
+            a, tile_rows, rq, n_splits, partial, 8 * nv, ta_rows_of(rq, a.heads / a.kv_heads), ta_vs(a.vdim, a.value_heads));
     LAYER_CHECK_LAUNCH("dl_talk_attention_tc");
     return 0;
 }

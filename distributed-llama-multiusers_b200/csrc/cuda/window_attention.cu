@@ -79,7 +79,8 @@ __global__ void __launch_bounds__(256) window_kv_write_kernel(DlWindowKvArgs a) 
 // threads at once; then a warp per (query or key) head: optional rotary on the first rope_dims dimensions (pairs
 // (i, i + rope_dims / 2) with rope_half, else (2i, 2i + 1); cos and sin of the row's angles are formed once, in f64),
 // THEN, with qk_norm, the head is divided by sqrt(mean(head^2) + eps): the queries in place, the keys on their way into
-// the cache.  The values are copied behind the keys.  With `talk` the head mix of the scores is folded into the queries:
+// the cache.  q_norm / k_norm (weights over all heads' columns): in front of the rotary, the row's whole query / key projection is
+// divided by its root mean square and multiplied by the weight.  The values are copied behind the keys.  With `talk` the head mix of the scores is folded into the queries:
 // q_mixed[h][c * dim + i] = sum over the query heads g of key/value head c of talk[h][g] q_g[i].
 // Dynamic shared memory: 2 (kv_heads + q_heads) dim + rope_dims + q_heads^2 floats.
 template <typename CT>
@@ -113,6 +114,20 @@ __global__ void __launch_bounds__(256) attn_kv_write_kernel(DlWindowKvArgs a) {
         st_f(line0 + g * head_step + a.dim + i, a.v[(size_t)m * a.ldv + t]);
     }
     __syncthreads();
+    if (a.q_norm != nullptr || a.k_norm != nullptr) {
+        __shared__ float red[32];
+        for (int part = 0; part < 2; ++part) {                // the keys, then the queries
+            const float* w = part ? a.q_norm : a.k_norm;
+            float* r = raw_s + (part ? (size_t)a.kv_heads * D : 0);
+            const int cnt = (part ? nq : nk) * D;
+            if (w == nullptr || cnt == 0) continue;
+            float ss = 0.f;
+            for (int t = threadIdx.x; t < cnt; t += blockDim.x) ss = fmaf(r[t], r[t], ss);
+            const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)cnt + a.eps);
+            for (int t = threadIdx.x; t < cnt; t += blockDim.x) r[t] = r[t] * inv * w[t];
+        }
+        __syncthreads();
+    }
     for (int h = (a.kv_heads - nk) + warp; h < a.kv_heads + nq; h += nw) {
         const bool is_k = h < a.kv_heads;
         const float* src = raw_s + (size_t)h * D;
@@ -179,7 +194,7 @@ extern "C" int dl_window_kv_write(const DlWindowKvArgs* args, int M, void* strea
         LAYER_CHECK_LAUNCH("dl_window_kv_write");
         return 0;
     }
-    if (a.qk_norm) { dl_set_error("dl_window_kv_write: qk_norm belongs to the separate-value form"); return -1; }
+    if (a.qk_norm || a.q_norm || a.k_norm) { dl_set_error("dl_window_kv_write: qk_norm, q_norm and k_norm belong to the separate-value form"); return -1; }
     if (a.rope_dims > a.dim || (a.rope_dims & 1) || a.rope_dims > 2 * WK_MAX_PAIRS || a.page_size != WA_PAGE) { dl_set_error("dl_window_kv_write: bad rotary or page size"); return -1; }
     cudaStream_t st = (cudaStream_t)stream;
     if (a.ctype == DL_T_BF16) window_kv_write_kernel<__nv_bfloat16><<<M, 256, 0, st>>>(a);
@@ -198,6 +213,8 @@ __global__ void window_attention_kernel(DlWindowAttnArgs a) {
     const int rep = a.heads / a.kv_heads, D = a.dim, RD = a.rope_dims, DV = a.vdim > 0 ? a.vdim : D;
     const int KH = a.key_heads > 1 ? a.key_heads : 1, QD = KH * D;      // head-mixed scores: a query meets the keys of all KH key/value heads side by side
     const int LD = D + (a.vdim > 0 ? a.vdim : RD), VT = LD - D, LP = QD + VT + 1;
+    const bool wide = a.value_heads > 1;               // this CTA: the group's weights against the values of key/value head vg
+    const int vg = wide ? blockIdx.z : g;
     const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* q_s = sm;                                   // [rep][QD]
     float* tile = q_s + (size_t)rep * QD;              // [WA_PAGE][QD keys | VT: the rest of head g's line | 1]
@@ -214,11 +231,12 @@ __global__ void window_attention_kernel(DlWindowAttnArgs a) {
         __syncthreads();
         const int page = a.block_table[(size_t)slot * a.max_pages + pg];
         const CT* src = (const CT*)a.cache + ((size_t)page * a.kv_heads + g) * WA_PAGE * LD;
+        const CT* src_v = (const CT*)a.cache + ((size_t)page * a.kv_heads + vg) * WA_PAGE * LD;
         const int j_lo = max(0, first - pg * WA_PAGE), j_hi = min(WA_PAGE, pos + 1 - pg * WA_PAGE);   // visible lines [j_lo, j_hi)
         for (int i = threadIdx.x; i < WA_PAGE * LD; i += blockDim.x) {
             const int j = i / LD, d = i - j * LD;
             if (KH > 1 && d < D) continue;             // the keys come from every key/value head, below
-            tile[j * LP + (d < D ? d : QD + d - D)] = (j >= j_lo && j < j_hi) ? ld_f(src + i) : 0.f;
+            tile[j * LP + (d < D ? d : QD + d - D)] = (j >= j_lo && j < j_hi) ? ld_f((d < D ? src : src_v) + i) : 0.f;
         }
         if (KH > 1) {
             for (int i = threadIdx.x; i < KH * WA_PAGE * D; i += blockDim.x) {
@@ -260,13 +278,15 @@ __global__ void window_attention_kernel(DlWindowAttnArgs a) {
         const int h = t / DV;
         float l = ml[2 * h + 1];
         if (a.sink) l += expf(a.sink[g * rep + h] - ml[2 * h]);
-        a.out[(size_t)m * a.ldo + (size_t)g * rep * DV + t] = acc[t] / l;
+        if (wide) a.out[(size_t)m * a.ldo + ((size_t)(g * rep + h) * a.kv_heads + vg) * DV + (t - h * DV)] = acc[t] / l;
+        else a.out[(size_t)m * a.ldo + (size_t)g * rep * DV + t] = acc[t] / l;
     }
 }
 
 static int window_args_ok(const DlWindowAttnArgs& a, const char* who) {
     if (a.heads < 1 || a.kv_heads < 1 || a.heads % a.kv_heads || a.dim < 1 || a.rope_dims > a.dim || a.window < 0 || a.page_size != WA_PAGE ||
-        a.vdim < 0 || a.chunk < 0 || (a.vdim > 0 && a.rope_dims != 0) || (a.key_heads > 1 && (a.key_heads != a.kv_heads || a.vdim < 1))) {
+        a.vdim < 0 || a.chunk < 0 || (a.vdim > 0 && a.rope_dims != 0) || (a.key_heads > 1 && (a.key_heads != a.kv_heads || a.vdim < 1)) ||
+        (a.value_heads > 1 && (a.value_heads != a.kv_heads || a.vdim < 1 || a.key_heads > 1))) {
         dl_set_error("%s: bad shape (heads %d / %d, dim %d, rotary %d, window %d, page %d)", who, a.heads, a.kv_heads, a.dim, a.rope_dims, a.window, a.page_size);
         return -1;
     }
@@ -281,7 +301,7 @@ extern "C" int dl_window_attention(const DlWindowAttnArgs* args, int M, void* st
     const size_t smem = ((size_t)rep * (QD + DV) + (size_t)WA_PAGE * (QD + LD - a.dim + 1) + (size_t)nw * WA_PAGE + 2 * (size_t)rep) * sizeof(float);
     if (smem > 227 * 1024) { dl_set_error("dl_window_attention: %d heads per group x dim %d need %zu bytes of shared memory", rep, a.dim, smem); return -1; }
     cudaStream_t st = (cudaStream_t)stream;
-    dim3 grid(M, a.kv_heads);
+    dim3 grid(M, a.kv_heads, a.value_heads > 1 ? a.value_heads : 1);
     cudaError_t e;
     if (a.ctype == DL_T_BF16) {
         e = cudaFuncSetAttribute(window_attention_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);

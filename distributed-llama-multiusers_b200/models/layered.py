@@ -8,11 +8,14 @@ meets the residual stream is the architecture's ``residual`` style (``RESIDUAL_S
                  which is how Venadra's pre-norm layers run (one stream, m = 1)
     "post":      x <- x + m * norm(sub(x))                               the sublayer reads the stream itself; the only
                  norm sits on its output (Darusun)
+    "parallel":  x <- x + mixer(norm1(x)) + ff(norm2(x))                 both of the same x; norm weights plain (Vopedra)
 
 What a design fixes without saying it in config.json (how its attention masks, whether its experts are gated, ...) is
 its entry of ``DESIGNS``; everything config.json gives is read from there.  A configuration with ``canon: {taps}`` puts a
 short causal convolution in front of every mixer: h <- h + conv(h) on the normed input, the last taps - 1 inputs kept per
-sequence slot and layer.
+sequence slot and layer.  ``loop: {start, stop, times}`` runs that slice of the list `times` times in a row on the same
+weights, every pass with caches and states of its own (parallel residual style; the embedding output and a vector
+``loop.step[pass]`` are added to the stream ahead of a pass).
 
 The mixers and feed-forwards are looked up by name (``MIXERS`` / ``FEED_FORWARDS`` below), so another design composes
 the same mechanisms with its own sizes and order; ``ARCHITECTURES`` in models/registry.py maps an architecture name to
@@ -28,9 +31,13 @@ this engine.  Mixers here:
   rotate-half layout in front of the unit norm; scores mixed across heads by a matrix `talk` before the softmax (folded
   into the queries, see WindowAttentionMixer); a layer that reads another layer's keys and values (``kv_from``);
 * ``lightning`` -- linear attention with a fixed decay per head and an f32 state [dim][vdim] per head and slot, SiLU on
-  q, k and v, an RMS norm over the concatenated heads and a sigmoid output gate.
+  q, k and v, an RMS norm over the concatenated heads and a sigmoid output gate;
+* ``mlstm`` -- a matrix memory with exponential input and forget gates per head, stabilised by a running maximum;
+* ``hgrn2`` -- linear attention whose forget gate per head and channel also decides what is written;
+* ``mamba1`` -- a selective state-space recurrence with a state per channel behind a short causal convolution;
+* ``parallel`` -- two mixers side by side on the same input, their outputs normed and averaged.
 
-Feed-forwards: ``dense`` (squared ReLU, PolyNorm, or xIELU) and ``moe`` (sigmoid-scored, group-limited routing over small
+Feed-forwards: ``dense`` (squared ReLU, PolyNorm, xIELU, or a GELU-gated unit) and ``moe`` (sigmoid-scored, group-limited routing over small
 squared-ReLU experts; or softmax-scored, renormalised routing over gated experts, with an optional router bias and a
 shared expert behind a sigmoid gate per token).  A layer with ``weights_of: j`` runs
 layer j's weights on a cache or state of its own (a looped layer).
@@ -69,6 +76,8 @@ class LayerSpec:
     mixer: dict
     mlp: Optional[dict]
     weights_of: Optional[int] = None       # run that layer's weights (norms, mixer, feed-forward) on a cache / state of its own
+    tensors: Optional[int] = None          # index in the tensor names l<i>.*, where it is not the place in the list (behind a loop)
+    opens: Optional[int] = None            # first layer of this pass of the loop
 
 
 # What a design fixes outside its config.json, by architecture name.  residual: how sublayers meet the residual stream.
@@ -78,7 +87,9 @@ class LayerSpec:
 # e<n>.gate; True: a sigma(1.702 a) (1 + b) with expert.limit, "silu": silu(a) b), bias (tensor `router.b`), shared (entry
 # `shared` of the mlp: one more gated expert for every token behind sigmoid(`shared.sg` . h)).  attention also: rot
 # ("interleaved" | "half": the pair layout of the rotary, which own values otherwise exclude), talk (tensor `talk`
-# [heads][heads] mixes the scores of the heads before the softmax).  latent: rot (the same), sink, gate ("full": one
+# [heads][heads] mixes the heads: "scores" before the softmax | "weights" after it), proj_norm (tensors q.norm, k.norm: an RMS
+# norm over the whole query / key projection ahead of the rotary).  dense_act also: "gelu_glu" (tensors gate, up).
+# embed_norm (tensor embed.norm: the embedding is normed).  parallel: the mixers of its two branches.  latent: rot (the same), sink, gate ("full": one
 # gate per output column | "head": one per head).  norm_weights "scalar": every norm over the width has one number.
 DESIGNS = {
     "Ribivik": {"residual": "sandwich"},
@@ -88,10 +99,14 @@ DESIGNS = {
                 "dense_act": "polynorm",
                 "moe": {"score": "softmax", "renorm": True, "gated": True}},
     "Darusun": {"residual": "post", "norm_weights": "scalar",
-                "attention": {"values": "own", "qk_norm": True, "rot": "half", "talk": True},
+                "attention": {"values": "own", "qk_norm": True, "rot": "half", "talk": "scores"},
                 "latent": {"rot": "interleaved", "sink": True, "gate": "head"},
                 "dense_act": "xielu",
                 "moe": {"score": "softmax", "renorm": True, "gated": "silu", "bias": True, "shared": True}},
+    "Vopedra": {"residual": "parallel", "embed_norm": True,
+                "attention": {"values": "own", "rot": "half", "talk": "weights", "proj_norm": True},
+                "parallel": {"left": "attention", "right": "hgrn2"},
+                "dense_act": "gelu_glu"},
 }
 RESIDUAL_STYLES = {name: d["residual"] for name, d in DESIGNS.items()}
 
@@ -112,6 +127,7 @@ class LayerListConfig:
     hyper_weights: bool = False            # the layers bring hc<q>.in / .out / .mix tensors (else the plain sum)
     canon_taps: int = 0                    # > 0: h <- h + conv(h) over the last `taps` normed inputs, in front of every mixer
     traits: dict = field(default_factory=dict)      # the design's entry of DESIGNS
+    loop_times: int = 0                    # passes of the loop (0: none); `layers` holds the runs of all passes
 
     # the serving code reads these names from every engine's header
     @property
@@ -130,13 +146,27 @@ class LayerListConfig:
             if l.weights_of is not None and (not 0 <= l.weights_of < len(layers) or layers[l.weights_of].weights_of is not None):
                 raise ValueError(f"layer {i}: weights_of {l.weights_of} is not a layer with weights of its own")
         arch = c["architecture"]
+        loop_times = 0
+        if c.get("loop"):
+            start, stop, loop_times = (int(c["loop"][k]) for k in ("start", "stop", "times"))
+            if not 0 <= start < stop <= len(layers) or loop_times < 1:
+                raise ValueError(f"loop {start} .. {stop} x {loop_times} does not fit {len(layers)} layers")
+            if any(l.weights_of is not None or l.mixer.get("kv_from") is not None for l in layers) or RESIDUAL_STYLES.get(arch) != "parallel":
+                raise ValueError("a loop is known for the parallel residual style and layers that name no other layer")
+            runs = []
+            for i, l in enumerate(layers[:stop] + layers[start:stop] * (loop_times - 1) + layers[stop:]):
+                t = (i - start) // (stop - start) if start <= i < start + (stop - start) * loop_times else None      # pass of the loop
+                src = start + (i - start) % (stop - start) if t is not None else i if i < start else i - (stop - start) * (loop_times - 1)
+                runs.append(LayerSpec(l.type, l.mixer, l.mlp, src if t else None, src, t if t is not None and src == start else None))
+            layers = runs
         return LayerListConfig(architecture=arch, width=int(c["width"]), vocab=int(c["vocab"]),
                                norm_eps=float(c["norm"]["eps"]), logit_softcap=float(c.get("logit_softcap") or 0.0),
                                layers=layers, residual=RESIDUAL_STYLES.get(arch, "sandwich"),
                                embed_scale=float((c.get("embedding") or {}).get("scale", 1.0)),
                                residual_mult=float(c.get("residual_mult", 1.0)),
                                streams=int(c.get("streams") or 1), hyper_weights=bool(c.get("streams")),
-                               canon_taps=int((c.get("canon") or {}).get("taps") or 0), traits=DESIGNS.get(arch, {}))
+                               canon_taps=int((c.get("canon") or {}).get("taps") or 0), traits=DESIGNS.get(arch, {}),
+                               loop_times=loop_times)
 
     @staticmethod
     def load(model_dir: str) -> "LayerListConfig":
@@ -194,6 +224,7 @@ class DenseWeight:
 TC_MIN_ROWS = int(os.environ.get("DLLAMA_LAYERS_TC_MIN_ROWS", "32"))
 CHUNKED_SCAN_MIN_ROWS = 256  # a batch holding this many rows of one sequence runs the recurrence chunk-parallel
 LIGHTNING_CHUNKED_MIN_ROWS = 128     # the same for linear attention (chunks of 64 rows)
+GATED_CHUNKED_MIN_ROWS = 128         # and for linear attention with data-dependent gates
 TC_HEADS_MIN_ROWS = 256      # per-head products (one small GEMM per head) take the tensor-core path from this many rows
 GRAPH_MAX_ROWS = 64          # batches up to this many rows are replayed from CUDA graphs
 WINDOW_MAX_SPLITS = 32       # most CTAs that share one tile's pages in the windowed-attention kernel
@@ -338,13 +369,22 @@ class DenseFeedForward:
     """Tensors <prefix>up, down:  W_down act(W_up h).  act = relu(.)^2, or (design trait dense_act "polynorm", tensor
     <prefix>act = [c1, c2, c3, c0]) PolyNorm: c0 + sum_p cp z^p / rms(z^p), p = 1..3, with the powers taken element-wise and
     the root mean square (eps inside) over a row; or ("xielu", tensor <prefix>act = [p, q]) xIELU: softplus(p) z^2 + z / 2 for
-    z > 0, (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 for z <= 0, in the up-projection's epilogue."""
+    z > 0, (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 for z <= 0, in the up-projection's epilogue; or ("gelu_glu", tensor
+    <prefix>gate) the gated unit gelu(W_gate h) * (W_up h), gelu in its tanh form, from ONE product: gate and up rows interleaved
+    (gate_0, up_0, gate_1, ...), so the epilogue sees a value's two products side by side."""
 
     def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str):
         self.eng = eng
         self.ff = int(m["ff"])
-        self.w_up, self.w_down = eng.dense_weight(eng.weight(prefix + "up")), eng.dense_weight(eng.weight(prefix + "down"))
         act = eng.cfg.traits.get("dense_act")
+        w_up = eng.weight(prefix + "up")
+        self.glu = act == "gelu_glu"
+        if self.glu:
+            w_gate = eng.weight(prefix + "gate")
+            if tuple(w_gate.shape) != (self.ff, eng.cfg.width) or w_up.shape != w_gate.shape:
+                raise ValueError(f"layer {index}: gate / up have shapes {tuple(w_gate.shape)} / {tuple(w_up.shape)}")
+            w_up = torch.stack([w_gate, w_up], dim=1).reshape(2 * self.ff, eng.cfg.width).contiguous()
+        self.w_up, self.w_down = eng.dense_weight(w_up), eng.dense_weight(eng.weight(prefix + "down"))
         self.poly = eng.vector(prefix + "act") if act == "polynorm" else None
         if self.poly is not None and tuple(self.poly.shape) != (4,):
             raise ValueError(f"layer {index}: {prefix}act has shape {tuple(self.poly.shape)}")
@@ -365,7 +405,9 @@ class DenseFeedForward:
     def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
         e, L = self.eng, self.eng.L
         up = e.buf("up", self.ff)
-        if self.poly is not None:
+        if self.glu:
+            e.mm(self.w_up, h, up, M, epi=L.DENSE_GLU_GELU, src="h")
+        elif self.poly is not None:
             e.mm(self.w_up, h, up, M, src="h")
             L.poly_norm(up, up, M, self.ff, self.poly, e.cfg.norm_eps)
         elif self.xielu is not None:
@@ -392,7 +434,11 @@ class WindowAttentionMixer:
       talk: <prefix>talk [heads][heads] mixes the heads' scaled scores before mask and softmax, score'_h = sum_g talk[h][g]
              score_g.  The mix is linear in the queries, so it is folded into them: with c(g) the key/value head of query
              head g,  score'_h = sum_c ( sum_{g: c(g) = c} talk[h][g] q_g ) . k_c  -- head h gets ONE query of kv_heads * dim
-             numbers that meets the keys of all key/value heads side by side; the values stay those of its own group.
+             numbers that meets the keys of all key/value heads side by side; the values stay those of its own group.  That is
+             talk "scores"; talk "weights" mixes the softmax weights instead, weight'_h = sum_g talk[h][g] weight_g, which is linear in
+             the outputs: every head's weights meet the values of all key/value heads side by side (kv_heads * vdim numbers
+             per head) and the head's outputs are summed with talk afterwards;
+      proj_norm: an RMS norm with weights <prefix>q.norm / k.norm over all heads' columns of q / k at once, BEFORE the rotary.
     A mixer entry with `kv_from: j` has no k / v tensors and no cache: it reads layer j's keys (as cached: rotated and
     normalised) and values with queries, mask and the rest of its own."""
 
@@ -441,8 +487,18 @@ class WindowAttentionMixer:
             self.talk = eng.vector(prefix + "talk") if tr.get("talk") else None
             if self.talk is not None and tuple(self.talk.shape) != (H, H):
                 raise ValueError(f"layer {index}: talk has shape {tuple(self.talk.shape)}")
+            self.q_norm = self.k_norm = None
+            if tr.get("proj_norm"):
+                self.q_norm = eng.vector(prefix + "q.norm")
+                self.k_norm = eng.vector(prefix + "k.norm") if self.kv_from is None else None
+                if not self.own_v or self.q_norm.numel() != H * d or (self.k_norm is not None and self.k_norm.numel() != G * d):
+                    raise ValueError(f"layer {index}: q.norm / k.norm do not fit {H} / {G} heads of {d}")
         else:
             self.w_qk, self.w_o, self.w_g, self.sink, self.talk = share.w_qk, share.w_o, share.w_g, share.sink, share.talk
+            self.q_norm, self.k_norm = share.q_norm, share.k_norm
+        # heads mixed before the softmax: queries against all key heads; after it: weights against all value heads
+        self.key_heads = G if self.talk is not None and tr.get("talk") == "scores" else 0
+        self.value_heads = G if self.talk is not None and tr.get("talk") == "weights" else 0
         self.owns_weights = share is None
         self.line = d + (dv if self.own_v else self.rope_dims)
         # a kv_from layer is bound to its owner's cache once all layers exist
@@ -454,19 +510,21 @@ class WindowAttentionMixer:
         attn_tc = eng.round_x and os.environ.get("DLLAMA_LAYERS_ATTN_TC", "1") != "0"
         if attn_tc and dv == d and self.talk is None and L.window_tc_supported(H, G, d, 0 if self.own_v else self.rope_dims, eng.wdtype):
             self.tc_rq = L.window_tc_rows(H, G)
-        elif attn_tc and self.own_v and self.softcap == 0.0 and L.talk_tc_supported(H, G, d, dv, G if self.talk is not None else 0, eng.wdtype):
+        elif attn_tc and self.own_v and self.softcap == 0.0 and L.talk_tc_supported(H, G, d, dv, self.key_heads, eng.wdtype, self.value_heads):
             # values wider or narrower than the keys, head-mixed scores: the tile kernel of talk_attention.cu
             # tiles of 128 stacked (row, head) pairs for long portions, of 16 for decoding, 64 where those do not fit
-            kh = G if self.talk is not None else 0
-            self.tc_rq, self.tc_rq_small, self.tc_talk = L.talk_tc_rows(H, G, d, dv, kh, 1 << 30), L.talk_tc_rows(H, G, d, dv, kh, 1), True
-            self.partial_floats = L.talk_tc_partial_floats(WINDOW_CTAS_PER_SM * eng.n_sms, 1, 1, dv, self.tc_rq, H)
+            kh, vh = self.key_heads, self.value_heads
+            self.tc_rq, self.tc_rq_small, self.tc_talk = L.talk_tc_rows(H, G, d, dv, kh, 1 << 30, vh), L.talk_tc_rows(H, G, d, dv, kh, 1, vh), True
+            self.partial_floats = L.talk_tc_partial_floats(WINDOW_CTAS_PER_SM * eng.n_sms, 1, 1, dv, self.tc_rq, H, vh)
 
     def scratch(self) -> Dict[str, int]:
         n = {"qk": (self.H + self.G) * self.dim + (self.G * self.vdim if self.own_v else 0), "o": self.H * self.vdim}
         if self.w_g is not None:
             n["og"] = self.H * self.vdim
-        if self.talk is not None:
+        if self.key_heads:
             n["qmix"] = self.H * self.G * self.dim
+        if self.value_heads:
+            n["owide"] = self.H * self.G * self.vdim
         return n
 
     def bind(self, mixers: list):
@@ -493,18 +551,22 @@ class WindowAttentionMixer:
         # one launch: the keys (and values) go into the cache and the queries are rotated / normalised in place (and mixed)
         q_in = qk
         if self.own_v:
-            if self.talk is not None:
+            if self.key_heads:
                 q_in = e.buf("qmix", H * G * d)
             L.window_kv_write(qk[:, H * d:] if own_kv else None, M, G, d, rd, self.freqs, self.rope_mag, e.pos, e.slot, e.block_table,
                               self.cache, q=qk, q_heads=H, v=qk[:, nqk:] if own_kv else None, vdim=dv, qk_norm=self.qk_norm,
-                              eps=e.cfg.norm_eps, rope_half=self.own_rot == "half", talk=self.talk, q_mixed=q_in if self.talk is not None else None)
+                              eps=e.cfg.norm_eps, rope_half=self.own_rot == "half", talk=self.talk if self.key_heads else None,
+                              q_mixed=q_in if self.key_heads else None, q_norm=self.q_norm, k_norm=self.k_norm)
             rd = 0                            # the attention kernels meet keys that are complete: nothing of a line is shared with its value
         else:
             L.window_kv_write(qk[:, H * d:], M, G, d, rd, self.freqs, self.rope_mag, e.pos, e.slot, e.block_table, self.cache,
                               q=qk, q_heads=H)
         opts = dict(vdim=dv if self.own_v else 0, chunk=self.chunk, sink=self.sink)
-        if self.talk is not None:
+        if self.key_heads:
             opts["key_heads"] = G
+        if self.value_heads:
+            opts["value_heads"] = G
+            o = e.buf("owide", H * G * dv)
         if self.tc_rq:
             rq = self.tc_rq_small if self.tc_rq_small and e.longest <= self.tc_rq_small else self.tc_rq
             tile_rows, n_tiles = e.window_tiles(rq)
@@ -519,18 +581,23 @@ class WindowAttentionMixer:
             partial = e.window_partial(d, self.partial_floats) if n_splits > 1 else None
             if self.tc_talk:
                 L.talk_attention_tc(q_in, o, H, G, d, dv, self.scale, self.window, e.pos, e.slot, e.block_table, self.cache, tile_rows,
-                                    n_tiles, rq, n_splits, partial, chunk=self.chunk, sink=self.sink, key_heads=opts.get("key_heads", 0))
+                                    n_tiles, rq, n_splits, partial, chunk=self.chunk, sink=self.sink, key_heads=opts.get("key_heads", 0),
+                                    value_heads=opts.get("value_heads", 0))
             else:
                 L.window_attention_tc(qk, o, H, G, d, rd, self.scale, self.softcap, self.window, e.pos, e.slot, e.block_table,
                                       self.cache, tile_rows, n_tiles, rq, n_splits, partial, **opts)
         else:
             L.window_attention(q_in, o, M, H, G, d, rd, self.scale, self.softcap, self.window, e.pos, e.slot, e.block_table,
                                self.cache, **opts)
+        image = None
+        if self.value_heads:              # the heads' outputs mixed, straight into the output projection's operand image where it takes one
+            image, wide, o = e.image("tmp", M) if self.w_g is None else None, o, e.buf("o", H * dv)
+            L.talk_mix(wide, self.talk, M, H, G, dv, o, image=image)
         if self.w_g is not None:
             og = e.buf("og", H * dv)
             e.mm(self.w_g, h, og, M, epi=L.DENSE_SIGMOID_MUL, aux=o, src="h")
             o = og
-        e.mm(self.w_o, o, y, M)
+        e.mm(self.w_o, o, y, M, ready=image is not None)
 
 
 class LightningMixer:
@@ -582,6 +649,209 @@ class LightningMixer:
         L.rms_norm(ys, yn, M, H * dv, e.cfg.norm_eps, w=self.norm)
         e.mm(self.w_g, h, og, M, epi=L.DENSE_SIGMOID_MUL, aux=yn, src="h")
         e.mm(self.w_o, og, y, M)
+
+
+class MLstmMixer:
+    """A matrix memory with exponential gates (mLSTM).  Tensors <prefix>q, k, v, i, i.b, f, f.b, g, norm, o.  Sizes: heads, dim,
+    vdim, gate_cap.  Per head, with q scaled by dim^(-1/2) and c = gate_cap:  a = c tanh((W_i h + b_i) / c),
+    b = log sigmoid(c tanh((W_f h + b_f) / c)); a running maximum u <- max(b + u, a) that starts at 0 keeps the exponentials <= 1:
+        S <- e^(b + u_old - u) S + e^(a - u) k v^T,  n likewise with k alone,  o = S^T q / (max(|n . q|, e^-u) + 1e-6)
+    (S, n and u: f32, one per slot and head); every head's o is divided by its root mean square, times <prefix>norm [heads * vdim]
+    and sigmoid(W_g h), then W_o.  ONE product gives q, k, v, the output gate and both gates' inputs."""
+
+    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["MLstmMixer"] = None):
+        self.eng, self.index = eng, index
+        self.H, self.dim, self.vdim, self.cap = int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"])
+        H, d, dv = self.H, self.dim, self.vdim
+        if not eng.L.gated_supported(d, dv):
+            raise ValueError(f"layer {index}: the matrix memory takes head sizes up to 512 ({d})")
+        self.owns_weights = share is None
+        if share is None:
+            W, V, D = eng.weight, eng.vector, eng.dense_weight
+            parts = [W(prefix + n) for n in ("q", "k", "v", "g", "i", "f")]
+            rows = (H * d, H * d, H * dv, H * dv, H, H)
+            if any(tuple(t.shape) != (r, eng.cfg.width) for t, r in zip(parts, rows)):
+                raise ValueError(f"layer {index}: q, k, v, g, i, f have shapes {[tuple(t.shape) for t in parts]}")
+            self.w_in, self.w_o = D(torch.cat(parts, 0).contiguous()), D(W(prefix + "o"))
+            self.bi, self.bf, self.norm = V(prefix + "i.b"), V(prefix + "f.b"), V(prefix + "norm")
+            if self.bi.numel() != H or self.bf.numel() != H or self.norm.numel() != H * dv:
+                raise ValueError(f"layer {index}: i.b, f.b or norm do not fit {H} heads of {dv}")
+        else:
+            self.w_in, self.w_o, self.bi, self.bf, self.norm = share.w_in, share.w_o, share.bi, share.bf, share.norm
+        f32 = dict(dtype=torch.float32, device=eng.device)
+        self.state, self.n_state = torch.zeros(eng.n_slots, H, d, dv, **f32), torch.zeros(eng.n_slots, H, d, **f32)
+        self.u_state = torch.zeros(eng.n_slots, H, **f32)
+        self.chunked = eng.L.gated_chunked_supported(d, dv, False)
+
+    def scratch(self) -> Dict[str, int]:
+        return {"mx": self.w_in.N, "ys": self.H * self.vdim, "yn": self.H * self.vdim, "gates": 4 * self.H}
+
+    def bind(self, mixers: list):
+        pass
+
+    def weight_bytes(self) -> int:
+        return self.w_in.nbytes() + self.w_o.nbytes() if self.owns_weights else 0
+
+    def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
+        e, L = self.eng, self.eng.L
+        H, d, dv = self.H, self.dim, self.vdim
+        mx, ys, yn = e.buf("mx", self.w_in.N), e.buf("ys", H * dv), e.buf("yn", H * dv)
+        keep, put, floor, den = (e.buf("gates", 4 * H).view(-1)[i * e.max_rows * H:(i + 1) * e.max_rows * H] for i in range(4))     # [rows][heads] each
+        e.mm(self.w_in, h, mx, M, src="h")
+        k0, v0, g0, i0 = H * d, 2 * H * d, H * (2 * d + dv), H * (2 * d + 2 * dv)
+        L.mlstm_gates(e.mamba_batch, e.n_seq, mx[:, i0:], mx[:, i0 + H:], self.bi, self.bf, self.cap, self.u_state, keep, put, floor, H)
+        L.gated_scan(e.mamba_batch, e.n_seq, mx, mx[:, v0:], ys, self.state, H, d, dv, q_scale=d ** -0.5, k=mx[:, k0:], log_keep=keep,
+                     put=put, den=den, n_state=self.n_state, **e.gated_chunking(self))
+        image = e.image("tmp", M)
+        L.head_norm(ys, M, H, dv, e.cfg.norm_eps, self.norm, yn, den=den, floor=floor, gate=mx[:, g0:], image=image)
+        e.mm(self.w_o, yn, y, M, ready=image is not None)
+
+
+class Hgrn2Mixer:
+    """Linear attention whose forget gate decides what is written (HGRN2).  Tensors <prefix>q, f, f.b, lower, v, norm, o.  Sizes:
+    heads, dim, vdim.  q = SiLU(W_q h), v = W_v h, per head and channel g = l + (1 - l) sigmoid(W_f h + b) with l = <prefix>lower
+    [heads * dim];  S <- diag(g) S + (1 - g) v^T (f32, one [dim][vdim] per slot and head),  o = S^T q;  every head's o gets an RMS
+    norm with <prefix>norm [vdim] (shared by the heads), then W_o."""
+
+    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["Hgrn2Mixer"] = None):
+        self.eng, self.index = eng, index
+        self.H, self.dim, self.vdim = int(m["heads"]), int(m["dim"]), int(m["vdim"])
+        H, d, dv = self.H, self.dim, self.vdim
+        if not eng.L.gated_supported(d, dv):
+            raise ValueError(f"layer {index}: gated linear attention takes head sizes up to 512 ({d})")
+        self.owns_weights = share is None
+        if share is None:
+            W, V, D = eng.weight, eng.vector, eng.dense_weight
+            parts = [W(prefix + n) for n in ("q", "f", "v")]
+            if any(tuple(t.shape) != (r, eng.cfg.width) for t, r in zip(parts, (H * d, H * d, H * dv))):
+                raise ValueError(f"layer {index}: q, f, v have shapes {[tuple(t.shape) for t in parts]}")
+            self.w_in, self.w_o = D(torch.cat(parts, 0).contiguous()), D(W(prefix + "o"))
+            self.f_bias, self.lower, self.norm = V(prefix + "f.b"), V(prefix + "lower"), V(prefix + "norm")
+            if self.f_bias.numel() != H * d or self.lower.numel() != H * d or self.norm.numel() != dv:
+                raise ValueError(f"layer {index}: f.b, lower or norm do not fit {H} heads of {d} / {dv}")
+        else:
+            self.w_in, self.w_o, self.f_bias, self.lower, self.norm = share.w_in, share.w_o, share.f_bias, share.lower, share.norm
+        self.state = torch.zeros(eng.n_slots, H, d, dv, dtype=torch.float32, device=eng.device)
+        self.chunked = eng.L.gated_chunked_supported(d, dv, True)
+
+    def scratch(self) -> Dict[str, int]:
+        return {"mx": self.w_in.N, "ys": self.H * self.vdim, "yn": self.H * self.vdim}
+
+    def bind(self, mixers: list):
+        pass
+
+    def weight_bytes(self) -> int:
+        return self.w_in.nbytes() + self.w_o.nbytes() if self.owns_weights else 0
+
+    def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
+        e, L = self.eng, self.eng.L
+        H, d, dv = self.H, self.dim, self.vdim
+        mx, ys, yn = e.buf("mx", self.w_in.N), e.buf("ys", H * dv), e.buf("yn", H * dv)
+        e.mm(self.w_in, h, mx, M, src="h")
+        L.gated_scan(e.mamba_batch, e.n_seq, mx, mx[:, 2 * H * d:], ys, self.state, H, d, dv, q_silu=True, f=mx[:, H * d:],
+                     f_bias=self.f_bias, lower=self.lower, **e.gated_chunking(self))
+        image = e.image("tmp", M)
+        L.head_norm(ys, M, H, dv, e.cfg.norm_eps, self.norm, yn, image=image)
+        e.mm(self.w_o, yn, y, M, ready=image is not None)
+
+
+class Mamba1Mixer:
+    """Selective scan with a state per channel (Mamba).  Tensors <prefix>in, conv, conv.b, x, dt, dt.b, A_log, D, o.  Sizes: inner,
+    state, conv (taps), dt_rank.  [x | z] = W_in h; x <- SiLU of a causal convolution per channel; [dt | B | C] = W_x x;
+    step = softplus(W_dt dt + b);  S[c][n] <- exp(-step_c e^A_log[c][n]) S[c][n] + step_c x_c B_n,  y_c = S[c] . C + D_c x_c;
+    W_o (y * SiLU(z)).  Per slot: S [inner][state] and the convolution's last taps - 1 inputs, f32."""
+
+    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["Mamba1Mixer"] = None):
+        self.eng, self.index = eng, index
+        self.inner, self.N, self.rank, self.taps = int(m["inner"]), int(m["state"]), int(m["dt_rank"]), int(m["conv"])
+        if not eng.L.selective_supported(self.N):
+            raise ValueError(f"layer {index}: the selective scan takes up to 128 state entries per channel ({self.N})")
+        self.owns_weights = share is None
+        if share is None:
+            W, V, D = eng.weight, eng.vector, eng.dense_weight
+            w_in, w_x, w_dt = W(prefix + "in"), W(prefix + "x"), W(prefix + "dt")
+            self.w_conv, self.b_conv = W(prefix + "conv"), W(prefix + "conv.b")
+            if tuple(w_in.shape) != (2 * self.inner, eng.cfg.width) or tuple(w_x.shape) != (self.rank + 2 * self.N, self.inner) or \
+                    tuple(w_dt.shape) != (self.inner, self.rank) or tuple(self.w_conv.shape) != (self.inner, self.taps):
+                raise ValueError(f"layer {index}: in, x, dt, conv have shapes {[tuple(t.shape) for t in (w_in, w_x, w_dt, self.w_conv)]}")
+            self.w_in, self.w_x, self.w_dt, self.w_o = D(w_in), D(w_x), D(w_dt), D(W(prefix + "o"))
+            self.dt_bias, self.A_log, self.D = V(prefix + "dt.b"), V(prefix + "A_log"), V(prefix + "D")
+            if tuple(self.A_log.shape) != (self.inner, self.N):
+                raise ValueError(f"layer {index}: A_log has shape {tuple(self.A_log.shape)}")
+        else:
+            for n in ("w_in", "w_x", "w_dt", "w_o", "w_conv", "b_conv", "dt_bias", "A_log", "D"):
+                setattr(self, n, getattr(share, n))
+        f32 = dict(dtype=torch.float32, device=eng.device)
+        self.state = torch.zeros(eng.n_slots, self.inner, self.N, **f32)
+        self.conv_state = torch.zeros(eng.n_slots, max(1, self.taps - 1), self.inner, **f32)
+
+    def scratch(self) -> Dict[str, int]:
+        return {"zx": 2 * self.inner, "xbc": self.inner, "dbc": self.rank + 2 * self.N, "dtr": self.inner, "ys": self.inner}
+
+    def bind(self, mixers: list):
+        pass
+
+    def weight_bytes(self) -> int:
+        if not self.owns_weights:
+            return 0
+        return self.w_in.nbytes() + self.w_x.nbytes() + self.w_dt.nbytes() + self.w_o.nbytes() + self.w_conv.numel() * self.w_conv.element_size()
+
+    def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
+        e, L = self.eng, self.eng.L
+        I, N, r = self.inner, self.N, self.rank
+        zx, xc, dbc, dtr, ys = e.buf("zx", 2 * I), e.buf("xbc", I), e.buf("dbc", r + 2 * N), e.buf("dtr", I), e.buf("ys", I)
+        e.mm(self.w_in, h, zx, M, src="h")
+        L.causal_conv(e.mamba_batch, M, e.n_seq, zx, self.w_conv, self.conv_state, xc, bias=self.b_conv, act=True)
+        e.mm(self.w_x, xc, dbc, M)
+        e.mm(self.w_dt, dbc, dtr, M)
+        image = e.image("tmp", M)
+        L.selective_scan(e.mamba_batch, e.n_seq, xc, dtr, dbc[:, r:], dbc[:, r + N:], self.dt_bias, self.A_log, self.D, self.state, ys, I, N,
+                         z=zx[:, I:], image=image)
+        e.mm(self.w_o, ys, y, M, ready=image is not None)
+
+
+class ParallelMixer:
+    """Two mixers side by side on the same input (the design's `parallel` trait names them; their tensors sit under <prefix>left. and
+    <prefix>right.): half the sum of their outputs, each first RMS-normed over the width with <prefix>left.out / right.out.  The
+    norms, the average and the sum into the residual stream are part of the stream's step (forward_branches)."""
+
+    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["ParallelMixer"] = None):
+        self.eng = eng
+        kinds = eng.cfg.traits["parallel"]
+        self.left, self.right = (MIXERS[kinds[s]](eng, index, m[s], f"{prefix}{s}.", share=getattr(share, s) if share is not None else None)
+                                 for s in ("left", "right"))
+        if share is None:       # the factor 1/2 rides on the norms' weights (exact: a power of two)
+            self.out_l, self.out_r = ((0.5 * eng.norm_weight(f"{prefix}{s}.out")).contiguous() for s in ("left", "right"))
+        else:
+            self.out_l, self.out_r = share.out_l, share.out_r
+
+    def parts(self) -> list:
+        return [self.left, self.right]
+
+    def scratch(self) -> Dict[str, int]:
+        n = {"br_l": self.eng.cfg.width, "br_r": self.eng.cfg.width}
+        for p in self.parts():
+            for name, w in p.scratch().items():
+                n[name] = max(n.get(name, 0), w)
+        return n
+
+    def bind(self, mixers: list):
+        for p in self.parts():
+            p.bind(mixers)
+
+    def weight_bytes(self) -> int:
+        return sum(p.weight_bytes() for p in self.parts())
+
+    def forward_branches(self, h: torch.Tensor, M: int) -> list:
+        """[(branch output, weight of its norm)]: the mixer's output is the sum of the normed branches."""
+        bl, br = self.eng.buf("br_l"), self.eng.buf("br_r")
+        self.left.forward(h, bl, M)
+        self.right.forward(h, br, M)
+        return [(bl, self.out_l), (br, self.out_r)]
+
+    def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
+        e = self.eng
+        e.L.residual_step(M, e.cfg.width, e.cfg.norm_eps, normed=self.forward_branches(h, M), x=y)
 
 
 class RoutedExperts:
@@ -679,7 +949,8 @@ class RoutedExperts:
 
 
 MIXERS = {"latent_attention": LatentAttentionMixer, "mamba2": Mamba2Mixer, "attention": WindowAttentionMixer,
-          "lightning": LightningMixer}
+          "lightning": LightningMixer, "mlstm": MLstmMixer, "hgrn2": Hgrn2Mixer, "mamba1": Mamba1Mixer, "parallel": ParallelMixer}
+SHARING_MIXERS = ("attention", "lightning", "mlstm", "hgrn2", "mamba1", "parallel")      # run another layer's weights on a cache / state of their own
 FEED_FORWARDS = {"dense": DenseFeedForward, "moe": RoutedExperts}
 
 
@@ -699,7 +970,8 @@ class _HyperWeights:
 
 class _Layer:
     def __init__(self, eng: "LayerListEngine", i: int, spec: LayerSpec, owner: Optional["_Layer"] = None):
-        p = f"l{i}."
+        p = f"l{i if spec.tensors is None else spec.tensors}."
+        self.opens = spec.opens
         if spec.type not in MIXERS:
             raise ValueError(f"layer {i}: unknown mixer type {spec.type!r}")
         sandwich, post = eng.cfg.residual == "sandwich", eng.cfg.residual == "post"
@@ -708,8 +980,8 @@ class _Layer:
         self.canon_state = torch.zeros(eng.n_slots, max(taps - 1, 1), eng.cfg.width, dtype=torch.float32, device=eng.device) if taps > 0 else None
         if owner is not None:
             # the owner's weights on a cache / state of this layer's own
-            if spec.type not in ("attention", "lightning") or sandwich:
-                raise ValueError(f"layer {i}: weights_of is only known for attention and lightning mixers of hyper-style models")
+            if spec.type not in SHARING_MIXERS or sandwich:
+                raise ValueError(f"layer {i}: running another layer's weights is not known for {spec.type} mixers or the sandwich residual style")
             self.mixer = MIXERS[spec.type](eng, i, spec.mixer, "", share=owner.mixer)
             self.ff = owner.ff
             for n in ("norm1", "norm1b", "norm2", "norm2b", "hc1", "hc2", "canon1"):
@@ -791,11 +1063,18 @@ class LayerListEngine:
                     built[i] = _Layer(self, i, spec, owner)
             self.layers: List[_Layer] = [built[i] for i in range(len(self.cfg.layers))]
             self.final_norm, self.head = self.norm_weight("final.norm"), self.dense_weight(self.weight("head"))
+            self.embed_norm = self.norm_weight("embed.norm") if self.cfg.traits.get("embed_norm") else None
+            self.loop_step = None
+            if self.cfg.loop_times:
+                self.loop_step = self.vector("loop.step")
+                if tuple(self.loop_step.shape) != (self.cfg.loop_times, self.cfg.width):
+                    raise ValueError(f"loop.step has shape {tuple(self.loop_step.shape)}")
         finally:
             self._st.close()
         mixers = [l.mixer for l in self.layers]
         for mx in mixers:
             mx.bind(mixers)
+        mixers = [part for mx in mixers for part in (mx.parts() if isinstance(mx, ParallelMixer) else [mx])]
         # latent attention on the tensor cores (bf16 caches): rows of a sequence are tiled so that rows x heads <= 32
         att = [mx for mx in mixers if isinstance(mx, LatentAttentionMixer)]
         self.attn_rq = 0
@@ -826,8 +1105,16 @@ class LayerListEngine:
         if lt and R >= LIGHTNING_CHUNKED_MIN_ROWS and os.environ.get("DLLAMA_LAYERS_CHUNKED_SCAN", "1") != "0":
             self._lightning_scratch = torch.zeros(max(L.lightning_chunk_floats(R, self.n_slots, mx.H, mx.dim, mx.vdim) for mx in lt),
                                                   dtype=torch.float32, device=dev)
-        if self.cfg.residual == "post" and self.cfg.streams != 1:
-            raise ValueError("the post-norm residual style keeps one residual stream")
+        # the same with data-dependent gates
+        gt = [mx for mx in mixers if isinstance(mx, (MLstmMixer, Hgrn2Mixer)) and mx.chunked]
+        self.gated_chunks, self._gated_scratch, self._gated_slots = 0, None, R // L.GATED_CHUNK + self.n_slots
+        if gt and R >= GATED_CHUNKED_MIN_ROWS and os.environ.get("DLLAMA_LAYERS_CHUNKED_SCAN", "1") != "0":
+            self._gated_scratch = torch.zeros(max(L.gated_chunk_floats(R, self.n_slots, mx.H, mx.dim, mx.vdim) for mx in gt),
+                                              dtype=torch.float32, device=dev)
+        if self.cfg.residual in ("post", "parallel") and self.cfg.streams != 1:
+            raise ValueError(f"the {self.cfg.residual} residual style keeps one residual stream")
+        if (self.embed_norm is not None) != (self.cfg.residual == "parallel"):
+            raise ValueError("a normed embedding belongs to the parallel residual style")
         if self.cfg.canon_taps and self.cfg.residual != "hyper":
             raise ValueError("a convolution in front of the mixers is only wired into the pre-norm / hyper residual style")
         # scratch: one f32 buffer per name, as wide as the widest user
@@ -843,13 +1130,15 @@ class LayerListEngine:
         self._xh = {}
         if self.tc:       # activation slabs: one kept for a sublayer's input (several products read it), one for the rest
             n = L.xh_bytes(self._kmax, self.ncap)
-            self._xh = {k: torch.zeros(n, dtype=torch.uint8, device=dev) for k in ("h", "tmp")}
+            self._xh = {k: torch.zeros(n, dtype=torch.uint8, device=dev) for k in ("h", "tmp") + (("h2",) if self.cfg.residual == "parallel" else ())}
         if self.cfg.streams > L.HC_MAX_STREAMS:
             raise ValueError(f"{self.cfg.streams} streams: the kernels keep at most {L.HC_MAX_STREAMS} copies of the residual stream")
         self.x = torch.zeros(R, self.cfg.streams * self.cfg.width, dtype=torch.float32, device=dev)      # row = [streams][width]
         self.hn = torch.zeros(R, self.cfg.width, dtype=torch.float32, device=dev)
         self.hc = torch.zeros(R, self.cfg.width, dtype=torch.float32, device=dev) if self.cfg.canon_taps else None
         self.y = torch.zeros(R, self.cfg.width, dtype=torch.float32, device=dev)
+        if self.cfg.residual == "parallel":       # the embedding output, the feed-forward's input and output
+            self.x0, self.hn2, self.y2 = (torch.zeros(R, self.cfg.width, dtype=torch.float32, device=dev) for _ in range(3))
         self.logits = torch.zeros(R, self.cfg.vocab, dtype=torch.float32, device=dev)
         self.out_tokens = torch.zeros(R, dtype=torch.int32, device=dev)
         self.h_out_tokens = torch.zeros(R, dtype=torch.int32).pin_memory()
@@ -884,7 +1173,7 @@ class LayerListEngine:
         self.block_table = torch.zeros(self.n_slots, self.max_pages, dtype=torch.int32, device=dev)
         self.h_block_table = torch.zeros(self.n_slots, self.max_pages, dtype=torch.int32).pin_memory()
         self._staging_ev: Optional[torch.cuda.Event] = None
-        self._xh_h_ready = False
+        self._xh_h_ready, self._xh_h = False, "h"
         # decode-sized batches replay a CUDA graph per batch shape (rows, sequences, wanted logits, attention tiling):
         # a step is ~25 small launches per layer, and the host cannot issue them as fast as the GPU retires them
         self.use_graphs = bool(use_graphs) and os.environ.get("DLLAMA_LAYERS_GRAPHS", "1") != "0"
@@ -923,15 +1212,16 @@ class LayerListEngine:
         return DenseWeight(t, self.tc)
 
     def mm(self, w: DenseWeight, x: torch.Tensor, y: torch.Tensor, M: int, epi: int = 0, aux=None, param: float = 0.0,
-           src: str = "tmp", param2: float = 0.0):
+           src: str = "tmp", param2: float = 0.0, ready: bool = False):
         """y[:M] = epi(x[:M] @ w^T).  src="h": x is the current sublayer input; its tensor-core image is made by the
-        first product that reads it (begin_sublayer() marks it stale) and shared by the others."""
+        first product that reads it (begin_sublayer() marks it stale) and shared by the others.  ready: the launch that
+        produced x left it as the image of `src` (see image())."""
         L = self.L
         if w.wh is None or M < TC_MIN_ROWS:
             L.dense(w.t, x, y, M, self.round_x, epi=epi, aux=aux, param=param, param2=param2)
             return
-        xh = self._xh[src]
-        if src != "h" or not self._xh_h_ready:
+        xh = self._xh[self._xh_h if src == "h" else src]
+        if not ready and (src != "h" or not self._xh_h_ready):
             L.xh_from_rows(x, M, w.K, self.ncap, xh)
             self._xh_h_ready = src == "h" or self._xh_h_ready
         L.dense_tc(w.wh, w.N, w.K, xh, self.ncap, y, M, epi=epi, aux=aux, param=param, param2=param2)
@@ -952,6 +1242,17 @@ class LayerListEngine:
         if not self._n_chunks or not self.L.mamba_chunked_supported(mx.P, mx.N):
             return None
         return (self.chunk_seq, self.chunk_off, self._n_chunks) + self._chunk_scratch
+
+    def image(self, name: str, M: int):
+        """(activation image, its row capacity) if products over M rows read bf16 images, so that a kernel can leave its
+        result in the next product's operand layout; None where they read f32 rows."""
+        return (self._xh[name], self.ncap) if self.tc and M >= TC_MIN_ROWS else None
+
+    def gated_chunking(self, mx) -> dict:
+        """The chunking of this batch for a gated linear-attention scan (empty: token by token)."""
+        if not mx.chunked or not self.gated_chunks:
+            return {}
+        return dict(max_chunks=self.gated_chunks, scratch=self._gated_scratch, chunk_slots=self._gated_slots)
 
     def lightning_scratch(self, mx):
         return self._lightning_scratch
@@ -975,8 +1276,9 @@ class LayerListEngine:
         o = self._wtile_off[rq]
         return self.desc[o:], self._wtile_n[rq]
 
-    def begin_sublayer(self):
-        self._xh_h_ready = False
+    def begin_sublayer(self, image: str = "h", ready: bool = False):
+        """A sublayer starts: its input's tensor-core image is `image`, complete already if `ready`."""
+        self._xh_h, self._xh_h_ready = image, ready
 
     def buf(self, name: str, width: Optional[int] = None) -> torch.Tensor:
         """Scratch `name` as [max_rows][width] (default: the width it was sized for)."""
@@ -1064,6 +1366,9 @@ class LayerListEngine:
         self.lightning_chunks = 0
         if self._lightning_scratch is not None and longest >= LIGHTNING_CHUNKED_MIN_ROWS:
             self.lightning_chunks = (longest + self.L.LIGHTNING_CHUNK - 1) // self.L.LIGHTNING_CHUNK
+        self.gated_chunks = 0
+        if self._gated_scratch is not None and longest >= GATED_CHUNKED_MIN_ROWS:
+            self.gated_chunks = (longest + self.L.GATED_CHUNK - 1) // self.L.GATED_CHUNK
         self._n_chunks = 0
         if self._chunk_scratch is not None and longest >= CHUNKED_SCAN_MIN_ROWS:
             co, nc, ch = self._chunks_off, 0, self.L.MAMBA_CHUNK
@@ -1089,7 +1394,10 @@ class LayerListEngine:
         L, cfg, eps = self.L, self.cfg, self.cfg.norm_eps
         x, hn, y, W = self.x, self.hn, self.y, self.cfg.width
         L.embed_rows(self.embed, self.tokens, x, M, cfg.embed_scale, cfg.streams)
-        if cfg.residual == "hyper":
+        head_ready = False
+        if cfg.residual == "parallel":
+            head_ready = self._launch_parallel_layers(M, n_logits)
+        elif cfg.residual == "hyper":
             self._launch_hyper_layers(M)
             if n_logits:      # the copies summed, the model's norm, only the wanted rows
                 L.hyper_step(x, n_logits, cfg.streams, W, h=hn, norm_w=self.final_norm, eps=eps, rows=self.logit_rows)
@@ -1123,11 +1431,47 @@ class LayerListEngine:
             if n_logits:
                 L.rms_norm(x, hn, n_logits, W, eps, w=self.final_norm, plus_one=True, rows=self.logit_rows)
         if n_logits:
-            self.begin_sublayer()
+            self.begin_sublayer(ready=head_ready)
             if cfg.logit_softcap > 0:
-                self.mm(self.head, hn, self.logits, n_logits, epi=L.DENSE_SOFTCAP, param=cfg.logit_softcap)
+                self.mm(self.head, hn, self.logits, n_logits, epi=L.DENSE_SOFTCAP, param=cfg.logit_softcap, src="h")
             else:
-                self.mm(self.head, hn, self.logits, n_logits)
+                self.mm(self.head, hn, self.logits, n_logits, src="h")
+
+    def _launch_parallel_layers(self, M: int, n_logits: int) -> bool:
+        """Layers whose mixer and feed-forward read the same residual stream through a norm each.  One launch per layer sums
+        the last layer's outputs into the stream (branches normed on the way; ahead of a pass of the loop also the embedding
+        output and the pass's vector) and leaves both normed copies, as bf16 images where the products read those.  Returns
+        whether the last norm left the head's operand image."""
+        L, cfg = self.L, self.cfg
+        x, x0, W, eps = self.x, self.x0, cfg.width, cfg.norm_eps
+        L.rms_norm(x, x0, M, W, eps, w=self.embed_norm)                       # the embedding output
+        src, adds, normed = x0, [], []
+        img1, img2 = self.image("h", M), self.image("h2", M)
+        for l in self.layers:
+            if l.opens:
+                adds = adds + [x0]
+            L.residual_step(M, W, eps, x_in=src, adds=adds, normed=normed, vec=self.loop_step[l.opens] if l.opens is not None else None,
+                            x=x, outs=[(l.norm1, img1 or self.hn)] + ([(l.norm2, img2 or self.hn2)] if l.ff is not None else []))
+            src, adds, normed = x, [], []
+            self.begin_sublayer("h", ready=img1 is not None)
+            if isinstance(l.mixer, ParallelMixer):
+                normed = l.mixer.forward_branches(self.hn, M)
+            else:
+                l.mixer.forward(self.hn, self.y, M)
+                adds.append(self.y)
+            if l.ff is not None:
+                self.begin_sublayer("h2", ready=img2 is not None)
+                l.ff.forward(self.hn2, self.y2, M)
+                adds.append(self.y2)
+            if self.layer_probe is not None:
+                L.residual_step(M, W, eps, x_in=src, adds=adds, normed=normed, x=x)
+                adds, normed = [], []
+                self.layer_probe.append(x[:M].clone())
+        if not n_logits:
+            return False
+        img = self.image("h", n_logits)
+        L.residual_step(n_logits, W, eps, x_in=src, adds=adds, normed=normed, rows=self.logit_rows, outs=[(self.final_norm, img or self.hn)])
+        return img is not None
 
     def _launch_hyper_layers(self, M: int):
         """Sublayer after sublayer on the copies of the residual stream.  The write of one sublayer's output and the read
@@ -1263,6 +1607,35 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
         t[prefix + "out"] = (1.0 + torch.randn(S, generator=g) * 0.2).to(torch.bfloat16)
         t[prefix + "mix"] = (torch.eye(S) * 0.9 + torch.randn(S, S, generator=g) * 0.1).to(torch.bfloat16)
 
+    def attention(p, m):
+        H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m.get("vdim", m["dim"])
+        t[p + "q"] = mat(H * d, W, 2.0)
+        if m.get("kv_from") is None:
+            t[p + "k"] = mat(G * d, W, 2.0)
+        t[p + "o"] = mat(W, H * dv)
+        if m.get("kv_from") is None and att.get("values") == "own":
+            t[p + "v"] = mat(G * dv, W)
+        if att.get("talk"):     # near the identity, with cross-talk between all heads
+            t[p + "talk"] = (torch.eye(H) + torch.randn(H, H, generator=g) * 0.3).to(torch.bfloat16)
+        if att.get("sink"):
+            t[p + "sink"] = (torch.randn(H, generator=g)).to(torch.bfloat16)
+        if att.get("gate"):
+            t[p + "g"] = mat(H * dv, W)
+        if att.get("proj_norm"):
+            t[p + "q.norm"], t[p + "k.norm"] = 1 + small(H * d), 1 + small(G * d)
+
+    def hgrn2(p, m):
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        t[p + "q"], t[p + "f"], t[p + "v"] = mat(H * d, W, 2.0), mat(H * d, W, 1.5), mat(H * dv, W, 1.5)
+        t[p + "f.b"] = (torch.rand(H * d, generator=g) * 4).to(torch.bfloat16)
+        t[p + "lower"] = (torch.rand(H * d, generator=g) * 0.9).to(torch.bfloat16)
+        t[p + "norm"], t[p + "o"] = 1 + small(dv), mat(W, H * dv)
+
+    if traits.get("embed_norm"):
+        t["embed.norm"] = norm_w()
+    if config.get("loop"):
+        t["loop.step"] = (torch.randn(int(config["loop"]["times"]), W, generator=g) * 0.3).to(torch.bfloat16)
+
     for i, l in enumerate(config["layers"]):
         p, m = f"l{i}.", l["mixer"]
         if l.get("weights_of") is not None:
@@ -1294,19 +1667,27 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
             t[p + "mix.D"], t[p + "mix.norm"] = 1 + small(H), 1 + small(inner)
             t[p + "mix.o"] = mat(W, inner)
         elif l["type"] == "attention":
-            H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m.get("vdim", m["dim"])
-            t[p + "mix.q"] = mat(H * d, W, 2.0)
-            if m.get("kv_from") is None:
-                t[p + "mix.k"] = mat(G * d, W, 2.0)
-            t[p + "mix.o"] = mat(W, H * dv)
-            if m.get("kv_from") is None and att.get("values") == "own":
-                t[p + "mix.v"] = mat(G * dv, W)
-            if att.get("talk"):     # near the identity, with cross-talk between all heads
-                t[p + "mix.talk"] = (torch.eye(H) + torch.randn(H, H, generator=g) * 0.3).to(torch.bfloat16)
-            if att.get("sink"):
-                t[p + "mix.sink"] = (torch.randn(H, generator=g)).to(torch.bfloat16)
-            if att.get("gate"):
-                t[p + "mix.g"] = mat(H * dv, W)
+            attention(p + "mix.", m)
+        elif l["type"] == "hgrn2":
+            hgrn2(p + "mix.", m)
+        elif l["type"] == "parallel":
+            attention(p + "mix.left.", m["left"])
+            hgrn2(p + "mix.right.", m["right"])
+            t[p + "mix.left.out"], t[p + "mix.right.out"] = 1 + small(W), 1 + small(W)
+        elif l["type"] == "mlstm":
+            H, d, dv = m["heads"], m["dim"], m["vdim"]
+            t[p + "mix.q"], t[p + "mix.k"], t[p + "mix.v"] = mat(H * d, W, 2.0), mat(H * d, W, 2.0), mat(H * dv, W, 1.5)
+            t[p + "mix.g"], t[p + "mix.o"], t[p + "mix.norm"] = mat(H * dv, W), mat(W, H * dv), 1 + small(H * dv)
+            t[p + "mix.i"], t[p + "mix.f"] = mat(H, W, 2.0), mat(H, W, 2.0)
+            t[p + "mix.i.b"], t[p + "mix.f.b"] = small(H, 0.5), (2 + torch.rand(H, generator=g) * 3).to(torch.bfloat16)
+        elif l["type"] == "mamba1":
+            inner, r, N, K = m["inner"], m["dt_rank"], m["state"], m["conv"]
+            t[p + "mix.in"] = mat(2 * inner, W, 1.5)
+            t[p + "mix.conv"], t[p + "mix.conv.b"] = mat(inner, K, 1.5), small(inner)
+            t[p + "mix.x"], t[p + "mix.dt"] = mat(r + 2 * N, inner, 1.5), mat(inner, r)
+            t[p + "mix.dt.b"] = (torch.rand(inner, generator=g) * 3 - 4).to(torch.bfloat16)
+            t[p + "mix.A_log"] = (torch.log(1.0 + torch.arange(N, dtype=torch.float32))[None, :] + torch.randn(inner, N, generator=g) * 0.2).to(torch.bfloat16)
+            t[p + "mix.D"], t[p + "mix.o"] = 1 + small(inner), mat(W, inner)
         elif l["type"] == "lightning":
             H, d, dv = m["heads"], m["dim"], m["vdim"]
             t[p + "mix.q"], t[p + "mix.k"], t[p + "mix.v"] = mat(H * d, W, 2.0), mat(H * d, W, 2.0), mat(H * dv, W, 2.0)
@@ -1334,6 +1715,8 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
                         t[p + f"mlp.e{n}.gate"] = mat(ff, W, 1.5)
             else:
                 t[p + "mlp.up"], t[p + "mlp.down"] = mat(l["mlp"]["ff"], W), mat(W, l["mlp"]["ff"])
+                if traits.get("dense_act") == "gelu_glu":
+                    t[p + "mlp.gate"] = mat(l["mlp"]["ff"], W, 1.5)
                 if traits.get("dense_act") == "polynorm":
                     t[p + "mlp.act"] = torch.tensor([0.6, 0.3, 0.15, 0.05]).add(torch.randn(4, generator=g) * 0.05).to(torch.bfloat16)
                 elif traits.get("dense_act") == "xielu":
@@ -1415,3 +1798,17 @@ def example_config_darusun(width: int = 160, vocab: int = 320, heads: int = 6, k
               {"type": "latent_attention", "mixer": dict(lat), "mlp": dict(moe)},
               {"type": "attention", "mixer": dict(attn, kv_from=0), "mlp": dict(moe)}]
     return {"architecture": "Darusun", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.6, "layers": layers}
+
+
+def example_config_vopedra(width: int = 160, vocab: int = 320, heads: int = 3) -> dict:
+    """A small Vopedra-shaped configuration: parallel-residual layers; a selective scan without a feed-forward, then a matrix
+    memory and a layer of two branches (attention whose softmax weights are mixed across heads, HGRN2) run twice, then a matrix
+    memory of other sizes."""
+    dense = {"kind": "dense", "ff": 2 * width}
+    left = {"heads": 2 * heads, "kv_heads": heads, "dim": 24, "vdim": 40, "scale": 0.2, "rot": {"base": 10000.0, "dims": 16}}
+    layers = [{"type": "mamba1", "mixer": {"inner": 2 * width, "state": 12, "conv": 4, "dt_rank": 9}, "mlp": None},
+              {"type": "mlstm", "mixer": {"heads": heads, "dim": 20, "vdim": 36, "gate_cap": 9.0}, "mlp": dict(dense)},
+              {"type": "parallel", "mixer": {"left": left, "right": {"heads": heads, "dim": 28, "vdim": 16}}, "mlp": dict(dense)},
+              {"type": "mlstm", "mixer": {"heads": 1, "dim": 40, "vdim": 24, "gate_cap": 15.0}, "mlp": {"kind": "dense", "ff": width}}]
+    return {"architecture": "Vopedra", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "loop": {"start": 1, "stop": 3, "times": 2},
+            "layers": layers}

@@ -10,10 +10,10 @@ from typing import Optional
 import torch
 
 from . import lib
-from .lib import (DENSE_GLU_CLAMP, DENSE_GLU_SILU, DENSE_MUL, DENSE_RELU2, DENSE_ROWGATE_ADD, DENSE_SIGMOID_MUL, DENSE_SILU, DENSE_SOFTCAP, DENSE_STORE,  # noqa: F401
+from .lib import (DENSE_GLU_CLAMP, DENSE_GLU_GELU, DENSE_GLU_SILU, DENSE_MUL, DENSE_RELU2, DENSE_ROWGATE_ADD, DENSE_SIGMOID_MUL, DENSE_SILU, DENSE_SOFTCAP, DENSE_STORE,  # noqa: F401
                   DENSE_XIELU, EPI_DENSE, T_BF16, T_F32,
-                  DlConvArgs, DlDenseArgs, DlEpilogue, DlHyperArgs, DlLatentAttnArgs, DlLightningArgs, DlLatentKvArgs, DlLatentTiles, DlMambaBatch, DlMambaChunks, DlMambaScanArgs, DlMoeArgs,
-                  DlMoePlanArgs, DlMoeSelectArgs, DlNormArgs, DlWindowAttnArgs, DlWindowKvArgs, check_layers, layers_lib)
+                  DlConvArgs, DlDenseArgs, DlEpilogue, DlGatedArgs, DlHeadNormArgs, DlHyperArgs, DlLatentAttnArgs, DlLightningArgs, DlLatentKvArgs, DlLatentTiles, DlMambaBatch, DlMambaChunks, DlMambaScanArgs, DlMoeArgs,
+                  DlMlstmGatesArgs, DlMoePlanArgs, DlMoeSelectArgs, DlNormArgs, DlResidualArgs, DlSelectiveArgs, DlWindowAttnArgs, DlWindowKvArgs, check_layers, layers_lib)
 
 PAGE_SIZE = 32
 HC_MAX_STREAMS = 16          # DL_HC_MAX_STREAMS of the hyper-connection kernel
@@ -257,6 +257,128 @@ def lightning_scan(batch: DlMambaBatch, n_seq: int, q: torch.Tensor, k: torch.Te
     lib.count_launch()
 
 
+# ---- linear attention with data-dependent gates ------------------------------------------------------------------------
+GATED_CHUNK = 64             # DL_GATED_CHUNK: rows of a sequence per chunk of the chunked scan
+
+
+def gated_supported(dim: int, vdim: int) -> bool:
+    return layers_lib().dl_gated_scan_supported(dim, vdim) == 0
+
+
+def gated_chunked_supported(dim: int, vdim: int, channel: bool) -> bool:
+    return layers_lib().dl_gated_scan_chunked_supported(dim, vdim, 1 if channel else 0) == 0
+
+
+def gated_chunk_floats(M: int, n_seq: int, n_heads: int, dim: int, vdim: int) -> int:
+    return int(layers_lib().dl_gated_chunk_floats(M, n_seq, n_heads, dim, vdim))
+
+
+def gated_scan(batch: DlMambaBatch, n_seq: int, q: torch.Tensor, v: torch.Tensor, y: torch.Tensor, state: torch.Tensor, n_heads: int,
+               dim: int, vdim: int, q_scale: float = 1.0, q_silu: bool = False, f: Optional[torch.Tensor] = None,
+               f_bias: Optional[torch.Tensor] = None, lower: Optional[torch.Tensor] = None, k: Optional[torch.Tensor] = None,
+               log_keep: Optional[torch.Tensor] = None, put: Optional[torch.Tensor] = None, den: Optional[torch.Tensor] = None,
+               n_state: Optional[torch.Tensor] = None, max_chunks: int = 0, scratch: Optional[torch.Tensor] = None, chunk_slots: int = 0):
+    """With f (raw gate, f_bias and lower [heads * dim]): S <- diag(g) S + (1 - g) v^T, g = lower + (1 - lower) sigmoid(f + f_bias).
+    With k, log_keep, put [M][heads]: S <- e^log_keep S + put k v^T, n likewise with k alone, den [M][heads] = n . q.
+    y = S^T q, q = silu(q) or q_scale * q; state [slots][heads][dim][vdim] f32 (n_state [slots][heads][dim]).  max_chunks > 0 (with
+    scratch for chunk_slots chunks): the chunk-parallel form for long portions."""
+    a = DlGatedArgs()
+    a.q, a.ldq, a.q_scale, a.q_silu = q.data_ptr(), q.stride(0), q_scale, 1 if q_silu else 0
+    a.k, a.ldk, a.v, a.ldv = _p(k), (k.stride(0) if k is not None else 0), v.data_ptr(), v.stride(0)
+    a.f, a.ldf, a.f_bias, a.lower = _p(f), (f.stride(0) if f is not None else 0), _p(f_bias), _p(lower)
+    a.log_keep, a.put, a.den = _p(log_keep), _p(put), _p(den)
+    a.y, a.ld_y, a.state, a.n_state = y.data_ptr(), y.stride(0), state.data_ptr(), _p(n_state)
+    a.n_heads, a.dim, a.vdim = n_heads, dim, vdim
+    if max_chunks > 0:
+        assert scratch.numel() >= chunk_slots * n_heads * dim * (vdim + 2)
+        check_layers(layers_lib().dl_gated_scan_chunked(batch, n_seq, max_chunks, a, scratch.data_ptr(), chunk_slots, _stream()),
+                     "dl_gated_scan_chunked")
+        lib.count_launch(3)
+        return
+    check_layers(layers_lib().dl_gated_scan(batch, n_seq, a, _stream()), "dl_gated_scan")
+    lib.count_launch()
+
+
+def mlstm_gates(batch: DlMambaBatch, n_seq: int, zi: torch.Tensor, zf: torch.Tensor, bi: torch.Tensor, bf: torch.Tensor, cap: float,
+                u_state: torch.Tensor, log_keep: torch.Tensor, put: torch.Tensor, floor: torch.Tensor, n_heads: int):
+    """Log decays, input weights and e^-u of the matrix memory with a running maximum u (u_state [slots][heads])."""
+    assert zi.stride(0) == zf.stride(0)
+    a = DlMlstmGatesArgs()
+    a.zi, a.zf, a.ld, a.bi, a.bf, a.cap = zi.data_ptr(), zf.data_ptr(), zi.stride(0), bi.data_ptr(), bf.data_ptr(), cap
+    a.u_state, a.log_keep, a.put, a.floor_, a.n_heads = u_state.data_ptr(), log_keep.data_ptr(), put.data_ptr(), floor.data_ptr(), n_heads
+    check_layers(layers_lib().dl_mlstm_gates(batch, n_seq, a, _stream()), "dl_mlstm_gates")
+    lib.count_launch()
+
+
+def head_norm(y: torch.Tensor, M: int, n_heads: int, vdim: int, eps: float, w: torch.Tensor, out: Optional[torch.Tensor],
+              den: Optional[torch.Tensor] = None, floor: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, image=None):
+    """Per head: y / (max(|den|, floor) + 1e-6), RMS norm with weight w ([vdim] or [n_heads * vdim]), times sigmoid(gate); to out or
+    into image = (activation image, ncap)."""
+    assert w.numel() in (vdim, n_heads * vdim)
+    a = DlHeadNormArgs()
+    a.y, a.ld_y, a.den, a.floor_ = y.data_ptr(), y.stride(0), _p(den), _p(floor)
+    a.w, a.w_full = w.data_ptr(), 1 if w.numel() == n_heads * vdim and n_heads > 1 else 0
+    a.gate, a.ld_gate = _p(gate), (gate.stride(0) if gate is not None else 0)
+    xh, ncap = image or (None, 0)
+    a.xh, a.ncap = _p(xh), ncap
+    if xh is None:
+        a.out, a.ld_out = out.data_ptr(), out.stride(0)
+    a.M, a.n_heads, a.vdim, a.eps = M, n_heads, vdim, eps
+    check_layers(layers_lib().dl_head_norm(a, _stream()), "dl_head_norm")
+    lib.count_launch()
+
+
+def selective_supported(state: int) -> bool:
+    return layers_lib().dl_selective_scan_supported(state) == 0
+
+
+def selective_scan(batch: DlMambaBatch, n_seq: int, x: torch.Tensor, dt: torch.Tensor, B: torch.Tensor, C: torch.Tensor,
+                   dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor, state_pool: torch.Tensor, y: Optional[torch.Tensor],
+                   inner: int, state: int, z: Optional[torch.Tensor] = None, image=None):
+    """Selective scan with a state per channel; dt raw (bias and softplus inside); out y (f32) or image = (activation image, ncap)."""
+    assert B.stride(0) == C.stride(0)
+    a = DlSelectiveArgs()
+    a.x, a.ld_x, a.dt, a.ld_dt = x.data_ptr(), x.stride(0), dt.data_ptr(), dt.stride(0)
+    a.B, a.C, a.ld_bc, a.z, a.ld_z = B.data_ptr(), C.data_ptr(), B.stride(0), _p(z), (z.stride(0) if z is not None else 0)
+    a.dt_bias, a.A_log, a.D, a.state_pool = dt_bias.data_ptr(), A_log.data_ptr(), D.data_ptr(), state_pool.data_ptr()
+    xh, ncap = image or (None, 0)
+    a.xh, a.ncap = _p(xh), ncap
+    if xh is None:
+        a.y, a.ld_y = y.data_ptr(), y.stride(0)
+    a.inner, a.state = inner, state
+    check_layers(layers_lib().dl_selective_scan(batch, n_seq, a, _stream()), "dl_selective_scan")
+    lib.count_launch()
+
+
+def residual_step(M: int, dim: int, eps: float, x_in: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, adds=(),
+                  normed=(), vec: Optional[torch.Tensor] = None, x: Optional[torch.Tensor] = None, outs=()):
+    """x[m] = x_in + sum of `adds` + sum of w * unit(v) over (v, w) in `normed`, all of row rows ? rows[m] : m, + vec; then per (w, h)
+    of `outs` h[m] = w * unit(x[m]), h an f32 buffer or an (activation image, ncap) pair.  At most three adds, two of the rest."""
+    a = DlResidualArgs()
+    a.x_in, a.ld_in, a.rows = _p(x_in), (x_in.stride(0) if x_in is not None else 0), _p(rows)
+    adds, normed, outs = list(adds), list(normed), list(outs)
+    assert len(adds) <= 3 and len(normed) <= 2 and len(outs) <= 2
+    for n, t in zip(("add1", "add2", "add3"), adds):
+        setattr(a, n, t.data_ptr())
+        setattr(a, "ld_" + n, t.stride(0))
+    for n, (t, w) in zip("ab", normed):
+        setattr(a, "norm_" + n, t.data_ptr())
+        setattr(a, "w_" + n, w.data_ptr())
+        setattr(a, "ld_" + n, t.stride(0))
+    a.vec, a.x, a.ldx = _p(vec), _p(x), (x.stride(0) if x is not None else 0)
+    for n, (w, h) in zip("12", outs):
+        setattr(a, "w" + n, w.data_ptr())
+        if isinstance(h, tuple):
+            setattr(a, "xh" + n, h[0].data_ptr())
+            a.ncap = h[1]
+        else:
+            setattr(a, "h" + n, h.data_ptr())
+            a.ldh = h.stride(0)
+    a.M, a.dim, a.eps = M, dim, eps
+    check_layers(layers_lib().dl_residual_step(a, _stream()), "dl_residual_step")
+    lib.count_launch()
+
+
 MAMBA_CHUNK = 128            # rows of a sequence per chunk of the chunked scan
 
 
@@ -305,11 +427,13 @@ def hyper_step(x: torch.Tensor, M: int, streams: int, dim: int, y: Optional[torc
 def window_kv_write(k: Optional[torch.Tensor], M: int, kv_heads: int, dim: int, rope_dims: int, freqs: torch.Tensor, rope_scale: float,
                     pos, slot, block_table: torch.Tensor, cache: torch.Tensor, q: Optional[torch.Tensor] = None, q_heads: int = 0,
                     v: Optional[torch.Tensor] = None, vdim: int = 0, qk_norm: bool = False, eps: float = 0.0, rope_half: bool = False,
-                    talk: Optional[torch.Tensor] = None, q_mixed: Optional[torch.Tensor] = None):
+                    talk: Optional[torch.Tensor] = None, q_mixed: Optional[torch.Tensor] = None,
+                    q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None):
     """Keys into the paged cache (rotated key + unrotated head per line); with q [M][q_heads * dim] the queries are
     rotated in place by the same launch.  With v [M][kv_heads * vdim] the line is key + value; rotary (pairs (i, i + dims / 2)
     with rope_half, else (2i, 2i + 1)) comes first, then qk_norm divides every query and key head by its root mean square.
-    talk [q_heads][q_heads] f32 with q_mixed [M][q_heads * kv_heads * dim]: the head mix of the scores, folded into the queries."""
+    talk [q_heads][q_heads] f32 with q_mixed [M][q_heads * kv_heads * dim]: the head mix of the scores, folded into the queries.
+    q_norm [q_heads * dim] / k_norm [kv_heads * dim] f32: an RMS norm over a row's whole projection, in front of the rotary."""
     a = DlWindowKvArgs()
     a.k, a.ld, a.kv_heads, a.dim, a.rope_dims = _p(k), (k.stride(0) if k is not None else 0), kv_heads, dim, rope_dims
     a.q, a.ldq, a.q_heads = _p(q), (q.stride(0) if q is not None else 0), q_heads
@@ -320,12 +444,13 @@ def window_kv_write(k: Optional[torch.Tensor], M: int, kv_heads: int, dim: int, 
     a.v, a.ldv, a.vdim = _p(v), (v.stride(0) if v is not None else 0), vdim
     a.qk_norm, a.eps = 1 if qk_norm else 0, eps
     a.rope_half, a.talk, a.q_mixed, a.ld_qm = 1 if rope_half else 0, _p(talk), _p(q_mixed), (q_mixed.stride(0) if q_mixed is not None else 0)
+    a.q_norm, a.k_norm = _p(q_norm), _p(k_norm)
     check_layers(layers_lib().dl_window_kv_write(a, M, _stream()), "dl_window_kv_write")
     lib.count_launch()
 
 
 def _window_args(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache,
-                 vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0):
+                 vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0, value_heads: int = 0):
     a = DlWindowAttnArgs()
     a.q, a.ldq, a.out, a.ldo = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0)
     a.heads, a.kv_heads, a.dim, a.rope_dims = heads, kv_heads, dim, rope_dims
@@ -333,17 +458,19 @@ def _window_args(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window
     a.pos, a.slot, a.block_table = pos.data_ptr(), slot.data_ptr(), block_table.data_ptr()
     a.max_pages, a.page_size = block_table.shape[1], PAGE_SIZE
     a.cache, a.ctype = cache.data_ptr(), _type(cache)
-    a.vdim, a.chunk, a.sink, a.key_heads = vdim, chunk, _p(sink), key_heads
+    a.vdim, a.chunk, a.sink, a.key_heads, a.value_heads = vdim, chunk, _p(sink), key_heads, value_heads
     return a
 
 
 def window_attention(q: torch.Tensor, out: torch.Tensor, M: int, heads: int, kv_heads: int, dim: int, rope_dims: int,
                      scale: float, softcap: float, window: int, pos, slot, block_table: torch.Tensor, cache: torch.Tensor,
-                     vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0):
+                     vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0, value_heads: int = 0):
     """The per-row kernel (either cache type, f32 arithmetic).  vdim > 0: values of their own behind the keys; chunk > 0:
     only keys of the row's own chunk of positions are visible; sink [heads]: joins the softmax denominator; key_heads =
-    kv_heads: q is [M][heads][kv_heads * dim] (head-mixed queries) against the keys of all key/value heads side by side."""
-    a = _window_args(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache, vdim, chunk, sink, key_heads)
+    kv_heads: q is [M][heads][kv_heads * dim] (head-mixed queries) against the keys of all key/value heads side by side;
+    value_heads = kv_heads: out is [M][heads][kv_heads * vdim], every head's weights against the values of all key/value heads."""
+    a = _window_args(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache, vdim, chunk, sink, key_heads,
+                     value_heads)
     check_layers(layers_lib().dl_window_attention(a, M, _stream()), "dl_window_attention")
     lib.count_launch()
 
@@ -376,47 +503,58 @@ def window_attention_tc(q: torch.Tensor, out: torch.Tensor, heads: int, kv_heads
     lib.count_launch(2 if n_splits > 1 else 1)
 
 
-def talk_tc_supported(heads: int, kv_heads: int, dim: int, vdim: int, key_heads: int, cache_dtype) -> bool:
+def talk_tc_supported(heads: int, kv_heads: int, dim: int, vdim: int, key_heads: int, cache_dtype, value_heads: int = 0) -> bool:
     ctype = T_BF16 if cache_dtype == torch.bfloat16 else T_F32
-    return layers_lib().dl_talk_attention_tc_supported(heads, kv_heads, dim, vdim, key_heads, ctype) == 0
+    return layers_lib().dl_talk_attention_tc_supported(heads, kv_heads, dim, vdim, key_heads, value_heads, ctype) == 0
 
 
-def talk_tc_rows(heads: int, kv_heads: int, dim: int, vdim: int, key_heads: int, longest: int) -> int:
+def talk_tc_rows(heads: int, kv_heads: int, dim: int, vdim: int, key_heads: int, longest: int, value_heads: int = 0) -> int:
     """Rows of one sequence per tile of the kernel for portions of up to `longest` rows: the tile stacks 16 (decoding), 64
     or 128 (row, head-of-a-group) pairs, whichever fits the shared memory."""
-    return int(layers_lib().dl_talk_tc_tile_rows(heads, kv_heads, dim, vdim, key_heads, longest)) // (heads // kv_heads)
+    return int(layers_lib().dl_talk_tc_tile_rows(heads, kv_heads, dim, vdim, key_heads, value_heads, longest)) // (heads // kv_heads)
 
 
-def talk_tc_partial_floats(n_tiles: int, kv_heads: int, n_splits: int, vdim: int, rq: int, heads: int) -> int:
+def talk_tc_partial_floats(n_tiles: int, kv_heads: int, n_splits: int, vdim: int, rq: int, heads: int, value_heads: int = 0) -> int:
     stacked = rq * (heads // kv_heads)
-    return int(layers_lib().dl_talk_tc_partial_floats(n_tiles, kv_heads, n_splits, vdim, 16 if stacked <= 16 else 64 if stacked <= 64 else 128))
+    return int(layers_lib().dl_talk_tc_partial_floats(n_tiles, kv_heads, n_splits, vdim, value_heads, 16 if stacked <= 16 else 64 if stacked <= 64 else 128))
 
 
 def talk_attention_tc(q: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int,
                       pos, slot, block_table: torch.Tensor, cache: torch.Tensor, tile_rows: torch.Tensor, n_tiles: int, rq: int,
                       n_splits: int = 1, partial: Optional[torch.Tensor] = None, chunk: int = 0, sink: Optional[torch.Tensor] = None,
-                      key_heads: int = 0):
+                      key_heads: int = 0, value_heads: int = 0):
     """The tile kernel for values of their own width and (key_heads = kv_heads) head-mixed queries [M][heads][kv_heads * dim]
-    against the keys of all key/value heads side by side.  Tiles and page shares as in window_attention_tc."""
-    a = _window_args(q, out, heads, kv_heads, dim, 0, scale, 0.0, window, pos, slot, block_table, cache, vdim, chunk, sink, key_heads)
+    against the keys of all key/value heads side by side, or (value_heads = kv_heads) every head's weights against the values
+    of all key/value heads, out [M][heads][kv_heads * vdim].  Tiles and page shares as in window_attention_tc."""
+    a = _window_args(q, out, heads, kv_heads, dim, 0, scale, 0.0, window, pos, slot, block_table, cache, vdim, chunk, sink, key_heads, value_heads)
     if n_splits > 1:
-        assert partial is not None and partial.numel() >= talk_tc_partial_floats(n_tiles, kv_heads, n_splits, vdim, rq, heads)
+        assert partial is not None and partial.numel() >= talk_tc_partial_floats(n_tiles, kv_heads, n_splits, vdim, rq, heads, value_heads)
     check_layers(layers_lib().dl_talk_attention_tc(a, tile_rows.data_ptr(), n_tiles, rq, n_splits, _p(partial), _stream()),
                  "dl_talk_attention_tc")
     lib.count_launch(2 if n_splits > 1 else 1)
 
 
 def talk_attention_tiles(q, out, heads, kv_heads, dim, vdim, scale, window, pos, slot, block_table, cache, tiles, rq: int, n_splits: int = 1,
-                         chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0):
+                         chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0, value_heads: int = 0):
     """Convenience for callers with host-side tiles (lists of up to rq row indices of one sequence, consecutive positions)."""
     t = torch.full((len(tiles), rq), -1, dtype=torch.int32)
     for i, rows in enumerate(tiles):
         t[i, :len(rows)] = torch.tensor(rows, dtype=torch.int32)
     partial = None
     if n_splits > 1:
-        partial = torch.zeros(talk_tc_partial_floats(len(tiles), kv_heads, n_splits, vdim, rq, heads), dtype=torch.float32, device=q.device)
+        partial = torch.zeros(talk_tc_partial_floats(len(tiles), kv_heads, n_splits, vdim, rq, heads, value_heads), dtype=torch.float32, device=q.device)
     talk_attention_tc(q, out, heads, kv_heads, dim, vdim, scale, window, pos, slot, block_table, cache, t.to(q.device), len(tiles), rq,
-                      n_splits, partial, chunk, sink, key_heads)
+                      n_splits, partial, chunk, sink, key_heads, value_heads)
+
+
+def talk_mix(wide: torch.Tensor, talk: torch.Tensor, M: int, heads: int, kv_heads: int, vdim: int, out: Optional[torch.Tensor],
+             image=None):
+    """out[m][h] = sum_g talk[h][g] wide[m][g][c(h)], wide [M][heads][kv_heads][vdim]; image = (activation image, ncap) instead of out."""
+    xh, ncap = image or (None, 0)
+    assert talk.dtype == torch.float32 and talk.is_contiguous() and wide.stride(0) == heads * kv_heads * vdim
+    check_layers(layers_lib().dl_talk_mix(wide.data_ptr(), talk.data_ptr(), M, heads, kv_heads, vdim, _p(out) if xh is None else None,
+                                          out.stride(0) if xh is None else 0, _p(xh), ncap, _stream()), "dl_talk_mix")
+    lib.count_launch()
 
 
 def window_attention_tiles(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache, tiles,

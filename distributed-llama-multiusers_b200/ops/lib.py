@@ -215,7 +215,7 @@ def check(rc: int, what: str = ""):
 # ---- hyper-connections, routed experts)
 T_F32, T_BF16 = 0, 1
 DENSE_STORE, DENSE_RELU2, DENSE_SIGMOID_MUL, DENSE_SOFTCAP, DENSE_SILU, DENSE_GLU_CLAMP = 0, 1, 2, 3, 4, 5
-DENSE_MUL, DENSE_XIELU, DENSE_ROWGATE_ADD, DENSE_GLU_SILU = 6, 7, 8, 9
+DENSE_MUL, DENSE_XIELU, DENSE_ROWGATE_ADD, DENSE_GLU_SILU, DENSE_GLU_GELU = 6, 7, 8, 9, 10
 
 
 class DlDenseArgs(C.Structure):
@@ -298,7 +298,8 @@ class DlWindowKvArgs(C.Structure):
                 ("pos", C.c_void_p), ("slot", C.c_void_p), ("block_table", C.c_void_p),
                 ("max_pages", C.c_int), ("page_size", C.c_int), ("cache", C.c_void_p), ("ctype", C.c_int),
                 ("v", C.c_void_p), ("ldv", C.c_longlong), ("vdim", C.c_int), ("qk_norm", C.c_int), ("eps", C.c_float),
-                ("rope_half", C.c_int), ("talk", C.c_void_p), ("q_mixed", C.c_void_p), ("ld_qm", C.c_longlong)]
+                ("rope_half", C.c_int), ("talk", C.c_void_p), ("q_mixed", C.c_void_p), ("ld_qm", C.c_longlong),
+                ("q_norm", C.c_void_p), ("k_norm", C.c_void_p)]
 
 
 class DlWindowAttnArgs(C.Structure):
@@ -308,7 +309,7 @@ class DlWindowAttnArgs(C.Structure):
                 ("scale", C.c_float), ("softcap", C.c_float), ("window", C.c_int),
                 ("pos", C.c_void_p), ("slot", C.c_void_p), ("block_table", C.c_void_p),
                 ("max_pages", C.c_int), ("page_size", C.c_int), ("cache", C.c_void_p), ("ctype", C.c_int),
-                ("vdim", C.c_int), ("chunk", C.c_int), ("sink", C.c_void_p), ("key_heads", C.c_int)]
+                ("vdim", C.c_int), ("chunk", C.c_int), ("sink", C.c_void_p), ("key_heads", C.c_int), ("value_heads", C.c_int)]
 
 
 class DlConvArgs(C.Structure):
@@ -325,6 +326,49 @@ class DlLightningArgs(C.Structure):
                 ("ldq", C.c_longlong), ("ldk", C.c_longlong), ("ldv", C.c_longlong),
                 ("decay", C.c_void_p), ("y", C.c_void_p), ("ld_y", C.c_longlong), ("state", C.c_void_p),
                 ("n_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int)]
+
+
+class DlGatedArgs(C.Structure):
+    """Mirror of ``DlGatedArgs``."""
+    _fields_ = [("q", C.c_void_p), ("ldq", C.c_longlong), ("q_scale", C.c_float), ("q_silu", C.c_int),
+                ("k", C.c_void_p), ("ldk", C.c_longlong), ("v", C.c_void_p), ("ldv", C.c_longlong),
+                ("f", C.c_void_p), ("ldf", C.c_longlong), ("f_bias", C.c_void_p), ("lower", C.c_void_p),
+                ("log_keep", C.c_void_p), ("put", C.c_void_p), ("y", C.c_void_p), ("ld_y", C.c_longlong), ("den", C.c_void_p),
+                ("state", C.c_void_p), ("n_state", C.c_void_p), ("n_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int)]
+
+
+class DlMlstmGatesArgs(C.Structure):
+    """Mirror of ``DlMlstmGatesArgs``."""
+    _fields_ = [("zi", C.c_void_p), ("zf", C.c_void_p), ("ld", C.c_longlong), ("bi", C.c_void_p), ("bf", C.c_void_p),
+                ("cap", C.c_float), ("u_state", C.c_void_p), ("log_keep", C.c_void_p), ("put", C.c_void_p), ("floor_", C.c_void_p),
+                ("n_heads", C.c_int)]
+
+
+class DlHeadNormArgs(C.Structure):
+    """Mirror of ``DlHeadNormArgs``."""
+    _fields_ = [("y", C.c_void_p), ("ld_y", C.c_longlong), ("den", C.c_void_p), ("floor_", C.c_void_p), ("w", C.c_void_p),
+                ("w_full", C.c_int), ("gate", C.c_void_p), ("ld_gate", C.c_longlong), ("out", C.c_void_p), ("ld_out", C.c_longlong),
+                ("xh", C.c_void_p), ("ncap", C.c_int), ("M", C.c_int), ("n_heads", C.c_int), ("vdim", C.c_int), ("eps", C.c_float)]
+
+
+class DlSelectiveArgs(C.Structure):
+    """Mirror of ``DlSelectiveArgs``."""
+    _fields_ = [("x", C.c_void_p), ("ld_x", C.c_longlong), ("dt", C.c_void_p), ("ld_dt", C.c_longlong),
+                ("B", C.c_void_p), ("C", C.c_void_p), ("ld_bc", C.c_longlong), ("z", C.c_void_p), ("ld_z", C.c_longlong),
+                ("dt_bias", C.c_void_p), ("A_log", C.c_void_p), ("D", C.c_void_p), ("state_pool", C.c_void_p),
+                ("y", C.c_void_p), ("ld_y", C.c_longlong), ("xh", C.c_void_p), ("ncap", C.c_int),
+                ("inner", C.c_int), ("state", C.c_int)]
+
+
+class DlResidualArgs(C.Structure):
+    """Mirror of ``DlResidualArgs``."""
+    _fields_ = [("x_in", C.c_void_p), ("ld_in", C.c_longlong), ("rows", C.c_void_p),
+                ("add1", C.c_void_p), ("add2", C.c_void_p), ("add3", C.c_void_p),
+                ("ld_add1", C.c_longlong), ("ld_add2", C.c_longlong), ("ld_add3", C.c_longlong),
+                ("norm_a", C.c_void_p), ("w_a", C.c_void_p), ("norm_b", C.c_void_p), ("w_b", C.c_void_p),
+                ("ld_a", C.c_longlong), ("ld_b", C.c_longlong), ("vec", C.c_void_p), ("x", C.c_void_p), ("ldx", C.c_longlong),
+                ("w1", C.c_void_p), ("h1", C.c_void_p), ("xh1", C.c_void_p), ("w2", C.c_void_p), ("h2", C.c_void_p), ("xh2", C.c_void_p),
+                ("ldh", C.c_longlong), ("ncap", C.c_int), ("M", C.c_int), ("dim", C.c_int), ("eps", C.c_float)]
 
 
 class DlMoeSelectArgs(C.Structure):
@@ -390,10 +434,11 @@ def layers_lib():
     L.dl_window_attention_tc.argtypes = [C.POINTER(DlWindowAttnArgs), vp, i32, i32, i32, vp, vp]
     L.dl_window_tc_partial_floats.argtypes = [i32, i32, i32, i32]
     L.dl_window_tc_partial_floats.restype = i64
-    L.dl_talk_attention_tc_supported.argtypes = [i32, i32, i32, i32, i32, i32]
+    L.dl_talk_attention_tc_supported.argtypes = [i32] * 7
     L.dl_talk_attention_tc.argtypes = [C.POINTER(DlWindowAttnArgs), vp, i32, i32, i32, vp, vp]
-    L.dl_talk_tc_partial_floats.argtypes = [i32, i32, i32, i32, i32]
-    L.dl_talk_tc_tile_rows.argtypes = [i32, i32, i32, i32, i32, i32]
+    L.dl_talk_tc_partial_floats.argtypes = [i32] * 6
+    L.dl_talk_tc_tile_rows.argtypes = [i32] * 7
+    L.dl_talk_mix.argtypes = [vp, vp, i32, i32, i32, i32, vp, i64, vp, i32, vp]
     L.dl_talk_tc_partial_floats.restype = i64
     L.dl_mamba_conv.argtypes = [C.POINTER(DlMambaBatch), i32, i32, vp, i64, i32, vp, vp, i32, vp, vp, i32, i32, vp]
     L.dl_mamba_scan.argtypes = [C.POINTER(DlMambaBatch), i32, C.POINTER(DlMambaScanArgs), vp]
@@ -408,6 +453,17 @@ def layers_lib():
     L.dl_lightning_scan_chunked_supported.restype = i32
     L.dl_lightning_chunk_floats.argtypes = [i32, i32, i32, i32, i32]
     L.dl_lightning_chunk_floats.restype = i64
+    L.dl_gated_scan.argtypes = [C.POINTER(DlMambaBatch), i32, C.POINTER(DlGatedArgs), vp]
+    L.dl_gated_scan_chunked.argtypes = [C.POINTER(DlMambaBatch), i32, i32, C.POINTER(DlGatedArgs), vp, i32, vp]
+    L.dl_gated_scan_supported.argtypes = [i32, i32]
+    L.dl_gated_scan_chunked_supported.argtypes = [i32, i32, i32]
+    L.dl_gated_chunk_floats.argtypes = [i32, i32, i32, i32, i32]
+    L.dl_gated_chunk_floats.restype = i64
+    L.dl_mlstm_gates.argtypes = [C.POINTER(DlMambaBatch), i32, C.POINTER(DlMlstmGatesArgs), vp]
+    L.dl_head_norm.argtypes = [C.POINTER(DlHeadNormArgs), vp]
+    L.dl_selective_scan.argtypes = [C.POINTER(DlMambaBatch), i32, C.POINTER(DlSelectiveArgs), vp]
+    L.dl_selective_scan_supported.argtypes = [i32]
+    L.dl_residual_step.argtypes = [C.POINTER(DlResidualArgs), vp]
     L.dl_wh_bytes.restype = i64
     L.dl_wh_bytes.argtypes = [i32, i32]
     L.dl_wh_from_dense.argtypes = [vp, i32, i32, i64, vp, vp]
@@ -421,7 +477,9 @@ def layers_lib():
                  "dl_mamba_conv", "dl_mamba_scan", "dl_mamba_scan_chunked", "dl_sample_rows", "dl_argmax", "dl_wh_from_dense", "dl_xh_from_rows",
                  "dl_gemm_wh_tc", "dl_hyper_step", "dl_window_kv_write", "dl_window_attention", "dl_moe_select", "dl_moe_rows", "dl_moe_plan",
                  "dl_moe_combine", "dl_xh_gather_rows", "dl_gemm_wh_tc_grouped", "dl_window_tc_rows", "dl_window_attention_tc_supported",
-                 "dl_window_attention_tc", "dl_talk_attention_tc_supported", "dl_talk_attention_tc", "dl_talk_tc_tile_rows", "dl_causal_conv", "dl_poly_norm", "dl_lightning_scan", "dl_lightning_scan_chunked"):
+                 "dl_window_attention_tc", "dl_talk_attention_tc_supported", "dl_talk_attention_tc", "dl_talk_tc_tile_rows", "dl_causal_conv", "dl_poly_norm", "dl_lightning_scan", "dl_lightning_scan_chunked",
+                 "dl_gated_scan", "dl_gated_scan_chunked", "dl_gated_scan_supported", "dl_gated_scan_chunked_supported", "dl_mlstm_gates", "dl_head_norm",
+                 "dl_selective_scan", "dl_selective_scan_supported", "dl_residual_step", "dl_talk_mix"):
         getattr(L, name).restype = i32
     _layers = L
     return L

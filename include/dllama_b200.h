@@ -29,7 +29,9 @@ enum { DL_DENSE_STORE = 0, DL_DENSE_RELU2 = 1, DL_DENSE_SIGMOID_MUL = 2, DL_DENS
        DL_DENSE_MUL = 6          /* aux[m][n] * (.)                                                                  */,
        DL_DENSE_XIELU = 7        /* z > 0: param z^2 + z / 2;  else: param2 (exp(z) - 1 - z) + z / 2                 */,
        DL_DENSE_ROWGATE_ADD = 8  /* y[m][n] + sigmoid(aux[m * ld_aux]) * (.): one gate per row, added to what y holds */,
-       DL_DENSE_GLU_SILU = 9     /* tensor-core epilogue only, columns paired like GLU_CLAMP: silu(gate) * up        */ };
+       DL_DENSE_GLU_SILU = 9     /* tensor-core epilogue only, columns paired like GLU_CLAMP: silu(gate) * up        */,
+       DL_DENSE_GLU_GELU = 10    /* columns paired like GLU_CLAMP (weight rows gate_0, up_0, gate_1, ...): gelu_tanh(gate) * up; every
+                                    product kernel has it, the output has half as many columns as the weight has rows   */ };
 
 typedef struct {
     int kind;
@@ -492,6 +494,87 @@ typedef struct {
 } DlHyperArgs;
 int dl_hyper_step(const DlHyperArgs* args /*host*/, void* stream);
 
+/* ---- linear attention with data-dependent gates (gated_scan.cu) -------------------------------------------------------
+ * Per head, state S [dim][vdim] f32 per slot, one row of the batch after another of a sequence (fresh at position 0):
+ *   channel form (f != NULL):  z = f + f_bias, g = lower + (1 - lower) sigmoid(z) per channel, S <- diag(g) S + (1 - g) v^T
+ *   head form (log_keep):      S <- e^log_keep S + put k v^T,  n <- e^log_keep n + put k,  den = n . q
+ * then y = S^T q with q = silu(q) (q_silu) or q_scale * q.  The gates of the head form come from dl_mlstm_gates. */
+typedef struct {
+    const float* q; long long ldq; float q_scale; int q_silu;
+    const float* k; long long ldk;           /* head form */
+    const float* v; long long ldv;
+    const float* f; long long ldf; const float* f_bias; const float* lower;   /* channel form; f_bias, lower [heads * dim] */
+    const float* log_keep; const float* put; /* head form: [M][heads] */
+    float* y; long long ld_y;                /* [M][heads * vdim] */
+    float* den;                              /* head form: [M][heads] */
+    float* state; float* n_state;            /* [n_slots][heads][dim][vdim], head form also [n_slots][heads][dim] */
+    int n_heads, dim, vdim;
+} DlGatedArgs;
+int dl_gated_scan_supported(int dim, int vdim);
+int dl_gated_scan(const DlMambaBatch* batch /*host*/, int n_seq, const DlGatedArgs* args /*host*/, void* stream);
+/* Long portions: chunks of DL_GATED_CHUNK rows of a sequence in parallel (three launches), as dl_lightning_scan_chunked */
+#define DL_GATED_CHUNK 64
+int dl_gated_scan_chunked_supported(int dim, int vdim, int channel);
+long long dl_gated_chunk_floats(int M, int n_seq, int n_heads, int dim, int vdim);
+int dl_gated_scan_chunked(const DlMambaBatch* batch /*host*/, int n_seq, int max_chunks, const DlGatedArgs* args /*host*/,
+                          float* scratch, int chunk_slots, void* stream);
+/* Gates of a matrix memory with a running maximum u (one f32 per slot and head, 0 ahead of the first row): a = cap tanh((zi +
+ * bi) / cap), b = log sigmoid(cap tanh((zf + bf) / cap)), u' = max(b + u, a), log_keep = b + u - u', put = e^(a - u'),
+ * floor = e^-u'.  zi, zf: [M] rows of n_heads numbers; outputs [M][n_heads]. */
+typedef struct {
+    const float* zi; const float* zf; long long ld;
+    const float* bi; const float* bf; float cap;
+    float* u_state;
+    float* log_keep; float* put; float* floor_;
+    int n_heads;
+} DlMlstmGatesArgs;
+int dl_mlstm_gates(const DlMambaBatch* batch /*host*/, int n_seq, const DlMlstmGatesArgs* args /*host*/, void* stream);
+/* Per row and head of vdim numbers: o = y / (max(|den|, floor) + 1e-6) (den NULL: y), then o / sqrt(mean(o^2) + eps) * w
+ * (w [vdim], or [n_heads * vdim] with w_full), then * sigmoid(gate) (gate NULL: none).  To out (f32) or, with xh, into the
+ * tcgen05 GEMM's activation image. */
+typedef struct {
+    const float* y; long long ld_y;
+    const float* den; const float* floor_;
+    const float* w; int w_full;
+    const float* gate; long long ld_gate;
+    float* out; long long ld_out; uint8_t* xh; int ncap;
+    int M, n_heads, vdim; float eps;
+} DlHeadNormArgs;
+int dl_head_norm(const DlHeadNormArgs* args /*host*/, void* stream);
+
+/* ---- selective scan with a state per channel (selective_scan.cu) -------------------------------------------------------
+ * step = softplus(dt + dt_bias);  S[c][n] <- exp(-step_c exp(A_log[c][n])) S[c][n] + step_c x_c B_n;
+ * y_c = (sum_n S[c][n] C_n + D_c x_c) * silu(z_c)  (z NULL: no gate).  State [n_slots][inner][state] f32. */
+typedef struct {
+    const float* x; long long ld_x;          /* [M][inner], convolved and activated */
+    const float* dt; long long ld_dt;        /* [M][inner] */
+    const float* B; const float* C; long long ld_bc;      /* [M] rows of `state` numbers */
+    const float* z; long long ld_z;
+    const float* dt_bias; const float* A_log; const float* D;      /* [inner], [inner][state], [inner] f32 */
+    float* state_pool;
+    float* y; long long ld_y; uint8_t* xh; int ncap;      /* y (f32) or, with xh, the activation image of the tcgen05 GEMM */
+    int inner, state;
+} DlSelectiveArgs;
+int dl_selective_scan_supported(int state);
+int dl_selective_scan(const DlMambaBatch* batch /*host*/, int n_seq, const DlSelectiveArgs* args /*host*/, void* stream);
+
+/* ---- one step of a residual stream (norms.cu) ------------------------------------------------------------------------
+ *   x[m] = x_in + add1 + add2 + add3 + w_a * unit(norm_a) + w_b * unit(norm_b) + vec    unit(v) = v / sqrt(mean(v^2) + eps)
+ *   h1[m] = w1 * unit(x[m]),  h2[m] = w2 * unit(x[m])       each to f32 rows or into an activation image (xh1 / xh2)
+ * Every term may be absent (NULL); x NULL: the sum is not stored; rows: all terms but vec are those of row rows[m] (a gather). */
+typedef struct {
+    const float* x_in; long long ld_in; const int* rows;
+    const float* add1; const float* add2; const float* add3; long long ld_add1, ld_add2, ld_add3;
+    const float* norm_a; const float* w_a; const float* norm_b; const float* w_b; long long ld_a, ld_b;
+    const float* vec;
+    float* x; long long ldx;
+    const float* w1; float* h1; uint8_t* xh1;
+    const float* w2; float* h2; uint8_t* xh2;
+    long long ldh; int ncap;
+    int M, dim; float eps;
+} DlResidualArgs;
+int dl_residual_step(const DlResidualArgs* args /*host*/, void* stream);
+
 /* ---- sliding-window grouped-query attention whose values are its keys (window_attention.cu) -------------------------
  * Cache line per token and key/value head: [ rot(k)[0 : dim] | k[0 : rope_dims] ]; cache [page][kv_head][page_size][dim +
  * rope_dims].  Rotary: interleaved pairs, angle pos * freqs[i] (f64 [rope_dims / 2]), cos and sin times rope_scale. */
@@ -515,6 +598,9 @@ typedef struct {
      * queries: q_mixed[m][h][c * dim + i] = sum_{g in group c} talk[h][g] q[m][g][i] (after rotary and norm), a query of
      * kv_heads * dim numbers per head that meets the concatenated keys of all key/value heads (DlWindowAttnArgs.key_heads) */
     const float* talk; float* q_mixed; long long ld_qm;
+    /* root mean square over the WHOLE query / key projection of a row (all heads' columns at once), in front of the rotary:
+     * x * w / sqrt(mean(x^2) + eps), w [q_heads * dim] / [kv_heads * dim] f32; NULL: none */
+    const float* q_norm; const float* k_norm;
 } DlWindowKvArgs;
 int dl_window_kv_write(const DlWindowKvArgs* args /*host*/, int M, void* stream);
 /* out[m][h] = sum_j softmax_j(cap(scale q[m][h] . key_j)) value_j over the positions j with 0 <= pos[m] - j < window
@@ -534,6 +620,9 @@ typedef struct {
     int key_heads;                            /* 0 / 1: a head's key is its key/value head's; kv_heads: q is [M][heads][kv_heads * dim] and
                                                  meets the keys of ALL key/value heads side by side (head-mixed scores, see DlWindowKvArgs.talk);
                                                  the values stay those of the head's own key/value head */
+    int value_heads;                          /* 0 / 1: a head's values are its key/value head's; kv_heads: every head's weights meet the
+                                                 values of ALL key/value heads, out [M][heads][kv_heads * vdim] (weights mixed across heads
+                                                 after the softmax, see dl_talk_mix).  Not together with key_heads */
 } DlWindowAttnArgs;
 int dl_window_attention(const DlWindowAttnArgs* args /*host*/, int M, void* stream);
 
@@ -591,12 +680,17 @@ int dl_window_attention_tc_supported(int heads, int kv_heads, int dim, int rope_
 long long dl_window_tc_partial_floats(int n_tiles, int kv_heads, int n_splits, int dim);
 int dl_window_attention_tc(const DlWindowAttnArgs* args /*host*/, const int* tile_rows, int n_tiles, int rq, int n_splits,
                            float* partial, void* stream);
+/* Attention weights mixed across heads AFTER the softmax: with wide[m][g][c * vdim + i] = sum_j p_g(j) v_c,j[i] (every head's
+ * weights against the values of all key/value heads), out[m][h * vdim + i] = sum_g talk[h][g] wide[m][g][c(h) * vdim + i],
+ * c(h) = h / (heads / kv_heads).  To out (f32) or, with xh, into the tcgen05 GEMM's activation image. */
+int dl_talk_mix(const float* wide, const float* talk, int M, int heads, int kv_heads, int vdim, float* out, long long ld_out,
+                uint8_t* xh, int ncap, void* stream);
 /* The tile kernel for values of a width of their own (vdim > 0, any multiple of 8 up to 128; rope_dims 0, no soft cap) and
  * for head-mixed scores (key_heads = kv_heads: q [M][heads][kv_heads * dim], talk_attention.cu).  Tiles as above. */
-int dl_talk_attention_tc_supported(int heads, int kv_heads, int dim, int vdim, int key_heads, int ctype);
+int dl_talk_attention_tc_supported(int heads, int kv_heads, int dim, int vdim, int key_heads, int value_heads, int ctype);
 /* stacked (row x head-of-a-group) rows per tile for portions of `longest` rows: 16 (decoding), 64 or 128; rq = that / (heads / kv_heads) */
-int dl_talk_tc_tile_rows(int heads, int kv_heads, int dim, int vdim, int key_heads, int longest);
-long long dl_talk_tc_partial_floats(int n_tiles, int kv_heads, int n_splits, int vdim, int tile_rows);
+int dl_talk_tc_tile_rows(int heads, int kv_heads, int dim, int vdim, int key_heads, int value_heads, int longest);
+long long dl_talk_tc_partial_floats(int n_tiles, int kv_heads, int n_splits, int vdim, int value_heads, int tile_rows);
 int dl_talk_attention_tc(const DlWindowAttnArgs* args /*host*/, const int* tile_rows, int n_tiles, int rq, int n_splits,
                          float* partial, void* stream);
 
