@@ -4,6 +4,7 @@
 // (rope / shift / silu / mul / cast / merge-add) exist on the hot path.
 #pragma once
 #include "common.cuh"
+#include <cuda_bf16.h>
 #include "../../../include/dllama_b200.h"
 
 // ---- Q80 block writers -------------------------------------------------------------------------
@@ -183,6 +184,7 @@ DL_DEVINL void epilogue_rows(const DlEpilogue& e, const float* out_s, int out_ld
                 const size_t ld = (size_t)e.ld;
                 float* d0 = e.dst[0] + (size_t)e.dst_off + (size_t)m0 * ld + col;
                 const float lim = e.dense_param;
+                uint8_t* xh = e.dense_xh;                              // the next product's bf16 activation image instead of f32 rows
                 const bool silu = e.dense_op == DL_DENSE_GLU_SILU;      // silu(gate) * up, no clamps
                 const bool gelu = e.dense_op == DL_DENSE_GLU_GELU;      // gelu_tanh(gate) * up
 #pragma unroll 4
@@ -190,7 +192,14 @@ DL_DEVINL void epilogue_rows(const DlEpilogue& e, const float* out_s, int out_ld
                     const float2 gu = *reinterpret_cast<const float2*>(out_s + m * out_ld + 2 * tid);
                     float g = gu.x, u = gu.y;
                     if (silu) { d0[m * ld] = g / (1.0f + expf(-g)) * u; continue; }
-                    if (gelu) { d0[m * ld] = act_gelu(g) * u; continue; }
+                    if (gelu) {
+                        const float v = act_gelu(g) * u;
+                        if (xh != nullptr)      // element (row, col) of the slabs [K tile of 128][8 rows][8 columns]
+                            *reinterpret_cast<__nv_bfloat16*>(xh + ((size_t)(col >> 7) * (e.dense_ncap >> 3) + ((m0 + m) >> 3)) * 2048 +
+                                                              ((col & 127) >> 3) * 128 + ((m0 + m) & 7) * 16 + (col & 7) * 2) = __float2bfloat16_rn(v);
+                        else d0[m * ld] = v;
+                        continue;
+                    }
                     if (lim > 0.0f) { g = fminf(g, lim); u = fminf(fmaxf(u, -lim), lim); }
                     d0[m * ld] = g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
                 }

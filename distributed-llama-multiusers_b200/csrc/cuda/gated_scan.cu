@@ -605,109 +605,155 @@ extern "C" int dl_gated_scan_chunked(const DlMambaBatch* batch, int n_seq, int m
 }
 
 // ------------------------------------------------------------------------------------------------
-// gates of the matrix memory: one warp per (sequence, head).  A token maps the running maximum u to max(b + u, a); such maps
-// compose (F, A) o (F', A') = (F + F', max(F' + A, A')), so 32 tokens are scanned by shuffles; four blocks of 32 tokens are
-// loaded together.
+// gates of the matrix memory: one CTA per (sequence, head).  A token maps the running maximum u to max(b + u, a); such maps
+// compose, (F, A) after (F', A') = (F + F', max(F + A', A)), so tokens are scanned in parallel: 32 by shuffles, four such
+// blocks per warp, the warps' totals through shared memory (8 warps for long portions, one for short ones).
 // ------------------------------------------------------------------------------------------------
-__global__ void __launch_bounds__(32) mlstm_gates_kernel(DlMambaBatch b, DlMlstmGatesArgs a) {
-    const int n = blockIdx.x, h = blockIdx.y, lane = threadIdx.x, H = a.n_heads;
+__global__ void __launch_bounds__(256) mlstm_gates_kernel(DlMambaBatch b, DlMlstmGatesArgs a) {
+    __shared__ float wF[8], wA[8];
+    const int n = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, H = a.n_heads;
     float* ug = a.u_state + (size_t)b.seq_slot[n] * H + h;
     float u = b.seq_pos0[n] == 0 ? 0.f : *ug;
     const float bi = a.bi[h], bf = a.bf[h], cap = a.cap;
     const int r0 = b.seq_start[n], r1 = b.seq_start[n + 1];
-    for (int rb = r0; rb < r1; rb += 128) {
+    for (int rb = r0; rb < r1; rb += nw * 128) {
+        const int w0 = rb + warp * 128;
         int row[4];
-        float zi[4], zf[4];
+        float lb[4], ai[4], F[4], A[4];
 #pragma unroll
-        for (int k = 0; k < 4; ++k) { const int r = rb + k * 32 + lane; row[k] = r < r1 ? b.seq_rows[r] : -1; }
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-            zi[k] = row[k] >= 0 ? a.zi[(size_t)row[k] * a.ld + h] : 0.f;
-            zf[k] = row[k] >= 0 ? a.zf[(size_t)row[k] * a.ld + h] : 0.f;
-        }
+        for (int k = 0; k < 4; ++k) { const int r = w0 + k * 32 + lane; row[k] = r < r1 ? b.seq_rows[r] : -1; }
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
-            if (rb + k * 32 >= r1) break;
-            const bool live = row[k] >= 0;
-            const float ai = cap * tanhf((zi[k] + bi) / cap);
-            const float lb = -softplus_f(-cap * tanhf((zf[k] + bf) / cap));
-            float F = live ? lb : 0.f, A = live ? ai : -INFINITY;      // a lane without a token: the identity
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float Fp = __shfl_up_sync(0xffffffffu, F, o), Ap = __shfl_up_sync(0xffffffffu, A, o);
-                if (lane >= o) { A = fmaxf(F + Ap, A); F += Fp; }
-            }
-            const float un = fmaxf(F + u, A);
-            float up = __shfl_up_sync(0xffffffffu, un, 1);
-            if (lane == 0) up = u;
-            if (live) {
-                const size_t at = (size_t)row[k] * H + h;
-                a.log_keep[at] = lb + up - un;
-                a.put[at] = expf(ai - un);
-                a.floor_[at] = expf(-un);
-            }
-            u = __shfl_sync(0xffffffffu, un, 31);
+            ai[k] = row[k] >= 0 ? a.zi[(size_t)row[k] * a.ld + h] : 0.f;
+            lb[k] = row[k] >= 0 ? a.zf[(size_t)row[k] * a.ld + h] : 0.f;
         }
+        float pF = 0.f, pA = -INFINITY;                       // this warp's tokens so far, composed
+        float tF[4], tA[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            tF[k] = pF; tA[k] = pA;
+            F[k] = 0.f; A[k] = -INFINITY;                     // a lane without a token: the identity
+            if (w0 + k * 32 < r1) {
+                ai[k] = cap * tanhf((ai[k] + bi) / cap);
+                lb[k] = -softplus_f(-cap * tanhf((lb[k] + bf) / cap));
+                if (row[k] >= 0) { F[k] = lb[k]; A[k] = ai[k]; }
+#pragma unroll
+                for (int o = 1; o < 32; o <<= 1) {
+                    const float Fp = __shfl_up_sync(0xffffffffu, F[k], o), Ap = __shfl_up_sync(0xffffffffu, A[k], o);
+                    if (lane >= o) { A[k] = fmaxf(F[k] + Ap, A[k]); F[k] += Fp; }
+                }
+                const float bF = __shfl_sync(0xffffffffu, F[k], 31), bA = __shfl_sync(0xffffffffu, A[k], 31);
+                pA = fmaxf(bF + pA, bA);
+                pF += bF;
+            }
+        }
+        __syncthreads();                                      // the last round's totals have been read
+        if (lane == 0) { wF[warp] = pF; wA[warp] = pA; }
+        __syncthreads();
+        float uw = u;                                         // u ahead of this warp's tokens, then behind the last warp's
+        for (int w = 0; w < nw; ++w) {
+            if (w == warp) {
+                float ub = uw;
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const float us = fmaxf(tF[k] + ub, tA[k]);                        // ahead of block k
+                    const float un = fmaxf(F[k] + us, A[k]);
+                    float up = __shfl_up_sync(0xffffffffu, un, 1);
+                    if (lane == 0) up = us;
+                    if (row[k] >= 0) {
+                        const size_t at = (size_t)row[k] * H + h;
+                        a.log_keep[at] = lb[k] + up - un;
+                        a.put[at] = expf(ai[k] - un);
+                        a.floor_[at] = expf(-un);
+                    }
+                }
+            }
+            uw = fmaxf(wF[w] + uw, wA[w]);
+        }
+        u = uw;
     }
-    if (lane == 0) *ug = u;
+    if (threadIdx.x == 0) *ug = u;
 }
 
-extern "C" int dl_mlstm_gates(const DlMambaBatch* batch, int n_seq, const DlMlstmGatesArgs* args, void* stream) {
+extern "C" int dl_mlstm_gates(const DlMambaBatch* batch, int n_seq, int longest, const DlMlstmGatesArgs* args, void* stream) {
     if (args->n_heads < 1 || !(args->cap > 0.f)) { dl_set_error("dl_mlstm_gates: bad shape"); return -1; }
     if (n_seq < 1) return 0;
-    mlstm_gates_kernel<<<dim3(n_seq, args->n_heads), 32, 0, (cudaStream_t)stream>>>(*batch, *args);
+    mlstm_gates_kernel<<<dim3(n_seq, args->n_heads), longest > 128 ? 256 : 32, 0, (cudaStream_t)stream>>>(*batch, *args);
     LAYER_CHECK_LAUNCH("dl_mlstm_gates");
     return 0;
 }
 
 // ------------------------------------------------------------------------------------------------
-// normalised heads: one warp per (row, head), up to 512 columns kept in registers between the sum and the scaling
+// normalised heads: one warp per (row, head); four columns per lane and step (sizes and rows that allow it), up to 512 columns
+// kept in registers between the sum and the scaling
 // ------------------------------------------------------------------------------------------------
 #define HN_WARPS 8
-#define HN_CACHE 16
+#define HN_CACHE 4                 // groups of four columns per lane
+template <bool VEC>
 __global__ void __launch_bounds__(HN_WARPS * 32) head_norm_kernel(DlHeadNormArgs a) {
     const int m = blockIdx.x, lane = threadIdx.x & 31, V = a.vdim;
     const int h = blockIdx.y * HN_WARPS + (threadIdx.x >> 5);
     if (a.xh && blockIdx.y == 0) xh_zero_tail(a.xh, a.ncap, m, a.n_heads * V, threadIdx.x, HN_WARPS * 32);
     if (h >= a.n_heads) return;
     const float* y = a.y + (size_t)m * a.ld_y + (size_t)h * V;
+    const float* w = a.w + (a.w_full ? (size_t)h * V : 0);
+    const float* g = a.gate ? a.gate + (size_t)m * a.ld_gate + (size_t)h * V : nullptr;
     float scale = 1.f;
     if (a.den) scale = 1.f / (fmaxf(fabsf(a.den[(size_t)m * a.n_heads + h]), a.floor_[(size_t)m * a.n_heads + h]) + 1e-6f);
-    const bool cached = V <= 32 * HN_CACHE;
-    float v[HN_CACHE];
-    float ss = 0.f;
-    if (cached) {
+    if (VEC) {
+        const int n4 = V >> 2;
+        float4 v[HN_CACHE], gv[HN_CACHE];
+        float ss = 0.f;
 #pragma unroll
         for (int k = 0; k < HN_CACHE; ++k) {
             const int i = lane + 32 * k;
-            v[k] = i < V ? y[i] * scale : 0.f;
-            ss = fmaf(v[k], v[k], ss);
+            v[k] = gv[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < n4) {
+                v[k] = reinterpret_cast<const float4*>(y)[i];
+                if (g) gv[k] = reinterpret_cast<const float4*>(g)[i];
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < HN_CACHE; ++k) {
+            v[k] = make_float4(v[k].x * scale, v[k].y * scale, v[k].z * scale, v[k].w * scale);
+            ss = dot4(v[k], v[k], ss);
+        }
+        const float inv = 1.f / sqrtf(warp_sum(ss) / (float)V + a.eps);
+#pragma unroll
+        for (int k = 0; k < HN_CACHE; ++k) {
+            const int i = lane + 32 * k;
+            if (i >= n4) continue;
+            const float4 wv = reinterpret_cast<const float4*>(w)[i];
+            float4 t = make_float4(v[k].x * inv * wv.x, v[k].y * inv * wv.y, v[k].z * inv * wv.z, v[k].w * inv * wv.w);
+            if (g) { t.x *= sigmoid_f(gv[k].x); t.y *= sigmoid_f(gv[k].y); t.z *= sigmoid_f(gv[k].z); t.w *= sigmoid_f(gv[k].w); }
+            if (a.xh) {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(t.x, t.y), hi = __floats2bfloat162_rn(t.z, t.w);
+                *reinterpret_cast<uint2*>(a.xh + xh_offset(a.ncap, m, h * V + i * 4)) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+            } else {
+                reinterpret_cast<float4*>(a.out + (size_t)m * a.ld_out + (size_t)h * V)[i] = t;
+            }
         }
     } else {
+        float ss = 0.f;
         for (int i = lane; i < V; i += 32) { const float t = y[i] * scale; ss = fmaf(t, t, ss); }
-    }
-    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)V + a.eps);
-    const float* w = a.w + (a.w_full ? (size_t)h * V : 0);
-    const float* g = a.gate ? a.gate + (size_t)m * a.ld_gate + (size_t)h * V : nullptr;
-    auto put = [&](int i, float t) {
-        t = t * inv * w[i];
-        if (g) t *= sigmoid_f(g[i]);
-        if (a.xh) xh_store(a.xh, a.ncap, m, h * V + i, t);
-        else a.out[(size_t)m * a.ld_out + (size_t)h * V + i] = t;
-    };
-    if (cached) {
-#pragma unroll
-        for (int k = 0; k < HN_CACHE; ++k)
-            if (lane + 32 * k < V) put(lane + 32 * k, v[k]);
-    } else {
-        for (int i = lane; i < V; i += 32) put(i, y[i] * scale);
+        const float inv = 1.f / sqrtf(warp_sum(ss) / (float)V + a.eps);
+        for (int i = lane; i < V; i += 32) {
+            float t = y[i] * scale * inv * w[i];
+            if (g) t *= sigmoid_f(g[i]);
+            if (a.xh) xh_store(a.xh, a.ncap, m, h * V + i, t);
+            else a.out[(size_t)m * a.ld_out + (size_t)h * V + i] = t;
+        }
     }
 }
 
 extern "C" int dl_head_norm(const DlHeadNormArgs* args, void* stream) {
     const DlHeadNormArgs& a = *args;
     if (a.M < 1 || a.n_heads < 1 || a.vdim < 1 || !a.w || (!a.out && !a.xh) || (a.den && !a.floor_)) { dl_set_error("dl_head_norm: bad arguments"); return -1; }
-    head_norm_kernel<<<dim3(a.M, (a.n_heads + HN_WARPS - 1) / HN_WARPS), HN_WARPS * 32, 0, (cudaStream_t)stream>>>(a);
+    const auto al = [](const void* p, long long ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
+    const bool vec = a.vdim % 4 == 0 && a.vdim <= 128 * HN_CACHE && al(a.y, a.ld_y) && al(a.w, 0) && al(a.gate, a.ld_gate) && al(a.out, a.ld_out);
+    const dim3 grid(a.M, (a.n_heads + HN_WARPS - 1) / HN_WARPS);
+    if (vec) head_norm_kernel<true><<<grid, HN_WARPS * 32, 0, (cudaStream_t)stream>>>(a);
+    else head_norm_kernel<false><<<grid, HN_WARPS * 32, 0, (cudaStream_t)stream>>>(a);
     LAYER_CHECK_LAUNCH("dl_head_norm");
     return 0;
 }

@@ -159,6 +159,7 @@ __global__ void __launch_bounds__(RS_THREADS) residual_step_kernel(DlResidualArg
         inv_a = 1.f / sqrtf(block_sum(sa, red) / (float)dim + a.eps);
         if (pb) inv_b = 1.f / sqrtf(block_sum(sb, red) / (float)dim + a.eps);
     }
+    const __nv_bfloat16* tb = a.table ? (const __nv_bfloat16*)a.table + src * a.ld_in : nullptr;
     const float* p1 = a.add1 ? a.add1 + src * a.ld_add1 : nullptr;
     const float* p2 = a.add2 ? a.add2 + src * a.ld_add2 : nullptr;
     const float* p3 = a.add3 ? a.add3 + src * a.ld_add3 : nullptr;
@@ -174,6 +175,7 @@ __global__ void __launch_bounds__(RS_THREADS) residual_step_kernel(DlResidualArg
         if (p2) t += p2[i];
         if (p3) t += p3[i];
         if (xi) t += xi[i];
+        if (tb) t += __bfloat162float(tb[i]);
         if (a.vec) t += a.vec[i];
         row_s[i] = t;
         if (a.x) a.x[(size_t)m * a.ldx + i] = t;
@@ -195,12 +197,123 @@ __global__ void __launch_bounds__(RS_THREADS) residual_step_kernel(DlResidualArg
     if (a.xh2) xh_zero_tail(a.xh2, a.ncap, m, dim, tid, RS_THREADS);
 }
 
+// the same with four columns per thread and step (dim % 4 == 0, aligned rows): every term of the row is loaded at once and stays in
+// registers, so a decoded row costs one round of loads and two block sums
+__device__ __forceinline__ float4 rs_add(float4 x, float4 y) { return make_float4(x.x + y.x, x.y + y.y, x.z + y.z, x.w + y.w); }
+__device__ __forceinline__ float rs_sq(float4 x, float acc) { return fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, acc)))); }
+__device__ __forceinline__ void rs_put(float* h, uint8_t* xh, int ncap, int m, long long ld, int i, float4 v) {
+    if (xh) {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+        *reinterpret_cast<uint2*>(xh + xh_offset(ncap, m, i * 4)) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+    } else {
+        reinterpret_cast<float4*>(h + (size_t)m * ld)[i] = v;
+    }
+}
+
+template <int NG>
+__global__ void __launch_bounds__(RS_THREADS) residual_step_vec_kernel(DlResidualArgs a) {
+    __shared__ float red[2 * (RS_THREADS / 32)];
+    const int m = blockIdx.x, dim = a.dim, n4 = dim >> 2, tid = threadIdx.x;
+    const size_t src = a.rows ? a.rows[m] : m;
+    float4 t[NG], u[NG], v[NG];
+    float sa = 0.f, sb = 0.f;
+#pragma unroll
+    for (int k = 0; k < NG; ++k) {
+        const int i = tid + k * RS_THREADS;
+        t[k] = u[k] = v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < n4) {
+            if (a.norm_a) u[k] = reinterpret_cast<const float4*>(a.norm_a + src * a.ld_a)[i];
+            if (a.norm_b) v[k] = reinterpret_cast<const float4*>(a.norm_b + src * a.ld_b)[i];
+            if (a.add1) t[k] = reinterpret_cast<const float4*>(a.add1 + src * a.ld_add1)[i];
+            if (a.add2) t[k] = rs_add(t[k], reinterpret_cast<const float4*>(a.add2 + src * a.ld_add2)[i]);
+            if (a.x_in) t[k] = rs_add(t[k], reinterpret_cast<const float4*>(a.x_in + src * a.ld_in)[i]);
+            if (a.table) {
+                const uint2 w = reinterpret_cast<const uint2*>((const __nv_bfloat16*)a.table + src * a.ld_in)[i];
+                t[k] = rs_add(t[k], make_float4(__uint_as_float(w.x << 16), __uint_as_float(w.x & 0xffff0000u), __uint_as_float(w.y << 16), __uint_as_float(w.y & 0xffff0000u)));
+            }
+            if (a.add3) t[k] = rs_add(t[k], reinterpret_cast<const float4*>(a.add3 + src * a.ld_add3)[i]);
+            if (a.vec) t[k] = rs_add(t[k], reinterpret_cast<const float4*>(a.vec)[i]);
+        }
+        sa = rs_sq(u[k], sa);
+        sb = rs_sq(v[k], sb);
+    }
+    const int warp = tid >> 5, lane = tid & 31;
+    if (a.norm_a) {
+        sa = warp_sum(sa);
+        sb = warp_sum(sb);
+        if (lane == 0) { red[warp] = sa; red[RS_THREADS / 32 + warp] = sb; }
+        __syncthreads();
+        sa = sb = 0.f;
+#pragma unroll
+        for (int w = 0; w < RS_THREADS / 32; ++w) { sa += red[w]; sb += red[RS_THREADS / 32 + w]; }
+        const float ia = 1.f / sqrtf(sa / (float)dim + a.eps), ib = 1.f / sqrtf(sb / (float)dim + a.eps);
+#pragma unroll
+        for (int k = 0; k < NG; ++k) {
+            const int i = tid + k * RS_THREADS;
+            if (i < n4) {
+                const float4 wa = reinterpret_cast<const float4*>(a.w_a)[i];
+                float4 n = make_float4(wa.x * (u[k].x * ia), wa.y * (u[k].y * ia), wa.z * (u[k].z * ia), wa.w * (u[k].w * ia));
+                if (a.norm_b) {
+                    const float4 wb = reinterpret_cast<const float4*>(a.w_b)[i];
+                    n = make_float4(fmaf(wb.x, v[k].x * ib, n.x), fmaf(wb.y, v[k].y * ib, n.y), fmaf(wb.z, v[k].z * ib, n.z), fmaf(wb.w, v[k].w * ib, n.w));
+                }
+                t[k] = rs_add(n, t[k]);
+            }
+        }
+        __syncthreads();
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NG; ++k) {
+        const int i = tid + k * RS_THREADS;
+        if (a.x && i < n4) reinterpret_cast<float4*>(a.x + (size_t)m * a.ldx)[i] = t[k];
+        ss = rs_sq(t[k], ss);
+    }
+    if (!a.w1) return;
+    ss = warp_sum(ss);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int w = 0; w < RS_THREADS / 32; ++w) ss += red[w];
+    const float inv = 1.f / sqrtf(ss / (float)dim + a.eps);
+#pragma unroll
+    for (int k = 0; k < NG; ++k) {
+        const int i = tid + k * RS_THREADS;
+        if (i < n4) {
+            const float4 w = reinterpret_cast<const float4*>(a.w1)[i];
+            const float4 n = make_float4(t[k].x * inv, t[k].y * inv, t[k].z * inv, t[k].w * inv);
+            rs_put(a.h1, a.xh1, a.ncap, m, a.ldh, i, make_float4(n.x * w.x, n.y * w.y, n.z * w.z, n.w * w.w));
+            if (a.w2) {
+                const float4 w2 = reinterpret_cast<const float4*>(a.w2)[i];
+                rs_put(a.h2, a.xh2, a.ncap, m, a.ldh, i, make_float4(n.x * w2.x, n.y * w2.y, n.z * w2.z, n.w * w2.w));
+            }
+        }
+    }
+    if (a.xh1) xh_zero_tail(a.xh1, a.ncap, m, dim, tid, RS_THREADS);
+    if (a.xh2) xh_zero_tail(a.xh2, a.ncap, m, dim, tid, RS_THREADS);
+}
+
 extern "C" int dl_residual_step(const DlResidualArgs* args, void* stream) {
     const DlResidualArgs& a = *args;
     if (a.M < 1 || a.dim < 1) { dl_set_error("dl_residual_step: bad shape"); return -1; }
     if ((a.norm_b && !a.norm_a) || (a.norm_a && !a.w_a) || (a.norm_b && !a.w_b) || (a.w2 && !a.w1) || (a.w1 && !a.h1 && !a.xh1) || (a.w2 && !a.h2 && !a.xh2)) {
         dl_set_error("dl_residual_step: terms do not fit together");
         return -1;
+    }
+    if (a.x_in && a.table) { dl_set_error("dl_residual_step: x_in and table"); return -1; }
+    const auto al = [](const void* p, long long ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
+    const bool vec = a.dim % 4 == 0 && a.dim <= 4 * RS_THREADS * 8 && al(a.x_in, a.ld_in) && al(a.table, a.ld_in) && al(a.add1, a.ld_add1) && al(a.add2, a.ld_add2) &&
+                     al(a.add3, a.ld_add3) && al(a.norm_a, a.ld_a) && al(a.norm_b, a.ld_b) && al(a.w_a, 0) && al(a.w_b, 0) && al(a.vec, 0) && al(a.x, a.ldx) &&
+                     al(a.w1, 0) && al(a.w2, 0) && al(a.h1, a.ldh) && al(a.h2, a.ldh);
+    if (vec) {
+        cudaStream_t st = (cudaStream_t)stream;
+        if (a.dim <= 4 * RS_THREADS) residual_step_vec_kernel<1><<<a.M, RS_THREADS, 0, st>>>(a);
+        else if (a.dim <= 8 * RS_THREADS) residual_step_vec_kernel<2><<<a.M, RS_THREADS, 0, st>>>(a);
+        else if (a.dim <= 16 * RS_THREADS) residual_step_vec_kernel<4><<<a.M, RS_THREADS, 0, st>>>(a);
+        else residual_step_vec_kernel<8><<<a.M, RS_THREADS, 0, st>>>(a);
+        LAYER_CHECK_LAUNCH("dl_residual_step");
+        return 0;
     }
     const size_t smem = (size_t)a.dim * (1 + (a.norm_a ? 1 : 0) + (a.norm_b ? 1 : 0)) * sizeof(float);
     if (smem > 200 * 1024) { dl_set_error("dl_residual_step: rows of %d do not fit shared memory", a.dim); return -1; }

@@ -31,6 +31,7 @@
 #define TA_PAGE 32
 #define TA_MAX_ROWS 128
 #define TA_MAX_SPLITS 32
+#define TA_MERGE 256            // outputs per CTA of the merge
 #define TA_LOG2E 1.4426950408889634f
 #define TA_LN2 0.6931471805599453f
 
@@ -269,7 +270,7 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
     }
 }
 
-// merge of the page shares: one CTA per (tile, key/value head, position of the tile).  The shares' maxima and sums are
+// merge of the page shares: one CTA per (tile, key/value head, position of the tile) and 256 (head, column) outputs.  The shares' maxima and sums are
 // gathered into shared memory, every (head, share) weight e^(m_k - m) / l is formed once, then a thread per (head,
 // column) sums the shares.
 __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, const int* __restrict__ tile_rows, int rq, int n_splits,
@@ -277,10 +278,11 @@ __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, con
     __shared__ float w_s[64 * TA_MAX_SPLITS], l_s[64 * TA_MAX_SPLITS];      // heads of one group x shares
     const bool wide = a.value_heads > 1;                      // blockIdx.y: (key/value head of the scores, block of vs value heads)
     const int nvb = wide ? (a.kv_heads + vs - 1) / vs : 1, DVH = wide ? DVP / vs : DVP;
-    const int tile = blockIdx.x, g = blockIdx.y / nvb, v0 = ((int)blockIdx.y - g * nvb) * vs, r = blockIdx.z, DV = a.vdim, rep = a.heads / a.kv_heads;
+    const int gv = blockIdx.y % (a.kv_heads * nvb), part = blockIdx.y / (a.kv_heads * nvb);
+    const int tile = blockIdx.x, g = gv / nvb, v0 = (gv - g * nvb) * vs, r = blockIdx.z, DV = a.vdim, rep = a.heads / a.kv_heads;
     const int m = tile_rows[(size_t)tile * rq + r];
     if (m < 0) return;
-    const float* base = partial + ((size_t)tile * a.kv_heads * nvb + blockIdx.y) * n_splits * TA_ROWS * (DVP + 2);
+    const float* base = partial + ((size_t)tile * a.kv_heads * nvb + gv) * n_splits * TA_ROWS * (DVP + 2);
     for (int idx = threadIdx.x; idx < rep * n_splits; idx += blockDim.x) {
         const int hg = idx / n_splits, k = idx - hg * n_splits;
         const float* p = base + ((size_t)k * TA_ROWS + r * rep + hg) * (DVP + 2);
@@ -303,7 +305,7 @@ __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, con
     }
     __syncthreads();
     const int nv = wide ? min(vs, a.kv_heads - v0) : 1, W = nv * DV;
-    for (int idx = threadIdx.x; idx < rep * W; idx += blockDim.x) {
+    for (int idx = part * TA_MERGE + threadIdx.x; idx < min(rep * W, (part + 1) * TA_MERGE); idx += blockDim.x) {
         const int hg = idx / W, c = idx - hg * W, vh = c / DV;
         const float* p = base + (size_t)(r * rep + hg) * (DVP + 2) + vh * DVH + (c - vh * DV);
         float acc = 0.f;                      // a share without pages left zeros and weighs 0: every load can go out at once
@@ -343,12 +345,64 @@ __global__ void __launch_bounds__(128) talk_mix_kernel(const float* __restrict__
         }
 }
 
+// the same with four columns per lane (vdim % 4 == 0): a CTA takes TM_ROWS rows of one key/value head c, a warp a row at a time; talk's
+// rows of group c sit transposed in shared memory, REP of them per load
+#define TM_ROWS 8
+template <int REP>
+__global__ void __launch_bounds__(128) talk_mix_vec_kernel(const float* __restrict__ wide, const float* __restrict__ talk, int M, int heads, int kv_heads,
+                                                           int vdim, float* __restrict__ out, long long ld_out, uint8_t* __restrict__ xh, int ncap) {
+    extern __shared__ __align__(16) float talk_s[];           // [heads][rep rounded up to REP]
+    const int c = blockIdx.y, rep = heads / kv_heads, RP = (rep + REP - 1) / REP * REP, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int i = threadIdx.x; i < heads * RP; i += blockDim.x) {
+        const int g = i / RP, r = i - g * RP;
+        talk_s[i] = r < rep ? talk[(size_t)(c * rep + r) * heads + g] : 0.f;
+    }
+    __syncthreads();
+    const size_t gs = (size_t)kv_heads * vdim;
+    for (int m = blockIdx.x * TM_ROWS + warp; m < min(M, (blockIdx.x + 1) * TM_ROWS); m += 4) {
+        if (xh && c == 0) xh_zero_tail(xh, ncap, m, heads * vdim, lane, 32);
+        const float* row = wide + (size_t)m * heads * gs + (size_t)c * vdim;
+        for (int i = lane * 4; i < vdim; i += 128)
+            for (int h0 = 0; h0 < rep; h0 += REP) {
+                float4 acc[REP];
+#pragma unroll
+                for (int r = 0; r < REP; ++r) acc[r] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+                for (int g = 0; g < heads; ++g) {
+                    const float4 v = *reinterpret_cast<const float4*>(row + (size_t)g * gs + i);
+#pragma unroll
+                    for (int r = 0; r < REP; ++r) {
+                        const float t = talk_s[g * RP + h0 + r];
+                        acc[r] = make_float4(fmaf(t, v.x, acc[r].x), fmaf(t, v.y, acc[r].y), fmaf(t, v.z, acc[r].z), fmaf(t, v.w, acc[r].w));
+                    }
+                }
+#pragma unroll
+                for (int r = 0; r < REP; ++r)
+                    if (h0 + r < rep) {
+                        const int k = (c * rep + h0 + r) * vdim + i;
+                        if (xh) *reinterpret_cast<uint2*>(xh + xh_offset(ncap, m, k)) = make_uint2(pack_bf16(acc[r].x, acc[r].y), pack_bf16(acc[r].z, acc[r].w));
+                        else *reinterpret_cast<float4*>(out + (size_t)m * ld_out + k) = acc[r];
+                    }
+            }
+    }
+}
+
 extern "C" int dl_talk_mix(const float* wide, const float* talk, int M, int heads, int kv_heads, int vdim, float* out, long long ld_out,
                            uint8_t* xh, int ncap, void* stream) {
     if (M < 1 || kv_heads < 1 || heads % kv_heads || vdim < 1 || (!out && !xh)) { dl_set_error("dl_talk_mix: bad shape"); return -1; }
     const dim3 grid(M, kv_heads);
     const int threads = vdim <= 32 ? 32 : vdim <= 64 ? 64 : 128, rep = heads / kv_heads;
     cudaStream_t st = (cudaStream_t)stream;
+    const size_t smem = (size_t)heads * (rep + 7) / 8 * 8 * sizeof(float) + 32 * heads;
+    if (vdim % 4 == 0 && ((uintptr_t)wide & 15) == 0 && (xh || (((uintptr_t)out & 15) == 0 && ld_out % 4 == 0)) && smem <= 48 * 1024) {
+        const dim3 gv((M + TM_ROWS - 1) / TM_ROWS, kv_heads);
+        if (rep <= 1) talk_mix_vec_kernel<1><<<gv, 128, smem, st>>>(wide, talk, M, heads, kv_heads, vdim, out, ld_out, xh, ncap);
+        else if (rep <= 2) talk_mix_vec_kernel<2><<<gv, 128, smem, st>>>(wide, talk, M, heads, kv_heads, vdim, out, ld_out, xh, ncap);
+        else if (rep <= 4) talk_mix_vec_kernel<4><<<gv, 128, smem, st>>>(wide, talk, M, heads, kv_heads, vdim, out, ld_out, xh, ncap);
+        else talk_mix_vec_kernel<8><<<gv, 128, smem, st>>>(wide, talk, M, heads, kv_heads, vdim, out, ld_out, xh, ncap);
+        LAYER_CHECK_LAUNCH("dl_talk_mix");
+        return 0;
+    }
     if (rep <= 2) talk_mix_kernel<2><<<grid, threads, 0, st>>>(wide, talk, heads, kv_heads, vdim, out, ld_out, xh, ncap);
     else if (rep <= 4) talk_mix_kernel<4><<<grid, threads, 0, st>>>(wide, talk, heads, kv_heads, vdim, out, ld_out, xh, ncap);
     else talk_mix_kernel<8><<<grid, threads, 0, st>>>(wide, talk, heads, kv_heads, vdim, out, ld_out, xh, ncap);
@@ -462,9 +516,11 @@ extern "C" int dl_talk_attention_tc(const DlWindowAttnArgs* args, const int* til
     TA_CASE(8, 16, true) TA_CASE(8, 32, true)
 #undef TA_CASE
     if (rc != 0) return rc;
-    if (n_splits > 1)
-        talk_merge_kernel<<<dim3(n_tiles, a.kv_heads * ta_nvb(a.vdim, a.value_heads), rq), 128, 0, st>>>(
-            a, tile_rows, rq, n_splits, partial, 8 * nv, ta_rows_of(rq, a.heads / a.kv_heads), ta_vs(a.vdim, a.value_heads));
+    if (n_splits > 1) {
+        const int vs = ta_vs(a.vdim, a.value_heads), parts = (a.heads / a.kv_heads * vs * a.vdim + TA_MERGE - 1) / TA_MERGE;
+        talk_merge_kernel<<<dim3(n_tiles, a.kv_heads * ta_nvb(a.vdim, a.value_heads) * parts, rq), 128, 0, st>>>(
+            a, tile_rows, rq, n_splits, partial, 8 * nv, ta_rows_of(rq, a.heads / a.kv_heads), vs);
+    }
     LAYER_CHECK_LAUNCH("dl_talk_attention_tc");
     return 0;
 }

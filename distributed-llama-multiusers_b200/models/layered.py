@@ -224,7 +224,7 @@ class DenseWeight:
 TC_MIN_ROWS = int(os.environ.get("DLLAMA_LAYERS_TC_MIN_ROWS", "32"))
 CHUNKED_SCAN_MIN_ROWS = 256  # a batch holding this many rows of one sequence runs the recurrence chunk-parallel
 LIGHTNING_CHUNKED_MIN_ROWS = 128     # the same for linear attention (chunks of 64 rows)
-GATED_CHUNKED_MIN_ROWS = 128         # and for linear attention with data-dependent gates
+GATED_CHUNKED_MIN_ROWS = 128         # and for linear attention with data-dependent gates and selective scans per channel
 TC_HEADS_MIN_ROWS = 256      # per-head products (one small GEMM per head) take the tensor-core path from this many rows
 GRAPH_MAX_ROWS = 64          # batches up to this many rows are replayed from CUDA graphs
 WINDOW_MAX_SPLITS = 32       # most CTAs that share one tile's pages in the windowed-attention kernel
@@ -406,8 +406,11 @@ class DenseFeedForward:
         e, L = self.eng, self.eng.L
         up = e.buf("up", self.ff)
         if self.glu:
-            e.mm(self.w_up, h, up, M, epi=L.DENSE_GLU_GELU, src="h")
-        elif self.poly is not None:
+            image = e.image("tmp", M) if self.ff % 128 == 0 else None
+            e.mm(self.w_up, h, up, M, epi=L.DENSE_GLU_GELU, src="h", image=image)
+            e.mm(self.w_down, up, y, M, ready=image is not None)
+            return
+        if self.poly is not None:
             e.mm(self.w_up, h, up, M, src="h")
             L.poly_norm(up, up, M, self.ff, self.poly, e.cfg.norm_eps)
         elif self.xielu is not None:
@@ -699,7 +702,8 @@ class MLstmMixer:
         keep, put, floor, den = (e.buf("gates", 4 * H).view(-1)[i * e.max_rows * H:(i + 1) * e.max_rows * H] for i in range(4))     # [rows][heads] each
         e.mm(self.w_in, h, mx, M, src="h")
         k0, v0, g0, i0 = H * d, 2 * H * d, H * (2 * d + dv), H * (2 * d + 2 * dv)
-        L.mlstm_gates(e.mamba_batch, e.n_seq, mx[:, i0:], mx[:, i0 + H:], self.bi, self.bf, self.cap, self.u_state, keep, put, floor, H)
+        L.mlstm_gates(e.mamba_batch, e.n_seq, mx[:, i0:], mx[:, i0 + H:], self.bi, self.bf, self.cap, self.u_state, keep, put, floor, H,
+                      e.longest)
         L.gated_scan(e.mamba_batch, e.n_seq, mx, mx[:, v0:], ys, self.state, H, d, dv, q_scale=d ** -0.5, k=mx[:, k0:], log_keep=keep,
                      put=put, den=den, n_state=self.n_state, **e.gated_chunking(self))
         image = e.image("tmp", M)
@@ -775,15 +779,17 @@ class Mamba1Mixer:
                     tuple(w_dt.shape) != (self.inner, self.rank) or tuple(self.w_conv.shape) != (self.inner, self.taps):
                 raise ValueError(f"layer {index}: in, x, dt, conv have shapes {[tuple(t.shape) for t in (w_in, w_x, w_dt, self.w_conv)]}")
             self.w_in, self.w_x, self.w_dt, self.w_o = D(w_in), D(w_x), D(w_dt), D(W(prefix + "o"))
-            self.dt_bias, self.A_log, self.D = V(prefix + "dt.b"), V(prefix + "A_log"), V(prefix + "D")
-            if tuple(self.A_log.shape) != (self.inner, self.N):
-                raise ValueError(f"layer {index}: A_log has shape {tuple(self.A_log.shape)}")
+            A_log, self.dt_bias, self.D = V(prefix + "A_log"), V(prefix + "dt.b"), V(prefix + "D")
+            if tuple(A_log.shape) != (self.inner, self.N):
+                raise ValueError(f"layer {index}: A_log has shape {tuple(A_log.shape)}")
+            self.A2 = (-torch.exp(A_log.double()) / math.log(2.0)).float().contiguous()      # decays are formed in base 2
         else:
-            for n in ("w_in", "w_x", "w_dt", "w_o", "w_conv", "b_conv", "dt_bias", "A_log", "D"):
+            for n in ("w_in", "w_x", "w_dt", "w_o", "w_conv", "b_conv", "dt_bias", "A2", "D"):
                 setattr(self, n, getattr(share, n))
         f32 = dict(dtype=torch.float32, device=eng.device)
         self.state = torch.zeros(eng.n_slots, self.inner, self.N, **f32)
         self.conv_state = torch.zeros(eng.n_slots, max(1, self.taps - 1), self.inner, **f32)
+        self.chunked = eng.L.selective_chunked_supported(self.N)
 
     def scratch(self) -> Dict[str, int]:
         return {"zx": 2 * self.inner, "xbc": self.inner, "dbc": self.rank + 2 * self.N, "dtr": self.inner, "ys": self.inner}
@@ -805,8 +811,8 @@ class Mamba1Mixer:
         e.mm(self.w_x, xc, dbc, M)
         e.mm(self.w_dt, dbc, dtr, M)
         image = e.image("tmp", M)
-        L.selective_scan(e.mamba_batch, e.n_seq, xc, dtr, dbc[:, r:], dbc[:, r + N:], self.dt_bias, self.A_log, self.D, self.state, ys, I, N,
-                         z=zx[:, I:], image=image)
+        L.selective_scan(e.mamba_batch, e.n_seq, xc, dtr, dbc[:, r:], dbc[:, r + N:], self.dt_bias, self.A2, self.D, self.state, ys, I, N,
+                         e.longest, z=zx[:, I:], image=image, **e.selective_chunking(self))
         e.mm(self.w_o, ys, y, M, ready=image is not None)
 
 
@@ -1111,6 +1117,10 @@ class LayerListEngine:
         if gt and R >= GATED_CHUNKED_MIN_ROWS and os.environ.get("DLLAMA_LAYERS_CHUNKED_SCAN", "1") != "0":
             self._gated_scratch = torch.zeros(max(L.gated_chunk_floats(R, self.n_slots, mx.H, mx.dim, mx.vdim) for mx in gt),
                                               dtype=torch.float32, device=dev)
+        st = [mx for mx in mixers if isinstance(mx, Mamba1Mixer) and mx.chunked]
+        self.selective_chunks, self._selective_scratch, self._selective_slots = 0, None, R // L.SELECTIVE_CHUNK + self.n_slots
+        if st and R >= GATED_CHUNKED_MIN_ROWS and os.environ.get("DLLAMA_LAYERS_CHUNKED_SCAN", "1") != "0":
+            self._selective_scratch = torch.zeros(self._selective_slots * max(mx.inner * (mx.N + 1) for mx in st), dtype=torch.float32, device=dev)
         if self.cfg.residual in ("post", "parallel") and self.cfg.streams != 1:
             raise ValueError(f"the {self.cfg.residual} residual style keeps one residual stream")
         if (self.embed_norm is not None) != (self.cfg.residual == "parallel"):
@@ -1212,10 +1222,10 @@ class LayerListEngine:
         return DenseWeight(t, self.tc)
 
     def mm(self, w: DenseWeight, x: torch.Tensor, y: torch.Tensor, M: int, epi: int = 0, aux=None, param: float = 0.0,
-           src: str = "tmp", param2: float = 0.0, ready: bool = False):
+           src: str = "tmp", param2: float = 0.0, ready: bool = False, image=None):
         """y[:M] = epi(x[:M] @ w^T).  src="h": x is the current sublayer input; its tensor-core image is made by the
         first product that reads it (begin_sublayer() marks it stale) and shared by the others.  ready: the launch that
-        produced x left it as the image of `src` (see image())."""
+        produced x left it as the image of `src` (see image()).  image: the result leaves as that image instead of y."""
         L = self.L
         if w.wh is None or M < TC_MIN_ROWS:
             L.dense(w.t, x, y, M, self.round_x, epi=epi, aux=aux, param=param, param2=param2)
@@ -1224,7 +1234,7 @@ class LayerListEngine:
         if not ready and (src != "h" or not self._xh_h_ready):
             L.xh_from_rows(x, M, w.K, self.ncap, xh)
             self._xh_h_ready = src == "h" or self._xh_h_ready
-        L.dense_tc(w.wh, w.N, w.K, xh, self.ncap, y, M, epi=epi, aux=aux, param=param, param2=param2)
+        L.dense_tc(w.wh, w.N, w.K, xh, self.ncap, y, M, epi=epi, aux=aux, param=param, param2=param2, image=image)
 
     def mm_heads(self, w: DenseWeight, x: torch.Tensor, y: torch.Tensor, M: int, x_head_stride: int, y_head_stride: int):
         """Per head h: y[:M, h*ys : h*ys+N] = x[:M, h*xs : h*xs+K] @ w[h]^T."""
@@ -1253,6 +1263,12 @@ class LayerListEngine:
         if not mx.chunked or not self.gated_chunks:
             return {}
         return dict(max_chunks=self.gated_chunks, scratch=self._gated_scratch, chunk_slots=self._gated_slots)
+
+    def selective_chunking(self, mx) -> dict:
+        """The same for a selective scan."""
+        if not mx.chunked or not self.selective_chunks:
+            return {}
+        return dict(max_chunks=self.selective_chunks, scratch=self._selective_scratch, chunk_slots=self._selective_slots)
 
     def lightning_scratch(self, mx):
         return self._lightning_scratch
@@ -1369,6 +1385,9 @@ class LayerListEngine:
         self.gated_chunks = 0
         if self._gated_scratch is not None and longest >= GATED_CHUNKED_MIN_ROWS:
             self.gated_chunks = (longest + self.L.GATED_CHUNK - 1) // self.L.GATED_CHUNK
+        self.selective_chunks = 0
+        if self._selective_scratch is not None and longest >= GATED_CHUNKED_MIN_ROWS:
+            self.selective_chunks = (longest + self.L.SELECTIVE_CHUNK - 1) // self.L.SELECTIVE_CHUNK
         self._n_chunks = 0
         if self._chunk_scratch is not None and longest >= CHUNKED_SCAN_MIN_ROWS:
             co, nc, ch = self._chunks_off, 0, self.L.MAMBA_CHUNK
@@ -1393,8 +1412,9 @@ class LayerListEngine:
     def _launch_forward(self, M: int, n_logits: int):
         L, cfg, eps = self.L, self.cfg, self.cfg.norm_eps
         x, hn, y, W = self.x, self.hn, self.y, self.cfg.width
-        L.embed_rows(self.embed, self.tokens, x, M, cfg.embed_scale, cfg.streams)
         head_ready = False
+        if cfg.residual != "parallel":
+            L.embed_rows(self.embed, self.tokens, x, M, cfg.embed_scale, cfg.streams)
         if cfg.residual == "parallel":
             head_ready = self._launch_parallel_layers(M, n_logits)
         elif cfg.residual == "hyper":
@@ -1444,7 +1464,7 @@ class LayerListEngine:
         whether the last norm left the head's operand image."""
         L, cfg = self.L, self.cfg
         x, x0, W, eps = self.x, self.x0, cfg.width, cfg.norm_eps
-        L.rms_norm(x, x0, M, W, eps, w=self.embed_norm)                       # the embedding output
+        L.residual_step(M, W, eps, x_in=self.embed, rows=self.tokens, outs=[(self.embed_norm, x0)])        # the embedding output
         src, adds, normed = x0, [], []
         img1, img2 = self.image("h", M), self.image("h2", M)
         for l in self.layers:

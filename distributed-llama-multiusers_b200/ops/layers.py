@@ -104,11 +104,15 @@ def xh_from_rows(x: torch.Tensor, M: int, K: int, ncap: int, xh: torch.Tensor):
 
 
 def dense_tc(wh: torch.Tensor, N: int, K: int, xh: torch.Tensor, ncap: int, y: torch.Tensor, M: int, epi: int = DENSE_STORE,
-             aux: Optional[torch.Tensor] = None, param: float = 0.0, param2: float = 0.0):
-    """y[:M, :N] = epi(x @ w^T) from the two operand images (bf16 x bf16 -> f32 in tensor memory)."""
+             aux: Optional[torch.Tensor] = None, param: float = 0.0, param2: float = 0.0, image=None):
+    """y[:M, :N] = epi(x @ w^T) from the two operand images (bf16 x bf16 -> f32 in tensor memory); DENSE_GLU_GELU may leave the
+    result in image = (activation image, ncap) instead of y."""
     e = DlEpilogue()
     e.kind, e.n_dst, e.ld, e.dst_off = EPI_DENSE, 1, y.stride(0), 0
     e.dst[0] = y.data_ptr()
+    if image is not None:
+        assert epi == DENSE_GLU_GELU and N // 2 % 128 == 0 and image[0].data_ptr() != xh.data_ptr()
+        e.dense_xh, e.dense_ncap = image[0].data_ptr(), image[1]
     e.dense_op, e.dense_param, e.dense_param2 = epi, param, param2
     e.dense_aux, e.dense_aux_ld = _p(aux), (aux.stride(0) if aux is not None else 0)
     check_layers(layers_lib().dl_gemm_wh_tc(wh.data_ptr(), N, _round_up(K, 128), xh.data_ptr(), ncap, M, e, 2, 0, _stream()),
@@ -300,13 +304,14 @@ def gated_scan(batch: DlMambaBatch, n_seq: int, q: torch.Tensor, v: torch.Tensor
 
 
 def mlstm_gates(batch: DlMambaBatch, n_seq: int, zi: torch.Tensor, zf: torch.Tensor, bi: torch.Tensor, bf: torch.Tensor, cap: float,
-                u_state: torch.Tensor, log_keep: torch.Tensor, put: torch.Tensor, floor: torch.Tensor, n_heads: int):
-    """Log decays, input weights and e^-u of the matrix memory with a running maximum u (u_state [slots][heads])."""
+                u_state: torch.Tensor, log_keep: torch.Tensor, put: torch.Tensor, floor: torch.Tensor, n_heads: int, longest: int):
+    """Log decays, input weights and e^-u of the matrix memory with a running maximum u (u_state [slots][heads]); longest: rows of
+    the longest portion of the batch."""
     assert zi.stride(0) == zf.stride(0)
     a = DlMlstmGatesArgs()
     a.zi, a.zf, a.ld, a.bi, a.bf, a.cap = zi.data_ptr(), zf.data_ptr(), zi.stride(0), bi.data_ptr(), bf.data_ptr(), cap
     a.u_state, a.log_keep, a.put, a.floor_, a.n_heads = u_state.data_ptr(), log_keep.data_ptr(), put.data_ptr(), floor.data_ptr(), n_heads
-    check_layers(layers_lib().dl_mlstm_gates(batch, n_seq, a, _stream()), "dl_mlstm_gates")
+    check_layers(layers_lib().dl_mlstm_gates(batch, n_seq, longest, a, _stream()), "dl_mlstm_gates")
     lib.count_launch()
 
 
@@ -328,34 +333,51 @@ def head_norm(y: torch.Tensor, M: int, n_heads: int, vdim: int, eps: float, w: t
     lib.count_launch()
 
 
+SELECTIVE_CHUNK = 64         # DL_SELECTIVE_CHUNK: rows of a sequence per chunk of the chunked selective scan
+
+
 def selective_supported(state: int) -> bool:
     return layers_lib().dl_selective_scan_supported(state) == 0
 
 
+def selective_chunked_supported(state: int) -> bool:
+    return layers_lib().dl_selective_scan_chunked_supported(state) == 0
+
+
 def selective_scan(batch: DlMambaBatch, n_seq: int, x: torch.Tensor, dt: torch.Tensor, B: torch.Tensor, C: torch.Tensor,
-                   dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor, state_pool: torch.Tensor, y: Optional[torch.Tensor],
-                   inner: int, state: int, z: Optional[torch.Tensor] = None, image=None):
-    """Selective scan with a state per channel; dt raw (bias and softplus inside); out y (f32) or image = (activation image, ncap)."""
+                   dt_bias: torch.Tensor, A2: torch.Tensor, D: torch.Tensor, state_pool: torch.Tensor, y: Optional[torch.Tensor],
+                   inner: int, state: int, longest: int, z: Optional[torch.Tensor] = None, image=None, max_chunks: int = 0,
+                   scratch: Optional[torch.Tensor] = None, chunk_slots: int = 0):
+    """Selective scan with a state per channel; dt raw (bias and softplus inside), A2 [inner][state] = -exp(A_log) / ln 2; out y (f32)
+    or image = (activation image, ncap).  longest: rows of the longest portion of the batch; max_chunks > 0 (with scratch for
+    chunk_slots chunks): the chunk-parallel form."""
     assert B.stride(0) == C.stride(0)
     a = DlSelectiveArgs()
     a.x, a.ld_x, a.dt, a.ld_dt = x.data_ptr(), x.stride(0), dt.data_ptr(), dt.stride(0)
     a.B, a.C, a.ld_bc, a.z, a.ld_z = B.data_ptr(), C.data_ptr(), B.stride(0), _p(z), (z.stride(0) if z is not None else 0)
-    a.dt_bias, a.A_log, a.D, a.state_pool = dt_bias.data_ptr(), A_log.data_ptr(), D.data_ptr(), state_pool.data_ptr()
+    a.dt_bias, a.A2, a.D, a.state_pool = dt_bias.data_ptr(), A2.data_ptr(), D.data_ptr(), state_pool.data_ptr()
     xh, ncap = image or (None, 0)
     a.xh, a.ncap = _p(xh), ncap
     if xh is None:
         a.y, a.ld_y = y.data_ptr(), y.stride(0)
     a.inner, a.state = inner, state
-    check_layers(layers_lib().dl_selective_scan(batch, n_seq, a, _stream()), "dl_selective_scan")
+    if max_chunks > 0:
+        assert scratch.numel() >= chunk_slots * inner * (state + 1)
+        check_layers(layers_lib().dl_selective_scan_chunked(batch, n_seq, max_chunks, a, scratch.data_ptr(), chunk_slots, _stream()),
+                     "dl_selective_scan_chunked")
+        lib.count_launch(3)
+        return
+    check_layers(layers_lib().dl_selective_scan(batch, n_seq, longest, a, _stream()), "dl_selective_scan")
     lib.count_launch()
 
 
-def residual_step(M: int, dim: int, eps: float, x_in: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, adds=(),
-                  normed=(), vec: Optional[torch.Tensor] = None, x: Optional[torch.Tensor] = None, outs=()):
+def residual_step(M: int, dim: int, eps: float, x_in: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, adds=(), normed=(), vec: Optional[torch.Tensor] = None, x: Optional[torch.Tensor] = None, outs=()):
     """x[m] = x_in + sum of `adds` + sum of w * unit(v) over (v, w) in `normed`, all of row rows ? rows[m] : m, + vec; then per (w, h)
     of `outs` h[m] = w * unit(x[m]), h an f32 buffer or an (activation image, ncap) pair.  At most three adds, two of the rest."""
     a = DlResidualArgs()
-    a.x_in, a.ld_in, a.rows = _p(x_in), (x_in.stride(0) if x_in is not None else 0), _p(rows)
+    a.ld_in, a.rows = (x_in.stride(0) if x_in is not None else 0), _p(rows)
+    if x_in is not None:         # f32 rows, or the bf16 rows of a table
+        setattr(a, "table" if x_in.dtype == torch.bfloat16 else "x_in", x_in.data_ptr())
     adds, normed, outs = list(adds), list(normed), list(outs)
     assert len(adds) <= 3 and len(normed) <= 2 and len(outs) <= 2
     for n, t in zip(("add1", "add2", "add3"), adds):

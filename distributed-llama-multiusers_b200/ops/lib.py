@@ -61,6 +61,8 @@ class DlEpilogue(C.Structure):
         ("dense_aux", C.c_void_p),
         ("dense_aux_ld", C.c_longlong),
         ("dense_param2", C.c_float),
+        ("dense_xh", C.c_void_p),
+        ("dense_ncap", C.c_int),
     ]
 
 
@@ -355,14 +357,14 @@ class DlSelectiveArgs(C.Structure):
     """Mirror of ``DlSelectiveArgs``."""
     _fields_ = [("x", C.c_void_p), ("ld_x", C.c_longlong), ("dt", C.c_void_p), ("ld_dt", C.c_longlong),
                 ("B", C.c_void_p), ("C", C.c_void_p), ("ld_bc", C.c_longlong), ("z", C.c_void_p), ("ld_z", C.c_longlong),
-                ("dt_bias", C.c_void_p), ("A_log", C.c_void_p), ("D", C.c_void_p), ("state_pool", C.c_void_p),
+                ("dt_bias", C.c_void_p), ("A2", C.c_void_p), ("D", C.c_void_p), ("state_pool", C.c_void_p),
                 ("y", C.c_void_p), ("ld_y", C.c_longlong), ("xh", C.c_void_p), ("ncap", C.c_int),
                 ("inner", C.c_int), ("state", C.c_int)]
 
 
 class DlResidualArgs(C.Structure):
     """Mirror of ``DlResidualArgs``."""
-    _fields_ = [("x_in", C.c_void_p), ("ld_in", C.c_longlong), ("rows", C.c_void_p),
+    _fields_ = [("x_in", C.c_void_p), ("ld_in", C.c_longlong), ("rows", C.c_void_p), ("table", C.c_void_p),
                 ("add1", C.c_void_p), ("add2", C.c_void_p), ("add3", C.c_void_p),
                 ("ld_add1", C.c_longlong), ("ld_add2", C.c_longlong), ("ld_add3", C.c_longlong),
                 ("norm_a", C.c_void_p), ("w_a", C.c_void_p), ("norm_b", C.c_void_p), ("w_b", C.c_void_p),
@@ -459,9 +461,11 @@ def layers_lib():
     L.dl_gated_scan_chunked_supported.argtypes = [i32, i32, i32]
     L.dl_gated_chunk_floats.argtypes = [i32, i32, i32, i32, i32]
     L.dl_gated_chunk_floats.restype = i64
-    L.dl_mlstm_gates.argtypes = [C.POINTER(DlMambaBatch), i32, C.POINTER(DlMlstmGatesArgs), vp]
+    L.dl_mlstm_gates.argtypes = [C.POINTER(DlMambaBatch), i32, i32, C.POINTER(DlMlstmGatesArgs), vp]
     L.dl_head_norm.argtypes = [C.POINTER(DlHeadNormArgs), vp]
-    L.dl_selective_scan.argtypes = [C.POINTER(DlMambaBatch), i32, C.POINTER(DlSelectiveArgs), vp]
+    L.dl_selective_scan.argtypes = [C.POINTER(DlMambaBatch), i32, i32, C.POINTER(DlSelectiveArgs), vp]
+    L.dl_selective_scan_chunked.argtypes = [C.POINTER(DlMambaBatch), i32, i32, C.POINTER(DlSelectiveArgs), vp, i32, vp]
+    L.dl_selective_scan_chunked_supported.argtypes = [i32]
     L.dl_selective_scan_supported.argtypes = [i32]
     L.dl_residual_step.argtypes = [C.POINTER(DlResidualArgs), vp]
     L.dl_wh_bytes.restype = i64
@@ -479,7 +483,7 @@ def layers_lib():
                  "dl_moe_combine", "dl_xh_gather_rows", "dl_gemm_wh_tc_grouped", "dl_window_tc_rows", "dl_window_attention_tc_supported",
                  "dl_window_attention_tc", "dl_talk_attention_tc_supported", "dl_talk_attention_tc", "dl_talk_tc_tile_rows", "dl_causal_conv", "dl_poly_norm", "dl_lightning_scan", "dl_lightning_scan_chunked",
                  "dl_gated_scan", "dl_gated_scan_chunked", "dl_gated_scan_supported", "dl_gated_scan_chunked_supported", "dl_mlstm_gates", "dl_head_norm",
-                 "dl_selective_scan", "dl_selective_scan_supported", "dl_residual_step", "dl_talk_mix"):
+                 "dl_selective_scan", "dl_selective_scan_supported", "dl_selective_scan_chunked", "dl_selective_scan_chunked_supported", "dl_residual_step", "dl_talk_mix"):
         getattr(L, name).restype = i32
     _layers = L
     return L

@@ -73,6 +73,8 @@ typedef struct {
     const float* dense_aux;
     long long dense_aux_ld;
     float dense_param2;
+    uint8_t* dense_xh;                /* DL_DENSE_GLU_GELU: the result leaves as the next product's bf16 activation image (its   */
+    int dense_ncap;                   /* width a multiple of 128; ncap rows) instead of f32 rows                                */
 } DlEpilogue;
 
 /* Fused activation producer for dl_gemv_q40: the kernel itself computes
@@ -528,7 +530,7 @@ typedef struct {
     float* log_keep; float* put; float* floor_;
     int n_heads;
 } DlMlstmGatesArgs;
-int dl_mlstm_gates(const DlMambaBatch* batch /*host*/, int n_seq, const DlMlstmGatesArgs* args /*host*/, void* stream);
+int dl_mlstm_gates(const DlMambaBatch* batch /*host*/, int n_seq, int longest, const DlMlstmGatesArgs* args /*host*/, void* stream);
 /* Per row and head of vdim numbers: o = y / (max(|den|, floor) + 1e-6) (den NULL: y), then o / sqrt(mean(o^2) + eps) * w
  * (w [vdim], or [n_heads * vdim] with w_full), then * sigmoid(gate) (gate NULL: none).  To out (f32) or, with xh, into the
  * tcgen05 GEMM's activation image. */
@@ -550,13 +552,21 @@ typedef struct {
     const float* dt; long long ld_dt;        /* [M][inner] */
     const float* B; const float* C; long long ld_bc;      /* [M] rows of `state` numbers */
     const float* z; long long ld_z;
-    const float* dt_bias; const float* A_log; const float* D;      /* [inner], [inner][state], [inner] f32 */
+    const float* dt_bias; const float* A2; const float* D;         /* [inner], [inner][state] = -exp(A_log) / ln 2, [inner] f32 */
     float* state_pool;
     float* y; long long ld_y; uint8_t* xh; int ncap;      /* y (f32) or, with xh, the activation image of the tcgen05 GEMM */
     int inner, state;
 } DlSelectiveArgs;
 int dl_selective_scan_supported(int state);
-int dl_selective_scan(const DlMambaBatch* batch /*host*/, int n_seq, const DlSelectiveArgs* args /*host*/, void* stream);
+/* longest: rows of the longest portion of the batch (1: the kernel for single decoded rows) */
+int dl_selective_scan(const DlMambaBatch* batch /*host*/, int n_seq, int longest, const DlSelectiveArgs* args /*host*/, void* stream);
+/* Long portions: chunks of DL_SELECTIVE_CHUNK rows of a sequence in parallel (three launches: every chunk's own state from zeros
+ * and its sum of steps, the prefix over a sequence's chunks, the chunks' outputs); scratch: chunk_slots * inner * (state + 1) f32
+ * with chunk_slots = M / DL_SELECTIVE_CHUNK + n_seq of the largest batch */
+#define DL_SELECTIVE_CHUNK 64
+int dl_selective_scan_chunked_supported(int state);
+int dl_selective_scan_chunked(const DlMambaBatch* batch /*host*/, int n_seq, int max_chunks, const DlSelectiveArgs* args /*host*/,
+                              float* scratch, int chunk_slots, void* stream);
 
 /* ---- one step of a residual stream (norms.cu) ------------------------------------------------------------------------
  *   x[m] = x_in + add1 + add2 + add3 + w_a * unit(norm_a) + w_b * unit(norm_b) + vec    unit(v) = v / sqrt(mean(v^2) + eps)
@@ -564,6 +574,7 @@ int dl_selective_scan(const DlMambaBatch* batch /*host*/, int n_seq, const DlSel
  * Every term may be absent (NULL); x NULL: the sum is not stored; rows: all terms but vec are those of row rows[m] (a gather). */
 typedef struct {
     const float* x_in; long long ld_in; const int* rows;
+    const void* table;                        /* instead of x_in: bf16 rows (an embedding table, rows = the tokens) */
     const float* add1; const float* add2; const float* add3; long long ld_add1, ld_add2, ld_add3;
     const float* norm_a; const float* w_a; const float* norm_b; const float* w_b; long long ld_a, ld_b;
     const float* vec;

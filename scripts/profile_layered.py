@@ -17,6 +17,16 @@
       the head-mixed attention tile kernel alone (2048 rows of one sequence, 16 / 4 heads, keys and values of 128, 64
       rotated dims, the head mix folded into queries of 4 x 128), timed with CUDA events:
         ncu --set full --clock-control none -k regex:talk_attention_mma -s 1 -c 1 -o out python scripts/profile_layered.py talk-attention
+  python scripts/profile_layered.py gated-scan
+      the chunk-parallel scans with data-dependent gates alone (2048 rows of one sequence; matrix memory with 8 heads of
+      128 x 256, HGRN2 with 16 heads of 128 x 128), then both token by token on 1 and 32 sequences of one row:
+        ncu --set full --clock-control none -k regex:gated_chunk_out -s 1 -c 2 -o out python scripts/profile_layered.py gated-scan
+  python scripts/profile_layered.py selective-scan
+      the selective scan alone (4096 channels of 16 state entries; 2048 rows of one sequence, then 32 sequences of one row):
+        ncu --set full --clock-control none -k regex:selective_scan -s 1 -c 1 -o out python scripts/profile_layered.py selective-scan
+  python scripts/profile_layered.py wide-attention
+      attention whose softmax weights are mixed across heads (2048 rows of one sequence, 16 / 4 heads of 128) and the mix alone:
+        ncu --set full --clock-control none -k regex:talk_attention_mma -s 1 -c 1 -o out python scripts/profile_layered.py wide-attention
 Run the plain command first; capture only if it exits 0.
 """
 import argparse
@@ -155,13 +165,104 @@ def lightning_scan(a):
             print("token-by-token scan, %d sequences of one row: %.1f us for %.1f MB of state read and written" % (m, ev0.elapsed_time(ev1) * 1e3, 2 * m * H * d * dv * 4 / 1e6))
 
 
+def _sequences(n_rows, n_seq):
+    """Batch descriptor of n_seq sequences of n_rows consecutive rows each (fresh if a sequence has more than one row)."""
+    import torch
+    from dllama_b200.ops import layers as L
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    M, p0 = n_rows * n_seq, 0 if n_rows > 1 else 5
+    keep = [i32([p0 + i % n_rows for i in range(M)]), i32([i // n_rows for i in range(M)]), i32([i * n_rows for i in range(n_seq + 1)]),
+            i32(list(range(M))), i32(list(range(n_seq))), i32([p0] * n_seq)]
+    return L.mamba_batch(*keep), keep
+
+
+def _timed(what, fn, repeats=4):
+    import torch
+    ev0, ev1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    for _ in range(repeats):
+        ev0.record()
+        fn()
+        ev1.record()
+        torch.cuda.synchronize()
+        print("%s: %.1f us" % (what, ev0.elapsed_time(ev1) * 1e3))
+
+
+def gated_scan(a):
+    import torch
+    from dllama_b200.ops import layers as L
+    n, users = 2048, 32
+    g = torch.Generator().manual_seed(1)
+    for name, H, d, dv in (("matrix memory", 8, 128, 256), ("HGRN2", 16, 128, 128)):
+        x = torch.randn(n, H * (2 * d + dv), generator=g).cuda()
+        y, den = torch.zeros(n, H * dv, device="cuda"), torch.zeros(n * H, device="cuda")
+        state, n_state, u = torch.zeros(users, H, d, dv, device="cuda"), torch.zeros(users, H, d, device="cuda"), torch.zeros(users, H, device="cuda")
+        z, bias = torch.randn(n, 2 * H, generator=g).cuda(), torch.full((H * d,), 2.0, device="cuda")
+        keep, put, floor = (torch.zeros(n * H, device="cuda") for _ in range(3))
+        slots = n // L.GATED_CHUNK + users
+        scratch = torch.zeros(L.gated_chunk_floats(n, users, H, d, dv), device="cuda")
+
+        def scan(b, n_seq, **kw):
+            if name == "HGRN2":
+                L.gated_scan(b, n_seq, x, x[:, 2 * H * d:], y, state, H, d, dv, q_silu=True, f=x[:, H * d:], f_bias=bias, lower=bias * 0.1, **kw)
+            else:
+                L.mlstm_gates(b, n_seq, z, z[:, H:], bias, bias, 15.0, u, keep, put, floor, H, n if n_seq == 1 and kw else 1)
+                L.gated_scan(b, n_seq, x, x[:, 2 * H * d:], y, state, H, d, dv, q_scale=d ** -0.5, k=x[:, H * d:], log_keep=keep, put=put,
+                             den=den, n_state=n_state, **kw)
+
+        b, hold = _sequences(n, 1)
+        _timed(f"{name}, chunked, {n} rows", lambda: scan(b, 1, max_chunks=n // L.GATED_CHUNK, scratch=scratch, chunk_slots=slots))
+        print("GFLOP (state update and read-out, 4 dim vdim per row and head): %.2f" % (n * H * 4 * d * dv / 1e9))
+        for m in (1, users):
+            b1, hold1 = _sequences(1, m)
+            _timed(f"{name}, token by token, {m} sequences of one row ({2 * m * H * d * dv * 4 / 1e6:.1f} MB of state)", lambda: scan(b1, m), 3)
+
+
+def selective_scan(a):
+    import torch
+    from dllama_b200.ops import layers as L
+    n, users, inner, N, r = 2048, 32, 4096, 16, 128
+    g = torch.Generator().manual_seed(1)
+    x, dt, z = (torch.randn(n, inner, generator=g).cuda() for _ in range(3))
+    dbc = torch.randn(n, r + 2 * N, generator=g).cuda()
+    A2, bias, D = -torch.exp(torch.randn(inner, N, generator=g) * 0.5).cuda(), torch.full((inner,), -3.0, device="cuda"), torch.ones(inner, device="cuda")
+    state, y = torch.zeros(users, inner, N, device="cuda"), torch.zeros(n, inner, device="cuda")
+    slots = n // L.SELECTIVE_CHUNK + 1
+    scratch = torch.zeros(slots * inner * (N + 1), device="cuda")
+    for rows, n_seq, chunked in ((n, 1, True), (n, 1, False), (1, users, False)):
+        b, hold = _sequences(rows, n_seq)
+        kw = dict(max_chunks=n // L.SELECTIVE_CHUNK, scratch=scratch, chunk_slots=slots) if chunked else {}
+        _timed(f"selective scan, {n_seq} sequences of {rows} rows{', chunked' if chunked else ''}",
+               lambda: L.selective_scan(b, n_seq, x, dt, dbc[:, r:], dbc[:, r + N:], bias, A2, D, state, y, inner, N, rows, z=z, **kw))
+
+
+def wide_attention(a):
+    import torch
+    from dllama_b200.ops import layers as L
+    H, G, d, dv, n = 16, 4, 128, 128, 2048
+    n_pages = n // 32
+    bt = torch.arange(n_pages, dtype=torch.int32).view(1, -1).cuda()
+    cache = torch.randn(n_pages, G, 32, d + dv, device="cuda").to(torch.bfloat16)
+    g = torch.Generator().manual_seed(1)
+    q, talk = torch.randn(n, H * d, generator=g).cuda(), (torch.eye(H) + torch.randn(H, H, generator=g) * 0.3).cuda()
+    pos, slot = torch.arange(n, dtype=torch.int32).cuda(), torch.zeros(n, dtype=torch.int32).cuda()
+    wide, out = torch.zeros(n, H * G * dv, device="cuda"), torch.zeros(n, H * dv, device="cuda")
+    rq = L.talk_tc_rows(H, G, d, dv, 0, n, G)
+    tiles = torch.arange(n, dtype=torch.int32).view(-1, rq).cuda()
+    _timed("attention, weights against all value heads, tiles of %d rows" % rq,
+           lambda: L.talk_attention_tc(q, wide, H, G, d, dv, 0.1, 0, pos, slot, bt, cache, tiles, n // rq, rq, 1, None, value_heads=G))
+    _timed("mix of the heads' outputs", lambda: L.talk_mix(wide, talk, n, H, G, dv, out))
+    pairs = n * (n + 1) // 2
+    print("FLOPs per launch (visible pairs, 2 * (128 + 4 * 128) per head): %.1f G" % (pairs * H * 2 * (d + G * dv) / 1e9))
+
+
 if __name__ == "__main__":
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("what", choices=("steps", "window-attention", "lightning-scan", "talk-attention"))
+    ap.add_argument("what", choices=("steps", "window-attention", "lightning-scan", "talk-attention", "gated-scan", "selective-scan", "wide-attention"))
     ap.add_argument("--design", default="sunesun", choices=("ribivik", "sunesun", "venadra", "darusun", "vopedra"))
     ap.add_argument("--size", default="w2048")
     ap.add_argument("--layers", type=int, default=4)
     ap.add_argument("--prompt", type=int, default=2048)
     ap.add_argument("--model-dir", default="/tmp")
     a = ap.parse_args()
-    {"steps": steps, "window-attention": window_attention, "lightning-scan": lightning_scan, "talk-attention": talk_attention}[a.what](a)
+    {"steps": steps, "window-attention": window_attention, "lightning-scan": lightning_scan, "talk-attention": talk_attention,
+     "gated-scan": gated_scan, "selective-scan": selective_scan, "wide-attention": wide_attention}[a.what](a)
