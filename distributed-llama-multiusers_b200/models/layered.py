@@ -1696,15 +1696,15 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
             t[p + "mix.left.out"], t[p + "mix.right.out"] = 1 + small(W), 1 + small(W)
         elif l["type"] == "mlstm":
             H, d, dv = m["heads"], m["dim"], m["vdim"]
-            t[p + "mix.q"], t[p + "mix.k"], t[p + "mix.v"] = mat(H * d, W, 2.0), mat(H * d, W, 2.0), mat(H * dv, W, 1.5)
+            t[p + "mix.q"], t[p + "mix.k"], t[p + "mix.v"] = mat(H * d, W), mat(H * d, W), mat(H * dv, W)
             t[p + "mix.g"], t[p + "mix.o"], t[p + "mix.norm"] = mat(H * dv, W), mat(W, H * dv), 1 + small(H * dv)
-            t[p + "mix.i"], t[p + "mix.f"] = mat(H, W, 2.0), mat(H, W, 2.0)
+            t[p + "mix.i"], t[p + "mix.f"] = mat(H, W), mat(H, W)
             t[p + "mix.i.b"], t[p + "mix.f.b"] = small(H, 0.5), (2 + torch.rand(H, generator=g) * 3).to(torch.bfloat16)
         elif l["type"] == "mamba1":
             inner, r, N, K = m["inner"], m["dt_rank"], m["state"], m["conv"]
-            t[p + "mix.in"] = mat(2 * inner, W, 1.5)
-            t[p + "mix.conv"], t[p + "mix.conv.b"] = mat(inner, K, 1.5), small(inner)
-            t[p + "mix.x"], t[p + "mix.dt"] = mat(r + 2 * N, inner, 1.5), mat(inner, r)
+            t[p + "mix.in"] = mat(2 * inner, W)
+            t[p + "mix.conv"], t[p + "mix.conv.b"] = mat(inner, K), small(inner)
+            t[p + "mix.x"], t[p + "mix.dt"] = mat(r + 2 * N, inner), mat(inner, r)
             t[p + "mix.dt.b"] = (torch.rand(inner, generator=g) * 3 - 4).to(torch.bfloat16)
             t[p + "mix.A_log"] = (torch.log(1.0 + torch.arange(N, dtype=torch.float32))[None, :] + torch.randn(inner, N, generator=g) * 0.2).to(torch.bfloat16)
             t[p + "mix.D"], t[p + "mix.o"] = 1 + small(inner), mat(W, inner)

@@ -211,3 +211,68 @@ def test_darusun_oracle_window_head_mix_routing_and_prefix_property():
     sel, w = D.route(z, 3)
     assert sel.tolist() == [[1, 3, 4]] and abs(float(w.sum()) - 1.0) < 1e-12 and abs(float(w[0, 0] / w[0, 2]) - math.exp(1.5)) < 1e-9
     assert abs(float(D.xielu(torch.tensor([2.0], dtype=torch.float64), 0.0, 0.0)) - (math.log(2.0) * 4 + 1)) < 1e-12
+
+
+def test_vopedra_configuration_runs_and_tensor_names(tmp_path):
+    from dllama_b200.models.layered import DESIGNS, example_config_vopedra
+    cfg = example_config_vopedra()
+    d = str(tmp_path / "d")
+    tensors = write_random_model(d, cfg, seed=1)
+    assert registry.architecture_of(d) == "Vopedra" and "Vopedra" in registry.ARCHITECTURES
+    c = LayerListConfig.load(d)
+    assert (c.residual, c.streams, c.canon_taps, c.logit_softcap, c.loop_times) == ("parallel", 1, 0, 0.0, 2)
+    assert c.traits is DESIGNS["Vopedra"] and c.traits["attention"]["talk"] == "weights" and c.norm_eps == 1e-6
+    # the slice [1, 3) runs twice: later passes name the first pass's run and keep the tensors' numbers; the layer behind the loop too
+    assert [(l.type, l.weights_of, l.tensors, l.opens) for l in c.layers] == [
+        ("mamba1", None, 0, None), ("mlstm", None, 1, 0), ("parallel", None, 2, None), ("mlstm", 1, 1, 1), ("parallel", 2, 2, None), ("mlstm", None, 3, None)]
+    assert tensors["loop.step"].shape == (2, 160) and tensors["embed.norm"].shape == (160,) and "l4.norm1" not in tensors and "l0.norm2" not in tensors
+    assert tensors["l0.mix.x"].shape == (9 + 24, 320) and tensors["l0.mix.A_log"].shape == (320, 12) and tensors["l0.mix.conv"].shape == (320, 4)
+    assert tensors["l1.mix.i"].shape == (3, 160) and tensors["l1.mix.norm"].shape == (3 * 36,) and tensors["l1.mlp.gate"].shape == (320, 160)
+    assert tensors["l2.mix.left.q.norm"].shape == (6 * 24,) and tensors["l2.mix.left.talk"].shape == (6, 6) and tensors["l2.mix.right.norm"].shape == (16,)
+    assert tensors["l2.mix.right.lower"].shape == (3 * 28,) and tensors["l2.mix.left.out"].shape == (160,)
+    for loop, order in ((None, [0, 1, 2, 3]), ((0, 4, 2), [0, 1, 2, 3, 0, 1, 2, 3]), ((3, 4, 3), [0, 1, 2, 3, 3, 3]), ((1, 2, 1), [0, 1, 2, 3])):
+        one = dict(cfg, loop=dict(zip(("start", "stop", "times"), loop)) if loop else None)
+        runs = LayerListConfig.from_dict(one).layers
+        assert [i if l.tensors is None else l.tensors for i, l in enumerate(runs)] == order
+        if loop:
+            assert [l.opens for l in runs if l.opens is not None] == list(range(loop[2])) and all((l.weights_of is None) == (order.index(l.tensors) == i) for i, l in enumerate(runs))
+    for loop in ((2, 2, 1), (0, 5, 1), (1, 3, 0)):
+        with pytest.raises(ValueError):
+            LayerListConfig.from_dict(dict(cfg, loop=dict(zip(("start", "stop", "times"), loop))))
+    with pytest.raises(ValueError):          # a loop belongs to designs whose stream is stepped once per layer
+        LayerListConfig.from_dict(dict(example_config(blocks=1), loop={"start": 0, "stop": 1, "times": 2}))
+
+
+def test_vopedra_oracle_mix_gates_state_carry_and_prefix_property():
+    """The oracle itself: appended tokens change nothing before them; an identity mix leaves plain attention and the mix of
+    the weights is the mix of the outputs over all value heads; states carried across a cut equal one walk; the matrix memory's
+    running maximum changes nothing but the floor of its denominator."""
+    import vopedra_oracle as V
+    from dllama_b200.models.layered import example_config_vopedra
+    cfg = example_config_vopedra(width=48, vocab=40, heads=2)
+    t = random_tensors(cfg, seed=2)
+    toks = torch.randint(0, 40, (23,), generator=torch.Generator().manual_seed(3)).tolist()
+    assert torch.allclose(V.model_logits(t, cfg, toks)[:9], V.model_logits(t, cfg, toks[:9]), atol=1e-9)
+    g = torch.Generator().manual_seed(5)
+    T, H, G, d, dv = 9, 4, 2, 6, 5
+    q, k, v = (torch.randn(T, n, m, generator=g, dtype=torch.float64) for n, m in ((H, d), (G, d), (G, dv)))
+    talk = torch.randn(H, H, generator=g, dtype=torch.float64)
+    mixed, plain = V.softmax_then_mix_rows(q, k, v, 0.7, talk), V.softmax_then_mix_rows(q, k, v, 0.7, torch.eye(H, dtype=torch.float64))
+    for h in range(H):
+        p = torch.softmax(0.7 * (k[:, h // 2] @ q[8, h]), -1)
+        assert torch.allclose(plain[8, h], p @ v[:, h // 2], atol=1e-12)
+    wide = torch.stack([torch.stack([torch.softmax(0.7 * (k[:, x // 2] @ q[8, x]), -1) @ v[:, c] for c in range(G)]) for x in range(H)])      # [heads, value heads, dv]
+    for h in range(H):
+        assert torch.allclose(mixed[8, h], (talk[h][:, None] * wide[:, h // 2]).sum(0), atol=1e-12)
+    kk, vv = torch.randn(T, H, d, generator=g, dtype=torch.float64), torch.randn(T, H, dv, generator=g, dtype=torch.float64)
+    f = torch.rand(T, H, d, generator=g, dtype=torch.float64)
+    whole, S = V.gated_rows(q, kk, vv, f)
+    first, S1 = V.gated_rows(q[:4], kk[:4], vv[:4], f[:4])
+    rest, S2 = V.gated_rows(q[4:], kk[4:], vv[4:], f[4:], S1)
+    assert torch.allclose(torch.cat([first, rest]), whole, atol=1e-12) and torch.allclose(S, S2, atol=1e-12)
+    a, b = V.mlstm_gates(torch.randn(T, H, generator=g, dtype=torch.float64) * 2, torch.randn(T, H, generator=g, dtype=torch.float64) + 2, 7.0)
+    o, (_, _, u) = V.mlstm_rows(q, kk, vv, a, b)
+    for h in range(H):                       # without the running maximum: weights e^(b_(j+1) + .. + b_i + a_j)
+        w = torch.exp(torch.stack([b[j + 1:, h].sum() + a[j, h] for j in range(T)]))
+        num, den = ((w * (kk[:, h] @ q[8, h]))[:, None] * vv[:, h]).sum(0), (w * (kk[:, h] @ q[8, h])).sum().abs()
+        assert torch.allclose(o[8, h], num / (torch.clamp(den, min=1.0) + 1e-6 * torch.exp(u[h])), rtol=1e-9, atol=1e-12)
