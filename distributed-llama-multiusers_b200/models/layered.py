@@ -53,6 +53,7 @@ and step sizes are f32.  ``dtype="float32"`` widens weights and caches to f32 an
 """
 from __future__ import annotations
 
+import contextlib
 import json
 import math
 import os
@@ -226,6 +227,7 @@ CHUNKED_SCAN_MIN_ROWS = 256  # a batch holding this many rows of one sequence ru
 LIGHTNING_CHUNKED_MIN_ROWS = 128     # the same for linear attention (chunks of 64 rows)
 GATED_CHUNKED_MIN_ROWS = 128         # and for linear attention with data-dependent gates and selective scans per channel
 TC_HEADS_MIN_ROWS = 256      # per-head products (one small GEMM per head) take the tensor-core path from this many rows
+BRANCH_MAX_ROWS = 1 << 30    # branches on the same input run on streams of their own up to this many rows
 GRAPH_MAX_ROWS = 64          # batches up to this many rows are replayed from CUDA graphs
 WINDOW_MAX_SPLITS = 32       # most CTAs that share one tile's pages in the windowed-attention kernel
 WINDOW_CTAS_PER_SM = 8       # pages are shared until about this many CTAs per SM run (one page in flight per CTA)
@@ -850,9 +852,12 @@ class ParallelMixer:
 
     def forward_branches(self, h: torch.Tensor, M: int) -> list:
         """[(branch output, weight of its norm)]: the mixer's output is the sum of the normed branches."""
-        bl, br = self.eng.buf("br_l"), self.eng.buf("br_r")
+        e = self.eng
+        bl, br = e.buf("br_l"), e.buf("br_r")
+        with e.side(1, M):
+            self.right.forward(h, br, M)
         self.left.forward(h, bl, M)
-        self.right.forward(h, br, M)
+        e.join(1, M)
         return [(bl, self.out_l), (br, self.out_r)]
 
     def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
@@ -1140,7 +1145,7 @@ class LayerListEngine:
         self._xh = {}
         if self.tc:       # activation slabs: one kept for a sublayer's input (several products read it), one for the rest
             n = L.xh_bytes(self._kmax, self.ncap)
-            self._xh = {k: torch.zeros(n, dtype=torch.uint8, device=dev) for k in ("h", "tmp") + (("h2",) if self.cfg.residual == "parallel" else ())}
+            self._xh = {k: torch.zeros(n, dtype=torch.uint8, device=dev) for k in ("h", "tmp") + (("h2", "tmp1", "tmp2") if self.cfg.residual == "parallel" else ())}
         if self.cfg.streams > L.HC_MAX_STREAMS:
             raise ValueError(f"{self.cfg.streams} streams: the kernels keep at most {L.HC_MAX_STREAMS} copies of the residual stream")
         self.x = torch.zeros(R, self.cfg.streams * self.cfg.width, dtype=torch.float32, device=dev)      # row = [streams][width]
@@ -1183,7 +1188,10 @@ class LayerListEngine:
         self.block_table = torch.zeros(self.n_slots, self.max_pages, dtype=torch.int32, device=dev)
         self.h_block_table = torch.zeros(self.n_slots, self.max_pages, dtype=torch.int32).pin_memory()
         self._staging_ev: Optional[torch.cuda.Event] = None
-        self._xh_h_ready, self._xh_h = False, "h"
+        self._xh_h_ready, self._xh_h, self._tmp = False, "h", "tmp"
+        # branches that read the same input (mixer and feed-forward, the two halves of a parallel mixer) run side by side
+        self.branch_max_rows = int(os.environ.get("DLLAMA_LAYERS_BRANCH_MAX_ROWS", str(BRANCH_MAX_ROWS)))
+        self._side_streams = [torch.cuda.Stream(device=dev) for _ in range(2)] if self.cfg.residual == "parallel" else []
         # decode-sized batches replay a CUDA graph per batch shape (rows, sequences, wanted logits, attention tiling):
         # a step is ~25 small launches per layer, and the host cannot issue them as fast as the GPU retires them
         self.use_graphs = bool(use_graphs) and os.environ.get("DLLAMA_LAYERS_GRAPHS", "1") != "0"
@@ -1230,7 +1238,7 @@ class LayerListEngine:
         if w.wh is None or M < TC_MIN_ROWS:
             L.dense(w.t, x, y, M, self.round_x, epi=epi, aux=aux, param=param, param2=param2)
             return
-        xh = self._xh[self._xh_h if src == "h" else src]
+        xh = self._xh[self._xh_h if src == "h" else self._tmp]
         if not ready and (src != "h" or not self._xh_h_ready):
             L.xh_from_rows(x, M, w.K, self.ncap, xh)
             self._xh_h_ready = src == "h" or self._xh_h_ready
@@ -1243,8 +1251,8 @@ class LayerListEngine:
             L.dense_heads(w.t, x, y, M, self.round_x, x_head_stride, y_head_stride)
             return
         for h in range(w.t.shape[0]):
-            L.xh_from_rows(x[:, h * x_head_stride:], M, w.K, self.ncap, self._xh["tmp"])
-            L.dense_tc(w.wh[h], w.N, w.K, self._xh["tmp"], self.ncap, y[:, h * y_head_stride:], M)
+            L.xh_from_rows(x[:, h * x_head_stride:], M, w.K, self.ncap, self._xh[self._tmp])
+            L.dense_tc(w.wh[h], w.N, w.K, self._xh[self._tmp], self.ncap, y[:, h * y_head_stride:], M)
 
     def mamba_chunks(self, mx):
         """The chunking of this batch for the two-pass scan, or None where the token-by-token scan runs (short portions,
@@ -1256,7 +1264,26 @@ class LayerListEngine:
     def image(self, name: str, M: int):
         """(activation image, its row capacity) if products over M rows read bf16 images, so that a kernel can leave its
         result in the next product's operand layout; None where they read f32 rows."""
-        return (self._xh[name], self.ncap) if self.tc and M >= TC_MIN_ROWS else None
+        return (self._xh[self._tmp if name == "tmp" else name], self.ncap) if self.tc and M >= TC_MIN_ROWS else None
+
+    @contextlib.contextmanager
+    def side(self, k: int, M: int):
+        """Launches inside go to side stream k, behind everything launched so far, with a "tmp" image of their own; join(k, M)
+        makes the current stream wait for them.  Batches of more than branch_max_rows rows stay on one stream."""
+        if M > self.branch_max_rows or not self._side_streams:
+            yield
+            return
+        self._side_streams[k].wait_stream(torch.cuda.current_stream())
+        tmp, self._tmp = self._tmp, f"tmp{k + 1}"
+        try:
+            with torch.cuda.stream(self._side_streams[k]):
+                yield
+        finally:
+            self._tmp = tmp
+
+    def join(self, k: int, M: int):
+        if M <= self.branch_max_rows and self._side_streams:
+            torch.cuda.current_stream().wait_stream(self._side_streams[k])
 
     def gated_chunking(self, mx) -> dict:
         """The chunking of this batch for a gated linear-attention scan (empty: token by token)."""
@@ -1473,6 +1500,10 @@ class LayerListEngine:
             L.residual_step(M, W, eps, x_in=src, adds=adds, normed=normed, vec=self.loop_step[l.opens] if l.opens is not None else None,
                             x=x, outs=[(l.norm1, img1 or self.hn)] + ([(l.norm2, img2 or self.hn2)] if l.ff is not None else []))
             src, adds, normed = x, [], []
+            if l.ff is not None:
+                self.begin_sublayer("h2", ready=img2 is not None)
+                with self.side(0, M):
+                    l.ff.forward(self.hn2, self.y2, M)
             self.begin_sublayer("h", ready=img1 is not None)
             if isinstance(l.mixer, ParallelMixer):
                 normed = l.mixer.forward_branches(self.hn, M)
@@ -1480,8 +1511,7 @@ class LayerListEngine:
                 l.mixer.forward(self.hn, self.y, M)
                 adds.append(self.y)
             if l.ff is not None:
-                self.begin_sublayer("h2", ready=img2 is not None)
-                l.ff.forward(self.hn2, self.y2, M)
+                self.join(0, M)
                 adds.append(self.y2)
             if self.layer_probe is not None:
                 L.residual_step(M, W, eps, x_in=src, adds=adds, normed=normed, x=x)
