@@ -73,7 +73,7 @@ def _run_gates(zi, zf, bi, bf, cap, slot, portions, n_slots=3, u0=None):
     return outs, u
 
 
-@pytest.mark.parametrize("cap", [3.0, 12.0, 30.0])
+@pytest.mark.parametrize("cap", [3.0, 11.0, 30.0])
 @pytest.mark.parametrize("portions", [[1], [1] * 40, [40, 1, 87, 2, 130], [300], [1500, 3]])
 def test_matrix_memory_gates(cap, portions):
     T, H = sum(portions), 3

@@ -143,7 +143,7 @@ def mlstm_mixer(t, p, m, h, eps):
 
 
 def causal_conv_rows(x, w, bias):
-    """x [T, C], w [C, taps] (last column: the current token's): zeros before the start."""
+    """x [T, C], w [C, taps]: tap j meets the input taps - 1 - j tokens back, nothing ahead of the first token."""
     T, taps = x.shape[0], w.shape[1]
     pad = torch.cat([torch.zeros(taps - 1, x.shape[1], dtype=F64), x], 0)
     return bias + sum(w[:, j] * pad[j:j + T] for j in range(taps))
