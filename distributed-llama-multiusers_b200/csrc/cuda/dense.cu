@@ -7,8 +7,8 @@
 //
 // Epilogues (what other models of this library fuse into their matmul kernels too): plain store, relu(.)^2,
 // aux * sigmoid(.) (an output gate), cap * tanh(. / cap) (logit soft-capping), . * sigmoid(.) (SiLU), aux * (.) (the second
-// half of a gated unit), xIELU (a quadratic for z > 0, an exponential for z <= 0, two constants), and a sum into Y behind one
-// sigmoid gate per row.
+// half of a gated unit), xIELU (a quadratic for z > 0, an exponential for z <= 0, two constants), a constant factor, and a sum
+// into Y behind one sigmoid gate per row.  A bias per output column, where given, is added first.
 #include "layer_common.cuh"
 #include "../../../include/dllama_b200.h"
 
@@ -19,6 +19,7 @@ __device__ __forceinline__ float dense_epi(float acc, int epi, float aux, float 
         case DL_DENSE_SOFTCAP: return param * tanhf(acc / param);
         case DL_DENSE_SILU: return silu_f(acc);
         case DL_DENSE_MUL: return aux * acc;
+        case DL_DENSE_SCALE: return param * acc;
         case DL_DENSE_XIELU: return acc > 0.f ? fmaf(param * acc, acc, 0.5f * acc) : fmaf(param2, expm1f(acc) - acc, 0.5f * acc);
         default: return acc;
     }
@@ -27,6 +28,7 @@ __device__ __forceinline__ float dense_epi(float acc, int epi, float aux, float 
 // element (m, n) of batch b leaves through the epilogue; the row-gated sum reads what Y holds first
 __device__ __forceinline__ void dense_store(const DlDenseArgs& a, int b, int m, int n, float acc) {
     float* y = a.Y + (size_t)b * a.y_bs + (size_t)m * a.ldy + n;
+    if (a.bias) acc += a.bias[(size_t)b * a.N + n];
     if (a.epi == DL_DENSE_ROWGATE_ADD) {
         *y = fmaf(sigmoid_f(a.aux[(size_t)b * a.aux_bs + (size_t)m * a.ld_aux]), acc, *y);
         return;
@@ -306,6 +308,7 @@ extern "C" int dl_dense(const DlDenseArgs* args, void* stream) {
     if (a.M < 1 || a.N < 1 || a.K < 1 || a.batch < 1) { dl_set_error("dl_dense: empty problem"); return -1; }
     if ((a.epi == DL_DENSE_SIGMOID_MUL || a.epi == DL_DENSE_MUL || a.epi == DL_DENSE_ROWGATE_ADD) && a.aux == nullptr) { dl_set_error("dl_dense: the gate epilogue needs aux"); return -1; }
     if (a.epi == DL_DENSE_GLU_CLAMP || a.epi == DL_DENSE_GLU_SILU) { dl_set_error("dl_dense: the paired-column epilogue belongs to the tensor-core GEMM"); return -1; }
+    if (a.bias && a.epi == DL_DENSE_GLU_GELU) { dl_set_error("dl_dense: paired columns take no bias"); return -1; }
     if (a.epi == DL_DENSE_GLU_GELU && (a.N & 1)) { dl_set_error("dl_dense: paired columns need an even number of weight rows"); return -1; }
     cudaStream_t st = (cudaStream_t)stream;
     if (a.wtype == DL_T_BF16) {

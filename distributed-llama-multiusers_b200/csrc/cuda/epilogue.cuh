@@ -213,14 +213,16 @@ DL_DEVINL void epilogue_rows(const DlEpilogue& e, const float* out_s, int out_ld
                 // one gate per row (ROWGATE_ADD) sits at aux[m * ald]; the other ops read aux[m * ald + column]
                 const float* aux = e.dense_aux != nullptr ? e.dense_aux + (size_t)m0 * ald + (op == DL_DENSE_ROWGATE_ADD ? 0 : grow) : nullptr;
                 const float prm = e.dense_param, prm2 = e.dense_param2;
+                const float bias = e.dense_bias != nullptr ? e.dense_bias[grow] : 0.0f;
 #pragma unroll 4
                 for (int m = m_first; m < M; m += m_step) {
-                    float v = out_s[m * out_ld + tid];
+                    float v = out_s[m * out_ld + tid] + bias;
                     if (op == DL_DENSE_RELU2) { v = fmaxf(v, 0.0f); v *= v; }
                     else if (op == DL_DENSE_SIGMOID_MUL) v = aux[m * ald] / (1.0f + expf(-v));
                     else if (op == DL_DENSE_SOFTCAP) v = prm * tanhf(v / prm);
                     else if (op == DL_DENSE_SILU) v = v / (1.0f + expf(-v));
                     else if (op == DL_DENSE_MUL) v = aux[m * ald] * v;
+                    else if (op == DL_DENSE_SCALE) v = prm * v;
                     else if (op == DL_DENSE_XIELU) v = v > 0.0f ? fmaf(prm * v, v, 0.5f * v) : fmaf(prm2, expm1f(v) - v, 0.5f * v);
                     else if (op == DL_DENSE_ROWGATE_ADD) v = fmaf(1.0f / (1.0f + expf(-aux[m * ald])), v, d0[m * ld]);
                     d0[m * ld] = v;

@@ -57,6 +57,41 @@ __global__ void __launch_bounds__(256) mamba_conv_kernel(DlMambaBatch b, const f
     }
 }
 
+// The same with heads of unit length: channels [0, unit_k) are heads of unit_dim channels, a warp each, which leave divided by
+// sqrt(sum of squares + 1e-6) (those of [0, unit_q) times unit_scale too); the other channels in groups of UNIT_REST, a warp each.
+#define UNIT_REST 128
+template <typename WT>
+__global__ void __launch_bounds__(256) conv_unit_kernel(DlMambaBatch b, DlConvArgs a) {
+    __shared__ const float* src[MB_MAX_TAPS];
+    const int m = blockIdx.x, taps = a.taps, lane = threadIdx.x & 31;
+    const WT* w = (const WT*)a.w;
+    const WT* bias = (const WT*)a.bias;
+    if (threadIdx.x < taps) {
+        const int n = b.row_seq[m], q = b.pos[m] - (taps - 1) + threadIdx.x, p0 = b.seq_pos0[n];
+        const float* p = nullptr;
+        if (q >= p0) p = a.in + (size_t)b.seq_rows[b.seq_start[n] + (q - p0)] * a.ld + a.in_off;
+        else if (q >= 0) p = a.conv_state + ((size_t)b.seq_slot[n] * (taps - 1) + (q - p0 + (taps - 1))) * a.channels;
+        src[threadIdx.x] = p;
+    }
+    __syncthreads();
+    const int heads = a.unit_k / a.unit_dim, item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int c0 = item < heads ? item * a.unit_dim : a.unit_k + (item - heads) * UNIT_REST;
+    const int c1 = item < heads ? c0 + a.unit_dim : min(c0 + UNIT_REST, a.channels);
+    float* out = a.out + (size_t)m * a.ld_out;
+    float ss = 0.f;
+    for (int ch = c0 + lane; ch < c1; ch += 32) {
+        float acc = bias ? ld_f(bias + ch) : 0.f;
+        for (int k = 0; k < taps; ++k)
+            if (src[k]) acc = fmaf(ld_f(w + (size_t)ch * taps + k), src[k][ch], acc);
+        if (a.act) acc = silu_f(acc);
+        out[ch] = acc;
+        ss = fmaf(acc, acc, ss);
+    }
+    if (item >= heads) return;
+    const float inv = (c0 < a.unit_q ? a.unit_scale : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
+    for (int ch = c0 + lane; ch < c1; ch += 32) out[ch] *= inv;          // a lane meets its own channels again
+}
+
 // carried inputs after the batch: positions last-(taps-2) .. last of each sequence (runs after the convolution)
 __global__ void __launch_bounds__(256) mamba_conv_carry_kernel(DlMambaBatch b, const float* __restrict__ in, long long ld, int in_off,
                                                                float* __restrict__ conv_state, int channels, int taps) {
@@ -79,7 +114,12 @@ extern "C" int dl_causal_conv(const DlMambaBatch* batch, int M, int n_seq, const
     if (a.out == a.in) { dl_set_error("dl_causal_conv: out must not alias in"); return -1; }
     cudaStream_t st = (cudaStream_t)stream;
     const int gy = (a.channels + 255) / 256;
-    if (a.wtype == DL_T_BF16)
+    if (a.unit_dim > 0) {
+        if (a.residual || a.unit_k % a.unit_dim || a.unit_q % a.unit_dim || a.unit_q > a.unit_k || a.unit_k > a.channels) { dl_set_error("dl_causal_conv: unit heads do not fit"); return -1; }
+        const int items = a.unit_k / a.unit_dim + (a.channels - a.unit_k + UNIT_REST - 1) / UNIT_REST;
+        if (a.wtype == DL_T_BF16) conv_unit_kernel<__nv_bfloat16><<<dim3(M, (items + 7) / 8), 256, 0, st>>>(*batch, a);
+        else conv_unit_kernel<float><<<dim3(M, (items + 7) / 8), 256, 0, st>>>(*batch, a);
+    } else if (a.wtype == DL_T_BF16)
         mamba_conv_kernel<<<dim3(M, gy), 256, 0, st>>>(*batch, a.in, a.ld, a.in_off, (const __nv_bfloat16*)a.w, (const __nv_bfloat16*)a.bias, a.conv_state,
                                                        a.out, a.ld_out, a.channels, a.taps, a.act, a.residual);
     else
@@ -99,6 +139,7 @@ extern "C" int dl_mamba_conv(const DlMambaBatch* batch, int M, int n_seq, const 
     DlConvArgs a;
     a.in = in; a.ld = ld; a.in_off = in_off; a.w = w; a.bias = bias; a.wtype = wtype; a.conv_state = conv_state;
     a.out = out; a.ld_out = channels; a.channels = channels; a.taps = taps; a.act = 1; a.residual = 0;
+    a.unit_dim = a.unit_q = a.unit_k = 0; a.unit_scale = 1.f;
     return dl_causal_conv(batch, M, n_seq, &a, stream);
 }
 

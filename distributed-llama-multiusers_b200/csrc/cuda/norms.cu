@@ -129,8 +129,8 @@ extern "C" int dl_poly_norm(const float* x, long long ldx, float* y, long long l
 }
 
 // ------------------------------------------------------------------------------------------------
-// One step of a residual stream: a row's sum (the stream, plain terms, terms normalised first, a vector for every row), then up
-// to two normed copies of it, as f32 rows or straight into the bf16 activation image of the products that read them.  One
+// One step of a residual stream: a row's sum (the stream, plain or scaled terms, terms normalised first, a vector for every row),
+// then up to two normed copies of it (root mean square, or layer norm with bias), as f32 rows or straight into the bf16 activation image of the products that read them.  One
 // CTA per row; the row stays in shared memory between the sums.  Three dependent passes at most: the roots of the normalised
 // terms, the sum and its root, the copies.
 // ------------------------------------------------------------------------------------------------
@@ -171,25 +171,33 @@ __global__ void __launch_bounds__(RS_THREADS) residual_step_kernel(DlResidualArg
             t = a.w_a[i] * (ra[i] * inv_a);
             if (a.norm_b) t = fmaf(a.w_b[i], rb[i] * inv_b, t);
         }
-        if (p1) t += p1[i];
-        if (p2) t += p2[i];
+        if (p1) t += a.add_scaled ? a.scale1 * p1[i] : p1[i];
+        if (p2) t += a.add_scaled ? a.scale2 * p2[i] : p2[i];
         if (p3) t += p3[i];
         if (xi) t += xi[i];
         if (tb) t += __bfloat162float(tb[i]);
         if (a.vec) t += a.vec[i];
         row_s[i] = t;
         if (a.x) a.x[(size_t)m * a.ldx + i] = t;
-        ss = fmaf(t, t, ss);
+        ss = a.layer_norm ? ss + t : fmaf(t, t, ss);
     }
     if (!a.w1) return;
-    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)dim + a.eps);
+    ss = block_sum(ss, red) / (float)dim;
+    float mean = 0.f;
+    if (a.layer_norm) {
+        mean = ss;
+        float sc = 0.f;
+        for (int i = tid; i < dim; i += RS_THREADS) { const float c = row_s[i] - mean; sc = fmaf(c, c, sc); }
+        ss = block_sum(sc, red) / (float)dim;
+    }
+    const float inv = 1.f / sqrtf(ss + a.eps);
 #pragma unroll 4
     for (int i = tid; i < dim; i += RS_THREADS) {
-        const float t = row_s[i] * inv;
-        const float u = t * a.w1[i];
+        const float t = (row_s[i] - mean) * inv;
+        const float u = fmaf(t, a.w1[i], a.b1 ? a.b1[i] : 0.f);
         if (a.xh1) xh_store(a.xh1, a.ncap, m, i, u); else a.h1[(size_t)m * a.ldh + i] = u;
         if (a.w2) {
-            const float v = t * a.w2[i];
+            const float v = fmaf(t, a.w2[i], a.b2 ? a.b2[i] : 0.f);
             if (a.xh2) xh_store(a.xh2, a.ncap, m, i, v); else a.h2[(size_t)m * a.ldh + i] = v;
         }
     }
@@ -225,7 +233,12 @@ __global__ void __launch_bounds__(RS_THREADS) residual_step_vec_kernel(DlResidua
             if (a.norm_a) u[k] = reinterpret_cast<const float4*>(a.norm_a + src * a.ld_a)[i];
             if (a.norm_b) v[k] = reinterpret_cast<const float4*>(a.norm_b + src * a.ld_b)[i];
             if (a.add1) t[k] = reinterpret_cast<const float4*>(a.add1 + src * a.ld_add1)[i];
-            if (a.add2) t[k] = rs_add(t[k], reinterpret_cast<const float4*>(a.add2 + src * a.ld_add2)[i]);
+            if (a.add_scaled) t[k] = make_float4(a.scale1 * t[k].x, a.scale1 * t[k].y, a.scale1 * t[k].z, a.scale1 * t[k].w);
+            if (a.add2) {
+                const float4 w = reinterpret_cast<const float4*>(a.add2 + src * a.ld_add2)[i];
+                const float s = a.add_scaled ? a.scale2 : 1.f;
+                t[k] = make_float4(fmaf(s, w.x, t[k].x), fmaf(s, w.y, t[k].y), fmaf(s, w.z, t[k].z), fmaf(s, w.w, t[k].w));
+            }
             if (a.x_in) t[k] = rs_add(t[k], reinterpret_cast<const float4*>(a.x_in + src * a.ld_in)[i]);
             if (a.table) {
                 const uint2 w = reinterpret_cast<const uint2*>((const __nv_bfloat16*)a.table + src * a.ld_in)[i];
@@ -267,9 +280,25 @@ __global__ void __launch_bounds__(RS_THREADS) residual_step_vec_kernel(DlResidua
     for (int k = 0; k < NG; ++k) {
         const int i = tid + k * RS_THREADS;
         if (a.x && i < n4) reinterpret_cast<float4*>(a.x + (size_t)m * a.ldx)[i] = t[k];
-        ss = rs_sq(t[k], ss);
+        ss = a.layer_norm ? ss + (t[k].x + t[k].y) + (t[k].z + t[k].w) : rs_sq(t[k], ss);
     }
     if (!a.w1) return;
+    if (a.layer_norm) {                       // the row minus its mean, then the sum of ITS squares
+        ss = warp_sum(ss);
+        if (lane == 0) red[RS_THREADS / 32 + warp] = ss;
+        __syncthreads();
+        float mean = 0.f;
+#pragma unroll
+        for (int w = 0; w < RS_THREADS / 32; ++w) mean += red[RS_THREADS / 32 + w];
+        mean /= (float)dim;
+        ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < NG; ++k)
+            if (tid + k * RS_THREADS < n4) {
+                t[k] = make_float4(t[k].x - mean, t[k].y - mean, t[k].z - mean, t[k].w - mean);
+                ss = rs_sq(t[k], ss);
+            }
+    }
     ss = warp_sum(ss);
     if (lane == 0) red[warp] = ss;
     __syncthreads();
@@ -283,10 +312,12 @@ __global__ void __launch_bounds__(RS_THREADS) residual_step_vec_kernel(DlResidua
         if (i < n4) {
             const float4 w = reinterpret_cast<const float4*>(a.w1)[i];
             const float4 n = make_float4(t[k].x * inv, t[k].y * inv, t[k].z * inv, t[k].w * inv);
-            rs_put(a.h1, a.xh1, a.ncap, m, a.ldh, i, make_float4(n.x * w.x, n.y * w.y, n.z * w.z, n.w * w.w));
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), b1 = a.b1 ? reinterpret_cast<const float4*>(a.b1)[i] : zero;
+            rs_put(a.h1, a.xh1, a.ncap, m, a.ldh, i, make_float4(fmaf(n.x, w.x, b1.x), fmaf(n.y, w.y, b1.y), fmaf(n.z, w.z, b1.z), fmaf(n.w, w.w, b1.w)));
             if (a.w2) {
                 const float4 w2 = reinterpret_cast<const float4*>(a.w2)[i];
-                rs_put(a.h2, a.xh2, a.ncap, m, a.ldh, i, make_float4(n.x * w2.x, n.y * w2.y, n.z * w2.z, n.w * w2.w));
+                const float4 b2 = a.b2 ? reinterpret_cast<const float4*>(a.b2)[i] : zero;
+                rs_put(a.h2, a.xh2, a.ncap, m, a.ldh, i, make_float4(fmaf(n.x, w2.x, b2.x), fmaf(n.y, w2.y, b2.y), fmaf(n.z, w2.z, b2.z), fmaf(n.w, w2.w, b2.w)));
             }
         }
     }
@@ -305,7 +336,7 @@ extern "C" int dl_residual_step(const DlResidualArgs* args, void* stream) {
     const auto al = [](const void* p, long long ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
     const bool vec = a.dim % 4 == 0 && a.dim <= 4 * RS_THREADS * 8 && al(a.x_in, a.ld_in) && al(a.table, a.ld_in) && al(a.add1, a.ld_add1) && al(a.add2, a.ld_add2) &&
                      al(a.add3, a.ld_add3) && al(a.norm_a, a.ld_a) && al(a.norm_b, a.ld_b) && al(a.w_a, 0) && al(a.w_b, 0) && al(a.vec, 0) && al(a.x, a.ldx) &&
-                     al(a.w1, 0) && al(a.w2, 0) && al(a.h1, a.ldh) && al(a.h2, a.ldh);
+                     al(a.w1, 0) && al(a.w2, 0) && al(a.b1, 0) && al(a.b2, 0) && al(a.h1, a.ldh) && al(a.h2, a.ldh);
     if (vec) {
         cudaStream_t st = (cudaStream_t)stream;
         if (a.dim <= 4 * RS_THREADS) residual_step_vec_kernel<1><<<a.M, RS_THREADS, 0, st>>>(a);

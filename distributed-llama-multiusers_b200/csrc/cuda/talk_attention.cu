@@ -21,7 +21,7 @@
 // multiplies the heads of key/value head g, and the page staged for all of them holds every head's keys and values once.  Per page of 32 tokens it stages the keys of every key/value head and the values
 // of head g (cp.async, two buffers: page k + 1 is in flight while page k is multiplied), then per warp
 //     S[16 x 32]  = Q[16 x KH * DP] . K[32 x KH * DP]^T      Q (bf16, staged once per tile) and K by ldmatrix
-//     scale, mask, online softmax in f32 and base 2
+//     scale, soft cap, distance bias, mask, online softmax in f32 and base 2
 //     O[16 x DVP] += P[16 x 32] . V[32 x DVP]                  P from the score registers, V by ldmatrix.trans
 // mma.sync m16n8k16 bf16, f32 accumulators.  DP / DVP: dim / vdim rounded up to the template's sizes, the padding kept at
 // zero in shared memory.  Few tiles (decoding): n_splits CTAs share a tile's pages and talk_merge_kernel combines them.
@@ -38,6 +38,12 @@
 __device__ __forceinline__ float ta_ex2(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+__device__ __forceinline__ float ta_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
 
@@ -90,7 +96,9 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
         pg_hi = min(pg_hi, pg_lo + per - 1);
     }
     const bool active = ALLG ? warp < a.kv_heads * nvb : (warp < NR && warp * 16 < n_rows * rep);
-    const float c1 = a.scale * TA_LOG2E;
+    // soft cap as in window_attention.cu: cap tanh(x / cap) = cap (1 - 2 / (e^(2x / cap) + 1)), in base 2
+    const bool capped = a.softcap > 0.f, biased = a.slope != nullptr;
+    const float c1 = capped ? a.scale * 2.f / a.softcap * TA_LOG2E : a.scale * TA_LOG2E, capK = a.softcap * TA_LOG2E;
 
     // this thread's two stacked rows: s = position-in-tile * rep + head-in-group
     const int s0 = wrow * 16 + gid, s1 = s0 + 8;
@@ -99,6 +107,7 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
     const int pos0 = p_first + r0, pos1 = p_first + r1;
     const int cs0 = a.chunk > 0 ? pos0 / a.chunk * a.chunk : 0, cs1 = a.chunk > 0 ? pos1 / a.chunk * a.chunk : 0;
     const int cs_last = a.chunk > 0 ? p_last / a.chunk * a.chunk : 0;
+    const float sl0 = biased ? a.slope[g * rep + s0 % rep] * TA_LOG2E : 0.f, sl1 = biased ? a.slope[g * rep + s1 % rep] * TA_LOG2E : 0.f;
     // the tile's queries, rounded to bf16, zero-padded per key head
     for (int idx = threadIdx.x; idx < (ALLG ? a.kv_heads : 1) * TA_ROWS * (QDP / 4); idx += THREADS) {
         const int sr = idx / (QDP / 4), col = (idx - sr * (QDP / 4)) * 4;
@@ -170,8 +179,10 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 float s2 = sc[n][e] * c1;
+                const int j = pg_first + n * 8 + tig * 2 + (e & 1);
+                if (capped) s2 = fmaf(-2.f * capK, ta_rcp(ta_ex2(s2) + 1.f), capK);
+                if (biased) s2 = e < 2 ? fmaf(-sl0, (float)(pos0 - j), s2) : fmaf(-sl1, (float)(pos1 - j), s2);
                 if (!whole) {
-                    const int j = pg_first + n * 8 + tig * 2 + (e & 1);
                     const int pr = (e < 2) ? pos0 : pos1;
                     const bool vis = ((e < 2) ? ok0 : ok1) && j <= pr && (a.window == 0 || pr - j < a.window) && j >= ((e < 2) ? cs0 : cs1);
                     s2 = vis ? s2 : -INFINITY;
@@ -240,7 +251,7 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
     }
     if (ok0) {
         float* dst = a.out + (size_t)s_row[r0] * a.ldo + (size_t)(g * rep + s0 % rep) * (WIDE ? a.kv_heads * DV : DV);
-        const float inv = 1.f / l0;
+        const float inv = (a.gate ? sigmoid_f(a.gate[(size_t)s_row[r0] * a.ld_gate + g * rep + s0 % rep]) : 1.f) / l0;
         if (WIDE) {
 #pragma unroll
             for (int v = 0; v < NV; ++v) {
@@ -255,7 +266,7 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
     }
     if (ok1) {
         float* dst = a.out + (size_t)s_row[r1] * a.ldo + (size_t)(g * rep + s1 % rep) * (WIDE ? a.kv_heads * DV : DV);
-        const float inv = 1.f / l1;
+        const float inv = (a.gate ? sigmoid_f(a.gate[(size_t)s_row[r1] * a.ld_gate + g * rep + s1 % rep]) : 1.f) / l1;
         if (WIDE) {
 #pragma unroll
             for (int v = 0; v < NV; ++v) {
@@ -300,7 +311,7 @@ __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, con
             w_s[hg * n_splits + k] = e;
         }
         if (a.sink) l += expf(a.sink[g * rep + hg] - mx);
-        const float inv = 1.f / l;
+        const float inv = (a.gate ? sigmoid_f(a.gate[(size_t)m * a.ld_gate + g * rep + hg]) : 1.f) / l;
         for (int k = 0; k < n_splits; ++k) w_s[hg * n_splits + k] *= inv;
     }
     __syncthreads();
@@ -495,7 +506,7 @@ static int launch_talk(const DlWindowAttnArgs& a, const int* tile_rows, int n_ti
 extern "C" int dl_talk_attention_tc(const DlWindowAttnArgs* args, const int* tile_rows, int n_tiles, int rq, int n_splits,
                                     float* partial, void* stream) {
     const DlWindowAttnArgs& a = *args;
-    if (a.page_size != TA_PAGE || a.softcap != 0.f || a.rope_dims != 0 || a.window < 0 || a.chunk < 0 ||
+    if (a.page_size != TA_PAGE || (a.gate && a.value_heads > 1) || a.rope_dims != 0 || a.window < 0 || a.chunk < 0 ||
         dl_talk_attention_tc_supported(a.heads, a.kv_heads, a.dim, a.vdim, a.key_heads, a.value_heads, a.ctype) != 0 || rq < 1 ||
         rq * (a.heads / a.kv_heads) > TA_MAX_ROWS || (a.ldq & 3) || (a.ldo & 1) || ((uintptr_t)a.q & 15) || ((uintptr_t)a.out & 7)) {
         dl_set_error("dl_talk_attention_tc: sizes not supported (heads %d / %d, dim %d, vdim %d, key heads %d, value heads %d, rq %d)", a.heads, a.kv_heads, a.dim, a.vdim, a.key_heads, a.value_heads, rq);

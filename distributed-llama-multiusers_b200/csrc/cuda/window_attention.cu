@@ -15,7 +15,8 @@
 // written by attn_kv_write_kernel, which can divide every query and key head by its root mean square first.  Two more
 // options of the score side: a chunked mask (chunk > 0: j is visible to i only if floor(j / chunk) == floor(i / chunk);
 // the borders are multiples of `chunk` in sequence positions, wherever a portion starts) and a sink per head: the softmax
-// denominator gets one more term exp(sink_h) that pulls weight away from the keys and contributes no value.
+// denominator gets one more term exp(sink_h) that pulls weight away from the keys and contributes no value.  A distance bias
+// per head (slope_h (i - j), taken off after the cap) and a sigmoid gate per row and head on the output are further options.
 //
 // Kernels: the cache writer, which also turns the queries in place (one launch, cos and sin formed once per row and
 // pair); the per-row attention kernel (exact f32 arithmetic on either cache type; one CTA per
@@ -80,7 +81,7 @@ __global__ void __launch_bounds__(256) window_kv_write_kernel(DlWindowKvArgs a) 
 // (i, i + rope_dims / 2) with rope_half, else (2i, 2i + 1); cos and sin of the row's angles are formed once, in f64),
 // THEN, with qk_norm, the head is divided by sqrt(mean(head^2) + eps): the queries in place, the keys on their way into
 // the cache.  q_norm / k_norm (weights over all heads' columns): in front of the rotary, the row's whole query / key projection is
-// divided by its root mean square and multiplied by the weight.  The values are copied behind the keys.  With `talk` the head mix of the scores is folded into the queries:
+// divided by its root mean square and multiplied by the weight; with head_norm every head by its own (weights of one head's size).  The values are copied behind the keys.  With `talk` the head mix of the scores is folded into the queries:
 // q_mixed[h][c * dim + i] = sum over the query heads g of key/value head c of talk[h][g] q_g[i].
 // Dynamic shared memory: 2 (kv_heads + q_heads) dim + rope_dims + q_heads^2 floats.
 template <typename CT>
@@ -114,7 +115,17 @@ __global__ void __launch_bounds__(256) attn_kv_write_kernel(DlWindowKvArgs a) {
         st_f(line0 + g * head_step + a.dim + i, a.v[(size_t)m * a.ldv + t]);
     }
     __syncthreads();
-    if (a.q_norm != nullptr || a.k_norm != nullptr) {
+    if (a.head_norm) {
+        for (int h = (a.kv_heads - nk) + warp; h < a.kv_heads + nq; h += nw) {      // the warp that turns the head below
+            const float* w = h < a.kv_heads ? a.k_norm : a.q_norm;
+            float* r = raw_s + (size_t)h * D;
+            float ss = 0.f;
+            for (int i = lane; i < D; i += 32) ss = fmaf(r[i], r[i], ss);
+            const float inv = 1.f / sqrtf(warp_sum(ss) / (float)D + a.eps);
+            for (int i = lane; i < D; i += 32) r[i] = r[i] * inv * w[i];
+        }
+        __syncwarp();
+    } else if (a.q_norm != nullptr || a.k_norm != nullptr) {
         __shared__ float red[32];
         for (int part = 0; part < 2; ++part) {                // the keys, then the queries
             const float* w = part ? a.q_norm : a.k_norm;
@@ -178,6 +189,7 @@ extern "C" int dl_window_kv_write(const DlWindowKvArgs* args, int M, void* strea
     if (a.vdim > 0) {
         if ((a.k == nullptr) != (a.v == nullptr) || (a.k == nullptr && a.q == nullptr)) { dl_set_error("dl_window_kv_write: keys and values come together, or the queries alone"); return -1; }
         if (a.rope_dims < 0 || a.rope_dims > a.dim || (a.rope_dims & 1) || a.vdim < 1 || a.page_size != WA_PAGE) { dl_set_error("dl_window_kv_write: bad sizes (rope_dims %d, dim %d, vdim %d)", a.rope_dims, a.dim, a.vdim); return -1; }
+        if (a.head_norm && ((a.q && !a.q_norm) || (a.k && !a.k_norm))) { dl_set_error("dl_window_kv_write: head_norm needs q_norm and k_norm"); return -1; }
         if (a.talk != nullptr && (a.q == nullptr || a.q_mixed == nullptr || a.q_heads % a.kv_heads)) { dl_set_error("dl_window_kv_write: the head mix needs q, q_mixed and whole groups of heads"); return -1; }
         const int nq_ = a.q ? a.q_heads : 0;
         const size_t smem = ((size_t)2 * (a.kv_heads + nq_) * a.dim + a.rope_dims + (a.talk ? (size_t)nq_ * nq_ : 0)) * sizeof(float);
@@ -254,6 +266,7 @@ __global__ void window_attention_kernel(DlWindowAttnArgs a) {
             for (int d = 0; d < QD; ++d) s = fmaf(qh[d], row[d], s);
             s *= a.scale;
             if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+            if (a.slope) s -= a.slope[g * rep + h] * (float)(pos - pg * WA_PAGE - lane);
             if (!vis) s = -INFINITY;
             const float m_old = ml[2 * h], m_new = fmaxf(m_old, warp_max(s));
             const float p = vis ? expf(s - m_new) : 0.f;
@@ -278,6 +291,7 @@ __global__ void window_attention_kernel(DlWindowAttnArgs a) {
         const int h = t / DV;
         float l = ml[2 * h + 1];
         if (a.sink) l += expf(a.sink[g * rep + h] - ml[2 * h]);
+        if (a.gate) l /= sigmoid_f(a.gate[(size_t)m * a.ld_gate + g * rep + h]);
         if (wide) a.out[(size_t)m * a.ldo + ((size_t)(g * rep + h) * a.kv_heads + vg) * DV + (t - h * DV)] = acc[t] / l;
         else a.out[(size_t)m * a.ldo + (size_t)g * rep * DV + t] = acc[t] / l;
     }
@@ -286,7 +300,7 @@ __global__ void window_attention_kernel(DlWindowAttnArgs a) {
 static int window_args_ok(const DlWindowAttnArgs& a, const char* who) {
     if (a.heads < 1 || a.kv_heads < 1 || a.heads % a.kv_heads || a.dim < 1 || a.rope_dims > a.dim || a.window < 0 || a.page_size != WA_PAGE ||
         a.vdim < 0 || a.chunk < 0 || (a.vdim > 0 && a.rope_dims != 0) || (a.key_heads > 1 && (a.key_heads != a.kv_heads || a.vdim < 1)) ||
-        (a.value_heads > 1 && (a.value_heads != a.kv_heads || a.vdim < 1 || a.key_heads > 1))) {
+        (a.value_heads > 1 && (a.value_heads != a.kv_heads || a.vdim < 1 || a.key_heads > 1 || a.gate))) {
         dl_set_error("%s: bad shape (heads %d / %d, dim %d, rotary %d, window %d, page %d)", who, a.heads, a.kv_heads, a.dim, a.rope_dims, a.window, a.page_size);
         return -1;
     }
@@ -381,7 +395,7 @@ __global__ void __launch_bounds__(128, 4) window_attention_mma_kernel(DlWindowAt
         pg_hi = min(pg_hi, pg_lo + per - 1);
     }
     const bool active = warp * 16 < n_rows * rep;
-    const bool capped = a.softcap > 0.f;
+    const bool capped = a.softcap > 0.f, biased = a.slope != nullptr;
     const float c1 = capped ? a.scale * 2.f / a.softcap * WM_LOG2E : a.scale * WM_LOG2E;
     const float capK = a.softcap * WM_LOG2E;
 
@@ -392,6 +406,7 @@ __global__ void __launch_bounds__(128, 4) window_attention_mma_kernel(DlWindowAt
     const int pos0 = p_first + r0, pos1 = p_first + r1;
     const int cs0 = a.chunk > 0 ? pos0 / a.chunk * a.chunk : 0, cs1 = a.chunk > 0 ? pos1 / a.chunk * a.chunk : 0;      // first position of the row's chunk
     const int cs_last = a.chunk > 0 ? p_last / a.chunk * a.chunk : 0;
+    const float sl0 = biased ? a.slope[g * rep + s0 % rep] * WM_LOG2E : 0.f, sl1 = biased ? a.slope[g * rep + s1 % rep] * WM_LOG2E : 0.f;
     // the tile's queries, rounded to bf16, into shared memory (A fragments come from there by ldmatrix: registers are
     // what limits the CTAs per SM)
     for (int idx = threadIdx.x; idx < WM_ROWS * (D / 4); idx += 128) {
@@ -453,8 +468,9 @@ __global__ void __launch_bounds__(128, 4) window_attention_mma_kernel(DlWindowAt
             for (int e = 0; e < 4; ++e) {
                 float s2 = sc[n][e] * c1;
                 if (capped) s2 = fmaf(-2.f * capK, fast_rcp(fast_ex2(s2) + 1.f), capK);
+                const int j = pg_first + n * 8 + tig * 2 + (e & 1);
+                if (biased) s2 = e < 2 ? fmaf(-sl0, (float)(pos0 - j), s2) : fmaf(-sl1, (float)(pos1 - j), s2);
                 if (!whole) {
-                    const int j = pg_first + n * 8 + tig * 2 + (e & 1);
                     const int pr = (e < 2) ? pos0 : pos1;
                     const bool vis = ((e < 2) ? ok0 : ok1) && j <= pr && (a.window == 0 || pr - j < a.window) && j >= ((e < 2) ? cs0 : cs1);
                     s2 = vis ? s2 : -INFINITY;
@@ -524,13 +540,13 @@ __global__ void __launch_bounds__(128, 4) window_attention_mma_kernel(DlWindowAt
     }
     if (ok0) {
         float* dst = a.out + (size_t)s_row[r0] * a.ldo + (size_t)(g * rep + s0 % rep) * D;
-        const float inv = 1.f / l0;
+        const float inv = (a.gate ? sigmoid_f(a.gate[(size_t)s_row[r0] * a.ld_gate + g * rep + s0 % rep]) : 1.f) / l0;
 #pragma unroll
         for (int v = 0; v < NV; ++v) *reinterpret_cast<float2*>(dst + v * 8 + tig * 2) = make_float2(o[v][0] * inv, o[v][1] * inv);
     }
     if (ok1) {
         float* dst = a.out + (size_t)s_row[r1] * a.ldo + (size_t)(g * rep + s1 % rep) * D;
-        const float inv = 1.f / l1;
+        const float inv = (a.gate ? sigmoid_f(a.gate[(size_t)s_row[r1] * a.ld_gate + g * rep + s1 % rep]) : 1.f) / l1;
 #pragma unroll
         for (int v = 0; v < NV; ++v) *reinterpret_cast<float2*>(dst + v * 8 + tig * 2) = make_float2(o[v][2] * inv, o[v][3] * inv);
     }
@@ -564,7 +580,7 @@ __global__ void __launch_bounds__(128) window_merge_kernel(DlWindowAttnArgs a, c
             w_s[hg * n_splits + k] = e;
         }
         if (a.sink) l += expf(a.sink[g * rep + hg] - mx);
-        const float inv = 1.f / l;
+        const float inv = (a.gate ? sigmoid_f(a.gate[(size_t)m * a.ld_gate + g * rep + hg]) : 1.f) / l;
         for (int k = 0; k < n_splits; ++k) w_s[hg * n_splits + k] *= inv;
     }
     __syncthreads();

@@ -63,6 +63,7 @@ class DlEpilogue(C.Structure):
         ("dense_param2", C.c_float),
         ("dense_xh", C.c_void_p),
         ("dense_ncap", C.c_int),
+        ("dense_bias", C.c_void_p),
     ]
 
 
@@ -217,7 +218,8 @@ def check(rc: int, what: str = ""):
 # ---- hyper-connections, routed experts)
 T_F32, T_BF16 = 0, 1
 DENSE_STORE, DENSE_RELU2, DENSE_SIGMOID_MUL, DENSE_SOFTCAP, DENSE_SILU, DENSE_GLU_CLAMP = 0, 1, 2, 3, 4, 5
-DENSE_MUL, DENSE_XIELU, DENSE_ROWGATE_ADD, DENSE_GLU_SILU, DENSE_GLU_GELU = 6, 7, 8, 9, 10
+DENSE_MUL, DENSE_XIELU, DENSE_ROWGATE_ADD, DENSE_GLU_SILU, DENSE_GLU_GELU, DENSE_SCALE = 6, 7, 8, 9, 10, 11
+GATE_LOWER, GATE_ROOT_SIGMOID, GATE_EXP_EXP, GATE_SOFTPLUS = 0, 1, 2, 3
 
 
 class DlDenseArgs(C.Structure):
@@ -228,7 +230,7 @@ class DlDenseArgs(C.Structure):
                 ("M", C.c_int), ("N", C.c_int), ("K", C.c_int), ("batch", C.c_int),
                 ("round_x", C.c_int), ("epi", C.c_int),
                 ("aux", C.c_void_p), ("ld_aux", C.c_longlong), ("aux_bs", C.c_longlong),
-                ("param", C.c_float), ("param2", C.c_float)]
+                ("param", C.c_float), ("param2", C.c_float), ("bias", C.c_void_p)]
 
 
 class DlNormArgs(C.Structure):
@@ -301,7 +303,7 @@ class DlWindowKvArgs(C.Structure):
                 ("max_pages", C.c_int), ("page_size", C.c_int), ("cache", C.c_void_p), ("ctype", C.c_int),
                 ("v", C.c_void_p), ("ldv", C.c_longlong), ("vdim", C.c_int), ("qk_norm", C.c_int), ("eps", C.c_float),
                 ("rope_half", C.c_int), ("talk", C.c_void_p), ("q_mixed", C.c_void_p), ("ld_qm", C.c_longlong),
-                ("q_norm", C.c_void_p), ("k_norm", C.c_void_p)]
+                ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("head_norm", C.c_int)]
 
 
 class DlWindowAttnArgs(C.Structure):
@@ -311,7 +313,8 @@ class DlWindowAttnArgs(C.Structure):
                 ("scale", C.c_float), ("softcap", C.c_float), ("window", C.c_int),
                 ("pos", C.c_void_p), ("slot", C.c_void_p), ("block_table", C.c_void_p),
                 ("max_pages", C.c_int), ("page_size", C.c_int), ("cache", C.c_void_p), ("ctype", C.c_int),
-                ("vdim", C.c_int), ("chunk", C.c_int), ("sink", C.c_void_p), ("key_heads", C.c_int), ("value_heads", C.c_int)]
+                ("vdim", C.c_int), ("chunk", C.c_int), ("sink", C.c_void_p), ("key_heads", C.c_int), ("value_heads", C.c_int),
+                ("slope", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_longlong)]
 
 
 class DlConvArgs(C.Structure):
@@ -319,7 +322,8 @@ class DlConvArgs(C.Structure):
     _fields_ = [("in_", C.c_void_p), ("ld", C.c_longlong), ("in_off", C.c_int),
                 ("w", C.c_void_p), ("bias", C.c_void_p), ("wtype", C.c_int), ("conv_state", C.c_void_p),
                 ("out", C.c_void_p), ("ld_out", C.c_longlong),
-                ("channels", C.c_int), ("taps", C.c_int), ("act", C.c_int), ("residual", C.c_int)]
+                ("channels", C.c_int), ("taps", C.c_int), ("act", C.c_int), ("residual", C.c_int),
+                ("unit_dim", C.c_int), ("unit_q", C.c_int), ("unit_k", C.c_int), ("unit_scale", C.c_float)]
 
 
 class DlLightningArgs(C.Structure):
@@ -335,8 +339,17 @@ class DlGatedArgs(C.Structure):
     _fields_ = [("q", C.c_void_p), ("ldq", C.c_longlong), ("q_scale", C.c_float), ("q_silu", C.c_int),
                 ("k", C.c_void_p), ("ldk", C.c_longlong), ("v", C.c_void_p), ("ldv", C.c_longlong),
                 ("f", C.c_void_p), ("ldf", C.c_longlong), ("f_bias", C.c_void_p), ("lower", C.c_void_p),
+                ("gate", C.c_int), ("inv_tau", C.c_float), ("rate", C.c_void_p), ("bonus", C.c_void_p), ("beta", C.c_void_p), ("ld_beta", C.c_longlong),
+                ("k_heads", C.c_int),
                 ("log_keep", C.c_void_p), ("put", C.c_void_p), ("y", C.c_void_p), ("ld_y", C.c_longlong), ("den", C.c_void_p),
                 ("state", C.c_void_p), ("n_state", C.c_void_p), ("n_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int)]
+
+
+class DlShiftArgs(C.Structure):
+    """Mirror of ``DlShiftArgs``."""
+    _fields_ = [("h", C.c_void_p), ("ldh", C.c_longlong), ("mu", C.c_void_p), ("n_mix", C.c_int), ("width", C.c_int),
+                ("out", C.c_void_p), ("out_step", C.c_longlong), ("ld_out", C.c_longlong),
+                ("xh", C.c_void_p), ("xh_step", C.c_longlong), ("ncap", C.c_int), ("state", C.c_void_p)]
 
 
 class DlMlstmGatesArgs(C.Structure):
@@ -350,7 +363,8 @@ class DlHeadNormArgs(C.Structure):
     """Mirror of ``DlHeadNormArgs``."""
     _fields_ = [("y", C.c_void_p), ("ld_y", C.c_longlong), ("den", C.c_void_p), ("floor_", C.c_void_p), ("w", C.c_void_p),
                 ("w_full", C.c_int), ("gate", C.c_void_p), ("ld_gate", C.c_longlong), ("out", C.c_void_p), ("ld_out", C.c_longlong),
-                ("xh", C.c_void_p), ("ncap", C.c_int), ("M", C.c_int), ("n_heads", C.c_int), ("vdim", C.c_int), ("eps", C.c_float)]
+                ("xh", C.c_void_p), ("ncap", C.c_int), ("M", C.c_int), ("n_heads", C.c_int), ("vdim", C.c_int), ("eps", C.c_float),
+                ("gate_silu", C.c_int)]
 
 
 class DlSelectiveArgs(C.Structure):
@@ -370,7 +384,9 @@ class DlResidualArgs(C.Structure):
                 ("norm_a", C.c_void_p), ("w_a", C.c_void_p), ("norm_b", C.c_void_p), ("w_b", C.c_void_p),
                 ("ld_a", C.c_longlong), ("ld_b", C.c_longlong), ("vec", C.c_void_p), ("x", C.c_void_p), ("ldx", C.c_longlong),
                 ("w1", C.c_void_p), ("h1", C.c_void_p), ("xh1", C.c_void_p), ("w2", C.c_void_p), ("h2", C.c_void_p), ("xh2", C.c_void_p),
-                ("ldh", C.c_longlong), ("ncap", C.c_int), ("M", C.c_int), ("dim", C.c_int), ("eps", C.c_float)]
+                ("ldh", C.c_longlong), ("ncap", C.c_int), ("M", C.c_int), ("dim", C.c_int), ("eps", C.c_float),
+                ("layer_norm", C.c_int), ("b1", C.c_void_p), ("b2", C.c_void_p),
+                ("add_scaled", C.c_int), ("scale1", C.c_float), ("scale2", C.c_float)]
 
 
 class DlMoeSelectArgs(C.Structure):
@@ -461,6 +477,11 @@ def layers_lib():
     L.dl_gated_scan_chunked_supported.argtypes = [i32, i32, i32]
     L.dl_gated_chunk_floats.argtypes = [i32, i32, i32, i32, i32]
     L.dl_gated_chunk_floats.restype = i64
+    L.dl_delta_scan_chunked_supported.argtypes = [i32, i32]
+    L.dl_delta_chunk_floats.argtypes = [i32, i32, i32, i32, i32]
+    L.dl_delta_chunk_floats.restype = i64
+    L.dl_delta_scan_chunked.argtypes = [C.POINTER(DlMambaBatch), i32, i32, C.POINTER(DlGatedArgs), vp, i32, vp, i64, vp]
+    L.dl_token_shift.argtypes = [C.POINTER(DlMambaBatch), i32, C.POINTER(DlShiftArgs), vp]
     L.dl_mlstm_gates.argtypes = [C.POINTER(DlMambaBatch), i32, i32, C.POINTER(DlMlstmGatesArgs), vp]
     L.dl_head_norm.argtypes = [C.POINTER(DlHeadNormArgs), vp]
     L.dl_selective_scan.argtypes = [C.POINTER(DlMambaBatch), i32, i32, C.POINTER(DlSelectiveArgs), vp]
@@ -483,7 +504,7 @@ def layers_lib():
                  "dl_moe_combine", "dl_xh_gather_rows", "dl_gemm_wh_tc_grouped", "dl_window_tc_rows", "dl_window_attention_tc_supported",
                  "dl_window_attention_tc", "dl_talk_attention_tc_supported", "dl_talk_attention_tc", "dl_talk_tc_tile_rows", "dl_causal_conv", "dl_poly_norm", "dl_lightning_scan", "dl_lightning_scan_chunked",
                  "dl_gated_scan", "dl_gated_scan_chunked", "dl_gated_scan_supported", "dl_gated_scan_chunked_supported", "dl_mlstm_gates", "dl_head_norm",
-                 "dl_selective_scan", "dl_selective_scan_supported", "dl_selective_scan_chunked", "dl_selective_scan_chunked_supported", "dl_residual_step", "dl_talk_mix"):
+                 "dl_delta_scan_chunked", "dl_delta_scan_chunked_supported", "dl_token_shift", "dl_selective_scan", "dl_selective_scan_supported", "dl_selective_scan_chunked", "dl_selective_scan_chunked_supported", "dl_residual_step", "dl_talk_mix"):
         getattr(L, name).restype = i32
     _layers = L
     return L

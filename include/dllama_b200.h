@@ -31,7 +31,8 @@ enum { DL_DENSE_STORE = 0, DL_DENSE_RELU2 = 1, DL_DENSE_SIGMOID_MUL = 2, DL_DENS
        DL_DENSE_ROWGATE_ADD = 8  /* y[m][n] + sigmoid(aux[m * ld_aux]) * (.): one gate per row, added to what y holds */,
        DL_DENSE_GLU_SILU = 9     /* tensor-core epilogue only, columns paired like GLU_CLAMP: silu(gate) * up        */,
        DL_DENSE_GLU_GELU = 10    /* columns paired like GLU_CLAMP (weight rows gate_0, up_0, gate_1, ...): gelu_tanh(gate) * up; every
-                                    product kernel has it, the output has half as many columns as the weight has rows   */ };
+                                    product kernel has it, the output has half as many columns as the weight has rows   */,
+       DL_DENSE_SCALE = 11       /* param * (.)                                                                      */ };
 
 typedef struct {
     int kind;
@@ -75,6 +76,7 @@ typedef struct {
     float dense_param2;
     uint8_t* dense_xh;                /* DL_DENSE_GLU_GELU: the result leaves as the next product's bf16 activation image (its   */
     int dense_ncap;                   /* width a multiple of 128; ncap rows) instead of f32 rows                                */
+    const float* dense_bias;          /* [rows of the weight] or NULL: added to the value before the op (not with the paired-column ops) */
 } DlEpilogue;
 
 /* Fused activation producer for dl_gemv_q40: the kernel itself computes
@@ -324,7 +326,8 @@ int dl_peer_barrier(uint32_t* const* flags_on_peers /*host array*/, uint32_t* my
  * operand is rounded to bf16 on load (bf16 mode).  DL_DENSE_SIGMOID_MUL: aux[m][n] * sigmoid(.);
  * DL_DENSE_SOFTCAP: param * tanh(. / param); DL_DENSE_SILU: . * sigmoid(.); DL_DENSE_MUL: aux[m][n] * (.);
  * DL_DENSE_XIELU: param z^2 + z / 2 for z > 0, else param2 (exp(z) - 1 - z) + z / 2;
- * DL_DENSE_ROWGATE_ADD: Y[m][n] + sigmoid(aux[m * ld_aux]) * (.) (Y is read, then written). */
+ * DL_DENSE_ROWGATE_ADD: Y[m][n] + sigmoid(aux[m * ld_aux]) * (.) (Y is read, then written).
+ * bias (NULL: none): added to the product before the op; not with the paired-column ops. */
 typedef struct {
     const void* W; int wtype; long long ldw, w_bs;
     const float* X; long long ldx, x_bs;
@@ -335,6 +338,7 @@ typedef struct {
     const float* aux; long long ld_aux, aux_bs;
     float param;
     float param2;
+    const float* bias;                       /* [batch][N] f32 */
 } DlDenseArgs;
 int dl_dense(const DlDenseArgs* args /*host*/, void* stream);
 /* x[m][c][dim] = scale * table[tokens[m]] for c < copies */
@@ -427,13 +431,15 @@ int dl_mamba_conv(const DlMambaBatch* batch /*host*/, int M, int n_seq, const fl
                   const void* w, const void* bias, int wtype, float* conv_state, float* out, int channels, int taps,
                   void* stream);
 /* The general form: out[m][ch] = act(bias[ch] + conv) (+ in[m][ch] if residual); bias may be NULL; act 0: none, 1: silu.
- * out must not alias in. */
+ * out must not alias in.  unit_dim > 0: channels [0, unit_k) are heads of unit_dim channels; every head leaves divided by
+ * sqrt(sum of its squares + 1e-6), the heads of channels [0, unit_q) also multiplied by unit_scale. */
 typedef struct {
     const float* in; long long ld; int in_off;
     const void* w; const void* bias; int wtype;     /* w [channels][taps] */
     float* conv_state;                              /* [n_slots][taps - 1][channels] f32 */
     float* out; long long ld_out;
     int channels, taps, act, residual;
+    int unit_dim, unit_q, unit_k; float unit_scale;
 } DlConvArgs;
 int dl_causal_conv(const DlMambaBatch* batch /*host*/, int M, int n_seq, const DlConvArgs* args /*host*/, void* stream);
 typedef struct {
@@ -498,7 +504,13 @@ int dl_hyper_step(const DlHyperArgs* args /*host*/, void* stream);
 
 /* ---- linear attention with data-dependent gates (gated_scan.cu) -------------------------------------------------------
  * Per head, state S [dim][vdim] f32 per slot, one row of the batch after another of a sequence (fresh at position 0):
- *   channel form (f != NULL):  z = f + f_bias, g = lower + (1 - lower) sigmoid(z) per channel, S <- diag(g) S + (1 - g) v^T
+ *   channel form (f != NULL):  z = f + f_bias per channel (f_bias may be NULL), a decay g per channel by `gate`:
+ *     DL_GATE_LOWER         g = lower + (1 - lower) sigmoid(z), S <- diag(g) S + (1 - g) v^T   (no k)
+ *     DL_GATE_ROOT_SIGMOID  g = sigmoid(z)^(1 / tau)            S <- diag(g) S + k v^T
+ *     DL_GATE_EXP_EXP       g = exp(-exp(z))                    the same
+ *     DL_GATE_SOFTPLUS      g = exp(-rate_h softplus(z))        the same
+ *   bonus != NULL: the row reads the state ahead of its own update, y = S_old^T q + (sum_d q bonus k) v
+ *   beta != NULL (delta rule): S <- diag(g) S, u = sigmoid(beta_h) (v - S^T k), S <- S + k u^T
  *   head form (log_keep):      S <- e^log_keep S + put k v^T,  n <- e^log_keep n + put k,  den = n . q
  * then y = S^T q with q = silu(q) (q_silu) or q_scale * q.  The gates of the head form come from dl_mlstm_gates. */
 typedef struct {
@@ -506,12 +518,17 @@ typedef struct {
     const float* k; long long ldk;           /* head form */
     const float* v; long long ldv;
     const float* f; long long ldf; const float* f_bias; const float* lower;   /* channel form; f_bias, lower [heads * dim] */
+    int gate; float inv_tau; const float* rate;      /* channel form: DL_GATE_*; 1 / tau; rate [heads] f32 */
+    const float* bonus;                      /* [heads * dim] or NULL */
+    const float* beta; long long ld_beta;    /* [M] rows of `heads` numbers, or NULL */
+    int k_heads;                             /* q and k have this many heads (0: n_heads); head h reads head h / (n_heads / k_heads) */
     const float* log_keep; const float* put; /* head form: [M][heads] */
     float* y; long long ld_y;                /* [M][heads * vdim] */
     float* den;                              /* head form: [M][heads] */
     float* state; float* n_state;            /* [n_slots][heads][dim][vdim], head form also [n_slots][heads][dim] */
     int n_heads, dim, vdim;
 } DlGatedArgs;
+enum { DL_GATE_LOWER = 0, DL_GATE_ROOT_SIGMOID = 1, DL_GATE_EXP_EXP = 2, DL_GATE_SOFTPLUS = 3 };
 int dl_gated_scan_supported(int dim, int vdim);
 int dl_gated_scan(const DlMambaBatch* batch /*host*/, int n_seq, const DlGatedArgs* args /*host*/, void* stream);
 /* Long portions: chunks of DL_GATED_CHUNK rows of a sequence in parallel (three launches), as dl_lightning_scan_chunked */
@@ -520,6 +537,23 @@ int dl_gated_scan_chunked_supported(int dim, int vdim, int channel);
 long long dl_gated_chunk_floats(int M, int n_seq, int n_heads, int dim, int vdim);
 int dl_gated_scan_chunked(const DlMambaBatch* batch /*host*/, int n_seq, int max_chunks, const DlGatedArgs* args /*host*/,
                           float* scratch, int chunk_slots, void* stream);
+/* The delta rule in chunks (delta_scan.cu), three launches: every chunk's triangular system, the walk over a sequence's chunks,
+ * the chunks' outputs.  u: [M] rows of heads * vdim f32 (the corrected values); scratch: dl_delta_chunk_floats() f32. */
+int dl_delta_scan_chunked_supported(int dim, int vdim);
+long long dl_delta_chunk_floats(int M, int n_seq, int n_heads, int dim, int vdim);
+int dl_delta_scan_chunked(const DlMambaBatch* batch /*host*/, int n_seq, int max_chunks, const DlGatedArgs* args /*host*/,
+                          float* scratch, int chunk_slots, float* u, long long ld_u, void* stream);
+/* Mixes of a row with the row ahead of it in its sequence (zeros ahead of the first): mix s of row m = h + (h_prev - h) mu[s],
+ * to out[s * out_step + m * ld_out] (f32) or, with xh, into activation images xh_step bytes apart.  state [n_slots][width] f32
+ * carries every slot's last h and is updated. */
+typedef struct {
+    const float* h; long long ldh;
+    const float* mu; int n_mix, width;       /* [n_mix][width] f32 */
+    float* out; long long out_step, ld_out;
+    uint8_t* xh; long long xh_step; int ncap;
+    float* state;
+} DlShiftArgs;
+int dl_token_shift(const DlMambaBatch* batch /*host*/, int M, const DlShiftArgs* args /*host*/, void* stream);
 /* Gates of a matrix memory with a running maximum u (one f32 per slot and head, 0 ahead of the first row): a = cap tanh((zi +
  * bi) / cap), b = log sigmoid(cap tanh((zf + bf) / cap)), u' = max(b + u, a), log_keep = b + u - u', put = e^(a - u'),
  * floor = e^-u'.  zi, zf: [M] rows of n_heads numbers; outputs [M][n_heads]. */
@@ -532,8 +566,8 @@ typedef struct {
 } DlMlstmGatesArgs;
 int dl_mlstm_gates(const DlMambaBatch* batch /*host*/, int n_seq, int longest, const DlMlstmGatesArgs* args /*host*/, void* stream);
 /* Per row and head of vdim numbers: o = y / (max(|den|, floor) + 1e-6) (den NULL: y), then o / sqrt(mean(o^2) + eps) * w
- * (w [vdim], or [n_heads * vdim] with w_full), then * sigmoid(gate) (gate NULL: none).  To out (f32) or, with xh, into the
- * tcgen05 GEMM's activation image. */
+ * (w [vdim], or [n_heads * vdim] with w_full), then * sigmoid(gate), or gate * sigmoid(gate) with gate_silu (gate NULL: none).
+ * To out (f32) or, with xh, into the tcgen05 GEMM's activation image. */
 typedef struct {
     const float* y; long long ld_y;
     const float* den; const float* floor_;
@@ -541,6 +575,7 @@ typedef struct {
     const float* gate; long long ld_gate;
     float* out; long long ld_out; uint8_t* xh; int ncap;
     int M, n_heads, vdim; float eps;
+    int gate_silu;
 } DlHeadNormArgs;
 int dl_head_norm(const DlHeadNormArgs* args /*host*/, void* stream);
 
@@ -571,7 +606,9 @@ int dl_selective_scan_chunked(const DlMambaBatch* batch /*host*/, int n_seq, int
 /* ---- one step of a residual stream (norms.cu) ------------------------------------------------------------------------
  *   x[m] = x_in + add1 + add2 + add3 + w_a * unit(norm_a) + w_b * unit(norm_b) + vec    unit(v) = v / sqrt(mean(v^2) + eps)
  *   h1[m] = w1 * unit(x[m]),  h2[m] = w2 * unit(x[m])       each to f32 rows or into an activation image (xh1 / xh2)
- * Every term may be absent (NULL); x NULL: the sum is not stored; rows: all terms but vec are those of row rows[m] (a gather). */
+ * Every term may be absent (NULL); x NULL: the sum is not stored; rows: all terms but vec are those of row rows[m] (a gather).
+ * add_scaled: scale1 * add1 + scale2 * add2 instead of their plain sum.  layer_norm: h1[m] = w1 * c / sqrt(mean(c^2) + eps) + b1
+ * with c = x[m] - mean(x[m]), h2 likewise. */
 typedef struct {
     const float* x_in; long long ld_in; const int* rows;
     const void* table;                        /* instead of x_in: bf16 rows (an embedding table, rows = the tokens) */
@@ -583,6 +620,8 @@ typedef struct {
     const float* w2; float* h2; uint8_t* xh2;
     long long ldh; int ncap;
     int M, dim; float eps;
+    int layer_norm; const float* b1; const float* b2;
+    int add_scaled; float scale1, scale2;
 } DlResidualArgs;
 int dl_residual_step(const DlResidualArgs* args /*host*/, void* stream);
 
@@ -612,6 +651,7 @@ typedef struct {
     /* root mean square over the WHOLE query / key projection of a row (all heads' columns at once), in front of the rotary:
      * x * w / sqrt(mean(x^2) + eps), w [q_heads * dim] / [kv_heads * dim] f32; NULL: none */
     const float* q_norm; const float* k_norm;
+    int head_norm;                            /* 1: q_norm / k_norm are [dim] and every head is normed by itself, in front of the rotary */
 } DlWindowKvArgs;
 int dl_window_kv_write(const DlWindowKvArgs* args /*host*/, int M, void* stream);
 /* out[m][h] = sum_j softmax_j(cap(scale q[m][h] . key_j)) value_j over the positions j with 0 <= pos[m] - j < window
@@ -634,6 +674,8 @@ typedef struct {
     int value_heads;                          /* 0 / 1: a head's values are its key/value head's; kv_heads: every head's weights meet the
                                                  values of ALL key/value heads, out [M][heads][kv_heads * vdim] (weights mixed across heads
                                                  after the softmax, see dl_talk_mix).  Not together with key_heads */
+    const float* slope;                       /* [heads] or NULL: slope[h] * (pos[m] - j) is taken off the (capped) score of position j */
+    const float* gate; long long ld_gate;     /* [M] rows of `heads` numbers or NULL: head h leaves multiplied by sigmoid(gate[m][h]) */
 } DlWindowAttnArgs;
 int dl_window_attention(const DlWindowAttnArgs* args /*host*/, int M, void* stream);
 
@@ -696,7 +738,7 @@ int dl_window_attention_tc(const DlWindowAttnArgs* args /*host*/, const int* til
  * c(h) = h / (heads / kv_heads).  To out (f32) or, with xh, into the tcgen05 GEMM's activation image. */
 int dl_talk_mix(const float* wide, const float* talk, int M, int heads, int kv_heads, int vdim, float* out, long long ld_out,
                 uint8_t* xh, int ncap, void* stream);
-/* The tile kernel for values of a width of their own (vdim > 0, any multiple of 8 up to 128; rope_dims 0, no soft cap) and
+/* The tile kernel for values of a width of their own (vdim > 0, any multiple of 8 up to 128; rope_dims 0) and
  * for head-mixed scores (key_heads = kv_heads: q [M][heads][kv_heads * dim], talk_attention.cu).  Tiles as above. */
 int dl_talk_attention_tc_supported(int heads, int kv_heads, int dim, int vdim, int key_heads, int value_heads, int ctype);
 /* stacked (row x head-of-a-group) rows per tile for portions of `longest` rows: 16 (decoding), 64 or 128; rq = that / (heads / kv_heads) */
