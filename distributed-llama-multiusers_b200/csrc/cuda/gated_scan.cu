@@ -1,7 +1,10 @@
 // Linear attention whose decay depends on the data.  Per head, state S [dim][vdim] f32, one per sequence slot:
 //   channel form:  S <- diag(f_t) S + (1 - f_t) v_t^T                    f = lower + (1 - lower) sigmoid(z + bias), per channel of q
+//                  S <- diag(f_t) S + k_t v_t^T                          other gates (DL_GATE_*) come with keys of their own
+//   ahead form:    channel form that reads first: y_t = S_(t-1)^T q_t + (sum_d q_t bonus k_t) v_t
+//   delta form:    S <- diag(f_t) S, u = sigmoid(beta_t) (v_t - S^T k_t), S <- S + k_t u^T  (its chunked kernels: delta_scan.cu)
 //   head form:     S <- e^l_t S + p_t k_t v_t^T,  n <- e^l_t n + p_t k_t   one log decay l and one weight p per head and token
-//   both:          y_t = S_t^T q_t  (and den_t = n_t . q_t in the head form)
+//   all but ahead: y_t = S_t^T q_t  (and den_t = n_t . q_t in the head form)
 // Everything is f32.  A batch is any mix of sequences with one or more consecutive rows each (DlMambaBatch); a sequence
 // whose first row is position 0 starts from zeros whatever its slot held.
 //
@@ -14,46 +17,29 @@
 // sub-blocks of 16; between two sub-blocks the decay splits into three factors <= 1 (from the column's row to the end of its
 // block, over the blocks between, from the start of the row's block to the row), inside a sub-block it is the running
 // product itself.  Per head the log decays of a chunk are summed in f64.
-#include "layer_common.cuh"
-#include "../../../include/dllama_b200.h"
+#include "gated_common.cuh"
 
 #define GT_TB 8                   // tokens staged per barrier pair of the token-by-token kernel
 #define GT_COLS 32                // columns of S per CTA of the token-by-token kernel
-#define GC DL_GATED_CHUNK
-#define GC_THREADS 256
-#define GC_AS 68                  // row stride of the score matrix
-
-__device__ __forceinline__ float gated_q(const DlGatedArgs& a, size_t row, int i) {
-    const float v = a.q[row * a.ldq + i];
-    if (!a.q_silu) return v * a.q_scale;
-    float s, c;
-    sigmoid_pair_f(v, s, c);
-    return v * s;
-}
-// channel form: f and 1 - f of channel i (over all heads)
-__device__ __forceinline__ void gated_f(const DlGatedArgs& a, size_t row, int i, float& f, float& k) {
-    float s, c;
-    sigmoid_pair_f(a.f[row * a.ldf + i] + a.f_bias[i], s, c);
-    const float l = a.lower[i];
-    f = fmaf(1.f - l, s, l);
-    k = (1.f - l) * c;
-}
 
 // ------------------------------------------------------------------------------------------------
 // token by token: a CTA owns GT_COLS columns of one head's S; thread (column, dq) keeps the rows d with (d / 4) % 4 == dq of its
 // column (NR registers; rows in groups of four so that q, k and f leave shared memory as 16-byte words), the four threads
 // of a column are neighbouring lanes and sum their shares of y by two shuffles.  In the head form column `vdim` is n: its
-// value is 1 for every token and its output is den.
+// value is 1 for every token and its output is den.  Ahead form: the bonus term is one number per token (bs).  Delta form:
+// the column's share of S^T k is summed over the four lanes before the update.
 // ------------------------------------------------------------------------------------------------
-template <int NR, bool CH>
-__global__ void __launch_bounds__(GT_COLS * 4) gated_scan_kernel(DlMambaBatch b, DlGatedArgs a) {
+template <int NR, int MODE>
+__global__ void __launch_bounds__(GT_COLS * 4, NR <= 32 ? 3 : 1) gated_scan_kernel(DlMambaBatch b, DlGatedArgs a) {
     constexpr int DP = NR * 4;
+    constexpr bool CH = MODE != GATED_HEAD;
     extern __shared__ __align__(16) float sm[];
     const int n = blockIdx.x, h = blockIdx.y, dq = threadIdx.x & 3, c = blockIdx.z * GT_COLS + (threadIdx.x >> 2);
-    const int D = a.dim, V = a.vdim, H = a.n_heads;
+    const int D = a.dim, V = a.vdim, H = a.n_heads, hk = gated_k_head(a, h);
     float* qs = sm;                             // [GT_TB][DP]
     float* ks = qs + GT_TB * DP;                // [GT_TB][DP]
-    float* fs = ks + GT_TB * DP;                // channel form: [GT_TB][DP]; head form: [GT_TB] decays
+    float* fs = ks + GT_TB * DP;                // per channel: [GT_TB][DP]; head form: [GT_TB] decays
+    float* bs = fs + GT_TB * DP;                // ahead form: [GT_TB] sums of q bonus k; delta form: [GT_TB] sigmoid(beta)
     const size_t sh = (size_t)b.seq_slot[n] * H + h;
     const bool fresh = b.seq_pos0[n] == 0, is_n = !CH && c == V, live = c < V || is_n;
     float* Sg = is_n ? a.n_state + sh * D : a.state + sh * D * V + c;       // row d at Sg[d * step]
@@ -71,31 +57,68 @@ __global__ void __launch_bounds__(GT_COLS * 4) gated_scan_kernel(DlMambaBatch b,
         for (int t = threadIdx.x / 32; t < nt; t += GT_COLS * 4 / 32) {
             const size_t row = b.seq_rows[rb + t];
             const float put = CH ? 0.f : a.put[row * H + h];
+            float bonus = 0.f;
             for (int d = threadIdx.x & 31; d < DP; d += 32) {
                 float q = 0.f, k = 0.f, f = 0.f;
                 if (d < D) {
-                    q = gated_q(a, row, h * D + d);
-                    if (CH) gated_f(a, row, h * D + d, f, k);
+                    q = gated_q(a, row, hk * D + d);
+                    if (CH) gated_fk(a, row, h, hk, d, f, k);
                     else k = put * a.k[row * a.ldk + h * D + d];
+                    if (MODE == GATED_AHEAD) bonus = fmaf(q * a.bonus[h * D + d], k, bonus);
                 }
                 qs[t * DP + d] = q;
                 ks[t * DP + d] = k;
                 if (CH) fs[t * DP + d] = f;
             }
-            if (!CH && (threadIdx.x & 31) == 0) fs[t] = expf(a.log_keep[row * H + h]);
+            if (MODE == GATED_AHEAD) bonus = warp_sum(bonus);
+            if ((threadIdx.x & 31) == 0) {
+                if (!CH) fs[t] = expf(a.log_keep[row * H + h]);
+                if (MODE == GATED_AHEAD) bs[t] = bonus;
+                if (MODE == GATED_DELTA) bs[t] = sigmoid_f(a.beta[row * a.ld_beta + h]);
+            }
         }
         __syncthreads();
         for (int t = 0; t < nt; ++t) {
             const size_t row = b.seq_rows[rb + t];
-            const float v = c < V ? a.v[row * a.ldv + h * V + c] : 1.f;
+            float v = c < V ? a.v[row * a.ldv + h * V + c] : 1.f;
             const float keep = CH ? 0.f : fs[t];
             float y0 = 0.f, y1 = 0.f;
+            if (MODE == GATED_DELTA) {          // v becomes u, the state is decayed already
+                float d0 = 0.f, d1 = 0.f;
+#pragma unroll
+                for (int i = 0; i < NR; i += 4) {
+                    const int at = t * DP + i * 4 + dq * 4;
+                    const float4 k = *reinterpret_cast<const float4*>(ks + at), f = *reinterpret_cast<const float4*>(fs + at);
+                    s[i] *= f.x;         d0 = fmaf(s[i], k.x, d0);
+                    s[i + 1] *= f.y;     d1 = fmaf(s[i + 1], k.y, d1);
+                    s[i + 2] *= f.z;     d0 = fmaf(s[i + 2], k.z, d0);
+                    s[i + 3] *= f.w;     d1 = fmaf(s[i + 3], k.w, d1);
+                }
+                d0 += d1;
+                d0 += __shfl_xor_sync(0xffffffffu, d0, 1);
+                d0 += __shfl_xor_sync(0xffffffffu, d0, 2);
+                v = bs[t] * (v - d0);
+            }
 #pragma unroll
             for (int i = 0; i < NR; i += 4) {
                 const int at = t * DP + i * 4 + dq * 4;
                 const float4 q = *reinterpret_cast<const float4*>(qs + at), k = *reinterpret_cast<const float4*>(ks + at);
                 float4 f = make_float4(keep, keep, keep, keep);
+                if (MODE == GATED_DELTA) {
+                    s[i] = fmaf(k.x, v, s[i]);               y0 = fmaf(s[i], q.x, y0);
+                    s[i + 1] = fmaf(k.y, v, s[i + 1]);       y1 = fmaf(s[i + 1], q.y, y1);
+                    s[i + 2] = fmaf(k.z, v, s[i + 2]);       y0 = fmaf(s[i + 2], q.z, y0);
+                    s[i + 3] = fmaf(k.w, v, s[i + 3]);       y1 = fmaf(s[i + 3], q.w, y1);
+                    continue;
+                }
                 if (CH) f = *reinterpret_cast<const float4*>(fs + at);
+                if (MODE == GATED_AHEAD) {
+                    y0 = fmaf(s[i], q.x, y0);                s[i] = fmaf(f.x, s[i], k.x * v);
+                    y1 = fmaf(s[i + 1], q.y, y1);            s[i + 1] = fmaf(f.y, s[i + 1], k.y * v);
+                    y0 = fmaf(s[i + 2], q.z, y0);            s[i + 2] = fmaf(f.z, s[i + 2], k.z * v);
+                    y1 = fmaf(s[i + 3], q.w, y1);            s[i + 3] = fmaf(f.w, s[i + 3], k.w * v);
+                    continue;
+                }
                 s[i] = fmaf(f.x, s[i], k.x * v);             y0 = fmaf(s[i], q.x, y0);
                 s[i + 1] = fmaf(f.y, s[i + 1], k.y * v);     y1 = fmaf(s[i + 1], q.y, y1);
                 s[i + 2] = fmaf(f.z, s[i + 2], k.z * v);     y0 = fmaf(s[i + 2], q.z, y0);
@@ -104,6 +127,7 @@ __global__ void __launch_bounds__(GT_COLS * 4) gated_scan_kernel(DlMambaBatch b,
             float y = y0 + y1;
             y += __shfl_xor_sync(0xffffffffu, y, 1);
             y += __shfl_xor_sync(0xffffffffu, y, 2);
+            if (MODE == GATED_AHEAD) y = fmaf(bs[t], v, y);
             if (live && dq == 0) {
                 if (is_n) a.den[row * H + h] = y;
                 else a.y[row * a.ld_y + h * V + c] = y;
@@ -119,22 +143,25 @@ __global__ void __launch_bounds__(GT_COLS * 4) gated_scan_kernel(DlMambaBatch b,
     }
 }
 
-static int gated_args_ok(const DlGatedArgs& a, const char* who) {
-    const bool ch = a.f != nullptr;
-    if (a.n_heads < 1 || a.dim < 1 || a.vdim < 1 || a.dim > 512) { dl_set_error("%s: bad shape (heads %d, dim %d, vdim %d)", who, a.n_heads, a.dim, a.vdim); return -1; }
-    if (ch ? (!a.f_bias || !a.lower) : (!a.k || !a.log_keep || !a.put || !a.den || !a.n_state)) { dl_set_error("%s: the gates are incomplete", who); return -1; }
-    return 0;
-}
-
 extern "C" int dl_gated_scan_supported(int dim, int vdim) { return dim >= 1 && dim <= 512 && vdim >= 1 ? 0 : -1; }
 
+template <int NR, int MODE>
+static int launch_gated_mode(const DlMambaBatch& b, int n_seq, const DlGatedArgs& a, cudaStream_t st) {
+    constexpr bool CH = MODE != GATED_HEAD;
+    const size_t smem = ((size_t)(CH ? 3 : 2) * GT_TB * NR * 4 + GT_TB) * sizeof(float);
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(gated_scan_kernel<NR, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) { dl_set_error("dl_gated_scan: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
+    }
+    gated_scan_kernel<NR, MODE><<<dim3(n_seq, a.n_heads, (a.vdim + (CH ? 0 : 1) + GT_COLS - 1) / GT_COLS), GT_COLS * 4, smem, st>>>(b, a);
+    return 0;
+}
 template <int NR>
-static void launch_gated(const DlMambaBatch& b, int n_seq, const DlGatedArgs& a, cudaStream_t st) {
-    const bool ch = a.f != nullptr;
-    const size_t smem = ((size_t)(ch ? 3 : 2) * GT_TB * NR * 4 + GT_TB) * sizeof(float);
-    const dim3 grid(n_seq, a.n_heads, (a.vdim + (ch ? 0 : 1) + GT_COLS - 1) / GT_COLS);
-    if (ch) gated_scan_kernel<NR, true><<<grid, GT_COLS * 4, smem, st>>>(b, a);
-    else gated_scan_kernel<NR, false><<<grid, GT_COLS * 4, smem, st>>>(b, a);
+static int launch_gated(const DlMambaBatch& b, int n_seq, const DlGatedArgs& a, cudaStream_t st) {
+    if (a.f == nullptr) return launch_gated_mode<NR, GATED_HEAD>(b, n_seq, a, st);
+    if (a.beta != nullptr) return launch_gated_mode<NR, GATED_DELTA>(b, n_seq, a, st);
+    if (a.bonus != nullptr) return launch_gated_mode<NR, GATED_AHEAD>(b, n_seq, a, st);
+    return launch_gated_mode<NR, GATED_CHANNEL>(b, n_seq, a, st);
 }
 
 extern "C" int dl_gated_scan(const DlMambaBatch* batch, int n_seq, const DlGatedArgs* args, void* stream) {
@@ -142,16 +169,10 @@ extern "C" int dl_gated_scan(const DlMambaBatch* batch, int n_seq, const DlGated
     if (gated_args_ok(a, "dl_gated_scan")) return -1;
     if (n_seq < 1) return 0;
     cudaStream_t st = (cudaStream_t)stream;
-    if (a.dim <= 32) launch_gated<8>(*batch, n_seq, a, st);
-    else if (a.dim <= 64) launch_gated<16>(*batch, n_seq, a, st);
-    else if (a.dim <= 128) launch_gated<32>(*batch, n_seq, a, st);
-    else if (a.dim <= 256) launch_gated<64>(*batch, n_seq, a, st);
-    else {                                      // 48 KB + 32 B of staged tokens at most in the channel form
-        const size_t smem = ((size_t)3 * GT_TB * 512 + GT_TB) * sizeof(float);
-        cudaError_t e = cudaFuncSetAttribute(gated_scan_kernel<128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) { dl_set_error("dl_gated_scan: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
-        launch_gated<128>(*batch, n_seq, a, st);
-    }
+    const int rc = a.dim <= 32 ? launch_gated<8>(*batch, n_seq, a, st) : a.dim <= 64 ? launch_gated<16>(*batch, n_seq, a, st) :
+                   a.dim <= 128 ? launch_gated<32>(*batch, n_seq, a, st) : a.dim <= 256 ? launch_gated<64>(*batch, n_seq, a, st) :
+                   launch_gated<128>(*batch, n_seq, a, st);
+    if (rc != 0) return rc;
     LAYER_CHECK_LAUNCH("dl_gated_scan");
     return 0;
 }
@@ -160,30 +181,6 @@ extern "C" int dl_gated_scan(const DlMambaBatch* batch, int n_seq, const DlGated
 // chunked.  Chunk c of sequence n covers rows seq_start[n] + c GC ..; its scratch slot is seq_start[n] / GC + n + c.
 // Scratch: states [slots][H][D][V] | decay of the whole chunk [slots][H][D] (head form: entry 0 of D) | n sums [slots][H][D].
 // ------------------------------------------------------------------------------------------------
-struct GatedScratch { float* S; float* dec; float* ns; };
-
-__device__ __forceinline__ bool gated_chunk_of(const DlMambaBatch& b, int n, int c, int& row0, int& len, int& ci) {
-    const int s0 = b.seq_start[n], total = b.seq_start[n + 1] - s0;
-    if (c * GC >= total) return false;
-    row0 = s0 + c * GC;
-    len = min(GC, total - c * GC);
-    ci = s0 / GC + n + c;
-    return true;
-}
-
-// V columns c0 .. c0 + 127 of the chunk's values into [GC][128] (zeros beyond the chunk or the head's width)
-__device__ __forceinline__ void gated_stage_v(const DlGatedArgs& a, const int* rows, int len, int h, int c0, float* vt) {
-    const int lane = threadIdx.x & 31;
-    for (int j = threadIdx.x >> 5; j < GC; j += GC_THREADS / 32) {
-        const float* src = j < len ? a.v + (size_t)rows[j] * a.ldv + (size_t)h * a.vdim + c0 : nullptr;
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-            const int cc = lane + 32 * u;
-            vt[j * 128 + cc] = (src && c0 + cc < a.vdim) ? src[cc] : 0.f;
-        }
-    }
-}
-
 // pass 1: a chunk's own sum of (decay to the chunk's end * k_j) v_j^T, and the decay of the whole chunk
 template <bool CH>
 __global__ void __launch_bounds__(GC_THREADS) gated_chunk_state_kernel(DlMambaBatch b, DlGatedArgs a, GatedScratch sc) {
@@ -194,7 +191,7 @@ __global__ void __launch_bounds__(GC_THREADS) gated_chunk_state_kernel(DlMambaBa
     const int n = blockIdx.x, c = blockIdx.y, h = blockIdx.z;
     int row0, len, ci;
     if (!gated_chunk_of(b, n, c, row0, len, ci)) return;
-    const int D = a.dim, V = a.vdim, H = a.n_heads, D8 = (D + 7) & ~7;
+    const int D = a.dim, V = a.vdim, H = a.n_heads, D8 = (D + 7) & ~7, hk = gated_k_head(a, h);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* ks = sm;                             // [GC][D8]
     float* vt = ks + (size_t)GC * D8;           // channel form: the decays [GC][D8] first; then value tiles [GC][128]
@@ -214,7 +211,7 @@ __global__ void __launch_bounds__(GC_THREADS) gated_chunk_state_kernel(DlMambaBa
         for (int d = lane; d < D8; d += 32) {
             float k = 0.f, f = 1.f;
             if (j < len && d < D) {
-                if (CH) gated_f(a, row, h * D + d, f, k);
+                if (CH) gated_fk(a, row, h, hk, d, f, k);
                 else k = w_s[j] * a.k[row * a.ldk + h * D + d];
             }
             ks[j * D8 + d] = k;
@@ -308,13 +305,11 @@ __global__ void __launch_bounds__(256) gated_chunk_prefix_kernel(DlMambaBatch b,
     *Sg = R;
 }
 
-__device__ __forceinline__ float dot4(float4 x, float4 y, float acc) { return fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, acc)))); }
-__device__ __forceinline__ float4 mul4(float4 x, float4 y) { return make_float4(x.x * y.x, x.y * y.y, x.z * y.z, x.w * y.w); }
-
 // pass 3: the outputs of a chunk.  Shared memory: Q [GC][DP] | K [GC][DP], later tiles of V and of the carried state
 // [GC][128] | F [GC][DP] (channel form), later the scores A [GC][GC_AS] | block decays [4][DP].
-template <bool CH>
+template <int MODE>
 __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaBatch b, DlGatedArgs a, GatedScratch sc) {
+    constexpr bool CH = MODE != GATED_HEAD;
     extern __shared__ __align__(16) float sm[];
     __shared__ int rows[GC];
     __shared__ float put_s[GC], carry_s[GC];
@@ -322,7 +317,7 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
     const int n = blockIdx.x, c = blockIdx.y, h = blockIdx.z;
     int row0, len, ci;
     if (!gated_chunk_of(b, n, c, row0, len, ci)) return;
-    const int D = a.dim, V = a.vdim, H = a.n_heads, D4 = (D + 3) & ~3, DP = D4 + 4;
+    const int D = a.dim, V = a.vdim, H = a.n_heads, D4 = (D + 3) & ~3, DP = D4 + 4, hk = gated_k_head(a, h);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tb = threadIdx.x >> 4, cb = threadIdx.x & 15;
     float* Q = sm;
     float* K = Q + (size_t)GC * DP;
@@ -345,8 +340,8 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
         for (int d = lane; d < D4; d += 32) {
             float q = 0.f, k = 0.f, f = 1.f;
             if (j < len && d < D) {
-                q = gated_q(a, row, h * D + d);
-                if (CH) gated_f(a, row, h * D + d, f, k);
+                q = gated_q(a, row, hk * D + d);
+                if (CH) gated_fk(a, row, h, hk, d, f, k);
                 else k = a.k[row * a.ldk + h * D + d];
             }
             Q[j * DP + d] = q;
@@ -360,98 +355,8 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
     __syncthreads();
     if (!CH && threadIdx.x < GC) { g_s[threadIdx.x] = gsum; carry_s[threadIdx.x] = expf((float)gsum); }
     if (CH) {
-        // inside a sub-block: for column j the running product k_j f_(j+1) .. f_i, lanes along d.  Two warps per sub-block
-        // take its columns in turn; a lane's shares for all rows i are reduced together (16 values over 32 lanes).
-        const int blk = warp >> 1;
-        const float* Qb = Q + (size_t)blk * 16 * DP;
-        const float* Kb = K + (size_t)blk * 16 * DP;
-        const float* Fb = F + (size_t)blk * 16 * DP;
-        float diag[8];
-#pragma unroll 1
-        for (int jj = 0; jj < 8; ++jj) {
-            const int j = jj * 2 + (warp & 1);
-            float acc[16];
-#pragma unroll
-            for (int i = 0; i < 16; ++i) acc[i] = 0.f;
-            for (int d = lane; d < D4; d += 32) {
-                float p = Kb[j * DP + d];
-#pragma unroll
-                for (int i = 0; i < 16; ++i)
-                    if (i >= j) {
-                        if (i > j) p *= Fb[i * DP + d];
-                        acc[i] = fmaf(Qb[i * DP + d], p, acc[i]);
-                    }
-            }
-#pragma unroll
-            for (int o = 16, m = 8; o >= 2; o >>= 1, m >>= 1) {
-                const bool hi = lane & o;
-#pragma unroll
-                for (int t = 0; t < m; ++t) {
-                    const float keep = hi ? acc[t + m] : acc[t], send = hi ? acc[t] : acc[t + m];
-                    acc[t] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-                }
-            }
-            acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1);
-            // this lane now holds row i = lane / 2 of column j
-#pragma unroll
-            for (int u = 0; u < 8; ++u)
-                if (u == jj) diag[u] = acc[0];
-        }
-        __syncthreads();
-        // rows scaled by the decay from their block's start (Q) / to their block's end (K); T: a block's whole decay
-        for (int t = threadIdx.x; t < 4 * D4; t += GC_THREADS) {
-            const int bk = t / D4, d = t - bk * D4;
-            float p = 1.f;
-#pragma unroll
-            for (int i = 0; i < 16; ++i) {
-                p *= F[(bk * 16 + i) * DP + d];
-                Q[(bk * 16 + i) * DP + d] *= p;
-            }
-            T[bk * DP + d] = p;
-            p = 1.f;
-#pragma unroll
-            for (int i = 15; i >= 0; --i) {
-                K[(bk * 16 + i) * DP + d] *= p;
-                p *= F[(bk * 16 + i) * DP + d];
-            }
-        }
-        __syncthreads();
-        // between sub-blocks: thread (i, j) = (tb, cb) of the six block pairs
-        float a10 = 0.f, a20 = 0.f, a21 = 0.f, a30 = 0.f, a31 = 0.f, a32 = 0.f;
-        for (int d = 0; d < D4; d += 4) {
-            const float4 q1 = *reinterpret_cast<const float4*>(Q + (16 + tb) * DP + d), q2 = *reinterpret_cast<const float4*>(Q + (32 + tb) * DP + d);
-            const float4 q3 = *reinterpret_cast<const float4*>(Q + (48 + tb) * DP + d);
-            const float4 k0 = *reinterpret_cast<const float4*>(K + cb * DP + d), k1 = *reinterpret_cast<const float4*>(K + (16 + cb) * DP + d);
-            const float4 k2 = *reinterpret_cast<const float4*>(K + (32 + cb) * DP + d);
-            const float4 t1 = *reinterpret_cast<const float4*>(T + DP + d), t2 = *reinterpret_cast<const float4*>(T + 2 * DP + d);
-            const float4 k0t = mul4(k0, t1), k1t = mul4(k1, t2);
-            a10 = dot4(q1, k0, a10);
-            a21 = dot4(q2, k1, a21);
-            a32 = dot4(q3, k2, a32);
-            a20 = dot4(q2, k0t, a20);
-            a31 = dot4(q3, k1t, a31);
-            a30 = dot4(q3, mul4(k0t, t2), a30);
-        }
-        __syncthreads();                          // F is done with: A takes its place
-        A[(16 + tb) * GC_AS + cb] = a10;
-        A[(32 + tb) * GC_AS + cb] = a20;
-        A[(32 + tb) * GC_AS + 16 + cb] = a21;
-        A[(48 + tb) * GC_AS + cb] = a30;
-        A[(48 + tb) * GC_AS + 16 + cb] = a31;
-        A[(48 + tb) * GC_AS + 32 + cb] = a32;
-#pragma unroll
-        for (int jj = 0; jj < 8; ++jj) {
-            const int j = jj * 2 + (warp & 1), i = lane >> 1;
-            if ((lane & 1) == 0) A[(blk * 16 + i) * GC_AS + blk * 16 + j] = i >= j ? diag[jj] : 0.f;
-        }
-        // Q: the decay from the chunk's start
-        for (int t = threadIdx.x; t < 3 * D4; t += GC_THREADS) {
-            const int bk = t / D4 + 1, d = t - (bk - 1) * D4;
-            float p = T[d];
-            for (int u = 1; u < bk; ++u) p *= T[u * DP + d];
-#pragma unroll
-            for (int i = 0; i < 16; ++i) Q[(bk * 16 + i) * DP + d] *= p;
-        }
+        decayed_scores<MODE == GATED_AHEAD>(Q, K, F, T, D, D4, DP, MODE == GATED_AHEAD ? a.bonus + (size_t)h * D : nullptr,
+                                            [&](int i, int j, float v) { A[i * GC_AS + j] = i >= j ? v : 0.f; });
     } else {
         __syncthreads();
         // A[i][j] = e^(G_i - G_j) p_j q_i . k_j, rows tb * 4 + r, columns cb + 16 u
@@ -571,16 +476,26 @@ extern "C" long long dl_gated_chunk_floats(int M, int n_seq, int n_heads, int di
     return (long long)(M / GC + n_seq) * n_heads * dim * ((long long)vdim + 2);
 }
 
-template <bool CH>
+// pass 3 alone (the delta rule's outputs from its corrected values)
+int gated_chunk_out_channel(const DlMambaBatch& b, int n_seq, int max_chunks, const DlGatedArgs& a, const GatedScratch& sc, cudaStream_t st) {
+    const size_t smem = gated_out_smem(a.dim, true);
+    cudaError_t e = cudaFuncSetAttribute(gated_chunk_out_kernel<GATED_CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) { dl_set_error("gated_chunk_out: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
+    gated_chunk_out_kernel<GATED_CHANNEL><<<dim3(n_seq, max_chunks, a.n_heads), GC_THREADS, smem, st>>>(b, a, sc);
+    return 0;
+}
+
+template <int MODE>
 static int launch_gated_chunked(const DlMambaBatch& b, int n_seq, int max_chunks, const DlGatedArgs& a, const GatedScratch& sc, cudaStream_t st) {
+    constexpr bool CH = MODE != GATED_HEAD;
     const size_t smem1 = gated_state_smem(a.dim, CH), smem3 = gated_out_smem(a.dim, CH);
     cudaError_t e = cudaFuncSetAttribute(gated_chunk_state_kernel<CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(gated_chunk_out_kernel<CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gated_chunk_out_kernel<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
     if (e != cudaSuccess) { dl_set_error("dl_gated_scan_chunked: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
     const dim3 grid(n_seq, max_chunks, a.n_heads);
     gated_chunk_state_kernel<CH><<<grid, GC_THREADS, smem1, st>>>(b, a, sc);
     gated_chunk_prefix_kernel<CH><<<dim3(n_seq, a.n_heads, (a.dim * (a.vdim + (CH ? 0 : 1)) + 255) / 256), 256, 0, st>>>(b, a, sc);
-    gated_chunk_out_kernel<CH><<<grid, GC_THREADS, smem3, st>>>(b, a, sc);
+    gated_chunk_out_kernel<MODE><<<grid, GC_THREADS, smem3, st>>>(b, a, sc);
     return 0;
 }
 
@@ -590,6 +505,7 @@ extern "C" int dl_gated_scan_chunked(const DlMambaBatch* batch, int n_seq, int m
     const DlGatedArgs& a = *args;
     const bool ch = a.f != nullptr;
     if (gated_args_ok(a, "dl_gated_scan_chunked")) return -1;
+    if (a.beta) { dl_set_error("dl_gated_scan_chunked: the delta rule runs on dl_delta_scan_chunked"); return -1; }
     if (dl_gated_scan_chunked_supported(a.dim, a.vdim, ch) != 0 || scratch == nullptr) { dl_set_error("dl_gated_scan_chunked: sizes not supported (dim %d, vdim %d)", a.dim, a.vdim); return -1; }
     if (n_seq < 1 || max_chunks < 1) return 0;
     GatedScratch sc;
@@ -597,8 +513,9 @@ extern "C" int dl_gated_scan_chunked(const DlMambaBatch* batch, int n_seq, int m
     sc.S = scratch;
     sc.dec = sc.S + slots * a.n_heads * a.dim * a.vdim;
     sc.ns = sc.dec + slots * a.n_heads * a.dim;
-    const int rc = ch ? launch_gated_chunked<true>(*batch, n_seq, max_chunks, a, sc, (cudaStream_t)stream)
-                      : launch_gated_chunked<false>(*batch, n_seq, max_chunks, a, sc, (cudaStream_t)stream);
+    const int rc = !ch ? launch_gated_chunked<GATED_HEAD>(*batch, n_seq, max_chunks, a, sc, (cudaStream_t)stream) :
+                   a.bonus ? launch_gated_chunked<GATED_AHEAD>(*batch, n_seq, max_chunks, a, sc, (cudaStream_t)stream) :
+                             launch_gated_chunked<GATED_CHANNEL>(*batch, n_seq, max_chunks, a, sc, (cudaStream_t)stream);
     if (rc != 0) return rc;
     LAYER_CHECK_LAUNCH("dl_gated_scan_chunked");
     return 0;
@@ -725,7 +642,10 @@ __global__ void __launch_bounds__(HN_WARPS * 32) head_norm_kernel(DlHeadNormArgs
             if (i >= n4) continue;
             const float4 wv = reinterpret_cast<const float4*>(w)[i];
             float4 t = make_float4(v[k].x * inv * wv.x, v[k].y * inv * wv.y, v[k].z * inv * wv.z, v[k].w * inv * wv.w);
-            if (g) { t.x *= sigmoid_f(gv[k].x); t.y *= sigmoid_f(gv[k].y); t.z *= sigmoid_f(gv[k].z); t.w *= sigmoid_f(gv[k].w); }
+            if (g) {
+                if (a.gate_silu) { t.x *= gv[k].x; t.y *= gv[k].y; t.z *= gv[k].z; t.w *= gv[k].w; }
+                t.x *= sigmoid_f(gv[k].x); t.y *= sigmoid_f(gv[k].y); t.z *= sigmoid_f(gv[k].z); t.w *= sigmoid_f(gv[k].w);
+            }
             if (a.xh) {
                 __nv_bfloat162 lo = __floats2bfloat162_rn(t.x, t.y), hi = __floats2bfloat162_rn(t.z, t.w);
                 *reinterpret_cast<uint2*>(a.xh + xh_offset(a.ncap, m, h * V + i * 4)) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
@@ -739,7 +659,7 @@ __global__ void __launch_bounds__(HN_WARPS * 32) head_norm_kernel(DlHeadNormArgs
         const float inv = 1.f / sqrtf(warp_sum(ss) / (float)V + a.eps);
         for (int i = lane; i < V; i += 32) {
             float t = y[i] * scale * inv * w[i];
-            if (g) t *= sigmoid_f(g[i]);
+            if (g) t *= a.gate_silu ? silu_f(g[i]) : sigmoid_f(g[i]);
             if (a.xh) xh_store(a.xh, a.ncap, m, h * V + i, t);
             else a.out[(size_t)m * a.ld_out + (size_t)h * V + i] = t;
         }
