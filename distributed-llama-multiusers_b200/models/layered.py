@@ -8,14 +8,15 @@ meets the residual stream is the architecture's ``residual`` style (``RESIDUAL_S
                  which is how Venadra's pre-norm layers run (one stream, m = 1)
     "post":      x <- x + m * norm(sub(x))                               the sublayer reads the stream itself; the only
                  norm sits on its output (Darusun)
-    "parallel":  x <- x + mixer(norm1(x)) + ff(norm2(x))                 both of the same x; norm weights plain (Vopedra)
+    "parallel":  x <- x + mixer(norm1(x)) + ff(norm2(x))                 both of the same x; norm weights plain (Vopedra); or
+                 ONE norm whose output both read, a layer norm with bias (Silizen)
 
 What a design fixes without saying it in config.json (how its attention masks, whether its experts are gated, ...) is
 its entry of ``DESIGNS``; everything config.json gives is read from there.  A configuration with ``canon: {taps}`` puts a
 short causal convolution in front of every mixer: h <- h + conv(h) on the normed input, the last taps - 1 inputs kept per
 sequence slot and layer.  ``loop: {start, stop, times}`` runs that slice of the list `times` times in a row on the same
-weights, every pass with caches and states of its own (parallel residual style; the embedding output and a vector
-``loop.step[pass]`` are added to the stream ahead of a pass).
+weights, every pass with caches and states of its own (parallel residual style; ahead of a pass the embedding output and a
+vector ``loop.step[pass]`` are added to the stream, or a matrix ``loop.in`` maps stream and embedding output side by side).
 
 The mixers and feed-forwards are looked up by name (``MIXERS`` / ``FEED_FORWARDS`` below), so another design composes
 the same mechanisms with its own sizes and order; ``ARCHITECTURES`` in models/registry.py maps an architecture name to
@@ -29,13 +30,18 @@ this engine.  Mixers here:
   interleaved rotary positions with optional frequency interpolation, or none; soft-capped scores; queries and keys
   divided by their root mean square; a sink per head in the softmax denominator; a sigmoid output gate; rotary in the
   rotate-half layout in front of the unit norm; scores mixed across heads by a matrix `talk` before the softmax (folded
-  into the queries, see WindowAttentionMixer); a layer that reads another layer's keys and values (``kv_from``);
+  into the queries, see WindowAttentionMixer); a layer that reads another layer's keys and values (``kv_from``); norms per
+  query and key head with weights, projection biases, a distance bias per head, one output gate per head;
 * ``lightning`` -- linear attention with a fixed decay per head and an f32 state [dim][vdim] per head and slot, SiLU on
   q, k and v, an RMS norm over the concatenated heads and a sigmoid output gate;
 * ``mlstm`` -- a matrix memory with exponential input and forget gates per head, stabilised by a running maximum;
 * ``hgrn2`` -- linear attention whose forget gate per head and channel also decides what is written;
 * ``mamba1`` -- a selective state-space recurrence with a state per channel behind a short causal convolution;
-* ``parallel`` -- two mixers side by side on the same input, their outputs normed and averaged.
+* ``gated_linear`` -- linear attention with a data-dependent decay per head and key channel, read after the write;
+* ``delta`` -- the gated delta rule (decays per key channel, unit queries and keys behind a short convolution);
+* ``wkv`` -- RWKV time mixing: mixes with the row ahead, data-dependent decays, a bonus for the current token;
+* ``parallel``, ``parallel_2`` -- two mixers side by side on the same input, their outputs normed and averaged, or summed
+  with a constant factor each.
 
 Feed-forwards: ``dense`` (squared ReLU, PolyNorm, xIELU, or a GELU-gated unit) and ``moe`` (sigmoid-scored, group-limited routing over small
 squared-ReLU experts; or softmax-scored, renormalised routing over gated experts, with an optional router bias and a
@@ -54,6 +60,7 @@ and step sizes are f32.  ``dtype="float32"`` widens weights and caches to f32 an
 from __future__ import annotations
 
 import contextlib
+import functools
 import json
 import math
 import os
@@ -90,7 +97,12 @@ class LayerSpec:
 # ("interleaved" | "half": the pair layout of the rotary, which own values otherwise exclude), talk (tensor `talk`
 # [heads][heads] mixes the heads: "scores" before the softmax | "weights" after it), proj_norm (tensors q.norm, k.norm: an RMS
 # norm over the whole query / key projection ahead of the rotary).  dense_act also: "gelu_glu" (tensors gate, up).
-# embed_norm (tensor embed.norm: the embedding is normed).  parallel: the mixers of its two branches.  latent: rot (the same), sink, gate ("full": one
+# attention also: head_norm (tensors q.norm, k.norm [dim]: an RMS norm per head ahead of the rotary), bias (tensors q.b, k.b, v.b),
+# slopes (a distance bias 2^(-8 (h + 1) / heads) per head), sink "zero" (a sink whose score is 0), gate "head" (tensor `g` [heads]).
+# embed_norm (tensor embed.norm: the embedding is normed).  norm "layer": the norms over the width are layer norms with biases
+# (<name>.b).  one_norm: mixer and feed-forward read norm1's output.  loop_in: tensor loop.in [width][2 width] opens a pass.  tied_head: the
+# logits' matrix is the embedding.  parallel, parallel_2: the mixers of the two branches (with attention traits of their own where they
+# differ) and how they meet (combine "norms", the default, or "scales").    latent: rot (the same), sink, gate ("full": one
 # gate per output column | "head": one per head).  norm_weights "scalar": every norm over the width has one number.
 DESIGNS = {
     "Ribivik": {"residual": "sandwich"},
@@ -107,6 +119,12 @@ DESIGNS = {
     "Vopedra": {"residual": "parallel", "embed_norm": True,
                 "attention": {"values": "own", "rot": "half", "talk": "weights", "proj_norm": True},
                 "parallel": {"left": "attention", "right": "hgrn2"},
+                "dense_act": "gelu_glu"},
+    "Silizen": {"residual": "parallel", "norm": "layer", "one_norm": True, "loop_in": True, "tied_head": True,
+                "parallel": {"left": ("attention", {"values": "own", "rot": "half", "head_norm": True, "sink": "zero", "gate": "head"}),
+                             "right": "gated_linear", "combine": "scales"},
+                "parallel_2": {"left": ("attention", {"values": "own", "bias": True, "qk_norm": True, "slopes": True, "sink": "zero", "gate": "head"}),
+                               "right": "delta"},
                 "dense_act": "gelu_glu"},
 }
 RESIDUAL_STYLES = {name: d["residual"] for name, d in DESIGNS.items()}
@@ -129,6 +147,7 @@ class LayerListConfig:
     canon_taps: int = 0                    # > 0: h <- h + conv(h) over the last `taps` normed inputs, in front of every mixer
     traits: dict = field(default_factory=dict)      # the design's entry of DESIGNS
     loop_times: int = 0                    # passes of the loop (0: none); `layers` holds the runs of all passes
+    logit_scale: float = 1.0               # the logits are multiplied by it
 
     # the serving code reads these names from every engine's header
     @property
@@ -167,7 +186,7 @@ class LayerListConfig:
                                residual_mult=float(c.get("residual_mult", 1.0)),
                                streams=int(c.get("streams") or 1), hyper_weights=bool(c.get("streams")),
                                canon_taps=int((c.get("canon") or {}).get("taps") or 0), traits=DESIGNS.get(arch, {}),
-                               loop_times=loop_times)
+                               loop_times=loop_times, logit_scale=float(c.get("logit_scale", 1.0)))
 
     @staticmethod
     def load(model_dir: str) -> "LayerListConfig":
@@ -187,7 +206,9 @@ def rotary_frequencies(base: float, dims: int) -> torch.Tensor:
 
 
 def interpolated_rotary(base: float, dims: int, scaling: Optional[dict]):
-    """(frequencies f64 [dims / 2], magnitude).  Without `scaling`: the plain f_i and 1.  With scaling {factor, original,
+    """(frequencies f64 [dims / 2], magnitude).  Without `scaling`: the plain f_i and 1.  With scaling {factor, original, low,
+    high} by wavelength (Llama 3.1): r_i = original f_i / (2 pi), s_i = clamp((r_i - low) / (high - low), 0, 1),
+    f_i' = f_i / factor * (1 - s_i) + f_i s_i, magnitude 1.  With scaling {factor, original,
     fast, slow} the slow frequencies are divided by `factor`, the fast ones kept and those between blended (YaRN):
     with d(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(d(fast)), 0), hi = min(ceil(d(slow)), dims - 1),
     r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1):  f_i' = f_i / factor * r_i + f_i (1 - r_i); cos and sin are
@@ -196,6 +217,11 @@ def interpolated_rotary(base: float, dims: int, scaling: Optional[dict]):
     if not scaling:
         return f, 1.0
     factor, original = float(scaling["factor"]), float(scaling["original"])
+    if "low" in scaling:
+        low, high = float(scaling["low"]), float(scaling["high"])
+        r = original * f / (2.0 * math.pi)
+        s = ((r - low) / (high - low)).clamp(0.0, 1.0) if high > low else (r > high).to(torch.float64)
+        return f / factor * (1.0 - s) + f * s, 1.0
 
     def d(t):
         return dims * math.log(original / (2.0 * math.pi * float(t))) / (2.0 * math.log(base))
@@ -443,13 +469,20 @@ class WindowAttentionMixer:
              talk "scores"; talk "weights" mixes the softmax weights instead, weight'_h = sum_g talk[h][g] weight_g, which is linear in
              the outputs: every head's weights meet the values of all key/value heads side by side (kv_heads * vdim numbers
              per head) and the head's outputs are summed with talk afterwards;
-      proj_norm: an RMS norm with weights <prefix>q.norm / k.norm over all heads' columns of q / k at once, BEFORE the rotary.
+      proj_norm: an RMS norm with weights <prefix>q.norm / k.norm over all heads' columns of q / k at once, BEFORE the rotary;
+      head_norm: the same per head, weights [dim] shared by the heads;
+      bias: <prefix>q.b / k.b / v.b are added to the projections;
+      slopes: 2^(-8 (h + 1) / heads) * (i - j) is taken off head h's (capped) score;
+      sink "zero": a sink whose score is 0 (one more term 1 in the denominator), without a tensor;
+      gate "head": <prefix>g [heads][width], head h is multiplied by sigmoid(W_g h)_h; its rows ride in the q / k / v product and the
+             attention kernels apply it.
     A mixer entry with `kv_from: j` has no k / v tensors and no cache: it reads layer j's keys (as cached: rotated and
     normalised) and values with queries, mask and the rest of its own."""
 
-    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["WindowAttentionMixer"] = None):
+    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["WindowAttentionMixer"] = None,
+                 traits: Optional[dict] = None):
         self.eng, self.index = eng, index
-        tr = eng.cfg.traits.get("attention") or {}
+        tr = traits if traits is not None else eng.cfg.traits.get("attention") or {}
         self.own_v, self.qk_norm = tr.get("values", "keys") == "own", bool(tr.get("qk_norm"))
         self.H, self.G, self.dim = int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
         self.vdim = int(m.get("vdim", self.dim))
@@ -471,6 +504,10 @@ class WindowAttentionMixer:
         freqs, self.rope_mag = interpolated_rotary(float(rot["base"]), self.rope_dims, rot.get("scaling"))
         self.freqs = freqs.to(eng.device) if self.rope_dims else torch.zeros(1, dtype=torch.float64, device=eng.device)
         H, G, d, dv = self.H, self.G, self.dim, self.vdim
+        self.head_gate, self.head_norm = tr.get("gate") == "head", bool(tr.get("head_norm"))
+        self.slope = None
+        if tr.get("slopes"):
+            self.slope = torch.pow(2.0, -8.0 * (torch.arange(H, dtype=torch.float64) + 1) / H).float().to(eng.device)
         if share is None:
             W, D = eng.weight, eng.dense_weight
             wq = W(prefix + "q")
@@ -483,24 +520,40 @@ class WindowAttentionMixer:
                 if tuple(wv.shape) != (G * dv, eng.cfg.width):
                     raise ValueError(f"layer {index}: v has shape {tuple(wv.shape)}")
                 parts.append(wv)
+            self.bias = None
+            if tr.get("bias"):
+                bs = [eng.vector(prefix + n + ".b") for n in ("q", "k", "v")[:len(parts)]]
+                if any(b.numel() != w.shape[0] for b, w in zip(bs, parts)):
+                    raise ValueError(f"layer {index}: q.b / k.b / v.b do not fit their projections")
+                self.bias = torch.cat(bs + ([torch.zeros(H, device=eng.device)] if self.head_gate else []))
+            if self.head_gate:
+                wg = W(prefix + "g")
+                if not self.own_v or tuple(wg.shape) != (H, eng.cfg.width):
+                    raise ValueError(f"layer {index}: g has shape {tuple(wg.shape)}")
+                parts.append(wg)
             self.w_qk = D(torch.cat(parts, 0).contiguous())            # one product for queries, keys (and values)
             self.w_o = D(W(prefix + "o"))
-            self.w_g = D(W(prefix + "g")) if tr.get("gate") else None
-            self.sink = eng.vector(prefix + "sink") if tr.get("sink") else None
+            self.w_g = D(W(prefix + "g")) if tr.get("gate") and not self.head_gate else None
+            self.sink = torch.zeros(H, device=eng.device) if tr.get("sink") == "zero" else eng.vector(prefix + "sink") if tr.get("sink") else None
             if self.sink is not None and tuple(self.sink.shape) != (H,):
                 raise ValueError(f"layer {index}: sink has shape {tuple(self.sink.shape)}")
             self.talk = eng.vector(prefix + "talk") if tr.get("talk") else None
             if self.talk is not None and tuple(self.talk.shape) != (H, H):
                 raise ValueError(f"layer {index}: talk has shape {tuple(self.talk.shape)}")
             self.q_norm = self.k_norm = None
-            if tr.get("proj_norm"):
+            if self.head_norm:
+                self.q_norm = eng.vector(prefix + "q.norm")
+                self.k_norm = eng.vector(prefix + "k.norm") if self.kv_from is None else None
+                if not self.own_v or self.q_norm.numel() != d or (self.k_norm is not None and self.k_norm.numel() != d):
+                    raise ValueError(f"layer {index}: q.norm / k.norm do not fit heads of {d}")
+            elif tr.get("proj_norm"):
                 self.q_norm = eng.vector(prefix + "q.norm")
                 self.k_norm = eng.vector(prefix + "k.norm") if self.kv_from is None else None
                 if not self.own_v or self.q_norm.numel() != H * d or (self.k_norm is not None and self.k_norm.numel() != G * d):
                     raise ValueError(f"layer {index}: q.norm / k.norm do not fit {H} / {G} heads of {d}")
         else:
             self.w_qk, self.w_o, self.w_g, self.sink, self.talk = share.w_qk, share.w_o, share.w_g, share.sink, share.talk
-            self.q_norm, self.k_norm = share.q_norm, share.k_norm
+            self.q_norm, self.k_norm, self.bias = share.q_norm, share.k_norm, share.bias
         # heads mixed before the softmax: queries against all key heads; after it: weights against all value heads
         self.key_heads = G if self.talk is not None and tr.get("talk") == "scores" else 0
         self.value_heads = G if self.talk is not None and tr.get("talk") == "weights" else 0
@@ -515,15 +568,18 @@ class WindowAttentionMixer:
         attn_tc = eng.round_x and os.environ.get("DLLAMA_LAYERS_ATTN_TC", "1") != "0"
         if attn_tc and dv == d and self.talk is None and L.window_tc_supported(H, G, d, 0 if self.own_v else self.rope_dims, eng.wdtype):
             self.tc_rq = L.window_tc_rows(H, G)
-        elif attn_tc and self.own_v and self.softcap == 0.0 and L.talk_tc_supported(H, G, d, dv, self.key_heads, eng.wdtype, self.value_heads):
+        elif attn_tc and self.own_v and L.talk_tc_supported(H, G, d, dv, self.key_heads, eng.wdtype, self.value_heads):
             # values wider or narrower than the keys, head-mixed scores: the tile kernel of talk_attention.cu
             # tiles of 128 stacked (row, head) pairs for long portions, of 16 for decoding, 64 where those do not fit
             kh, vh = self.key_heads, self.value_heads
             self.tc_rq, self.tc_rq_small, self.tc_talk = L.talk_tc_rows(H, G, d, dv, kh, 1 << 30, vh), L.talk_tc_rows(H, G, d, dv, kh, 1, vh), True
             self.partial_floats = L.talk_tc_partial_floats(WINDOW_CTAS_PER_SM * eng.n_sms, 1, 1, dv, self.tc_rq, H, vh)
 
+    def qk_width(self) -> int:
+        return (self.w_qk.N + 3) // 4 * 4                     # rows start on 16 bytes
+
     def scratch(self) -> Dict[str, int]:
-        n = {"qk": (self.H + self.G) * self.dim + (self.G * self.vdim if self.own_v else 0), "o": self.H * self.vdim}
+        n = {"qk": self.qk_width(), "o": self.H * self.vdim}
         if self.w_g is not None:
             n["og"] = self.H * self.vdim
         if self.key_heads:
@@ -551,8 +607,8 @@ class WindowAttentionMixer:
         H, G, d, dv, rd = self.H, self.G, self.dim, self.vdim, self.rope_dims
         nqk = (H + G) * d
         own_kv = self.kv_from is None
-        qk, o = e.buf("qk", self.w_qk.N), e.buf("o", H * dv)
-        e.mm(self.w_qk, h, qk, M, src="h")
+        qk, o = e.buf("qk", self.qk_width()), e.buf("o", H * dv)
+        e.mm(self.w_qk, h, qk, M, src="h", bias=self.bias)
         # one launch: the keys (and values) go into the cache and the queries are rotated / normalised in place (and mixed)
         q_in = qk
         if self.own_v:
@@ -561,12 +617,13 @@ class WindowAttentionMixer:
             L.window_kv_write(qk[:, H * d:] if own_kv else None, M, G, d, rd, self.freqs, self.rope_mag, e.pos, e.slot, e.block_table,
                               self.cache, q=qk, q_heads=H, v=qk[:, nqk:] if own_kv else None, vdim=dv, qk_norm=self.qk_norm,
                               eps=e.cfg.norm_eps, rope_half=self.own_rot == "half", talk=self.talk if self.key_heads else None,
-                              q_mixed=q_in if self.key_heads else None, q_norm=self.q_norm, k_norm=self.k_norm)
+                              q_mixed=q_in if self.key_heads else None, q_norm=self.q_norm, k_norm=self.k_norm, head_norm=self.head_norm)
             rd = 0                            # the attention kernels meet keys that are complete: nothing of a line is shared with its value
         else:
             L.window_kv_write(qk[:, H * d:], M, G, d, rd, self.freqs, self.rope_mag, e.pos, e.slot, e.block_table, self.cache,
                               q=qk, q_heads=H)
-        opts = dict(vdim=dv if self.own_v else 0, chunk=self.chunk, sink=self.sink)
+        opts = dict(vdim=dv if self.own_v else 0, chunk=self.chunk, sink=self.sink, slope=self.slope,
+                    gate=qk[:, self.w_qk.N - H:] if self.head_gate else None)
         if self.key_heads:
             opts["key_heads"] = G
         if self.value_heads:
@@ -587,7 +644,7 @@ class WindowAttentionMixer:
             if self.tc_talk:
                 L.talk_attention_tc(q_in, o, H, G, d, dv, self.scale, self.window, e.pos, e.slot, e.block_table, self.cache, tile_rows,
                                     n_tiles, rq, n_splits, partial, chunk=self.chunk, sink=self.sink, key_heads=opts.get("key_heads", 0),
-                                    value_heads=opts.get("value_heads", 0))
+                                    value_heads=opts.get("value_heads", 0), softcap=self.softcap, slope=self.slope, gate=opts["gate"])
             else:
                 L.window_attention_tc(qk, o, H, G, d, rd, self.scale, self.softcap, self.window, e.pos, e.slot, e.block_table,
                                       self.cache, tile_rows, n_tiles, rq, n_splits, partial, **opts)
@@ -688,6 +745,9 @@ class MLstmMixer:
         self.u_state = torch.zeros(eng.n_slots, H, **f32)
         self.chunked = eng.L.gated_chunked_supported(d, dv, False)
 
+    def chunk_floats(self, rows: int, slots: int) -> int:
+        return self.eng.L.gated_chunk_floats(rows, slots, self.H, self.dim, self.vdim)
+
     def scratch(self) -> Dict[str, int]:
         return {"mx": self.w_in.N, "ys": self.H * self.vdim, "yn": self.H * self.vdim, "gates": 4 * self.H}
 
@@ -740,6 +800,9 @@ class Hgrn2Mixer:
         self.state = torch.zeros(eng.n_slots, H, d, dv, dtype=torch.float32, device=eng.device)
         self.chunked = eng.L.gated_chunked_supported(d, dv, True)
 
+    def chunk_floats(self, rows: int, slots: int) -> int:
+        return self.eng.L.gated_chunk_floats(rows, slots, self.H, self.dim, self.vdim)
+
     def scratch(self) -> Dict[str, int]:
         return {"mx": self.w_in.N, "ys": self.H * self.vdim, "yn": self.H * self.vdim}
 
@@ -758,6 +821,206 @@ class Hgrn2Mixer:
                      f_bias=self.f_bias, lower=self.lower, **e.gated_chunking(self))
         image = e.image("tmp", M)
         L.head_norm(ys, M, H, dv, e.cfg.norm_eps, self.norm, yn, image=image)
+        e.mm(self.w_o, yn, y, M, ready=image is not None)
+
+
+class GatedLinearMixer:
+    """Linear attention with a data-dependent decay per head and key channel.  Tensors <prefix>q, k, v, g, a1, a2, a2.b, norm, o.  Sizes:
+    heads, dim, vdim, tau.  q = W_q h / sqrt(dim), k, v;  f = sigmoid(W_a2 W_a1 h + b)^(1 / tau);  S <- diag(f) S + k v^T (f32, one
+    [dim][vdim] per slot and head),  o = S^T q;  every head's o gets an RMS norm with <prefix>norm [vdim] (shared by the heads), times
+    silu(W_g h), then W_o.  ONE product gives q, k, v, the output gate and the decays' low-rank inner vector."""
+
+    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["GatedLinearMixer"] = None):
+        self.eng, self.index = eng, index
+        self.H, self.dim, self.vdim, self.tau = int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["tau"])
+        H, d, dv = self.H, self.dim, self.vdim
+        if not eng.L.gated_supported(d, dv):
+            raise ValueError(f"layer {index}: gated linear attention takes head sizes up to 512 ({d})")
+        self.owns_weights = share is None
+        if share is None:
+            W, V, D = eng.weight, eng.vector, eng.dense_weight
+            parts = [W(prefix + n) for n in ("q", "k", "v", "g", "a1")]
+            w_a2 = W(prefix + "a2")
+            self.rank = int(w_a2.shape[1])
+            if any(tuple(t.shape) != (r, eng.cfg.width) for t, r in zip(parts, (H * d, H * d, H * dv, H * dv, self.rank))) or w_a2.shape[0] != H * d:
+                raise ValueError(f"layer {index}: q, k, v, g, a1, a2 have shapes {[tuple(t.shape) for t in parts + [w_a2]]}")
+            self.w_in, self.w_a2, self.w_o = D(torch.cat(parts, 0).contiguous()), D(w_a2), D(W(prefix + "o"))
+            self.a2_bias, self.norm = V(prefix + "a2.b"), V(prefix + "norm")
+            if self.a2_bias.numel() != H * d or self.norm.numel() != dv:
+                raise ValueError(f"layer {index}: a2.b or norm do not fit {H} heads of {d} / {dv}")
+        else:
+            for n in ("w_in", "w_a2", "w_o", "a2_bias", "norm", "rank"):
+                setattr(self, n, getattr(share, n))
+        self.state = torch.zeros(eng.n_slots, H, d, dv, dtype=torch.float32, device=eng.device)
+        self.chunked = eng.L.gated_chunked_supported(d, dv, True)
+
+    def chunk_floats(self, rows: int, slots: int) -> int:
+        return self.eng.L.gated_chunk_floats(rows, slots, self.H, self.dim, self.vdim)
+
+    def scratch(self) -> Dict[str, int]:
+        return {"mx": self.w_in.N, "az": self.H * self.dim, "ys": self.H * self.vdim, "yn": self.H * self.vdim}
+
+    def bind(self, mixers: list):
+        pass
+
+    def weight_bytes(self) -> int:
+        return self.w_in.nbytes() + self.w_a2.nbytes() + self.w_o.nbytes() if self.owns_weights else 0
+
+    def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
+        e, L = self.eng, self.eng.L
+        H, d, dv = self.H, self.dim, self.vdim
+        mx, az, ys, yn = e.buf("mx", self.w_in.N), e.buf("az", H * d), e.buf("ys", H * dv), e.buf("yn", H * dv)
+        k0, v0, g0, a0 = H * d, 2 * H * d, H * (2 * d + dv), H * (2 * d + 2 * dv)
+        e.mm(self.w_in, h, mx, M, src="h")
+        e.mm(self.w_a2, mx[:, a0:], az, M)
+        L.gated_scan(e.mamba_batch, e.n_seq, mx, mx[:, v0:], ys, self.state, H, d, dv, q_scale=d ** -0.5, k=mx[:, k0:], f=az, f_bias=self.a2_bias,
+                     gate=L.GATE_ROOT_SIGMOID, tau=self.tau, **e.gated_chunking(self))
+        image = e.image("tmp", M)
+        L.head_norm(ys, M, H, dv, e.cfg.norm_eps, self.norm, yn, gate=mx[:, g0:], gate_silu=True, image=image)
+        e.mm(self.w_o, yn, y, M, ready=image is not None)
+
+
+class DeltaMixer:
+    """The gated delta rule with decays per key channel.  Tensors <prefix>q, k, v, their .conv [channels][taps], b, A_log, a1, a2,
+    dt_bias, g1, g2, norm, o.  Sizes: heads, kv_heads (heads of q and k; head h uses h // (heads / kv_heads)), dim, vdim, conv (taps).
+    q, k, v = SiLU of a causal convolution per channel of their projections; q and k heads have length one, q / sqrt(dim) too;
+    f = exp(-e^A_log_h softplus(W_a2 W_a1 h + dt_bias)) [heads][dim];  S <- diag(f) S;  u = sigmoid(W_b h) (v - S^T k);  S <- S + k u^T;
+    o = S^T q;  every head's o gets an RMS norm with <prefix>norm [vdim], times sigmoid(W_g2 W_g1 h), then W_o.  Per slot: S [heads][dim]
+    [vdim] and the convolution's last taps - 1 inputs, f32.  ONE product gives everything that reads h."""
+
+    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["DeltaMixer"] = None):
+        self.eng, self.index = eng, index
+        self.H, self.G, self.dim, self.vdim, self.taps = int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]), int(m["vdim"]), int(m["conv"])
+        H, G, d, dv = self.H, self.G, self.dim, self.vdim
+        if not eng.L.gated_supported(d, dv) or H % G:
+            raise ValueError(f"layer {index}: {H} heads on {G} query / key heads of {d} (up to 512)")
+        self.channels = 2 * G * d + H * dv
+        self.owns_weights = share is None
+        if share is None:
+            W, V, D = eng.weight, eng.vector, eng.dense_weight
+            parts = [W(prefix + n) for n in ("q", "k", "v", "b", "a1", "g1")]
+            w_a2, w_g2 = W(prefix + "a2"), W(prefix + "g2")
+            self.ra, self.rg = int(w_a2.shape[1]), int(w_g2.shape[1])
+            rows = (G * d, G * d, H * dv, H, self.ra, self.rg)
+            if any(tuple(t.shape) != (r, eng.cfg.width) for t, r in zip(parts, rows)) or w_a2.shape[0] != H * d or w_g2.shape[0] != H * dv:
+                raise ValueError(f"layer {index}: q, k, v, b, a1, g1, a2, g2 have shapes {[tuple(t.shape) for t in parts + [w_a2, w_g2]]}")
+            self.w_conv = torch.cat([W(prefix + n + ".conv") for n in ("q", "k", "v")], 0).contiguous()
+            if tuple(self.w_conv.shape) != (self.channels, self.taps):
+                raise ValueError(f"layer {index}: the convolutions have shape {tuple(self.w_conv.shape)}")
+            self.w_in, self.w_a2, self.w_g2, self.w_o = D(torch.cat(parts, 0).contiguous()), D(w_a2), D(w_g2), D(W(prefix + "o"))
+            self.dt_bias, self.norm = V(prefix + "dt_bias"), V(prefix + "norm")
+            self.rate = torch.exp(V(prefix + "A_log").double()).float().contiguous()
+            if self.dt_bias.numel() != H * d or self.norm.numel() != dv or self.rate.numel() != H:
+                raise ValueError(f"layer {index}: dt_bias, norm or A_log do not fit {H} heads of {d} / {dv}")
+        else:
+            for n in ("w_in", "w_a2", "w_g2", "w_o", "w_conv", "dt_bias", "norm", "rate", "ra", "rg"):
+                setattr(self, n, getattr(share, n))
+        f32 = dict(dtype=torch.float32, device=eng.device)
+        self.state = torch.zeros(eng.n_slots, H, d, dv, **f32)
+        self.conv_state = torch.zeros(eng.n_slots, max(1, self.taps - 1), self.channels, **f32)
+        self.chunked = eng.L.delta_chunked_supported(d, dv)
+
+    def chunk_floats(self, rows: int, slots: int) -> int:
+        return self.eng.L.delta_chunk_floats(rows, slots, self.H, self.dim, self.vdim)
+
+    def scratch(self) -> Dict[str, int]:
+        H, d, dv = self.H, self.dim, self.vdim
+        return {"mx": self.w_in.N, "xbc": self.channels, "az": H * d, "gate2": H * dv, "ys": H * dv, "yn": H * dv, "du": H * dv if self.chunked else 0}
+
+    def bind(self, mixers: list):
+        pass
+
+    def weight_bytes(self) -> int:
+        if not self.owns_weights:
+            return 0
+        return sum(w.nbytes() for w in (self.w_in, self.w_a2, self.w_g2, self.w_o)) + self.w_conv.numel() * self.w_conv.element_size()
+
+    def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
+        e, L = self.eng, self.eng.L
+        H, G, d, dv = self.H, self.G, self.dim, self.vdim
+        mx, xc, az, g2, ys, yn = (e.buf(n, w) for n, w in (("mx", self.w_in.N), ("xbc", self.channels), ("az", H * d), ("gate2", H * dv),
+                                                           ("ys", H * dv), ("yn", H * dv)))
+        b0, a0 = self.channels, self.channels + H
+        e.mm(self.w_in, h, mx, M, src="h")
+        L.causal_conv(e.mamba_batch, M, e.n_seq, mx, self.w_conv, self.conv_state, xc, act=True, unit=(d, G * d, 2 * G * d, d ** -0.5))
+        e.mm(self.w_a2, mx[:, a0:], az, M)
+        e.mm(self.w_g2, mx[:, a0 + self.ra:], g2, M)
+        chunking = e.gated_chunking(self)
+        L.gated_scan(e.mamba_batch, e.n_seq, xc, xc[:, 2 * G * d:], ys, self.state, H, d, dv, k=xc[:, G * d:], f=az, f_bias=self.dt_bias,
+                     gate=L.GATE_SOFTPLUS, rate=self.rate, beta=mx[:, b0:], k_heads=G, u=e.buf("du", H * dv) if chunking else None, **chunking)
+        image = e.image("tmp", M)
+        L.head_norm(ys, M, H, dv, e.cfg.norm_eps, self.norm, yn, gate=g2, image=image)
+        e.mm(self.w_o, yn, y, M, ready=image is not None)
+
+
+class WkvMixer:
+    """RWKV time mixing.  Tensors <prefix>mu.r, mu.k, mu.v, mu.g, mu.w, r, k, v, g, w1, w2, w0, u, norm, o.  Sizes: heads, dim.  With
+    h' the row ahead in the sequence (zeros ahead of the first), mix_s = h + (h' - h) mu_s;  r, k, v = projections of theirs (heads x
+    dim);  f = exp(-exp(W_w2 tanh(W_w1 mix_w) + w0));  o = S^T r + (r . u k) v with the state ahead of the token, then
+    S <- diag(f) S + k v^T;  every head's o is divided by its root mean square, times <prefix>norm [heads * dim] and silu(W_g mix_g),
+    then W_o.  Per slot: S [heads][dim][dim] and the last h, f32.  Reads the rows of h, not their image (reads_rows)."""
+    MIXES = ("r", "k", "v", "g", "w")
+    reads_rows = True
+
+    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["WkvMixer"] = None):
+        self.eng, self.index = eng, index
+        self.H, self.dim = int(m["heads"]), int(m["dim"])
+        H, d, width = self.H, self.dim, eng.cfg.width
+        if not eng.L.gated_supported(d, d):
+            raise ValueError(f"layer {index}: time mixing takes head sizes up to 512 ({d})")
+        self.owns_weights = share is None
+        if share is None:
+            W, V, D = eng.weight, eng.vector, eng.dense_weight
+            parts, w1, w2 = [W(prefix + n) for n in ("r", "k", "v", "g")], W(prefix + "w1"), W(prefix + "w2")
+            self.rank = int(w1.shape[0])
+            if any(tuple(t.shape) != (H * d, width) for t in parts) or tuple(w1.shape) != (self.rank, width) or tuple(w2.shape) != (H * d, self.rank):
+                raise ValueError(f"layer {index}: r, k, v, g, w1, w2 have shapes {[tuple(t.shape) for t in parts + [w1, w2]]}")
+            self.w_rkvg, self.w_w1, self.w_w2, self.w_o = D(torch.stack(parts).contiguous()), D(w1), D(w2), D(W(prefix + "o"))
+            self.mu = torch.stack([V(prefix + "mu." + s) for s in self.MIXES]).contiguous()
+            self.w0, self.u, self.norm = V(prefix + "w0"), V(prefix + "u").reshape(-1).contiguous(), V(prefix + "norm")
+            if tuple(self.mu.shape) != (5, width) or any(t.numel() != H * d for t in (self.w0, self.u, self.norm)):
+                raise ValueError(f"layer {index}: mu, w0, u or norm do not fit {H} heads of {d}")
+        else:
+            for n in ("w_rkvg", "w_w1", "w_w2", "w_o", "mu", "w0", "u", "norm", "rank"):
+                setattr(self, n, getattr(share, n))
+        f32 = dict(dtype=torch.float32, device=eng.device)
+        self.state, self.shift_state = torch.zeros(eng.n_slots, H, d, d, **f32), torch.zeros(eng.n_slots, width, **f32)
+        self.chunked = eng.L.gated_chunked_supported(d, d, True)
+
+    def chunk_floats(self, rows: int, slots: int) -> int:
+        return self.eng.L.gated_chunk_floats(rows, slots, self.H, self.dim, self.dim)
+
+    def scratch(self) -> Dict[str, int]:
+        HD = self.H * self.dim
+        return {"shift": 5 * self.eng.cfg.width, "rkvg": 4 * HD, "w1": self.rank, "az": HD, "ys": HD, "yn": HD}
+
+    def bind(self, mixers: list):
+        pass
+
+    def weight_bytes(self) -> int:
+        return sum(w.nbytes() for w in (self.w_rkvg, self.w_w1, self.w_w2, self.w_o)) if self.owns_weights else 0
+
+    def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
+        e, L = self.eng, self.eng.L
+        H, d, width, R = self.H, self.dim, e.cfg.width, e.max_rows
+        HD = H * d
+        rkvg, w1, az, ys, yn = e.buf("rkvg", 4 * HD).view(4, R, HD), e.buf("w1", self.rank), e.buf("az", HD), e.buf("ys", HD), e.buf("yn", HD)
+        images = e.shift_images(M)
+        if images is not None:               # every mix straight into the operand image of the product that reads it
+            L.token_shift(e.mamba_batch, M, h, self.mu, self.shift_state, images=(images[0], images[0].numel(), e.ncap))
+            for s in range(4):
+                L.dense_tc(self.w_rkvg.wh[s], HD, width, images[s], e.ncap, rkvg[s], M)
+            L.dense_tc(self.w_w1.wh, self.rank, width, images[4], e.ncap, w1, M, epi=L.DENSE_SOFTCAP, param=1.0)        # cap 1: tanh
+        else:
+            mix = e.buf("shift", 5 * width).view(5, R, width)
+            L.token_shift(e.mamba_batch, M, h, self.mu, self.shift_state, out=mix)
+            L.dense_heads(self.w_rkvg.t, mix[0], rkvg[0], M, e.round_x, R * width, R * HD)
+            e.mm(self.w_w1, mix[4], w1, M, epi=L.DENSE_SOFTCAP, param=1.0)
+        e.mm(self.w_w2, w1, az, M)
+        L.gated_scan(e.mamba_batch, e.n_seq, rkvg[0], rkvg[2], ys, self.state, H, d, d, k=rkvg[1], f=az, f_bias=self.w0, gate=L.GATE_EXP_EXP,
+                     bonus=self.u, **e.gated_chunking(self))
+        image = e.image("tmp", M)
+        L.head_norm(ys, M, H, d, e.cfg.norm_eps, self.norm, yn, gate=rkvg[3], gate_silu=True, image=image)
         e.mm(self.w_o, yn, y, M, ready=image is not None)
 
 
@@ -819,16 +1082,26 @@ class Mamba1Mixer:
 
 
 class ParallelMixer:
-    """Two mixers side by side on the same input (the design's `parallel` trait names them; their tensors sit under <prefix>left. and
-    <prefix>right.): half the sum of their outputs, each first RMS-normed over the width with <prefix>left.out / right.out.  The
-    norms, the average and the sum into the residual stream are part of the stream's step (forward_branches)."""
+    """Two mixers side by side on the same input (the design's trait `kind` names them, an attention branch maybe with traits of its own;
+    their tensors sit under <prefix>left. and <prefix>right.).  combine "norms": half the sum of their outputs, each first RMS-normed over
+    the width with <prefix>left.out / right.out;  "scales": left_scale * left + right_scale * right, factors from the mixer entry.
+    Norms or factors and the sum into the residual stream are part of the stream's step (forward_branches)."""
 
-    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["ParallelMixer"] = None):
+    def __init__(self, eng: "LayerListEngine", index: int, m: dict, prefix: str, share: Optional["ParallelMixer"] = None, kind: str = "parallel"):
         self.eng = eng
-        kinds = eng.cfg.traits["parallel"]
-        self.left, self.right = (MIXERS[kinds[s]](eng, index, m[s], f"{prefix}{s}.", share=getattr(share, s) if share is not None else None)
-                                 for s in ("left", "right"))
-        if share is None:       # the factor 1/2 rides on the norms' weights (exact: a power of two)
+        spec = eng.cfg.traits.get(kind)
+        if spec is None:
+            raise ValueError(f"layer {index}: {eng.cfg.architecture} has no {kind!r} mixer")
+
+        def branch(s):
+            name, opts = (spec[s], {}) if isinstance(spec[s], str) else (spec[s][0], {"traits": spec[s][1]})
+            return MIXERS[name](eng, index, m[s], f"{prefix}{s}.", share=getattr(share, s) if share is not None else None, **opts)
+
+        self.left, self.right = branch("left"), branch("right")
+        self.scales = (float(m["left_scale"]), float(m["right_scale"])) if spec.get("combine") == "scales" else None
+        if self.scales is not None:
+            self.out_l = self.out_r = None
+        elif share is None:       # the factor 1/2 rides on the norms' weights (exact: a power of two)
             self.out_l, self.out_r = ((0.5 * eng.norm_weight(f"{prefix}{s}.out")).contiguous() for s in ("left", "right"))
         else:
             self.out_l, self.out_r = share.out_l, share.out_r
@@ -850,19 +1123,22 @@ class ParallelMixer:
     def weight_bytes(self) -> int:
         return sum(p.weight_bytes() for p in self.parts())
 
-    def forward_branches(self, h: torch.Tensor, M: int) -> list:
-        """[(branch output, weight of its norm)]: the mixer's output is the sum of the normed branches."""
+    def forward_branches(self, h: torch.Tensor, M: int) -> dict:
+        """The terms of residual_step() whose sum is the mixer's output: `normed` [(branch output, weight of its norm)], or `adds` with
+        their `scales`."""
         e = self.eng
         bl, br = e.buf("br_l"), e.buf("br_r")
         with e.side(1, M):
             self.right.forward(h, br, M)
         self.left.forward(h, bl, M)
         e.join(1, M)
-        return [(bl, self.out_l), (br, self.out_r)]
+        if self.scales is not None:
+            return {"adds": [bl, br], "scales": self.scales}
+        return {"normed": [(bl, self.out_l), (br, self.out_r)]}
 
     def forward(self, h: torch.Tensor, y: torch.Tensor, M: int):
         e = self.eng
-        e.L.residual_step(M, e.cfg.width, e.cfg.norm_eps, normed=self.forward_branches(h, M), x=y)
+        e.L.residual_step(M, e.cfg.width, e.cfg.norm_eps, x=y, **self.forward_branches(h, M))
 
 
 class RoutedExperts:
@@ -960,8 +1236,9 @@ class RoutedExperts:
 
 
 MIXERS = {"latent_attention": LatentAttentionMixer, "mamba2": Mamba2Mixer, "attention": WindowAttentionMixer,
-          "lightning": LightningMixer, "mlstm": MLstmMixer, "hgrn2": Hgrn2Mixer, "mamba1": Mamba1Mixer, "parallel": ParallelMixer}
-SHARING_MIXERS = ("attention", "lightning", "mlstm", "hgrn2", "mamba1", "parallel")      # run another layer's weights on a cache / state of their own
+          "lightning": LightningMixer, "mlstm": MLstmMixer, "hgrn2": Hgrn2Mixer, "mamba1": Mamba1Mixer, "gated_linear": GatedLinearMixer,
+          "delta": DeltaMixer, "wkv": WkvMixer, "parallel": ParallelMixer, "parallel_2": functools.partial(ParallelMixer, kind="parallel_2")}
+SHARING_MIXERS = ("attention", "lightning", "mlstm", "hgrn2", "mamba1", "gated_linear", "delta", "wkv", "parallel", "parallel_2")      # run another layer's weights on a cache / state of their own
 FEED_FORWARDS = {"dense": DenseFeedForward, "moe": RoutedExperts}
 
 
@@ -1000,7 +1277,7 @@ class _Layer:
             return
         self.mixer = MIXERS[spec.type](eng, i, spec.mixer, p + "mix.")
         # "post": the norm on a sublayer's output carries the residual multiplier, x <- x + (m g) * y / rms(y)
-        norm_w = (lambda name: (eng.norm_weight(name) * eng.cfg.residual_mult).contiguous()) if post else eng.norm_weight
+        norm_w = (lambda name: (eng.norm_weight(name) * eng.cfg.residual_mult).contiguous()) if post else eng.norm_params
         self.norm1 = norm_w(p + "norm1")
         self.canon1 = None
         if taps > 0:
@@ -1017,7 +1294,8 @@ class _Layer:
             if kind not in FEED_FORWARDS:
                 raise ValueError(f"layer {i}: unknown feed-forward kind {kind!r}")
             self.ff = FEED_FORWARDS[kind](eng, i, spec.mlp, p + "mlp.")
-            self.norm2 = norm_w(p + "norm2")
+            if not eng.cfg.traits.get("one_norm"):
+                self.norm2 = norm_w(p + "norm2")
             self.norm2b = eng.vector(p + "norm2b") if sandwich else None
             if not sandwich:
                 self.hc2 = _HyperWeights(eng, p + "hc2." if eng.cfg.hyper_weights else None)
@@ -1073,10 +1351,15 @@ class LayerListEngine:
                         raise ValueError(f"layer {i}: its entry differs from layer {spec.weights_of}, whose weights it uses")
                     built[i] = _Layer(self, i, spec, owner)
             self.layers: List[_Layer] = [built[i] for i in range(len(self.cfg.layers))]
-            self.final_norm, self.head = self.norm_weight("final.norm"), self.dense_weight(self.weight("head"))
+            self.final_norm = self.norm_params("final.norm")
+            self.head = self.dense_weight(self.embed if self.cfg.traits.get("tied_head") else self.weight("head"))
             self.embed_norm = self.norm_weight("embed.norm") if self.cfg.traits.get("embed_norm") else None
-            self.loop_step = None
-            if self.cfg.loop_times:
+            self.loop_step = self.loop_in = None
+            if self.cfg.loop_times and self.cfg.traits.get("loop_in"):
+                self.loop_in = self.dense_weight(self.weight("loop.in"))
+                if tuple(self.loop_in.t.shape) != (self.cfg.width, 2 * self.cfg.width):
+                    raise ValueError(f"loop.in has shape {tuple(self.loop_in.t.shape)}")
+            elif self.cfg.loop_times:
                 self.loop_step = self.vector("loop.step")
                 if tuple(self.loop_step.shape) != (self.cfg.loop_times, self.cfg.width):
                     raise ValueError(f"loop.step has shape {tuple(self.loop_step.shape)}")
@@ -1117,19 +1400,18 @@ class LayerListEngine:
             self._lightning_scratch = torch.zeros(max(L.lightning_chunk_floats(R, self.n_slots, mx.H, mx.dim, mx.vdim) for mx in lt),
                                                   dtype=torch.float32, device=dev)
         # the same with data-dependent gates
-        gt = [mx for mx in mixers if isinstance(mx, (MLstmMixer, Hgrn2Mixer)) and mx.chunked]
+        gt = [mx for mx in mixers if isinstance(mx, (MLstmMixer, Hgrn2Mixer, GatedLinearMixer, DeltaMixer, WkvMixer)) and mx.chunked]
         self.gated_chunks, self._gated_scratch, self._gated_slots = 0, None, R // L.GATED_CHUNK + self.n_slots
         if gt and R >= GATED_CHUNKED_MIN_ROWS and os.environ.get("DLLAMA_LAYERS_CHUNKED_SCAN", "1") != "0":
-            self._gated_scratch = torch.zeros(max(L.gated_chunk_floats(R, self.n_slots, mx.H, mx.dim, mx.vdim) for mx in gt),
-                                              dtype=torch.float32, device=dev)
+            self._gated_scratch = torch.zeros(max(mx.chunk_floats(R, self.n_slots) for mx in gt), dtype=torch.float32, device=dev)
         st = [mx for mx in mixers if isinstance(mx, Mamba1Mixer) and mx.chunked]
         self.selective_chunks, self._selective_scratch, self._selective_slots = 0, None, R // L.SELECTIVE_CHUNK + self.n_slots
         if st and R >= GATED_CHUNKED_MIN_ROWS and os.environ.get("DLLAMA_LAYERS_CHUNKED_SCAN", "1") != "0":
             self._selective_scratch = torch.zeros(self._selective_slots * max(mx.inner * (mx.N + 1) for mx in st), dtype=torch.float32, device=dev)
         if self.cfg.residual in ("post", "parallel") and self.cfg.streams != 1:
             raise ValueError(f"the {self.cfg.residual} residual style keeps one residual stream")
-        if (self.embed_norm is not None) != (self.cfg.residual == "parallel"):
-            raise ValueError("a normed embedding belongs to the parallel residual style")
+        if self.cfg.residual != "parallel" and any(self.cfg.traits.get(n) for n in ("embed_norm", "norm", "one_norm", "loop_in")):
+            raise ValueError("a normed embedding, layer norms, one norm per layer and loop.in belong to the parallel residual style")
         if self.cfg.canon_taps and self.cfg.residual != "hyper":
             raise ValueError("a convolution in front of the mixers is only wired into the pre-norm / hyper residual style")
         # scratch: one f32 buffer per name, as wide as the widest user
@@ -1146,6 +1428,10 @@ class LayerListEngine:
         if self.tc:       # activation slabs: one kept for a sublayer's input (several products read it), one for the rest
             n = L.xh_bytes(self._kmax, self.ncap)
             self._xh = {k: torch.zeros(n, dtype=torch.uint8, device=dev) for k in ("h", "tmp") + (("h2", "tmp1", "tmp2") if self.cfg.residual == "parallel" else ())}
+            self._shift_images = None
+            if any(isinstance(mx, WkvMixer) for mx in mixers):
+                n = L.xh_bytes(self.cfg.width, self.ncap)
+                self._shift_images = [t for t in torch.zeros(5, n, dtype=torch.uint8, device=dev)]
         if self.cfg.streams > L.HC_MAX_STREAMS:
             raise ValueError(f"{self.cfg.streams} streams: the kernels keep at most {L.HC_MAX_STREAMS} copies of the residual stream")
         self.x = torch.zeros(R, self.cfg.streams * self.cfg.width, dtype=torch.float32, device=dev)      # row = [streams][width]
@@ -1154,6 +1440,9 @@ class LayerListEngine:
         self.y = torch.zeros(R, self.cfg.width, dtype=torch.float32, device=dev)
         if self.cfg.residual == "parallel":       # the embedding output, the feed-forward's input and output
             self.x0, self.hn2, self.y2 = (torch.zeros(R, self.cfg.width, dtype=torch.float32, device=dev) for _ in range(3))
+            if self.loop_in is not None:      # [stream | embedding output], the operand of loop.in
+                self.x_x0 = torch.zeros(R, 2 * self.cfg.width, dtype=torch.float32, device=dev)
+                self.x0 = self.x_x0[:, self.cfg.width:]
         self.logits = torch.zeros(R, self.cfg.vocab, dtype=torch.float32, device=dev)
         self.out_tokens = torch.zeros(R, dtype=torch.int32, device=dev)
         self.h_out_tokens = torch.zeros(R, dtype=torch.int32).pin_memory()
@@ -1225,24 +1514,30 @@ class LayerListEngine:
             raise ValueError(f"{name} has shape {tuple(w.shape)}")
         return w
 
+    def norm_params(self, name: str):
+        """A norm over the width as residual_step() takes it: its weight, or (weight, bias) of a layer norm."""
+        if self.cfg.traits.get("norm") != "layer":
+            return self.norm_weight(name)
+        return self.norm_weight(name), self.norm_weight(name + ".b")
+
     def dense_weight(self, t: torch.Tensor) -> DenseWeight:
         self._kmax = max(self._kmax, int(t.shape[-1]))
         return DenseWeight(t, self.tc)
 
     def mm(self, w: DenseWeight, x: torch.Tensor, y: torch.Tensor, M: int, epi: int = 0, aux=None, param: float = 0.0,
-           src: str = "tmp", param2: float = 0.0, ready: bool = False, image=None):
-        """y[:M] = epi(x[:M] @ w^T).  src="h": x is the current sublayer input; its tensor-core image is made by the
+           src: str = "tmp", param2: float = 0.0, ready: bool = False, image=None, bias=None):
+        """y[:M] = epi(x[:M] @ w^T + bias).  src="h": x is the current sublayer input; its tensor-core image is made by the
         first product that reads it (begin_sublayer() marks it stale) and shared by the others.  ready: the launch that
         produced x left it as the image of `src` (see image()).  image: the result leaves as that image instead of y."""
         L = self.L
         if w.wh is None or M < TC_MIN_ROWS:
-            L.dense(w.t, x, y, M, self.round_x, epi=epi, aux=aux, param=param, param2=param2)
+            L.dense(w.t, x, y, M, self.round_x, epi=epi, aux=aux, param=param, param2=param2, bias=bias)
             return
         xh = self._xh[self._xh_h if src == "h" else self._tmp]
         if not ready and (src != "h" or not self._xh_h_ready):
             L.xh_from_rows(x, M, w.K, self.ncap, xh)
             self._xh_h_ready = src == "h" or self._xh_h_ready
-        L.dense_tc(w.wh, w.N, w.K, xh, self.ncap, y, M, epi=epi, aux=aux, param=param, param2=param2, image=image)
+        L.dense_tc(w.wh, w.N, w.K, xh, self.ncap, y, M, epi=epi, aux=aux, param=param, param2=param2, image=image, bias=bias)
 
     def mm_heads(self, w: DenseWeight, x: torch.Tensor, y: torch.Tensor, M: int, x_head_stride: int, y_head_stride: int):
         """Per head h: y[:M, h*ys : h*ys+N] = x[:M, h*xs : h*xs+K] @ w[h]^T."""
@@ -1265,6 +1560,10 @@ class LayerListEngine:
         """(activation image, its row capacity) if products over M rows read bf16 images, so that a kernel can leave its
         result in the next product's operand layout; None where they read f32 rows."""
         return (self._xh[self._tmp if name == "tmp" else name], self.ncap) if self.tc and M >= TC_MIN_ROWS else None
+
+    def shift_images(self, M: int):
+        """The five activation images of a time-mixing layer's mixes, or None where its products read f32 rows."""
+        return self._shift_images if self.tc and M >= TC_MIN_ROWS else None
 
     @contextlib.contextmanager
     def side(self, k: int, M: int):
@@ -1479,48 +1778,73 @@ class LayerListEngine:
                 L.rms_norm(x, hn, n_logits, W, eps, w=self.final_norm, plus_one=True, rows=self.logit_rows)
         if n_logits:
             self.begin_sublayer(ready=head_ready)
-            if cfg.logit_softcap > 0:
+            if cfg.logit_scale != 1.0:
+                self.mm(self.head, hn, self.logits, n_logits, epi=L.DENSE_SCALE, param=cfg.logit_scale, src="h")
+            elif cfg.logit_softcap > 0:
                 self.mm(self.head, hn, self.logits, n_logits, epi=L.DENSE_SOFTCAP, param=cfg.logit_softcap, src="h")
             else:
                 self.mm(self.head, hn, self.logits, n_logits, src="h")
 
     def _launch_parallel_layers(self, M: int, n_logits: int) -> bool:
-        """Layers whose mixer and feed-forward read the same residual stream through a norm each.  One launch per layer sums
-        the last layer's outputs into the stream (branches normed on the way; ahead of a pass of the loop also the embedding
-        output and the pass's vector) and leaves both normed copies, as bf16 images where the products read those.  Returns
-        whether the last norm left the head's operand image."""
+        """Layers whose mixer and feed-forward read the same residual stream through a norm each, or through one norm.  One launch
+        per layer sums the last layer's outputs into the stream (branches normed or scaled on the way; ahead of a pass of the loop
+        also the embedding output and the pass's vector) and leaves the normed copies, as bf16 images where the products read
+        those.  A pass that opens with loop.in needs the sum beside the embedding output first.  Returns whether the last norm
+        left the head's operand image."""
         L, cfg = self.L, self.cfg
         x, x0, W, eps = self.x, self.x0, cfg.width, cfg.norm_eps
-        L.residual_step(M, W, eps, x_in=self.embed, rows=self.tokens, outs=[(self.embed_norm, x0)])        # the embedding output
-        src, adds, normed = x0, [], []
+        one_norm, layer_norm = bool(cfg.traits.get("one_norm")), cfg.traits.get("norm") == "layer"
+        step = functools.partial(L.residual_step, dim=W, eps=eps, layer_norm=layer_norm)
+        # the embedding output
+        if self.embed_norm is not None:
+            L.residual_step(M, W, eps, x_in=self.embed, rows=self.tokens, outs=[(self.embed_norm, x0)])
+        else:
+            step(M, x_in=self.embed, rows=self.tokens, x=x0)
+        src, terms = x0, {}
         img1, img2 = self.image("h", M), self.image("h2", M)
         for l in self.layers:
-            if l.opens:
-                adds = adds + [x0]
-            L.residual_step(M, W, eps, x_in=src, adds=adds, normed=normed, vec=self.loop_step[l.opens] if l.opens is not None else None,
-                            x=x, outs=[(l.norm1, img1 or self.hn)] + ([(l.norm2, img2 or self.hn2)] if l.ff is not None else []))
-            src, adds, normed = x, [], []
+            vec = None
+            if l.opens is not None and self.loop_in is not None:
+                step(M, x_in=src, x=self.x_x0, **terms)
+                self.mm(self.loop_in, self.x_x0, x, M)
+                src, terms = x, {}
+            elif l.opens is not None:
+                vec = self.loop_step[l.opens]
+                if l.opens:
+                    terms = dict(terms, adds=list(terms.get("adds", [])) + [x0])
+            # a mixer that reads f32 rows gets them beside the image the feed-forward's product reads
+            rows = getattr(l.mixer, "reads_rows", False)
+            if one_norm:
+                outs = [(l.norm1, img1 or self.hn)] if not rows or l.ff is not None else []
+                if rows and (img1 or not outs):
+                    outs.append((l.norm1, self.hn))
+                ff_in, ff_image, ff_img = self.hn, "h", img1
+            else:
+                outs = [(l.norm1, self.hn if rows else img1 or self.hn)] + ([(l.norm2, img2 or self.hn2)] if l.ff is not None else [])
+                ff_in, ff_image, ff_img = self.hn2, "h2", img2
+            step(M, x_in=src, vec=vec, x=x if src is not x or terms or vec is not None else None, outs=outs, **terms)
+            src, terms = x, {}
             if l.ff is not None:
-                self.begin_sublayer("h2", ready=img2 is not None)
+                self.begin_sublayer(ff_image, ready=ff_img is not None)
                 with self.side(0, M):
-                    l.ff.forward(self.hn2, self.y2, M)
-            self.begin_sublayer("h", ready=img1 is not None)
+                    l.ff.forward(ff_in, self.y2, M)
+            self.begin_sublayer("h", ready=img1 is not None and not (rows and not one_norm))
             if isinstance(l.mixer, ParallelMixer):
-                normed = l.mixer.forward_branches(self.hn, M)
+                terms = l.mixer.forward_branches(self.hn, M)
             else:
                 l.mixer.forward(self.hn, self.y, M)
-                adds.append(self.y)
+                terms = {"adds": [self.y]}
             if l.ff is not None:
                 self.join(0, M)
-                adds.append(self.y2)
+                terms["adds"] = list(terms.get("adds", [])) + [self.y2]
             if self.layer_probe is not None:
-                L.residual_step(M, W, eps, x_in=src, adds=adds, normed=normed, x=x)
-                adds, normed = [], []
+                step(M, x_in=src, x=x, **terms)
+                terms = {}
                 self.layer_probe.append(x[:M].clone())
         if not n_logits:
             return False
         img = self.image("h", n_logits)
-        L.residual_step(n_logits, W, eps, x_in=src, adds=adds, normed=normed, rows=self.logit_rows, outs=[(self.final_norm, img or self.hn)])
+        step(n_logits, x_in=src, rows=self.logit_rows, outs=[(self.final_norm, img or self.hn)], **terms)
         return img is not None
 
     def _launch_hyper_layers(self, M: int):
@@ -1649,7 +1973,16 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
             return (1 + torch.randn((), generator=g) * 0.1).to(torch.bfloat16)
         return small(W) if sandwich else 1 + small(W)
 
-    t = {"embed": (torch.randn(V, W, generator=g)).to(torch.bfloat16), "head": mat(V, W), "final.norm": norm_w()}
+    t = {"embed": (torch.randn(V, W, generator=g)).to(torch.bfloat16)}
+    if not traits.get("tied_head"):
+        t["head"] = mat(V, W)
+
+    def norm(name):
+        t[name] = norm_w()
+        if traits.get("norm") == "layer":
+            t[name + ".b"] = small(W)
+
+    norm("final.norm")
 
     def hyper(prefix):
         # read weights around 1 / S, write weights around 1, a mixing matrix near the identity with some cross-talk
@@ -1657,7 +1990,7 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
         t[prefix + "out"] = (1.0 + torch.randn(S, generator=g) * 0.2).to(torch.bfloat16)
         t[prefix + "mix"] = (torch.eye(S) * 0.9 + torch.randn(S, S, generator=g) * 0.1).to(torch.bfloat16)
 
-    def attention(p, m):
+    def attention(p, m, att=att):
         H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m.get("vdim", m["dim"])
         t[p + "q"] = mat(H * d, W, 2.0)
         if m.get("kv_from") is None:
@@ -1667,10 +2000,15 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
             t[p + "v"] = mat(G * dv, W)
         if att.get("talk"):     # near the identity, with cross-talk between all heads
             t[p + "talk"] = (torch.eye(H) + torch.randn(H, H, generator=g) * 0.3).to(torch.bfloat16)
-        if att.get("sink"):
+        if att.get("sink") and att["sink"] != "zero":
             t[p + "sink"] = (torch.randn(H, generator=g)).to(torch.bfloat16)
         if att.get("gate"):
-            t[p + "g"] = mat(H * dv, W)
+            t[p + "g"] = mat(H if att["gate"] == "head" else H * dv, W)
+        if att.get("bias"):
+            for n, rows in (("q", H * d), ("k", G * d), ("v", G * dv)):
+                t[p + n + ".b"] = small(rows, 0.5)
+        if att.get("head_norm"):
+            t[p + "q.norm"], t[p + "k.norm"] = 1 + small(d), 1 + small(d)
         if att.get("proj_norm"):
             t[p + "q.norm"], t[p + "k.norm"] = 1 + small(H * d), 1 + small(G * d)
 
@@ -1681,16 +2019,46 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
         t[p + "lower"] = (torch.rand(H * d, generator=g) * 0.9).to(torch.bfloat16)
         t[p + "norm"], t[p + "o"] = 1 + small(dv), mat(W, H * dv)
 
+    def gated_linear(p, m):
+        H, d, dv, r = m["heads"], m["dim"], m["vdim"], m.get("rank", max(4, W // 16))
+        t[p + "q"], t[p + "k"], t[p + "v"], t[p + "g"] = mat(H * d, W, 2.0), mat(H * d, W), mat(H * dv, W), mat(H * dv, W)
+        t[p + "a1"], t[p + "a2"], t[p + "a2.b"] = mat(r, W), mat(H * d, r, 2.0), (torch.rand(H * d, generator=g) * 4).to(torch.bfloat16)
+        t[p + "norm"], t[p + "o"] = 1 + small(dv), mat(W, H * dv)
+
+    def delta(p, m):
+        H, G, d, dv, K, r = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"], m.get("rank", max(4, W // 16))
+        for n, rows in (("q", G * d), ("k", G * d), ("v", H * dv)):
+            t[p + n], t[p + n + ".conv"] = mat(rows, W, 1.5), mat(rows, K, 1.5)
+        t[p + "b"], t[p + "a1"], t[p + "a2"], t[p + "g1"], t[p + "g2"] = mat(H, W, 2.0), mat(r, W), mat(H * d, r), mat(r, W), mat(H * dv, r)
+        t[p + "A_log"] = torch.log(torch.rand(H, generator=g) * 1.5 + 0.25).to(torch.bfloat16)
+        t[p + "dt_bias"] = (torch.rand(H * d, generator=g) * 4 - 5).to(torch.bfloat16)
+        t[p + "norm"], t[p + "o"] = 1 + small(dv), mat(W, H * dv)
+
+    def wkv(p, m):
+        H, d, r = m["heads"], m["dim"], m.get("rank", max(4, W // 16))
+        for n in ("r", "k", "v", "g", "w"):
+            t[p + "mu." + n] = torch.rand(W, generator=g).to(torch.bfloat16)
+        for n in ("r", "k", "v", "g"):
+            t[p + n] = mat(H * d, W)
+        t[p + "w1"], t[p + "w2"], t[p + "w0"] = mat(r, W), mat(H * d, r), (torch.rand(H * d, generator=g) * 5 - 6).to(torch.bfloat16)
+        t[p + "u"], t[p + "norm"], t[p + "o"] = (torch.randn(H, d, generator=g) * 0.5).to(torch.bfloat16), 1 + small(H * d), mat(W, H * d)
+
+    def branch(spec, p, m):
+        kind, opts = (spec, {}) if isinstance(spec, str) else (spec[0], {"att": spec[1]})
+        {"attention": attention, "hgrn2": hgrn2, "gated_linear": gated_linear, "delta": delta}[kind](p, m, **opts)
+
     if traits.get("embed_norm"):
         t["embed.norm"] = norm_w()
-    if config.get("loop"):
+    if config.get("loop") and traits.get("loop_in"):
+        t["loop.in"] = mat(W, 2 * W)
+    elif config.get("loop"):
         t["loop.step"] = (torch.randn(int(config["loop"]["times"]), W, generator=g) * 0.3).to(torch.bfloat16)
 
     for i, l in enumerate(config["layers"]):
         p, m = f"l{i}.", l["mixer"]
         if l.get("weights_of") is not None:
             continue
-        t[p + "norm1"] = norm_w()
+        norm(p + "norm1")
         if taps:
             t[p + "canon1"] = mat(W, taps, 0.5)
         if sandwich:
@@ -1720,10 +2088,14 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
             attention(p + "mix.", m)
         elif l["type"] == "hgrn2":
             hgrn2(p + "mix.", m)
-        elif l["type"] == "parallel":
-            attention(p + "mix.left.", m["left"])
-            hgrn2(p + "mix.right.", m["right"])
-            t[p + "mix.left.out"], t[p + "mix.right.out"] = 1 + small(W), 1 + small(W)
+        elif l["type"] == "wkv":
+            wkv(p + "mix.", m)
+        elif l["type"] in ("parallel", "parallel_2"):
+            spec = traits[l["type"]]
+            branch(spec["left"], p + "mix.left.", m["left"])
+            branch(spec["right"], p + "mix.right.", m["right"])
+            if spec.get("combine") != "scales":
+                t[p + "mix.left.out"], t[p + "mix.right.out"] = 1 + small(W), 1 + small(W)
         elif l["type"] == "mlstm":
             H, d, dv = m["heads"], m["dim"], m["vdim"]
             t[p + "mix.q"], t[p + "mix.k"], t[p + "mix.v"] = mat(H * d, W), mat(H * d, W), mat(H * dv, W)
@@ -1745,7 +2117,8 @@ def random_tensors(config: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
         else:
             raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
         if l.get("mlp"):
-            t[p + "norm2"] = norm_w()
+            if not traits.get("one_norm"):
+                norm(p + "norm2")
             if sandwich:
                 t[p + "norm2b"] = small(W)
             elif S:
@@ -1862,3 +2235,20 @@ def example_config_vopedra(width: int = 160, vocab: int = 320, heads: int = 3) -
               {"type": "mlstm", "mixer": {"heads": 1, "dim": 40, "vdim": 24, "gate_cap": 15.0}, "mlp": {"kind": "dense", "ff": width}}]
     return {"architecture": "Vopedra", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "loop": {"start": 1, "stop": 3, "times": 2},
             "layers": layers}
+
+
+def example_config_silizen(width: int = 160, vocab: int = 320, heads: int = 3) -> dict:
+    """A small Silizen-shaped configuration: a time-mixing layer, then soft-capped attention beside gated linear attention and windowed
+    attention beside a gated delta rule (both run twice), then a time-mixing layer without a feed-forward."""
+    dense = {"kind": "dense", "ff": 2 * width}
+    left = {"heads": 2 * heads, "kv_heads": heads, "dim": 24, "vdim": 40, "scale": 0.2, "softcap": 20.0,
+            "rot": {"base": 10000.0, "dims": 16, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 256}}}
+    window = {"heads": 2 * heads, "kv_heads": heads, "dim": 32, "vdim": 32, "scale": 0.3, "mask": {"size": 40}}
+    layers = [{"type": "wkv", "mixer": {"heads": heads, "dim": 20}, "mlp": dict(dense)},
+              {"type": "parallel", "mlp": dict(dense), "mixer": {"left": left, "right": {"heads": heads, "dim": 28, "vdim": 16, "tau": 8.0},
+                                                                 "left_scale": 0.8, "right_scale": 1.1}},
+              {"type": "parallel_2", "mlp": {"kind": "dense", "ff": width},
+               "mixer": {"left": window, "right": {"heads": 2 * heads, "kv_heads": heads, "dim": 20, "vdim": 24, "conv": 3}}},
+              {"type": "wkv", "mixer": {"heads": 1, "dim": 36}, "mlp": None}]
+    return {"architecture": "Silizen", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "loop": {"start": 1, "stop": 3, "times": 2}, "layers": layers}

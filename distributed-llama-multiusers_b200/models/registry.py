@@ -22,6 +22,7 @@ ARCHITECTURES: Dict[str, Callable] = {
     "Sunesun": _layer_list,        # windowed attention (values = keys) + routed experts on hyper-connected residual streams
     "Venadra": _layer_list,        # lightning (linear) attention and chunked sink attention behind a short convolution, PolyNorm / gated experts
     "Darusun": _layer_list,        # post-norm layers: head-mixed grouped-query attention, windowed latent attention with sinks, xIELU / experts with a shared one
+    "Silizen": _layer_list,        # parallel-residual layers on one layer norm: soft-capped attention beside gated linear attention, windowed attention beside a gated delta rule, WKV time mixing
     "Vopedra": _layer_list,        # parallel-residual layers, some run several times: matrix memory, selective scan, attention beside HGRN2
 }
 

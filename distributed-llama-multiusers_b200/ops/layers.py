@@ -10,10 +10,10 @@ from typing import Optional
 import torch
 
 from . import lib
-from .lib import (DENSE_GLU_CLAMP, DENSE_GLU_GELU, DENSE_GLU_SILU, DENSE_MUL, DENSE_RELU2, DENSE_ROWGATE_ADD, DENSE_SIGMOID_MUL, DENSE_SILU, DENSE_SOFTCAP, DENSE_STORE,  # noqa: F401
-                  DENSE_XIELU, EPI_DENSE, T_BF16, T_F32,
+from .lib import (DENSE_GLU_CLAMP, DENSE_GLU_GELU, DENSE_GLU_SILU, DENSE_MUL, DENSE_RELU2, DENSE_ROWGATE_ADD, DENSE_SCALE, DENSE_SIGMOID_MUL, DENSE_SILU, DENSE_SOFTCAP, DENSE_STORE,  # noqa: F401
+                  DENSE_XIELU, EPI_DENSE, GATE_EXP_EXP, GATE_LOWER, GATE_ROOT_SIGMOID, GATE_SOFTPLUS, T_BF16, T_F32,
                   DlConvArgs, DlDenseArgs, DlEpilogue, DlGatedArgs, DlHeadNormArgs, DlHyperArgs, DlLatentAttnArgs, DlLightningArgs, DlLatentKvArgs, DlLatentTiles, DlMambaBatch, DlMambaChunks, DlMambaScanArgs, DlMoeArgs,
-                  DlMlstmGatesArgs, DlMoePlanArgs, DlMoeSelectArgs, DlNormArgs, DlResidualArgs, DlSelectiveArgs, DlWindowAttnArgs, DlWindowKvArgs, check_layers, layers_lib)
+                  DlMlstmGatesArgs, DlMoePlanArgs, DlMoeSelectArgs, DlNormArgs, DlResidualArgs, DlSelectiveArgs, DlShiftArgs, DlWindowAttnArgs, DlWindowKvArgs, check_layers, layers_lib)
 
 PAGE_SIZE = 32
 HC_MAX_STREAMS = 16          # DL_HC_MAX_STREAMS of the hyper-connection kernel
@@ -47,8 +47,8 @@ def embed_rows(table: torch.Tensor, tokens: torch.Tensor, x: torch.Tensor, M: in
 
 
 def dense(w: torch.Tensor, x: torch.Tensor, y: torch.Tensor, M: int, round_x: bool, epi: int = DENSE_STORE,
-          aux: Optional[torch.Tensor] = None, param: float = 0.0, param2: float = 0.0):
-    """y[:M] = epi(x[:M] @ w^T); w [N][K] (rows may be strided), x [.., >= K] and y [.., >= N] row-major f32."""
+          aux: Optional[torch.Tensor] = None, param: float = 0.0, param2: float = 0.0, bias: Optional[torch.Tensor] = None):
+    """y[:M] = epi(x[:M] @ w^T + bias); w [N][K] (rows may be strided), x [.., >= K] and y [.., >= N] row-major f32."""
     N, K = w.shape
     a = DlDenseArgs()
     a.W, a.wtype, a.ldw, a.w_bs = w.data_ptr(), _type(w), w.stride(0), 0
@@ -57,7 +57,7 @@ def dense(w: torch.Tensor, x: torch.Tensor, y: torch.Tensor, M: int, round_x: bo
     a.M, a.N, a.K, a.batch = M, N, K, 1
     a.round_x, a.epi = 1 if round_x else 0, epi
     a.aux, a.ld_aux, a.aux_bs = _p(aux), (aux.stride(0) if aux is not None else 0), 0
-    a.param, a.param2 = param, param2
+    a.param, a.param2, a.bias = param, param2, _p(bias)
     check_layers(layers_lib().dl_dense(a, _stream()), "dl_dense")
     lib.count_launch()
 
@@ -104,8 +104,8 @@ def xh_from_rows(x: torch.Tensor, M: int, K: int, ncap: int, xh: torch.Tensor):
 
 
 def dense_tc(wh: torch.Tensor, N: int, K: int, xh: torch.Tensor, ncap: int, y: torch.Tensor, M: int, epi: int = DENSE_STORE,
-             aux: Optional[torch.Tensor] = None, param: float = 0.0, param2: float = 0.0, image=None):
-    """y[:M, :N] = epi(x @ w^T) from the two operand images (bf16 x bf16 -> f32 in tensor memory); DENSE_GLU_GELU may leave the
+             aux: Optional[torch.Tensor] = None, param: float = 0.0, param2: float = 0.0, image=None, bias: Optional[torch.Tensor] = None):
+    """y[:M, :N] = epi(x @ w^T + bias) from the two operand images (bf16 x bf16 -> f32 in tensor memory); DENSE_GLU_GELU may leave the
     result in image = (activation image, ncap) instead of y."""
     e = DlEpilogue()
     e.kind, e.n_dst, e.ld, e.dst_off = EPI_DENSE, 1, y.stride(0), 0
@@ -113,7 +113,7 @@ def dense_tc(wh: torch.Tensor, N: int, K: int, xh: torch.Tensor, ncap: int, y: t
     if image is not None:
         assert epi == DENSE_GLU_GELU and N // 2 % 128 == 0 and image[0].data_ptr() != xh.data_ptr()
         e.dense_xh, e.dense_ncap = image[0].data_ptr(), image[1]
-    e.dense_op, e.dense_param, e.dense_param2 = epi, param, param2
+    e.dense_op, e.dense_param, e.dense_param2, e.dense_bias = epi, param, param2, _p(bias)
     e.dense_aux, e.dense_aux_ld = _p(aux), (aux.stride(0) if aux is not None else 0)
     check_layers(layers_lib().dl_gemm_wh_tc(wh.data_ptr(), N, _round_up(K, 128), xh.data_ptr(), ncap, M, e, 2, 0, _stream()),
                  "dl_gemm_wh_tc")
@@ -219,15 +219,19 @@ def mamba_conv(batch: DlMambaBatch, M: int, n_seq: int, zx: torch.Tensor, in_off
 
 
 def causal_conv(batch: DlMambaBatch, M: int, n_seq: int, x: torch.Tensor, w: torch.Tensor, conv_state: torch.Tensor,
-                out: torch.Tensor, bias: Optional[torch.Tensor] = None, act: bool = False, residual: bool = False, in_off: int = 0):
+                out: torch.Tensor, bias: Optional[torch.Tensor] = None, act: bool = False, residual: bool = False, in_off: int = 0,
+                unit=None):
     """out[m][ch] = act(bias + sum_k w[ch][k] x[position - (taps - 1) + k][ch]) (+ x[m][ch]); zeros before a sequence's
-    start; conv_state [slots][taps - 1][channels] carries every slot's last inputs and is updated."""
+    start; conv_state [slots][taps - 1][channels] carries every slot's last inputs and is updated.  unit = (head size, channels of
+    queries, channels of queries and keys, query factor): those channels leave as heads of length one, the queries times the factor."""
     channels, taps = w.shape
     a = DlConvArgs()
     a.in_, a.ld, a.in_off = x.data_ptr(), x.stride(0), in_off
     a.w, a.bias, a.wtype, a.conv_state = w.data_ptr(), _p(bias), _type(w), conv_state.data_ptr()
     a.out, a.ld_out = out.data_ptr(), out.stride(0)
     a.channels, a.taps, a.act, a.residual = channels, taps, 1 if act else 0, 1 if residual else 0
+    if unit is not None:
+        a.unit_dim, a.unit_q, a.unit_k, a.unit_scale = unit
     check_layers(layers_lib().dl_causal_conv(batch, M, n_seq, a, _stream()), "dl_causal_conv")
     lib.count_launch(2 if taps > 1 else 1)
 
@@ -281,9 +285,13 @@ def gated_scan(batch: DlMambaBatch, n_seq: int, q: torch.Tensor, v: torch.Tensor
                dim: int, vdim: int, q_scale: float = 1.0, q_silu: bool = False, f: Optional[torch.Tensor] = None,
                f_bias: Optional[torch.Tensor] = None, lower: Optional[torch.Tensor] = None, k: Optional[torch.Tensor] = None,
                log_keep: Optional[torch.Tensor] = None, put: Optional[torch.Tensor] = None, den: Optional[torch.Tensor] = None,
-               n_state: Optional[torch.Tensor] = None, max_chunks: int = 0, scratch: Optional[torch.Tensor] = None, chunk_slots: int = 0):
+               n_state: Optional[torch.Tensor] = None, gate: int = GATE_LOWER, tau: float = 1.0, rate: Optional[torch.Tensor] = None,
+               bonus: Optional[torch.Tensor] = None, beta: Optional[torch.Tensor] = None, k_heads: int = 0, u: Optional[torch.Tensor] = None, max_chunks: int = 0, scratch: Optional[torch.Tensor] = None, chunk_slots: int = 0):
     """With f (raw gate, f_bias and lower [heads * dim]): S <- diag(g) S + (1 - g) v^T, g = lower + (1 - lower) sigmoid(f + f_bias).
-    With k, log_keep, put [M][heads]: S <- e^log_keep S + put k v^T, n likewise with k alone, den [M][heads] = n . q.
+    gate: the decays g of the channel form (GATE_*; with tau or rate [heads]); all but GATE_LOWER have keys of their own, S <- diag(g) S + k v^T.
+    bonus [heads * dim]: a row reads the state ahead of its own update, y = S_old^T q + (q . bonus k) v.  beta [M] rows of raw write
+    strengths: the delta rule S <- diag(g) S, S <- S + k (sigmoid(beta) (v - S^T k))^T; chunked, it needs u [M][heads * vdim] f32.
+    k_heads: heads of q and k (0: n_heads).  With k, log_keep, put [M][heads]: S <- e^log_keep S + put k v^T, n likewise with k alone, den [M][heads] = n . q.
     y = S^T q, q = silu(q) or q_scale * q; state [slots][heads][dim][vdim] f32 (n_state [slots][heads][dim]).  max_chunks > 0 (with
     scratch for chunk_slots chunks): the chunk-parallel form for long portions."""
     a = DlGatedArgs()
@@ -293,6 +301,14 @@ def gated_scan(batch: DlMambaBatch, n_seq: int, q: torch.Tensor, v: torch.Tensor
     a.log_keep, a.put, a.den = _p(log_keep), _p(put), _p(den)
     a.y, a.ld_y, a.state, a.n_state = y.data_ptr(), y.stride(0), state.data_ptr(), _p(n_state)
     a.n_heads, a.dim, a.vdim = n_heads, dim, vdim
+    a.gate, a.inv_tau, a.rate, a.bonus, a.k_heads = gate, 1.0 / tau, _p(rate), _p(bonus), k_heads
+    a.beta, a.ld_beta = _p(beta), (beta.stride(0) if beta is not None else 0)
+    if max_chunks > 0 and beta is not None:
+        assert scratch.numel() >= chunk_slots * n_heads * (dim * (vdim + 2) + 2 * GATED_CHUNK * _round_up(dim, 4))
+        check_layers(layers_lib().dl_delta_scan_chunked(batch, n_seq, max_chunks, a, scratch.data_ptr(), chunk_slots, u.data_ptr(), u.stride(0),
+                                                        _stream()), "dl_delta_scan_chunked")
+        lib.count_launch(3)
+        return
     if max_chunks > 0:
         assert scratch.numel() >= chunk_slots * n_heads * dim * (vdim + 2)
         check_layers(layers_lib().dl_gated_scan_chunked(batch, n_seq, max_chunks, a, scratch.data_ptr(), chunk_slots, _stream()),
@@ -300,6 +316,28 @@ def gated_scan(batch: DlMambaBatch, n_seq: int, q: torch.Tensor, v: torch.Tensor
         lib.count_launch(3)
         return
     check_layers(layers_lib().dl_gated_scan(batch, n_seq, a, _stream()), "dl_gated_scan")
+    lib.count_launch()
+
+
+def delta_chunked_supported(dim: int, vdim: int) -> bool:
+    return layers_lib().dl_delta_scan_chunked_supported(dim, vdim) == 0
+
+
+def delta_chunk_floats(M: int, n_seq: int, n_heads: int, dim: int, vdim: int) -> int:
+    return int(layers_lib().dl_delta_chunk_floats(M, n_seq, n_heads, dim, vdim))
+
+
+def token_shift(batch: DlMambaBatch, M: int, h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, out: Optional[torch.Tensor] = None,
+                images=None):
+    """Mix s of row m = h + (h of the row ahead - h) mu[s], mu [mixes][width] f32; to out [mixes][>= M][width] f32, or into images =
+    (first image, bytes from one to the next, ncap).  state [slots][width] f32 carries every slot's last h and is updated."""
+    a = DlShiftArgs()
+    a.h, a.ldh, a.mu, a.n_mix, a.width, a.state = h.data_ptr(), h.stride(0), mu.data_ptr(), mu.shape[0], mu.shape[1], state.data_ptr()
+    if images is not None:
+        a.xh, a.xh_step, a.ncap = images[0].data_ptr(), images[1], images[2]
+    else:
+        a.out, a.out_step, a.ld_out = out.data_ptr(), out.stride(0), out.stride(1)
+    check_layers(layers_lib().dl_token_shift(batch, M, a, _stream()), "dl_token_shift")
     lib.count_launch()
 
 
@@ -316,14 +354,15 @@ def mlstm_gates(batch: DlMambaBatch, n_seq: int, zi: torch.Tensor, zf: torch.Ten
 
 
 def head_norm(y: torch.Tensor, M: int, n_heads: int, vdim: int, eps: float, w: torch.Tensor, out: Optional[torch.Tensor],
-              den: Optional[torch.Tensor] = None, floor: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, image=None):
-    """Per head: y / (max(|den|, floor) + 1e-6), RMS norm with weight w ([vdim] or [n_heads * vdim]), times sigmoid(gate); to out or
-    into image = (activation image, ncap)."""
+              den: Optional[torch.Tensor] = None, floor: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, image=None,
+              gate_silu: bool = False):
+    """Per head: y / (max(|den|, floor) + 1e-6), RMS norm with weight w ([vdim] or [n_heads * vdim]), times sigmoid(gate) (or
+    silu(gate)); to out or into image = (activation image, ncap)."""
     assert w.numel() in (vdim, n_heads * vdim)
     a = DlHeadNormArgs()
     a.y, a.ld_y, a.den, a.floor_ = y.data_ptr(), y.stride(0), _p(den), _p(floor)
     a.w, a.w_full = w.data_ptr(), 1 if w.numel() == n_heads * vdim and n_heads > 1 else 0
-    a.gate, a.ld_gate = _p(gate), (gate.stride(0) if gate is not None else 0)
+    a.gate, a.ld_gate, a.gate_silu = _p(gate), (gate.stride(0) if gate is not None else 0), 1 if gate_silu else 0
     xh, ncap = image or (None, 0)
     a.xh, a.ncap = _p(xh), ncap
     if xh is None:
@@ -371,9 +410,10 @@ def selective_scan(batch: DlMambaBatch, n_seq: int, x: torch.Tensor, dt: torch.T
     lib.count_launch()
 
 
-def residual_step(M: int, dim: int, eps: float, x_in: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, adds=(), normed=(), vec: Optional[torch.Tensor] = None, x: Optional[torch.Tensor] = None, outs=()):
+def residual_step(M: int, dim: int, eps: float, x_in: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, adds=(), normed=(), vec: Optional[torch.Tensor] = None, x: Optional[torch.Tensor] = None, outs=(), scales=None, layer_norm: bool = False):
     """x[m] = x_in + sum of `adds` + sum of w * unit(v) over (v, w) in `normed`, all of row rows ? rows[m] : m, + vec; then per (w, h)
-    of `outs` h[m] = w * unit(x[m]), h an f32 buffer or an (activation image, ncap) pair.  At most three adds, two of the rest."""
+    of `outs` h[m] = w * unit(x[m]), h an f32 buffer or an (activation image, ncap) pair.  At most three adds, two of the rest.
+    scales: factors of the first two adds.  layer_norm: an entry of `outs` is ((w, b), h) and h[m] = w * unit(x[m] - mean) + b."""
     a = DlResidualArgs()
     a.ld_in, a.rows = (x_in.stride(0) if x_in is not None else 0), _p(rows)
     if x_in is not None:         # f32 rows, or the bf16 rows of a table
@@ -388,7 +428,13 @@ def residual_step(M: int, dim: int, eps: float, x_in: Optional[torch.Tensor] = N
         setattr(a, "w_" + n, w.data_ptr())
         setattr(a, "ld_" + n, t.stride(0))
     a.vec, a.x, a.ldx = _p(vec), _p(x), (x.stride(0) if x is not None else 0)
+    if scales is not None:
+        a.add_scaled, (a.scale1, a.scale2) = 1, scales
+    a.layer_norm = 1 if layer_norm else 0
     for n, (w, h) in zip("12", outs):
+        if layer_norm:
+            w, bias = w
+            setattr(a, "b" + n, bias.data_ptr())
         setattr(a, "w" + n, w.data_ptr())
         if isinstance(h, tuple):
             setattr(a, "xh" + n, h[0].data_ptr())
@@ -450,12 +496,13 @@ def window_kv_write(k: Optional[torch.Tensor], M: int, kv_heads: int, dim: int, 
                     pos, slot, block_table: torch.Tensor, cache: torch.Tensor, q: Optional[torch.Tensor] = None, q_heads: int = 0,
                     v: Optional[torch.Tensor] = None, vdim: int = 0, qk_norm: bool = False, eps: float = 0.0, rope_half: bool = False,
                     talk: Optional[torch.Tensor] = None, q_mixed: Optional[torch.Tensor] = None,
-                    q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None):
+                    q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None, head_norm: bool = False):
     """Keys into the paged cache (rotated key + unrotated head per line); with q [M][q_heads * dim] the queries are
     rotated in place by the same launch.  With v [M][kv_heads * vdim] the line is key + value; rotary (pairs (i, i + dims / 2)
     with rope_half, else (2i, 2i + 1)) comes first, then qk_norm divides every query and key head by its root mean square.
     talk [q_heads][q_heads] f32 with q_mixed [M][q_heads * kv_heads * dim]: the head mix of the scores, folded into the queries.
-    q_norm [q_heads * dim] / k_norm [kv_heads * dim] f32: an RMS norm over a row's whole projection, in front of the rotary."""
+    q_norm [q_heads * dim] / k_norm [kv_heads * dim] f32: an RMS norm over a row's whole projection, in front of the rotary; with
+    head_norm they are [dim] and every head is normed by itself."""
     a = DlWindowKvArgs()
     a.k, a.ld, a.kv_heads, a.dim, a.rope_dims = _p(k), (k.stride(0) if k is not None else 0), kv_heads, dim, rope_dims
     a.q, a.ldq, a.q_heads = _p(q), (q.stride(0) if q is not None else 0), q_heads
@@ -466,13 +513,14 @@ def window_kv_write(k: Optional[torch.Tensor], M: int, kv_heads: int, dim: int, 
     a.v, a.ldv, a.vdim = _p(v), (v.stride(0) if v is not None else 0), vdim
     a.qk_norm, a.eps = 1 if qk_norm else 0, eps
     a.rope_half, a.talk, a.q_mixed, a.ld_qm = 1 if rope_half else 0, _p(talk), _p(q_mixed), (q_mixed.stride(0) if q_mixed is not None else 0)
-    a.q_norm, a.k_norm = _p(q_norm), _p(k_norm)
+    a.q_norm, a.k_norm, a.head_norm = _p(q_norm), _p(k_norm), 1 if head_norm else 0
     check_layers(layers_lib().dl_window_kv_write(a, M, _stream()), "dl_window_kv_write")
     lib.count_launch()
 
 
 def _window_args(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache,
-                 vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0, value_heads: int = 0):
+                 vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0, value_heads: int = 0,
+                 slope: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
     a = DlWindowAttnArgs()
     a.q, a.ldq, a.out, a.ldo = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0)
     a.heads, a.kv_heads, a.dim, a.rope_dims = heads, kv_heads, dim, rope_dims
@@ -481,18 +529,21 @@ def _window_args(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window
     a.max_pages, a.page_size = block_table.shape[1], PAGE_SIZE
     a.cache, a.ctype = cache.data_ptr(), _type(cache)
     a.vdim, a.chunk, a.sink, a.key_heads, a.value_heads = vdim, chunk, _p(sink), key_heads, value_heads
+    a.slope, a.gate, a.ld_gate = _p(slope), _p(gate), (gate.stride(0) if gate is not None else 0)
     return a
 
 
 def window_attention(q: torch.Tensor, out: torch.Tensor, M: int, heads: int, kv_heads: int, dim: int, rope_dims: int,
                      scale: float, softcap: float, window: int, pos, slot, block_table: torch.Tensor, cache: torch.Tensor,
-                     vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0, value_heads: int = 0):
+                     vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0, value_heads: int = 0,
+                     slope: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
     """The per-row kernel (either cache type, f32 arithmetic).  vdim > 0: values of their own behind the keys; chunk > 0:
     only keys of the row's own chunk of positions are visible; sink [heads]: joins the softmax denominator; key_heads =
     kv_heads: q is [M][heads][kv_heads * dim] (head-mixed queries) against the keys of all key/value heads side by side;
-    value_heads = kv_heads: out is [M][heads][kv_heads * vdim], every head's weights against the values of all key/value heads."""
+    value_heads = kv_heads: out is [M][heads][kv_heads * vdim], every head's weights against the values of all key/value heads.
+    slope [heads]: slope * distance is taken off a score; gate [M] rows of `heads` numbers: heads leave times sigmoid(gate)."""
     a = _window_args(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache, vdim, chunk, sink, key_heads,
-                     value_heads)
+                     value_heads, slope, gate)
     check_layers(layers_lib().dl_window_attention(a, M, _stream()), "dl_window_attention")
     lib.count_launch()
 
@@ -514,10 +565,12 @@ def window_tc_partial_floats(n_tiles: int, kv_heads: int, n_splits: int, dim: in
 def window_attention_tc(q: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dim: int, rope_dims: int, scale: float,
                         softcap: float, window: int, pos, slot, block_table: torch.Tensor, cache: torch.Tensor,
                         tile_rows: torch.Tensor, n_tiles: int, rq: int, n_splits: int = 1, partial: Optional[torch.Tensor] = None,
-                        vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None):
+                        vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None, slope: Optional[torch.Tensor] = None,
+                        gate: Optional[torch.Tensor] = None):
     """The tensor-core kernel over row tiles (tile_rows int32 [n_tiles][rq] on the device, -1 = no row).  n_splits > 1:
     that many CTAs share each tile's pages (few tiles: decoding) and a merge launch follows; partial: f32 scratch."""
-    a = _window_args(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache, vdim, chunk, sink)
+    a = _window_args(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache, vdim, chunk, sink,
+                     slope=slope, gate=gate)
     if n_splits > 1:
         assert partial is not None and partial.numel() >= window_tc_partial_floats(n_tiles, kv_heads, n_splits, dim)
     check_layers(layers_lib().dl_window_attention_tc(a, tile_rows.data_ptr(), n_tiles, rq, n_splits, _p(partial), _stream()),
@@ -544,11 +597,12 @@ def talk_tc_partial_floats(n_tiles: int, kv_heads: int, n_splits: int, vdim: int
 def talk_attention_tc(q: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int,
                       pos, slot, block_table: torch.Tensor, cache: torch.Tensor, tile_rows: torch.Tensor, n_tiles: int, rq: int,
                       n_splits: int = 1, partial: Optional[torch.Tensor] = None, chunk: int = 0, sink: Optional[torch.Tensor] = None,
-                      key_heads: int = 0, value_heads: int = 0):
+                      key_heads: int = 0, value_heads: int = 0, softcap: float = 0.0, slope: Optional[torch.Tensor] = None,
+                      gate: Optional[torch.Tensor] = None):
     """The tile kernel for values of their own width and (key_heads = kv_heads) head-mixed queries [M][heads][kv_heads * dim]
     against the keys of all key/value heads side by side, or (value_heads = kv_heads) every head's weights against the values
     of all key/value heads, out [M][heads][kv_heads * vdim].  Tiles and page shares as in window_attention_tc."""
-    a = _window_args(q, out, heads, kv_heads, dim, 0, scale, 0.0, window, pos, slot, block_table, cache, vdim, chunk, sink, key_heads, value_heads)
+    a = _window_args(q, out, heads, kv_heads, dim, 0, scale, softcap, window, pos, slot, block_table, cache, vdim, chunk, sink, key_heads, value_heads, slope, gate)
     if n_splits > 1:
         assert partial is not None and partial.numel() >= talk_tc_partial_floats(n_tiles, kv_heads, n_splits, vdim, rq, heads, value_heads)
     check_layers(layers_lib().dl_talk_attention_tc(a, tile_rows.data_ptr(), n_tiles, rq, n_splits, _p(partial), _stream()),
@@ -557,7 +611,8 @@ def talk_attention_tc(q: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: 
 
 
 def talk_attention_tiles(q, out, heads, kv_heads, dim, vdim, scale, window, pos, slot, block_table, cache, tiles, rq: int, n_splits: int = 1,
-                         chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0, value_heads: int = 0):
+                         chunk: int = 0, sink: Optional[torch.Tensor] = None, key_heads: int = 0, value_heads: int = 0, softcap: float = 0.0,
+                         slope: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
     """Convenience for callers with host-side tiles (lists of up to rq row indices of one sequence, consecutive positions)."""
     t = torch.full((len(tiles), rq), -1, dtype=torch.int32)
     for i, rows in enumerate(tiles):
@@ -566,7 +621,7 @@ def talk_attention_tiles(q, out, heads, kv_heads, dim, vdim, scale, window, pos,
     if n_splits > 1:
         partial = torch.zeros(talk_tc_partial_floats(len(tiles), kv_heads, n_splits, vdim, rq, heads, value_heads), dtype=torch.float32, device=q.device)
     talk_attention_tc(q, out, heads, kv_heads, dim, vdim, scale, window, pos, slot, block_table, cache, t.to(q.device), len(tiles), rq,
-                      n_splits, partial, chunk, sink, key_heads, value_heads)
+                      n_splits, partial, chunk, sink, key_heads, value_heads, softcap, slope, gate)
 
 
 def talk_mix(wide: torch.Tensor, talk: torch.Tensor, M: int, heads: int, kv_heads: int, vdim: int, out: Optional[torch.Tensor],
@@ -580,7 +635,8 @@ def talk_mix(wide: torch.Tensor, talk: torch.Tensor, M: int, heads: int, kv_head
 
 
 def window_attention_tiles(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache, tiles,
-                           n_splits: int = 1, vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None):
+                           n_splits: int = 1, vdim: int = 0, chunk: int = 0, sink: Optional[torch.Tensor] = None,
+                           slope: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
     """Convenience for callers with host-side tiles (lists of row indices of one sequence, consecutive positions)."""
     rq = window_tc_rows(heads, kv_heads)
     t = torch.full((len(tiles), rq), -1, dtype=torch.int32)
@@ -590,7 +646,7 @@ def window_attention_tiles(q, out, heads, kv_heads, dim, rope_dims, scale, softc
     if n_splits > 1:
         partial = torch.zeros(window_tc_partial_floats(len(tiles), kv_heads, n_splits, dim), dtype=torch.float32, device=q.device)
     window_attention_tc(q, out, heads, kv_heads, dim, rope_dims, scale, softcap, window, pos, slot, block_table, cache,
-                        t.to(q.device), len(tiles), rq, n_splits, partial, vdim, chunk, sink)
+                        t.to(q.device), len(tiles), rq, n_splits, partial, vdim, chunk, sink, slope, gate)
 
 
 # ---- routed experts ---------------------------------------------------------------------------------------------------
