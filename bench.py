@@ -51,14 +51,15 @@ def parse_args():
     ap.add_argument("--layered", default="", help="instead of the headline benchmark: prefill and decode throughput of the "
                     "layer-list design (Ribivik: Mamba-2 + latent attention, bf16) beside a Q40 Llama of equal width, "
                     "feed-forward size and depth, at these sizes (comma separated: w2048, w4096); prints one JSON line")
-    ap.add_argument("--layered-design", default="ribivik", choices=("ribivik", "sunesun", "venadra", "darusun", "vopedra"),
+    ap.add_argument("--layered-design", default="ribivik", choices=("ribivik", "sunesun", "venadra", "darusun", "vopedra", "silizen"),
                     help="--layered: which layer-list design runs beside the Llama arm (ribivik: Mamba-2 + latent attention; "
                          "sunesun: windowed attention whose values are its keys + routed experts on hyper-connected streams; "
                          "venadra: lightning and chunked sink attention, PolyNorm and gated experts; darusun: post-norm layers, "
                          "head-mixed attention, windowed latent attention, xIELU and experts with a shared one -- beside these two "
                          "also Sunesun, the closest layer-list design, at equal width, depth and experts; vopedra: matrix memory, "
                          "selective scan, attention with mixed softmax weights beside HGRN2, gated feed-forwards -- beside it Venadra "
-                         "(linear attention) and Darusun (head-mixed attention))")
+                         "(linear attention) and Darusun (head-mixed attention); silizen: time mixing, soft-capped attention beside gated "
+                         "linear attention, windowed attention beside a gated delta rule -- beside it Vopedra)")
     ap.add_argument("--layered-layers", type=int, default=4, help="--layered: layers of both models")
     ap.add_argument("--layered-prompt", type=int, default=2048, help="--layered: prompt length (one batch)")
     return ap.parse_args()
@@ -503,6 +504,23 @@ def vopedra_config(name: str, n_layers: int, vocab: int) -> dict:
     return {"architecture": "Vopedra", "width": W, "vocab": vocab, "norm": {"eps": 1e-5}, "layers": layers}
 
 
+def silizen_config(name: str, n_layers: int, vocab: int, window: int = 1024) -> dict:
+    """Width, heads and feed-forward of the Vopedra arm.  Layers in turn: time mixing, soft-capped attention (four key/value heads, 64
+    rotated dimensions) beside gated linear attention, windowed attention beside the gated delta rule, time mixing; no loop."""
+    import math
+    sz, ss = LAYERED_SIZES[name], SUNESUN_SIZES[name]
+    W = sz["width"]
+    attn = {"heads": ss["heads"], "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 1.0 / math.sqrt(128.0)}
+    left = dict(attn, softcap=50.0, rot={"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}})
+    heads = {"heads": W // 128, "dim": 128, "vdim": 128}
+    kinds = [("wkv", {"heads": W // 64, "dim": 64}),
+             ("parallel", {"left": left, "right": dict(heads, tau=16.0), "left_scale": 0.5, "right_scale": 0.5}),
+             ("parallel_2", {"left": dict(attn, mask={"size": window}), "right": dict(heads, kv_heads=W // 128, conv=4)}),
+             ("wkv", {"heads": W // 64, "dim": 64})]
+    layers = [{"type": kinds[i % 4][0], "mixer": dict(kinds[i % 4][1]), "mlp": {"kind": "dense", "ff": sz["ff"]}} for i in range(n_layers)]
+    return {"architecture": "Silizen", "width": W, "vocab": vocab, "norm": {"eps": 1e-5}, "logit_scale": 0.1, "layers": layers}
+
+
 def _time_ms(fn, warmup: int, steps: int):
     import torch
     for _ in range(warmup):
@@ -572,7 +590,7 @@ def run_layered(args):
         design = args.layered_design
         configs = {"ribivik": lambda: layered_config(sz, nl, vocab), "sunesun": lambda: sunesun_config(name, nl, vocab),
                    "venadra": lambda: venadra_config(name, nl, vocab), "darusun": lambda: darusun_config(name, nl, vocab),
-                   "vopedra": lambda: vopedra_config(name, nl, vocab)}
+                   "vopedra": lambda: vopedra_config(name, nl, vocab), "silizen": lambda: silizen_config(name, nl, vocab)}
 
         def layer_list_arm(dsg):
             d = os.path.join(args.model_dir, f"dllama_b200_{'layered' if dsg == 'ribivik' else dsg}_{name}_l{nl}")
@@ -588,7 +606,8 @@ def run_layered(args):
 
         r = layer_list_arm(design)
         beside = {"sunesun_bf16": layer_list_arm("sunesun")} if design in ("venadra", "darusun") else \
-            {d + "_bf16": layer_list_arm(d) for d in ("venadra", "darusun")} if design == "vopedra" else {}
+            {d + "_bf16": layer_list_arm(d) for d in ("venadra", "darusun")} if design == "vopedra" else \
+            {"vopedra_bf16": layer_list_arm("vopedra")} if design == "silizen" else {}
         shape = dict(dim=sz["width"], hidden_dim=sz["ff"], n_layers=nl, n_heads=sz["heads"], n_kv_heads=8, vocab_size=vocab,
                      max_seq_len=8192, rope_theta=10000, rope=None)
         path = os.path.join(args.model_dir, f"dllama_b200_llama_{name}_l{nl}_q40.m")

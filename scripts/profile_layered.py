@@ -21,6 +21,14 @@
       the chunk-parallel scans with data-dependent gates alone (2048 rows of one sequence; matrix memory with 8 heads of
       128 x 256, HGRN2 with 16 heads of 128 x 128), then both token by token on 1 and 32 sequences of one row:
         ncu --set full --clock-control none -k regex:gated_chunk_out -s 1 -c 2 -o out python scripts/profile_layered.py gated-scan
+  python scripts/profile_layered.py delta-scan
+      the recurrences with keys of their own alone (2048 rows of one sequence; gated linear attention and the gated delta rule with
+      16 heads of 128 x 128, time mixing with 32 heads of 64 x 64), then token by token on 1 and 32 sequences of one row:
+        ncu --set full --clock-control none -k regex:delta_chunk_ -s 2 -c 2 -o out python scripts/profile_layered.py delta-scan
+  python scripts/profile_layered.py biased-attention
+      the attention tile kernel with values of its own (2048 rows of one sequence, 16 / 4 heads of 128, sink, head gates), soft-capped
+      over all earlier positions, then with a distance bias in a window of 1024:
+        ncu --set full --clock-control none -k regex:window_attention_mma -s 1 -c 1 -o out python scripts/profile_layered.py biased-attention
   python scripts/profile_layered.py selective-scan
       the selective scan alone (4096 channels of 16 state entries; 2048 rows of one sequence, then 32 sequences of one row):
         ncu --set full --clock-control none -k regex:selective_scan -s 1 -c 1 -o out python scripts/profile_layered.py selective-scan
@@ -49,7 +57,7 @@ def steps(a):
     if not os.path.exists(os.path.join(d, "model.safetensors")):
         cfg = {"ribivik": lambda: bench.layered_config(bench.LAYERED_SIZES[a.size], nl, vocab), "sunesun": lambda: bench.sunesun_config(a.size, nl, vocab),
                "venadra": lambda: bench.venadra_config(a.size, nl, vocab), "darusun": lambda: bench.darusun_config(a.size, nl, vocab),
-               "vopedra": lambda: bench.vopedra_config(a.size, nl, vocab)}[a.design]()
+               "vopedra": lambda: bench.vopedra_config(a.size, nl, vocab), "silizen": lambda: bench.silizen_config(a.size, nl, vocab)}[a.design]()
         write_random_model(d, cfg, seed=1)
     torch.cuda.set_device(0)
     eng = registry.engine_for_dir(d, max_rows=T, n_slots=users, max_seq_len=T + 64, dtype="bfloat16")
@@ -217,6 +225,55 @@ def gated_scan(a):
             _timed(f"{name}, token by token, {m} sequences of one row ({2 * m * H * d * dv * 4 / 1e6:.1f} MB of state)", lambda: scan(b1, m), 3)
 
 
+def delta_scan(a):
+    import torch
+    from dllama_b200.ops import layers as L
+    n, users = 2048, 32
+    g = torch.Generator().manual_seed(1)
+    for name, H, d, dv in (("gated linear attention", 16, 128, 128), ("time mixing", 32, 64, 64), ("gated delta rule", 16, 128, 128)):
+        x = torch.randn(n, H * (3 * d + dv + 1), generator=g).cuda()
+        x[:, :2 * H * d] *= d ** -0.5
+        y, u, state, vec = torch.zeros(n, H * dv, device="cuda"), torch.zeros(n, H * dv, device="cuda"), torch.zeros(users, H, d, dv, device="cuda"), torch.zeros(H * d, device="cuda")
+        slots, z0 = n // L.GATED_CHUNK + users, H * (2 * d + dv)
+        kw = {"gated linear attention": dict(gate=L.GATE_ROOT_SIGMOID, tau=16.0), "time mixing": dict(gate=L.GATE_EXP_EXP, bonus=vec),
+              "gated delta rule": dict(gate=L.GATE_SOFTPLUS, rate=torch.ones(H, device="cuda"), beta=x[:, z0 + H * d:])}[name]
+        scratch = torch.zeros((L.delta_chunk_floats if "beta" in kw else L.gated_chunk_floats)(n, users, H, d, dv), device="cuda")
+
+        def scan(b, n_seq, **more):
+            L.gated_scan(b, n_seq, x, x[:, 2 * H * d:], y, state, H, d, dv, k=x[:, H * d:], f=x[:, z0:], f_bias=vec - 2, **kw, **more)
+
+        b, hold = _sequences(n, 1)
+        more = dict(u=u) if "beta" in kw else {}
+        _timed(f"{name}, chunked, {n} rows", lambda: scan(b, 1, max_chunks=n // L.GATED_CHUNK, scratch=scratch, chunk_slots=slots, **more))
+        for m in (1, users):
+            b1, hold1 = _sequences(1, m)
+            _timed(f"{name}, token by token, {m} sequences of one row ({2 * m * H * d * dv * 4 / 1e6:.1f} MB of state)", lambda: scan(b1, m), 3)
+
+
+def biased_attention(a):
+    import torch
+    from dllama_b200.ops import layers as L
+    H, G, d, n = 16, 4, 128, 2048
+    n_pages = n // 32
+    bt = torch.arange(n_pages, dtype=torch.int32).view(1, -1).cuda()
+    cache = torch.randn(n_pages, G, 32, 2 * d, device="cuda").to(torch.bfloat16)
+    g = torch.Generator().manual_seed(1)
+    q, gate = torch.randn(n, H * d, generator=g).cuda(), torch.randn(n, H, generator=g).cuda()
+    pos, slot = torch.arange(n, dtype=torch.int32).cuda(), torch.zeros(n, dtype=torch.int32).cuda()
+    out, sink, slope = torch.zeros(n, H * d, device="cuda"), torch.zeros(H, device="cuda"), torch.full((H,), 0.01, device="cuda")
+    rq = L.window_tc_rows(H, G)
+    tiles = torch.arange(n, dtype=torch.int32).view(-1, rq).cuda()
+    rq2 = L.talk_tc_rows(H, G, d, d, 0, n)
+    tiles2 = torch.arange(n, dtype=torch.int32).view(-1, rq2).cuda()
+    for what, cap, window, sl in (("soft-capped", 50.0, 0, None), ("distance bias, window 1024", 0.0, 1024, slope)):
+        _timed(f"windowed-attention kernel, {what}", lambda: L.window_attention_tc(q, out, H, G, d, 0, 0.09, cap, window, pos, slot, bt, cache, tiles, n // rq, rq,
+                                                                                  vdim=d, sink=sink, slope=sl, gate=gate))
+        _timed(f"own-width kernel, {what}", lambda: L.talk_attention_tc(q, out, H, G, d, d, 0.09, window, pos, slot, bt, cache, tiles2, n // rq2, rq2,
+                                                                       sink=sink, softcap=cap, slope=sl, gate=gate))
+        pairs = sum(min(i + 1, window or n) for i in range(n))
+        print("FLOPs per launch (visible pairs): %.1f G" % (pairs * H * 4 * d / 1e9))
+
+
 def selective_scan(a):
     import torch
     from dllama_b200.ops import layers as L
@@ -257,12 +314,12 @@ def wide_attention(a):
 
 if __name__ == "__main__":
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("what", choices=("steps", "window-attention", "lightning-scan", "talk-attention", "gated-scan", "selective-scan", "wide-attention"))
-    ap.add_argument("--design", default="sunesun", choices=("ribivik", "sunesun", "venadra", "darusun", "vopedra"))
+    ap.add_argument("what", choices=("steps", "window-attention", "lightning-scan", "talk-attention", "gated-scan", "delta-scan", "selective-scan", "wide-attention", "biased-attention"))
+    ap.add_argument("--design", default="sunesun", choices=("ribivik", "sunesun", "venadra", "darusun", "vopedra", "silizen"))
     ap.add_argument("--size", default="w2048")
     ap.add_argument("--layers", type=int, default=4)
     ap.add_argument("--prompt", type=int, default=2048)
     ap.add_argument("--model-dir", default="/tmp")
     a = ap.parse_args()
     {"steps": steps, "window-attention": window_attention, "lightning-scan": lightning_scan, "talk-attention": talk_attention,
-     "gated-scan": gated_scan, "selective-scan": selective_scan, "wide-attention": wide_attention}[a.what](a)
+     "gated-scan": gated_scan, "delta-scan": delta_scan, "biased-attention": biased_attention, "selective-scan": selective_scan, "wide-attention": wide_attention}[a.what](a)

@@ -87,21 +87,21 @@ def sink_attention_rows(q, k, v, scale, softcap=0.0, window=0, slopes=None, firs
     """q [T, H, d] and k [S, G, d] as they meet, v [S, G, dv]; query row t sits at position first + t.  The softmax's
     denominator has one more term exp(0)."""
     T, H, _ = q.shape
-    G, dv = v.shape[1:]
+    S, G, dv = v.shape
+    i, j = first + torch.arange(T)[:, None], torch.arange(S)[None, :]
+    seen = (j <= i) & (i - j < window) if window else j <= i
     out = torch.zeros(T, H, dv, dtype=F64)
-    for t in range(T):
-        i = first + t
-        lo = max(0, i - window + 1) if window else 0
-        for h in range(H):
-            g = h // (H // G)
-            s = k[lo:i + 1, g] @ q[t, h] * scale
-            if softcap:
-                s = softcap * torch.tanh(s / softcap)
-            if slopes is not None:
-                s = s - slopes[h] * (i - torch.arange(lo, i + 1, dtype=F64))
-            m = torch.clamp(s.max(), min=0.0)
-            e = torch.exp(s - m)
-            out[t, h] = (e / (torch.exp(-m) + e.sum())) @ v[lo:i + 1, g]
+    for h in range(H):
+        g = h // (H // G)
+        s = q[:, h] @ k[:, g].T * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        if slopes is not None:
+            s = s - slopes[h] * (i - j)
+        s = torch.where(seen, s, torch.tensor(-math.inf, dtype=F64))
+        m = s.amax(-1, keepdim=True).clamp(min=0.0)
+        e = torch.exp(s - m)
+        out[:, h] = (e / (torch.exp(-m) + e.sum(-1, keepdim=True))) @ v[:, g]
     return out
 
 
@@ -139,7 +139,7 @@ def gated_rows(q, k, v, f, S=None):
     out = torch.zeros(T, H, v.shape[-1], dtype=F64)
     for i in range(T):
         S = f[i][:, :, None] * S + k[i][:, :, None] * v[i][:, None, :]
-        out[i] = torch.einsum("hdv,hd->hv", S, q[i])
+        out[i] = (q[i][:, None, :] @ S)[:, 0]
     return out, S
 
 
@@ -173,9 +173,9 @@ def delta_rows(q, k, v, f, beta, S=None):
     out = torch.zeros(T, H, v.shape[-1], dtype=F64)
     for i in range(T):
         S = f[i][:, :, None] * S
-        u = beta[i][:, None] * (v[i] - torch.einsum("hdv,hd->hv", S, k[i]))
+        u = beta[i][:, None] * (v[i] - (k[i][:, None, :] @ S)[:, 0])
         S = S + k[i][:, :, None] * u[:, None, :]
-        out[i] = torch.einsum("hdv,hd->hv", S, q[i])
+        out[i] = (q[i][:, None, :] @ S)[:, 0]
     return out, S
 
 
@@ -201,7 +201,7 @@ def wkv_rows(r, k, v, f, u, S=None):
     S = torch.zeros(H, d, v.shape[-1], dtype=F64) if S is None else S.clone()
     out = torch.zeros(T, H, v.shape[-1], dtype=F64)
     for i in range(T):
-        out[i] = torch.einsum("hdv,hd->hv", S, r[i]) + (r[i] * u * k[i]).sum(-1, keepdim=True) * v[i]
+        out[i] = (r[i][:, None, :] @ S)[:, 0] + (r[i] * u * k[i]).sum(-1, keepdim=True) * v[i]
         S = f[i][:, :, None] * S + k[i][:, :, None] * v[i][:, None, :]
     return out, S
 
