@@ -13,8 +13,10 @@
 #include "mma_common.cuh"
 
 #define DR_CB 16                  // columns of the state per CTA of the walk
+#define DR_ROWS (2 * GC + 1)      // staged rows per chunk of the walk
 
-// scratch per chunk slot and head: GatedScratch's, then W [GC][D4] and the keys decayed to the chunk's end [GC][D4]
+// scratch per chunk slot and head: the states of GatedScratch, W [GC][D4], and the keys decayed to the chunk's end with the chunk's
+// whole decay as one more row, Ke [GC + 1][D4]
 struct DeltaScratch { GatedScratch g; float* W; float* Ke; };
 
 // one column of (I + N) X = b R by substitution, in place: x[i * ld], i < GC; Nt [GC][GC_AS] holds N transposed.  Rows in blocks of
@@ -60,7 +62,6 @@ __global__ void __launch_bounds__(GC_THREADS, 2) delta_chunk_system_kernel(DlMam
     int row0, len, ci;
     if (!gated_chunk_of(b, n, c, row0, len, ci)) return;
     const int D = a.dim, V = a.vdim, H = a.n_heads, D4 = (D + 3) & ~3, DP = D4 + 4, hk = gated_k_head(a, h);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* Q = sm;
     float* K = Q + (size_t)GC * DP;
     float* F = K + max((size_t)GC * DP, (size_t)GC * 128);
@@ -71,33 +72,24 @@ __global__ void __launch_bounds__(GC_THREADS, 2) delta_chunk_system_kernel(DlMam
         b_s[i] = i < len ? sigmoid_f(a.beta[(size_t)row * a.ld_beta + h]) : 0.f;
     }
     __syncthreads();
-    for (int j = warp; j < GC; j += GC_THREADS / 32) {
-#pragma unroll 4
-        for (int d = lane; d < D4; d += 32) {
-            float k = 0.f, f = 1.f;
-            if (j < len && d < D) gated_fk(a, rows[j], h, hk, d, f, k);
-            Q[j * DP + d] = k;
-            K[j * DP + d] = k;
-            F[j * DP + d] = f;
-        }
-    }
+    gated_stage_rows<false, true>(a, rows, len, h, hk, D4, DP, Q, K, F);
     __syncthreads();
     float* Nt = F;
     decayed_scores<false>(Q, K, F, T, D, D4, DP, nullptr, [&](int i, int j, float v) { if (i > j) Nt[j * GC_AS + i] = b_s[i] * v; });
-    float* Ke = sc.Ke + ((size_t)ci * H + h) * GC * D4;
+    float* Ke = sc.Ke + ((size_t)ci * H + h) * (GC + 1) * D4;
     for (int t = threadIdx.x; t < 4 * D4; t += GC_THREADS) {
         const int bk = t / D4, d = t - bk * D4;
         float p = 1.f;
         for (int v = bk + 1; v < 4; ++v) p *= T[v * DP + d];
 #pragma unroll
         for (int i = 0; i < 16; ++i) Ke[(size_t)(bk * 16 + i) * D4 + d] = K[(bk * 16 + i) * DP + d] * p;
-        if (bk == 0 && d < D) sc.g.dec[((size_t)ci * H + h) * D + d] = p * T[d];
+        if (bk == 0) Ke[(size_t)GC * D4 + d] = p * T[d];
     }
     __syncthreads();
     float* W = sc.W + ((size_t)ci * H + h) * GC * D4;
     for (int c0 = 0; c0 < V; c0 += 128) {
         const int cw = min(128, V - c0), off = c0 == 0 ? D4 : 0;      // the first round also solves for W
-        gated_stage_v(a, rows, len, h, c0, K);
+        gated_stage_v<128>(a, rows, len, h, c0, K);
         __syncthreads();
         for (int e = threadIdx.x; e < off + cw; e += GC_THREADS) {
             if (e < off) {
@@ -113,14 +105,14 @@ __global__ void __launch_bounds__(GC_THREADS, 2) delta_chunk_system_kernel(DlMam
     }
 }
 
-// pass 2.  Shared memory: [NB][W | keys to the end][GC][D4 + 4] | P [D4][DR_CB] | u [GC][DR_CB].
+// pass 2.  Shared memory: [NB][W [GC] | keys to the end, whole decay [GC + 1]][D4 + 4] | P [D4][DR_CB] | u [GC][DR_CB].
 __global__ void __launch_bounds__(256) delta_chunk_walk_kernel(DlMambaBatch b, DlGatedArgs a, DeltaScratch sc, float* __restrict__ u, long long ld_u, int NB) {
     extern __shared__ __align__(16) float sm[];
     const int n = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * DR_CB, tid = threadIdx.x;
     const int D = a.dim, V = a.vdim, H = a.n_heads, D4 = (D + 3) & ~3, DS = D4 + 4;
     const int s0 = b.seq_start[n], total = b.seq_start[n + 1] - s0, nc = (total + GC - 1) / GC;
     float* buf = sm;
-    float* P = buf + (size_t)NB * 2 * GC * DS;
+    float* P = buf + (size_t)NB * DR_ROWS * DS;
     float* us = P + (size_t)D4 * DR_CB;
     const size_t sh = (size_t)b.seq_slot[n] * H + h, ch0 = (size_t)(s0 / GC + n) * H + h;
     const bool fresh = b.seq_pos0[n] == 0;
@@ -129,15 +121,14 @@ __global__ void __launch_bounds__(256) delta_chunk_walk_kernel(DlMambaBatch b, D
         const int d = e / DR_CB, cc = e - d * DR_CB;
         P[e] = (!fresh && d < D && c0 + cc < V) ? Sg[(size_t)d * V + cc] : 0.f;
     }
-    const int q4 = D4 >> 2;
-    auto issue = [&](int c, int at) {
-        const size_t o = (ch0 + (size_t)c * H) * GC * D4;
-        float* dst = buf + (size_t)at * 2 * GC * DS;
-        for (int e = tid; e < GC * q4; e += 256) {
-            const int i = e / q4, p = (e - i * q4) * 4;
-            cp_async16(dst + (size_t)i * DS + p, sc.W + o + (size_t)i * D4 + p);
-            cp_async16(dst + (size_t)(GC + i) * DS + p, sc.Ke + o + (size_t)i * D4 + p);
-        }
+    auto issue = [&](int c, int at) {         // a warp per row
+        const size_t o = ch0 + (size_t)c * H;
+        const float* w = sc.W + o * GC * D4;
+        const float* ke = sc.Ke + o * (GC + 1) * D4 - (size_t)GC * D4;
+        float* dst = buf + (size_t)at * DR_ROWS * DS;
+        for (int p = (tid & 31) * 4; p < D4; p += 128)
+#pragma unroll 4
+            for (int i = tid >> 5; i < DR_ROWS; i += 8) cp_async16(dst + (size_t)i * DS + p, (i < GC ? w : ke) + (size_t)i * D4 + p);
     };
     const int ui = tid >> 2, uc = (tid & 3) * 4;               // step A: this thread's row and four columns of u
     const int half = tid >> 7, cols = DR_CB / 2;               // step B: half of the columns of rows d = tid % 128 + 128 x of P
@@ -155,7 +146,7 @@ __global__ void __launch_bounds__(256) delta_chunk_walk_kernel(DlMambaBatch b, D
         cp_async_wait_all();
         __syncthreads();                      // the chunk has landed, P is complete
         if (NB == 2 && c + 1 < nc) issue(c + 1, at ^ 1);
-        const float* W = buf + (size_t)at * 2 * GC * DS;
+        const float* W = buf + (size_t)at * DR_ROWS * DS;
         const float* Ke = W + (size_t)GC * DS;
         float* Pg = sc.g.S + (ch0 + (size_t)c * H) * D * V + c0;
         for (int e = tid; e < D * DR_CB; e += 256) {           // the state ahead of this chunk
@@ -163,6 +154,7 @@ __global__ void __launch_bounds__(256) delta_chunk_walk_kernel(DlMambaBatch b, D
             if (c0 + cc < V) Pg[(size_t)d * V + cc] = P[e];
         }
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
         for (int d = 0; d < D4; d += 4) {
             const float4 w = *reinterpret_cast<const float4*>(W + ui * DS + d);
             const float wv[4] = {w.x, w.y, w.z, w.w};
@@ -182,13 +174,13 @@ __global__ void __launch_bounds__(256) delta_chunk_walk_kernel(DlMambaBatch b, D
             if (ug && c0 + uc + x < V) ug[x] = t;
         }
         __syncthreads();
-        const float* dec = sc.g.dec + (ch0 + (size_t)c * H) * D;
+        const float* dec = Ke + (size_t)GC * DS;
         for (int d = tid & 127; d < D; d += 128) {
             float p[8];
             const float g = dec[d];
 #pragma unroll
             for (int x = 0; x < 8; ++x) p[x] = g * P[d * DR_CB + half * cols + x];
-#pragma unroll 4
+#pragma unroll 8
             for (int i = 0; i < GC; ++i) {
                 const float k = Ke[i * DS + d];
                 const float4 u0 = *reinterpret_cast<const float4*>(us + i * DR_CB + half * cols), u1 = *reinterpret_cast<const float4*>(us + i * DR_CB + half * cols + 4);
@@ -217,7 +209,7 @@ static size_t delta_system_smem(int dim) {
 }
 static size_t delta_walk_smem(int dim, int nb) {
     const size_t D4 = (dim + 3) & ~3;
-    return ((size_t)nb * 2 * GC * (D4 + 4) + D4 * DR_CB + (size_t)GC * DR_CB) * sizeof(float);
+    return ((size_t)nb * DR_ROWS * (D4 + 4) + D4 * DR_CB + (size_t)GC * DR_CB) * sizeof(float);
 }
 
 // 0 if the chunked kernels take these sizes
@@ -227,7 +219,7 @@ extern "C" int dl_delta_scan_chunked_supported(int dim, int vdim) {
 
 // f32 of scratch for a batch of M rows in n_seq sequences
 extern "C" long long dl_delta_chunk_floats(int M, int n_seq, int n_heads, int dim, int vdim) {
-    return (long long)(M / GC + n_seq) * n_heads * ((long long)dim * (vdim + 2) + 2 * GC * ((dim + 3) & ~3) + 3);
+    return (long long)(M / GC + n_seq) * n_heads * ((long long)dim * vdim + DR_ROWS * ((dim + 3) & ~3));
 }
 
 extern "C" int dl_delta_scan_chunked(const DlMambaBatch* batch, int n_seq, int max_chunks, const DlGatedArgs* args, float* scratch,
@@ -244,9 +236,8 @@ extern "C" int dl_delta_scan_chunked(const DlMambaBatch* batch, int n_seq, int m
     DeltaScratch sc;                          // the copied arrays first: they start on 16 bytes
     sc.W = scratch;
     sc.Ke = sc.W + slots * GC * D4;
-    sc.g.S = sc.Ke + slots * GC * D4;
-    sc.g.dec = sc.g.S + slots * a.dim * a.vdim;
-    sc.g.ns = nullptr;
+    sc.g.S = sc.Ke + slots * (GC + 1) * D4;
+    sc.g.dec = sc.g.ns = nullptr;
     const int nb = delta_walk_smem(a.dim, 2) <= DR_SMEM_MAX ? 2 : 1;
     const size_t smem1 = delta_system_smem(a.dim), smem2 = delta_walk_smem(a.dim, nb);
     cudaError_t e = cudaFuncSetAttribute(delta_chunk_system_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);

@@ -19,21 +19,31 @@ __device__ __forceinline__ float gated_q(const DlGatedArgs& a, size_t row, int i
     sigmoid_pair_f(v, s, c);
     return v * s;
 }
+// what a channel's gate reads besides the row: bias, lower bound, the head's rate
+struct GatedChannel { float bias, lower, rate; };
+__device__ __forceinline__ GatedChannel gated_channel(const DlGatedArgs& a, int h, int d) {
+    GatedChannel c;
+    c.bias = a.f_bias ? a.f_bias[h * a.dim + d] : 0.f;
+    c.lower = a.gate == DL_GATE_LOWER ? a.lower[h * a.dim + d] : 0.f;
+    c.rate = a.gate == DL_GATE_SOFTPLUS ? a.rate[h] : 0.f;
+    return c;
+}
+// decay f from the raw gate z; with DL_GATE_LOWER also the key k
+__device__ __forceinline__ void gated_form(const DlGatedArgs& a, const GatedChannel& c, float z, float& f, float& k) {
+    z += c.bias;
+    if (a.gate == DL_GATE_LOWER) {
+        float s, t;
+        sigmoid_pair_f(z, s, t);
+        f = fmaf(1.f - c.lower, s, c.lower);
+        k = (1.f - c.lower) * t;
+    } else {
+        f = a.gate == DL_GATE_ROOT_SIGMOID ? expf(-softplus_f(-z) * a.inv_tau) : a.gate == DL_GATE_EXP_EXP ? expf(-expf(z)) : expf(-c.rate * softplus_f(z));
+    }
+}
 // decay and key of channel d of head h (its keys are those of head hk)
 __device__ __forceinline__ void gated_fk(const DlGatedArgs& a, size_t row, int h, int hk, int d, float& f, float& k) {
-    const int i = h * a.dim + d;
-    float z = a.f[row * a.ldf + i];
-    if (a.f_bias) z += a.f_bias[i];
-    if (a.gate == DL_GATE_LOWER) {
-        float s, c;
-        sigmoid_pair_f(z, s, c);
-        const float l = a.lower[i];
-        f = fmaf(1.f - l, s, l);
-        k = (1.f - l) * c;
-        return;
-    }
-    k = a.k[row * a.ldk + hk * a.dim + d];
-    f = a.gate == DL_GATE_ROOT_SIGMOID ? expf(-softplus_f(-z) * a.inv_tau) : a.gate == DL_GATE_EXP_EXP ? expf(-expf(z)) : expf(-a.rate[h] * softplus_f(z));
+    k = a.gate == DL_GATE_LOWER ? 0.f : a.k[row * a.ldk + hk * a.dim + d];
+    gated_form(a, gated_channel(a, h, d), a.f[row * a.ldf + h * a.dim + d], f, k);
 }
 
 static inline int gated_args_ok(const DlGatedArgs& a, const char* who) {
@@ -58,15 +68,62 @@ __device__ __forceinline__ bool gated_chunk_of(const DlMambaBatch& b, int n, int
     return true;
 }
 
-// V columns c0 .. c0 + 127 of the chunk's values into [GC][128] (zeros beyond the chunk or the head's width)
+// V columns c0 .. c0 + VW - 1 (VW: 64 or 128) of the chunk's values into [GC][VW] (zeros beyond the chunk or the head's width); a warp's
+// eight rows are in flight together
+template <int VW>
 __device__ __forceinline__ void gated_stage_v(const DlGatedArgs& a, const int* rows, int len, int h, int c0, float* vt) {
-    const int lane = threadIdx.x & 31;
-    for (int j = threadIdx.x >> 5; j < GC; j += GC_THREADS / 32) {
-        const float* src = j < len ? a.v + (size_t)rows[j] * a.ldv + (size_t)h * a.vdim + c0 : nullptr;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    constexpr int NRW = GC * 32 / GC_THREADS;
 #pragma unroll
-        for (int u = 0; u < 4; ++u) {
-            const int cc = lane + 32 * u;
-            vt[j * 128 + cc] = (src && c0 + cc < a.vdim) ? src[cc] : 0.f;
+    for (int u = 0; u < VW / 32; ++u) {
+        const int cc = lane + 32 * u;
+        float v[NRW];
+#pragma unroll
+        for (int r = 0; r < NRW; ++r) {
+            const int j = warp + r * (GC_THREADS / 32);
+            v[r] = (j < len && c0 + cc < a.vdim) ? a.v[(size_t)rows[j] * a.ldv + (size_t)h * a.vdim + c0 + cc] : 0.f;
+        }
+#pragma unroll
+        for (int r = 0; r < NRW; ++r) vt[(warp + r * (GC_THREADS / 32)) * VW + cc] = v[r];
+    }
+}
+
+// keys, decays and (Q) queries of a chunk's rows into [GC][ld] each, columns [0, DP4); rows and columns that are not there: k = q = 0,
+// f = 1.  COPY: the keys also into Q.  A warp's eight rows are in flight together.
+template <bool WITH_Q, bool COPY>
+__device__ __forceinline__ void gated_stage_rows(const DlGatedArgs& a, const int* rows, int len, int h, int hk, int DP4, int ld, float* Q, float* K, float* F) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, D = a.dim;
+    constexpr int NRW = GC * 32 / GC_THREADS;
+    for (int d = lane; d < DP4; d += 32) {
+        float q[NRW], k[NRW], z[NRW];
+        GatedChannel c = {0.f, 0.f, 0.f};
+        if (d < D) c = gated_channel(a, h, d);
+#pragma unroll
+        for (int r = 0; r < NRW; ++r) {
+            const int j = warp + r * (GC_THREADS / 32);
+            const bool ok = j < len && d < D;
+            const size_t row = rows[j];
+            z[r] = ok ? a.f[row * a.ldf + h * D + d] : 0.f;
+            k[r] = ok && a.gate != DL_GATE_LOWER ? a.k[row * a.ldk + hk * D + d] : 0.f;
+            if (WITH_Q) q[r] = ok ? a.q[row * a.ldq + hk * D + d] : 0.f;
+        }
+#pragma unroll
+        for (int r = 0; r < NRW; ++r) {
+            const int j = warp + r * (GC_THREADS / 32);
+            float f = 1.f;
+            if (j < len && d < D) gated_form(a, c, z[r], f, k[r]);
+            K[j * ld + d] = k[r];
+            F[j * ld + d] = f;
+            if (COPY) Q[j * ld + d] = k[r];
+            if (WITH_Q) {
+                float v = q[r] * a.q_scale;
+                if (a.q_silu) {
+                    float s, t;
+                    sigmoid_pair_f(q[r], s, t);
+                    v = q[r] * s;
+                }
+                Q[j * ld + d] = v;
+            }
         }
     }
 }

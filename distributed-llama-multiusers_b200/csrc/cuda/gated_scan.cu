@@ -182,7 +182,8 @@ extern "C" int dl_gated_scan(const DlMambaBatch* batch, int n_seq, const DlGated
 // Scratch: states [slots][H][D][V] | decay of the whole chunk [slots][H][D] (head form: entry 0 of D) | n sums [slots][H][D].
 // ------------------------------------------------------------------------------------------------
 // pass 1: a chunk's own sum of (decay to the chunk's end * k_j) v_j^T, and the decay of the whole chunk
-template <bool CH>
+// RT x 4 NC elements of S per thread: tiles of 16 RT rows and 64 NC columns
+template <bool CH, int RT, int NC>
 __global__ void __launch_bounds__(GC_THREADS) gated_chunk_state_kernel(DlMambaBatch b, DlGatedArgs a, GatedScratch sc) {
     extern __shared__ __align__(16) float sm[];
     __shared__ int rows[GC];
@@ -194,7 +195,7 @@ __global__ void __launch_bounds__(GC_THREADS) gated_chunk_state_kernel(DlMambaBa
     const int D = a.dim, V = a.vdim, H = a.n_heads, D8 = (D + 7) & ~7, hk = gated_k_head(a, h);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* ks = sm;                             // [GC][D8]
-    float* vt = ks + (size_t)GC * D8;           // channel form: the decays [GC][D8] first; then value tiles [GC][128]
+    float* vt = ks + (size_t)GC * D8;           // channel form: the decays [GC][D8] first; then value tiles [GC][64 NC]
     if (threadIdx.x < GC) rows[threadIdx.x] = threadIdx.x < len ? b.seq_rows[row0 + threadIdx.x] : 0;
     if (!CH && threadIdx.x < GC) l_s[threadIdx.x] = threadIdx.x < len ? (double)a.log_keep[(size_t)b.seq_rows[row0 + threadIdx.x] * H + h] : 0.0;
     __syncthreads();
@@ -205,18 +206,11 @@ __global__ void __launch_bounds__(GC_THREADS) gated_chunk_state_kernel(DlMambaBa
         if (threadIdx.x == 0) sc.dec[((size_t)ci * H + h) * D] = expf((float)(g + l_s[0]));
     }
     if (!CH) __syncthreads();
-    for (int j = warp; j < GC; j += GC_THREADS / 32) {
+    if (CH) gated_stage_rows<false, false>(a, rows, len, h, hk, D8, D8, nullptr, ks, vt);
+    for (int j = warp; !CH && j < GC; j += GC_THREADS / 32) {
         const size_t row = rows[j];
 #pragma unroll 4
-        for (int d = lane; d < D8; d += 32) {
-            float k = 0.f, f = 1.f;
-            if (j < len && d < D) {
-                if (CH) gated_fk(a, row, h, hk, d, f, k);
-                else k = w_s[j] * a.k[row * a.ldk + h * D + d];
-            }
-            ks[j * D8 + d] = k;
-            if (CH) vt[j * D8 + d] = f;
-        }
+        for (int d = lane; d < D8; d += 32) ks[j * D8 + d] = j < len && d < D ? w_s[j] * a.k[row * a.ldk + h * D + d] : 0.f;
     }
     __syncthreads();
     if (CH) {
@@ -239,32 +233,40 @@ __global__ void __launch_bounds__(GC_THREADS) gated_chunk_state_kernel(DlMambaBa
     }
     float* out = sc.S + ((size_t)ci * H + h) * D * V;
     const int tb = threadIdx.x >> 4, cb = threadIdx.x & 15;
-    for (int c0 = 0; c0 < V; c0 += 128) {
+    for (int c0 = 0; c0 < V; c0 += 64 * NC) {
         __syncthreads();
-        gated_stage_v(a, rows, len, h, c0, vt);
+        gated_stage_v<64 * NC>(a, rows, len, h, c0, vt);
         __syncthreads();
-        for (int d0 = 0; d0 < D; d0 += 128) {
-            const int dt = d0 + tb * 8;          // this thread: 8 rows of S, columns cb * 4 .. + 3 and 64 + cb * 4 .. + 3 of the tile
+        for (int d0 = 0; d0 < D; d0 += 16 * RT) {
+            const int dt = d0 + tb * RT;         // this thread: RT rows of S, columns cb * 4 .. + 3 (and 64 + cb * 4 .. + 3) of the tile
             if (dt >= D8) continue;
-            float acc[8][8];
+            float acc[RT][4 * NC];
 #pragma unroll
-            for (int r = 0; r < 8; ++r)
+            for (int r = 0; r < RT; ++r)
 #pragma unroll
-                for (int u = 0; u < 8; ++u) acc[r][u] = 0.f;
+                for (int u = 0; u < 4 * NC; ++u) acc[r][u] = 0.f;
+#pragma unroll 2
             for (int j = 0; j < len; ++j) {
-                const float4 k0 = *reinterpret_cast<const float4*>(ks + j * D8 + dt), k1 = *reinterpret_cast<const float4*>(ks + j * D8 + dt + 4);
-                const float4 v0 = *reinterpret_cast<const float4*>(vt + j * 128 + cb * 4), v1 = *reinterpret_cast<const float4*>(vt + j * 128 + 64 + cb * 4);
-                const float kk[8] = {k0.x, k0.y, k0.z, k0.w, k1.x, k1.y, k1.z, k1.w};
-                const float vv[8] = {v0.x, v0.y, v0.z, v0.w, v1.x, v1.y, v1.z, v1.w};
+                float kk[RT], vv[4 * NC];
 #pragma unroll
-                for (int r = 0; r < 8; ++r)
+                for (int r = 0; r < RT; r += 4) {
+                    const float4 k = *reinterpret_cast<const float4*>(ks + j * D8 + dt + r);
+                    kk[r] = k.x; kk[r + 1] = k.y; kk[r + 2] = k.z; kk[r + 3] = k.w;
+                }
 #pragma unroll
-                    for (int u = 0; u < 8; ++u) acc[r][u] = fmaf(kk[r], vv[u], acc[r][u]);
+                for (int u = 0; u < NC; ++u) {
+                    const float4 v = *reinterpret_cast<const float4*>(vt + j * 64 * NC + u * 64 + cb * 4);
+                    vv[4 * u] = v.x; vv[4 * u + 1] = v.y; vv[4 * u + 2] = v.z; vv[4 * u + 3] = v.w;
+                }
+#pragma unroll
+                for (int r = 0; r < RT; ++r)
+#pragma unroll
+                    for (int u = 0; u < 4 * NC; ++u) acc[r][u] = fmaf(kk[r], vv[u], acc[r][u]);
             }
 #pragma unroll
-            for (int r = 0; r < 8; ++r)
+            for (int r = 0; r < RT; ++r)
 #pragma unroll
-                for (int u = 0; u < 8; ++u) {
+                for (int u = 0; u < 4 * NC; ++u) {
                     const int d = dt + r, cc = c0 + (u >> 2) * 64 + cb * 4 + (u & 3);
                     if (d < D && cc < V) out[(size_t)d * V + cc] = acc[r][u];
                 }
@@ -306,8 +308,8 @@ __global__ void __launch_bounds__(256) gated_chunk_prefix_kernel(DlMambaBatch b,
 }
 
 // pass 3: the outputs of a chunk.  Shared memory: Q [GC][DP] | K [GC][DP], later tiles of V and of the carried state
-// [GC][128] | F [GC][DP] (channel form), later the scores A [GC][GC_AS] | block decays [4][DP].
-template <int MODE>
+// [GC][64 NC] | F [GC][DP] (channel form), later the scores A [GC][GC_AS] | block decays [4][DP].
+template <int MODE, int NC>
 __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaBatch b, DlGatedArgs a, GatedScratch sc) {
     constexpr bool CH = MODE != GATED_HEAD;
     extern __shared__ __align__(16) float sm[];
@@ -321,7 +323,7 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tb = threadIdx.x >> 4, cb = threadIdx.x & 15;
     float* Q = sm;
     float* K = Q + (size_t)GC * DP;
-    float* F = K + max((size_t)GC * DP, (size_t)GC * 128);
+    float* F = K + max((size_t)GC * DP, (size_t)GC * 64 * NC);
     float* A = F;
     float* T = F + max(CH ? (size_t)GC * DP : 0, (size_t)GC * GC_AS);      // channel form: [4][DP]
     if (threadIdx.x < GC) {
@@ -334,19 +336,13 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
         }
     }
     __syncthreads();
-    for (int j = warp; j < GC; j += GC_THREADS / 32) {
+    if (CH) gated_stage_rows<true, false>(a, rows, len, h, hk, D4, DP, Q, K, F);
+    for (int j = warp; !CH && j < GC; j += GC_THREADS / 32) {
         const size_t row = rows[j];
 #pragma unroll 4
         for (int d = lane; d < D4; d += 32) {
-            float q = 0.f, k = 0.f, f = 1.f;
-            if (j < len && d < D) {
-                q = gated_q(a, row, hk * D + d);
-                if (CH) gated_fk(a, row, h, hk, d, f, k);
-                else k = a.k[row * a.ldk + h * D + d];
-            }
-            Q[j * DP + d] = q;
-            K[j * DP + d] = k;
-            if (CH) F[j * DP + d] = f;
+            Q[j * DP + d] = j < len && d < D ? gated_q(a, row, h * D + d) : 0.f;
+            K[j * DP + d] = j < len && d < D ? a.k[row * a.ldk + h * D + d] : 0.f;
         }
     }
     double gsum = 0.0;
@@ -398,18 +394,19 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
             if (lane == 0 && i < len) a.den[(size_t)rows[i] * H + h] = s;
         }
     }
-    // y = A V + Q P, V and P in tiles of 128 columns (P also 64 rows at a time) in the keys' place
+    // y = A V + Q P, V and P in tiles of 64 NC columns (P also 64 rows at a time) in the keys' place
     const float* P = sc.S + ((size_t)ci * H + h) * D * V;
     float* W = K;
-    for (int c0 = 0; c0 < V; c0 += 128) {
-        const int cw = min(128, V - c0);
-        float acc[4][8];
+    constexpr int VW = 64 * NC;
+    for (int c0 = 0; c0 < V; c0 += VW) {
+        const int cw = min(VW, V - c0);
+        float acc[4][4 * NC];
 #pragma unroll
         for (int r = 0; r < 4; ++r)
 #pragma unroll
-            for (int u = 0; u < 8; ++u) acc[r][u] = 0.f;
+            for (int u = 0; u < 4 * NC; ++u) acc[r][u] = 0.f;
         __syncthreads();
-        gated_stage_v(a, rows, len, h, c0, W);
+        gated_stage_v<VW>(a, rows, len, h, c0, W);
         __syncthreads();
         auto tile_mac = [&](const float* X, int ldx, int kn) {           // acc += X[rows][0 .. kn) . W[0 .. kn)[columns], kn a multiple of 4
             for (int k = 0; k < kn; k += 4) {
@@ -418,13 +415,17 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
                 for (int r = 0; r < 4; ++r) x[r] = *reinterpret_cast<const float4*>(X + (tb * 4 + r) * ldx + k);
 #pragma unroll
                 for (int kk = 0; kk < 4; ++kk) {
-                    const float4 w0 = *reinterpret_cast<const float4*>(W + (k + kk) * 128 + cb * 4), w1 = *reinterpret_cast<const float4*>(W + (k + kk) * 128 + 64 + cb * 4);
-                    const float wv[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+                    float wv[4 * NC];
+#pragma unroll
+                    for (int u = 0; u < NC; ++u) {
+                        const float4 w = *reinterpret_cast<const float4*>(W + (k + kk) * VW + u * 64 + cb * 4);
+                        wv[4 * u] = w.x; wv[4 * u + 1] = w.y; wv[4 * u + 2] = w.z; wv[4 * u + 3] = w.w;
+                    }
 #pragma unroll
                     for (int r = 0; r < 4; ++r) {
                         const float xv = kk == 0 ? x[r].x : kk == 1 ? x[r].y : kk == 2 ? x[r].z : x[r].w;
 #pragma unroll
-                        for (int u = 0; u < 8; ++u) acc[r][u] = fmaf(xv, wv[u], acc[r][u]);
+                        for (int u = 0; u < 4 * NC; ++u) acc[r][u] = fmaf(xv, wv[u], acc[r][u]);
                     }
                 }
             }
@@ -433,12 +434,13 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
         for (int d0 = 0; d0 < D; d0 += GC) {
             const int dn = min(GC, D - d0), dn4 = (dn + 3) & ~3;
             __syncthreads();
+#pragma unroll 4
             for (int d = warp; d < dn4; d += GC_THREADS / 32) {
+                float p[VW / 32];
 #pragma unroll
-                for (int u = 0; u < 4; ++u) {
-                    const int cc = lane + 32 * u;
-                    W[d * 128 + cc] = (d < dn && cc < cw) ? P[(size_t)(d0 + d) * V + c0 + cc] : 0.f;
-                }
+                for (int u = 0; u < VW / 32; ++u) p[u] = (d < dn && lane + 32 * u < cw) ? P[(size_t)(d0 + d) * V + c0 + lane + 32 * u] : 0.f;
+#pragma unroll
+                for (int u = 0; u < VW / 32; ++u) W[d * VW + lane + 32 * u] = p[u];
             }
             __syncthreads();
             if (tb * 4 < len) tile_mac(Q + d0, DP, dn4);
@@ -449,7 +451,7 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
             if (i >= len) continue;
             float* y = a.y + (size_t)rows[i] * a.ld_y + (size_t)h * V + c0;
 #pragma unroll
-            for (int u = 0; u < 8; ++u) {
+            for (int u = 0; u < 4 * NC; ++u) {
                 const int cc = (u >> 2) * 64 + cb * 4 + (u & 3);
                 if (cc < cw) y[cc] = acc[r][u];
             }
@@ -457,12 +459,13 @@ __global__ void __launch_bounds__(GC_THREADS, 2) gated_chunk_out_kernel(DlMambaB
     }
 }
 
-static size_t gated_state_smem(int dim, bool ch) {
-    const size_t D8 = (dim + 7) & ~7, vt = (ch && D8 > 128) ? D8 : 128;
+static int gated_nc(int vdim) { return vdim <= 64 ? 1 : 2; }         // column tiles of 64 or 128
+static size_t gated_state_smem(int dim, bool ch, int nc = 2) {
+    const size_t D8 = (dim + 7) & ~7, vw = 64 * nc, vt = (ch && D8 > vw) ? D8 : vw;
     return (size_t)GC * (D8 + vt) * sizeof(float);
 }
-static size_t gated_out_smem(int dim, bool ch) {
-    const size_t DP = ((dim + 3) & ~3) + 4, k = DP > 128 ? DP : 128, f = (ch && DP > GC_AS) ? DP : GC_AS;
+static size_t gated_out_smem(int dim, bool ch, int nc = 2) {
+    const size_t DP = ((dim + 3) & ~3) + 4, vw = 64 * nc, k = DP > vw ? DP : vw, f = (ch && DP > GC_AS) ? DP : GC_AS;
     return ((size_t)GC * (DP + k + f) + (ch ? 4 * DP : 0)) * sizeof(float);
 }
 
@@ -476,27 +479,38 @@ extern "C" long long dl_gated_chunk_floats(int M, int n_seq, int n_heads, int di
     return (long long)(M / GC + n_seq) * n_heads * dim * ((long long)vdim + 2);
 }
 
+template <int MODE, int NC>
+static int launch_gated_out(const DlMambaBatch& b, int n_seq, int max_chunks, const DlGatedArgs& a, const GatedScratch& sc, cudaStream_t st) {
+    const size_t smem = gated_out_smem(a.dim, MODE != GATED_HEAD, NC);
+    cudaError_t e = cudaFuncSetAttribute(gated_chunk_out_kernel<MODE, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) { dl_set_error("gated_chunk_out: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
+    gated_chunk_out_kernel<MODE, NC><<<dim3(n_seq, max_chunks, a.n_heads), GC_THREADS, smem, st>>>(b, a, sc);
+    return 0;
+}
+
 // pass 3 alone (the delta rule's outputs from its corrected values)
 int gated_chunk_out_channel(const DlMambaBatch& b, int n_seq, int max_chunks, const DlGatedArgs& a, const GatedScratch& sc, cudaStream_t st) {
-    const size_t smem = gated_out_smem(a.dim, true);
-    cudaError_t e = cudaFuncSetAttribute(gated_chunk_out_kernel<GATED_CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) { dl_set_error("gated_chunk_out: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
-    gated_chunk_out_kernel<GATED_CHANNEL><<<dim3(n_seq, max_chunks, a.n_heads), GC_THREADS, smem, st>>>(b, a, sc);
+    return gated_nc(a.vdim) == 1 ? launch_gated_out<GATED_CHANNEL, 1>(b, n_seq, max_chunks, a, sc, st) : launch_gated_out<GATED_CHANNEL, 2>(b, n_seq, max_chunks, a, sc, st);
+}
+
+template <bool CH, int RT, int NC>
+static int launch_gated_state(const DlMambaBatch& b, int n_seq, int max_chunks, const DlGatedArgs& a, const GatedScratch& sc, cudaStream_t st) {
+    const size_t smem = gated_state_smem(a.dim, CH, NC);
+    cudaError_t e = cudaFuncSetAttribute(gated_chunk_state_kernel<CH, RT, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) { dl_set_error("gated_chunk_state: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
+    gated_chunk_state_kernel<CH, RT, NC><<<dim3(n_seq, max_chunks, a.n_heads), GC_THREADS, smem, st>>>(b, a, sc);
     return 0;
 }
 
 template <int MODE>
 static int launch_gated_chunked(const DlMambaBatch& b, int n_seq, int max_chunks, const DlGatedArgs& a, const GatedScratch& sc, cudaStream_t st) {
     constexpr bool CH = MODE != GATED_HEAD;
-    const size_t smem1 = gated_state_smem(a.dim, CH), smem3 = gated_out_smem(a.dim, CH);
-    cudaError_t e = cudaFuncSetAttribute(gated_chunk_state_kernel<CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(gated_chunk_out_kernel<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
-    if (e != cudaSuccess) { dl_set_error("dl_gated_scan_chunked: shared memory attribute: %s", cudaGetErrorString(e)); return -(int)e; }
-    const dim3 grid(n_seq, max_chunks, a.n_heads);
-    gated_chunk_state_kernel<CH><<<grid, GC_THREADS, smem1, st>>>(b, a, sc);
+    const bool narrow = gated_nc(a.vdim) == 1, low = a.dim <= 64;
+    int rc = narrow ? (low ? launch_gated_state<CH, 4, 1>(b, n_seq, max_chunks, a, sc, st) : launch_gated_state<CH, 8, 1>(b, n_seq, max_chunks, a, sc, st))
+                    : (low ? launch_gated_state<CH, 4, 2>(b, n_seq, max_chunks, a, sc, st) : launch_gated_state<CH, 8, 2>(b, n_seq, max_chunks, a, sc, st));
+    if (rc != 0) return rc;
     gated_chunk_prefix_kernel<CH><<<dim3(n_seq, a.n_heads, (a.dim * (a.vdim + (CH ? 0 : 1)) + 255) / 256), 256, 0, st>>>(b, a, sc);
-    gated_chunk_out_kernel<MODE><<<grid, GC_THREADS, smem3, st>>>(b, a, sc);
-    return 0;
+    return narrow ? launch_gated_out<MODE, 1>(b, n_seq, max_chunks, a, sc, st) : launch_gated_out<MODE, 2>(b, n_seq, max_chunks, a, sc, st);
 }
 
 // max_chunks: the most chunks any sequence of the batch has; chunk_slots: M / GC + n_seq of the largest batch the scratch is for

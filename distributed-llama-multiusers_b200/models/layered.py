@@ -566,10 +566,11 @@ class WindowAttentionMixer:
         self.tc_rq, self.tc_rq_small, self.tc_talk = 0, 0, False
         self.partial_floats = 0                 # scratch of the page shares, if it is not the windowed kernel's
         attn_tc = eng.round_x and os.environ.get("DLLAMA_LAYERS_ATTN_TC", "1") != "0"
-        if attn_tc and dv == d and self.talk is None and L.window_tc_supported(H, G, d, 0 if self.own_v else self.rope_dims, eng.wdtype):
+        tile = attn_tc and self.own_v and L.talk_tc_supported(H, G, d, dv, self.key_heads, eng.wdtype, self.value_heads)
+        if attn_tc and not (tile and self.head_gate) and dv == d and self.talk is None and L.window_tc_supported(H, G, d, 0 if self.own_v else self.rope_dims, eng.wdtype):
             self.tc_rq = L.window_tc_rows(H, G)
-        elif attn_tc and self.own_v and L.talk_tc_supported(H, G, d, dv, self.key_heads, eng.wdtype, self.value_heads):
-            # values wider or narrower than the keys, head-mixed scores: the tile kernel of talk_attention.cu
+        elif tile:
+            # values wider or narrower than the keys, head-mixed scores, head gates: the tile kernel of talk_attention.cu
             # tiles of 128 stacked (row, head) pairs for long portions, of 16 for decoding, 64 where those do not fit
             kh, vh = self.key_heads, self.value_heads
             self.tc_rq, self.tc_rq_small, self.tc_talk = L.talk_tc_rows(H, G, d, dv, kh, 1 << 30, vh), L.talk_tc_rows(H, G, d, dv, kh, 1, vh), True
@@ -1008,15 +1009,21 @@ class WkvMixer:
         images = e.shift_images(M)
         if images is not None:               # every mix straight into the operand image of the product that reads it
             L.token_shift(e.mamba_batch, M, h, self.mu, self.shift_state, images=(images[0], images[0].numel(), e.ncap))
-            for s in range(4):
-                L.dense_tc(self.w_rkvg.wh[s], HD, width, images[s], e.ncap, rkvg[s], M)
-            L.dense_tc(self.w_w1.wh, self.rank, width, images[4], e.ncap, w1, M, epi=L.DENSE_SOFTCAP, param=1.0)        # cap 1: tanh
         else:
             mix = e.buf("shift", 5 * width).view(5, R, width)
             L.token_shift(e.mamba_batch, M, h, self.mu, self.shift_state, out=mix)
+        with e.side(1, M):                   # the decays' low-rank product beside the wide ones; cap 1: tanh
+            if images is not None:
+                L.dense_tc(self.w_w1.wh, self.rank, width, images[4], e.ncap, w1, M, epi=L.DENSE_SOFTCAP, param=1.0)
+            else:
+                e.mm(self.w_w1, mix[4], w1, M, epi=L.DENSE_SOFTCAP, param=1.0)
+            e.mm(self.w_w2, w1, az, M)
+        if images is not None:
+            for s in range(4):
+                L.dense_tc(self.w_rkvg.wh[s], HD, width, images[s], e.ncap, rkvg[s], M)
+        else:
             L.dense_heads(self.w_rkvg.t, mix[0], rkvg[0], M, e.round_x, R * width, R * HD)
-            e.mm(self.w_w1, mix[4], w1, M, epi=L.DENSE_SOFTCAP, param=1.0)
-        e.mm(self.w_w2, w1, az, M)
+        e.join(1, M)
         L.gated_scan(e.mamba_batch, e.n_seq, rkvg[0], rkvg[2], ys, self.state, H, d, d, k=rkvg[1], f=az, f_bias=self.w0, gate=L.GATE_EXP_EXP,
                      bonus=self.u, **e.gated_chunking(self))
         image = e.image("tmp", M)

@@ -304,7 +304,7 @@ def gated_scan(batch: DlMambaBatch, n_seq: int, q: torch.Tensor, v: torch.Tensor
     a.gate, a.inv_tau, a.rate, a.bonus, a.k_heads = gate, 1.0 / tau, _p(rate), _p(bonus), k_heads
     a.beta, a.ld_beta = _p(beta), (beta.stride(0) if beta is not None else 0)
     if max_chunks > 0 and beta is not None:
-        assert scratch.numel() >= chunk_slots * n_heads * (dim * (vdim + 2) + 2 * GATED_CHUNK * _round_up(dim, 4))
+        assert scratch.numel() >= chunk_slots * n_heads * (dim * vdim + (2 * GATED_CHUNK + 1) * _round_up(dim, 4))
         check_layers(layers_lib().dl_delta_scan_chunked(batch, n_seq, max_chunks, a, scratch.data_ptr(), chunk_slots, u.data_ptr(), u.stride(0),
                                                         _stream()), "dl_delta_scan_chunked")
         lib.count_launch(3)

@@ -132,7 +132,7 @@ def test_whole_prompts_match_the_oracle(model_a, dtype, tol, same):
     assert again.right.w_in is first.right.w_in and again.right.state is not first.right.state and again.left.cache is not first.left.cache
     assert eng.layers[6].mixer.shift_state is not eng.layers[3].mixer.shift_state and eng.layers[5].mixer.right.conv_state is not eng.layers[2].mixer.right.conv_state
     if dtype == "bfloat16":          # the tile kernels and the operand images are the ones that run
-        assert first.left.tc_talk and eng.layers[2].mixer.left.tc_rq and not eng.layers[2].mixer.left.tc_talk and eng.tc and eng.image("h", 64) is not None
+        assert first.left.tc_talk and eng.layers[2].mixer.left.tc_talk and eng.tc and eng.image("h", 64) is not None
     got = _replay(eng, reqs, _whole(reqs))
     assert eng.gated_chunks == 0 and eng._gated_scratch is not None
     for i in got:
