@@ -13,9 +13,10 @@
 #include "mma_common.cuh"
 
 #define DR_CB 16                  // columns of the state per CTA of the walk
-#define DR_ROWS (2 * GC + 1)      // staged rows per chunk of the walk
+#define DR_WS (GC + 4)            // row strides in shared memory: W transposed, the state
+#define DR_PS (DR_CB + 4)
 
-// scratch per chunk slot and head: the states of GatedScratch, W [GC][D4], and the keys decayed to the chunk's end with the chunk's
+// scratch per chunk slot and head: the states of GatedScratch, W transposed [D4][GC], and the keys decayed to the chunk's end with the chunk's
 // whole decay as one more row, Ke [GC + 1][D4]
 struct DeltaScratch { GatedScratch g; float* W; float* Ke; };
 
@@ -94,7 +95,8 @@ __global__ void __launch_bounds__(GC_THREADS, 2) delta_chunk_system_kernel(DlMam
         for (int e = threadIdx.x; e < off + cw; e += GC_THREADS) {
             if (e < off) {
                 solve_column(Q + e, DP, Nt, b_s);
-                for (int i = 0; i < GC; ++i) W[(size_t)i * D4 + e] = Q[i * DP + e];
+                for (int i = 0; i < GC; i += 4)
+                    *reinterpret_cast<float4*>(W + (size_t)e * GC + i) = make_float4(Q[i * DP + e], Q[(i + 1) * DP + e], Q[(i + 2) * DP + e], Q[(i + 3) * DP + e]);
             } else {
                 const int cc = e - off;
                 solve_column(K + cc, 128, Nt, b_s);
@@ -105,100 +107,140 @@ __global__ void __launch_bounds__(GC_THREADS, 2) delta_chunk_system_kernel(DlMam
     }
 }
 
-// pass 2.  Shared memory: [NB][W [GC] | keys to the end, whole decay [GC + 1]][D4 + 4] | P [D4][DR_CB] | u [GC][DR_CB].
+// pass 2.  Shared memory: [NB][W transposed [D4][DR_WS] | keys to the end and the whole decay [GC + 1][D4 + 4]] | P [D4][DR_PS] |
+// u [GC][DR_CB] | partial sums [8][GC][DR_CB].  W P: every warp takes each eighth row of P and forms all of the product (8 x 4 outputs
+// per lane), the eight sums meet in shared memory.  (keys)^T u: two halves of the rows, 4 x 4 outputs per thread.
 __global__ void __launch_bounds__(256) delta_chunk_walk_kernel(DlMambaBatch b, DlGatedArgs a, DeltaScratch sc, float* __restrict__ u, long long ld_u, int NB) {
     extern __shared__ __align__(16) float sm[];
-    const int n = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * DR_CB, tid = threadIdx.x;
-    const int D = a.dim, V = a.vdim, H = a.n_heads, D4 = (D + 3) & ~3, DS = D4 + 4;
+    const int n = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * DR_CB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int D = a.dim, V = a.vdim, H = a.n_heads, D4 = (D + 3) & ~3, DS = D4 + 4, stage = D4 * DR_WS + (GC + 1) * DS;
     const int s0 = b.seq_start[n], total = b.seq_start[n + 1] - s0, nc = (total + GC - 1) / GC;
-    float* buf = sm;
-    float* P = buf + (size_t)NB * DR_ROWS * DS;
-    float* us = P + (size_t)D4 * DR_CB;
+    float* P = sm + (size_t)NB * stage;
+    float* us = P + (size_t)D4 * DR_PS;
+    float* red = us + GC * DR_CB;
     const size_t sh = (size_t)b.seq_slot[n] * H + h, ch0 = (size_t)(s0 / GC + n) * H + h;
     const bool fresh = b.seq_pos0[n] == 0;
     float* Sg = a.state + sh * D * V + c0;
     for (int e = tid; e < D4 * DR_CB; e += 256) {
         const int d = e / DR_CB, cc = e - d * DR_CB;
-        P[e] = (!fresh && d < D && c0 + cc < V) ? Sg[(size_t)d * V + cc] : 0.f;
+        P[d * DR_PS + cc] = (!fresh && d < D && c0 + cc < V) ? Sg[(size_t)d * V + cc] : 0.f;
     }
-    auto issue = [&](int c, int at) {         // a warp per row
+    auto issue = [&](int c, int at) {
         const size_t o = ch0 + (size_t)c * H;
         const float* w = sc.W + o * GC * D4;
-        const float* ke = sc.Ke + o * (GC + 1) * D4 - (size_t)GC * D4;
-        float* dst = buf + (size_t)at * DR_ROWS * DS;
-        for (int p = (tid & 31) * 4; p < D4; p += 128)
+        const float* ke = sc.Ke + o * (GC + 1) * D4;
+        float* dw = sm + (size_t)at * stage;
+        float* dk = dw + (size_t)D4 * DR_WS;
 #pragma unroll 4
-            for (int i = tid >> 5; i < DR_ROWS; i += 8) cp_async16(dst + (size_t)i * DS + p, (i < GC ? w : ke) + (size_t)i * D4 + p);
+        for (int d = tid >> 4; d < D4; d += 16) cp_async16(dw + (size_t)d * DR_WS + (tid & 15) * 4, w + (size_t)d * GC + (tid & 15) * 4);      // half a warp per row
+        for (int p = lane * 4; p < D4; p += 128)
+#pragma unroll 4
+            for (int i = warp; i <= GC; i += 8) cp_async16(dk + (size_t)i * DS + p, ke + (size_t)i * D4 + p);
     };
-    const int ui = tid >> 2, uc = (tid & 3) * 4;               // step A: this thread's row and four columns of u
-    const int half = tid >> 7, cols = DR_CB / 2;               // step B: half of the columns of rows d = tid % 128 + 128 x of P
-    issue(0, 0);
-    for (int c = 0; c < nc; ++c) {
-        const int at = NB == 2 ? c & 1 : 0, len = min(GC, total - c * GC);
-        float own[4] = {0.f, 0.f, 0.f, 0.f};
-        float* ug = nullptr;
-        if (ui < len) {
-            ug = u + (size_t)b.seq_rows[s0 + c * GC + ui] * ld_u + (size_t)h * V + c0 + uc;
+    const int ui = tid >> 2, uc = (tid & 3) * 4;               // this thread's row and four columns of u
+    auto row_of = [&](int c) { return c < nc && c * GC + ui < total ? b.seq_rows[s0 + c * GC + ui] : -1; };
+    auto load_own = [&](int row, float* own) {
 #pragma unroll
-            for (int x = 0; x < 4; ++x)
-                if (c0 + uc + x < V) own[x] = ug[x];
-        }
+        for (int x = 0; x < 4; ++x) own[x] = row >= 0 && c0 + uc + x < V ? u[(size_t)row * ld_u + (size_t)h * V + c0 + uc + x] : 0.f;
+    };
+    const int rg = lane >> 2, cg = lane & 3;                   // W P: rows rg * 8 .. + 7, columns cg * 4 .. + 3
+    const int half = tid >> 7, kd = lane * 4, kc = ((tid >> 5) & 3) * 4;      // keys^T u: half of the rows, P rows kd .. + 3 (+ 128 m), columns kc .. + 3
+    float own[4];
+    int row = row_of(0);
+    issue(0, 0);
+    load_own(row, own);
+    for (int c = 0; c < nc; ++c) {
+        const int at = NB == 2 ? c & 1 : 0;
+        const int row_next = row_of(c + 1);
         cp_async_wait_all();
         __syncthreads();                      // the chunk has landed, P is complete
         if (NB == 2 && c + 1 < nc) issue(c + 1, at ^ 1);
-        const float* W = buf + (size_t)at * DR_ROWS * DS;
-        const float* Ke = W + (size_t)GC * DS;
+        const float* Wt = sm + (size_t)at * stage;
+        const float* Ke = Wt + (size_t)D4 * DR_WS;
         float* Pg = sc.g.S + (ch0 + (size_t)c * H) * D * V + c0;
         for (int e = tid; e < D * DR_CB; e += 256) {           // the state ahead of this chunk
             const int d = e / DR_CB, cc = e - d * DR_CB;
-            if (c0 + cc < V) Pg[(size_t)d * V + cc] = P[e];
+            if (c0 + cc < V) Pg[(size_t)d * V + cc] = P[d * DR_PS + cc];
         }
-        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        {
+            float acc[8][4];
+#pragma unroll
+            for (int r = 0; r < 8; ++r) acc[r][0] = acc[r][1] = acc[r][2] = acc[r][3] = 0.f;
 #pragma unroll 4
-        for (int d = 0; d < D4; d += 4) {
-            const float4 w = *reinterpret_cast<const float4*>(W + ui * DS + d);
-            const float wv[4] = {w.x, w.y, w.z, w.w};
+            for (int d = warp; d < D4; d += 8) {
+                const float4 w0 = *reinterpret_cast<const float4*>(Wt + d * DR_WS + rg * 8), w1 = *reinterpret_cast<const float4*>(Wt + d * DR_WS + rg * 8 + 4);
+                const float4 p = *reinterpret_cast<const float4*>(P + d * DR_PS + cg * 4);
+                const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
 #pragma unroll
-            for (int x = 0; x < 4; ++x) {
-                const float4 p = *reinterpret_cast<const float4*>(P + (d + x) * DR_CB + uc);
-                acc[0] = fmaf(wv[x], p.x, acc[0]);
-                acc[1] = fmaf(wv[x], p.y, acc[1]);
-                acc[2] = fmaf(wv[x], p.z, acc[2]);
-                acc[3] = fmaf(wv[x], p.w, acc[3]);
+                for (int r = 0; r < 8; ++r) {
+                    acc[r][0] = fmaf(w[r], p.x, acc[r][0]);
+                    acc[r][1] = fmaf(w[r], p.y, acc[r][1]);
+                    acc[r][2] = fmaf(w[r], p.z, acc[r][2]);
+                    acc[r][3] = fmaf(w[r], p.w, acc[r][3]);
+                }
             }
-        }
 #pragma unroll
-        for (int x = 0; x < 4; ++x) {
-            const float t = own[x] - acc[x];
-            us[ui * DR_CB + uc + x] = ui < len ? t : 0.f;
-            if (ug && c0 + uc + x < V) ug[x] = t;
+            for (int r = 0; r < 8; ++r)
+                *reinterpret_cast<float4*>(red + warp * GC * DR_CB + (rg * 8 + r) * DR_CB + cg * 4) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+        }
+        __syncthreads();
+        {
+            float t[4] = {own[0], own[1], own[2], own[3]};
+#pragma unroll
+            for (int w = 0; w < 8; ++w) {
+                const float4 r = *reinterpret_cast<const float4*>(red + w * GC * DR_CB + tid * 4);
+                t[0] -= r.x; t[1] -= r.y; t[2] -= r.z; t[3] -= r.w;
+            }
+            *reinterpret_cast<float4*>(us + tid * 4) = row >= 0 ? make_float4(t[0], t[1], t[2], t[3]) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int x = 0; x < 4; ++x)
+                if (row >= 0 && c0 + uc + x < V) u[(size_t)row * ld_u + (size_t)h * V + c0 + uc + x] = t[x];
+            row = row_next;
+            load_own(row, own);               // the next chunk's
         }
         __syncthreads();
         const float* dec = Ke + (size_t)GC * DS;
-        for (int d = tid & 127; d < D; d += 128) {
-            float p[8];
-            const float g = dec[d];
+        for (int d = kd; d < D4; d += 128) {
+            float acc[4][4];
 #pragma unroll
-            for (int x = 0; x < 8; ++x) p[x] = g * P[d * DR_CB + half * cols + x];
+            for (int r = 0; r < 4; ++r) acc[r][0] = acc[r][1] = acc[r][2] = acc[r][3] = 0.f;
 #pragma unroll 8
-            for (int i = 0; i < GC; ++i) {
-                const float k = Ke[i * DS + d];
-                const float4 u0 = *reinterpret_cast<const float4*>(us + i * DR_CB + half * cols), u1 = *reinterpret_cast<const float4*>(us + i * DR_CB + half * cols + 4);
-                p[0] = fmaf(k, u0.x, p[0]); p[1] = fmaf(k, u0.y, p[1]); p[2] = fmaf(k, u0.z, p[2]); p[3] = fmaf(k, u0.w, p[3]);
-                p[4] = fmaf(k, u1.x, p[4]); p[5] = fmaf(k, u1.y, p[5]); p[6] = fmaf(k, u1.z, p[6]); p[7] = fmaf(k, u1.w, p[7]);
+            for (int i = half * (GC / 2); i < (half + 1) * (GC / 2); ++i) {
+                const float4 k = *reinterpret_cast<const float4*>(Ke + i * DS + d), x = *reinterpret_cast<const float4*>(us + i * DR_CB + kc);
+                const float kk[4] = {k.x, k.y, k.z, k.w};
+#pragma unroll
+                for (int r = 0; r < 4; ++r) {
+                    acc[r][0] = fmaf(kk[r], x.x, acc[r][0]);
+                    acc[r][1] = fmaf(kk[r], x.y, acc[r][1]);
+                    acc[r][2] = fmaf(kk[r], x.z, acc[r][2]);
+                    acc[r][3] = fmaf(kk[r], x.w, acc[r][3]);
+                }
             }
 #pragma unroll
-            for (int x = 0; x < 8; ++x) P[d * DR_CB + half * cols + x] = p[x];
+            for (int r = 0; r < 4; ++r) {
+                float4* at_p = reinterpret_cast<float4*>(P + (d + r) * DR_PS + kc);
+                float4* at_r = reinterpret_cast<float4*>(red + ((d + r) * 4 + (kc >> 2)) * 4);
+                if (half) {
+                    *at_r = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+                } else {
+                    const float4 q = *at_p;
+                    const float g = dec[d + r];
+                    *at_p = make_float4(fmaf(g, q.x, acc[r][0]), fmaf(g, q.y, acc[r][1]), fmaf(g, q.z, acc[r][2]), fmaf(g, q.w, acc[r][3]));
+                }
+            }
         }
-        if (NB == 1 && c + 1 < nc) {
-            __syncthreads();
-            issue(c + 1, 0);
+        __syncthreads();
+        for (int e = tid; e < D4 * DR_CB / 4; e += 256) {       // the second half's sums
+            float4* at_p = reinterpret_cast<float4*>(P + (e >> 2) * DR_PS + (e & 3) * 4);
+            const float4 q = *at_p, r = *reinterpret_cast<const float4*>(red + e * 4);
+            *at_p = make_float4(q.x + r.x, q.y + r.y, q.z + r.z, q.w + r.w);
         }
+        if (NB == 1 && c + 1 < nc) issue(c + 1, 0);
     }
     __syncthreads();
     for (int e = tid; e < D * DR_CB; e += 256) {
         const int d = e / DR_CB, cc = e - d * DR_CB;
-        if (c0 + cc < V) Sg[(size_t)d * V + cc] = P[e];
+        if (c0 + cc < V) Sg[(size_t)d * V + cc] = P[d * DR_PS + cc];
     }
 }
 
@@ -209,7 +251,7 @@ static size_t delta_system_smem(int dim) {
 }
 static size_t delta_walk_smem(int dim, int nb) {
     const size_t D4 = (dim + 3) & ~3;
-    return ((size_t)nb * DR_ROWS * (D4 + 4) + D4 * DR_CB + (size_t)GC * DR_CB) * sizeof(float);
+    return ((size_t)nb * (D4 * DR_WS + (GC + 1) * (D4 + 4)) + D4 * DR_PS + (size_t)9 * GC * DR_CB) * sizeof(float);
 }
 
 // 0 if the chunked kernels take these sizes
@@ -219,7 +261,7 @@ extern "C" int dl_delta_scan_chunked_supported(int dim, int vdim) {
 
 // f32 of scratch for a batch of M rows in n_seq sequences
 extern "C" long long dl_delta_chunk_floats(int M, int n_seq, int n_heads, int dim, int vdim) {
-    return (long long)(M / GC + n_seq) * n_heads * ((long long)dim * vdim + DR_ROWS * ((dim + 3) & ~3));
+    return (long long)(M / GC + n_seq) * n_heads * ((long long)dim * vdim + (2 * GC + 1) * ((dim + 3) & ~3));
 }
 
 extern "C" int dl_delta_scan_chunked(const DlMambaBatch* batch, int n_seq, int max_chunks, const DlGatedArgs* args, float* scratch,

@@ -281,12 +281,11 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
     }
 }
 
-// merge of the page shares: one CTA per (tile, key/value head, position of the tile) and 256 (head, column) outputs.  The shares' maxima and sums are
-// gathered into shared memory, every (head, share) weight e^(m_k - m) / l is formed once, then a thread per (head,
-// column) sums the shares.
+// merge of the page shares: one CTA per (tile, key/value head, position of the tile) and 256 (head, column) outputs.  Every (head,
+// share) weight e^(m_k - m) / l is formed once, by a warp per head, then a thread per (head, column) sums the shares.
 __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, const int* __restrict__ tile_rows, int rq, int n_splits,
                                                          const float* __restrict__ partial, int DVP, int TA_ROWS, int vs) {
-    __shared__ float w_s[64 * TA_MAX_SPLITS], l_s[64 * TA_MAX_SPLITS];      // heads of one group x shares
+    __shared__ float w_s[64 * TA_MAX_SPLITS];                 // heads of one group x shares
     const bool wide = a.value_heads > 1;                      // blockIdx.y: (key/value head of the scores, block of vs value heads)
     const int nvb = wide ? (a.kv_heads + vs - 1) / vs : 1, DVH = wide ? DVP / vs : DVP;
     const int gv = blockIdx.y % (a.kv_heads * nvb), part = blockIdx.y / (a.kv_heads * nvb);
@@ -294,25 +293,15 @@ __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, con
     const int m = tile_rows[(size_t)tile * rq + r];
     if (m < 0) return;
     const float* base = partial + ((size_t)tile * a.kv_heads * nvb + gv) * n_splits * TA_ROWS * (DVP + 2);
-    for (int idx = threadIdx.x; idx < rep * n_splits; idx += blockDim.x) {
-        const int hg = idx / n_splits, k = idx - hg * n_splits;
-        const float* p = base + ((size_t)k * TA_ROWS + r * rep + hg) * (DVP + 2);
-        w_s[idx] = p[DVP];
-        l_s[idx] = p[DVP + 1];
-    }
-    __syncthreads();
-    for (int hg = threadIdx.x; hg < rep; hg += blockDim.x) {
-        float mx = -INFINITY, l = 0.f;
-        for (int k = 0; k < n_splits; ++k) mx = fmaxf(mx, w_s[hg * n_splits + k]);
-        for (int k = 0; k < n_splits; ++k) {
-            const float mk = w_s[hg * n_splits + k];
-            const float e = mk == -INFINITY ? 0.f : expf(mk - mx);
-            l += l_s[hg * n_splits + k] * e;
-            w_s[hg * n_splits + k] = e;
-        }
-        if (a.sink) l += expf(a.sink[g * rep + hg] - mx);
-        const float inv = (a.gate ? sigmoid_f(a.gate[(size_t)m * a.ld_gate + g * rep + hg]) : 1.f) / l;
-        for (int k = 0; k < n_splits; ++k) w_s[hg * n_splits + k] *= inv;
+    for (int hg = threadIdx.x >> 5; hg < rep; hg += blockDim.x >> 5) {        // a warp per head, a lane per share
+        const int k = threadIdx.x & 31;
+        const float* p = base + ((size_t)k * TA_ROWS + r * rep + hg) * (DVP + 2) + DVP;
+        const float mk = k < n_splits ? p[0] : -INFINITY, lk = k < n_splits ? p[1] : 0.f;
+        const float sink = a.sink ? a.sink[g * rep + hg] : 0.f, gate = a.gate ? sigmoid_f(a.gate[(size_t)m * a.ld_gate + g * rep + hg]) : 1.f;
+        const float mx = warp_max(mk), e = mk == -INFINITY ? 0.f : expf(mk - mx);
+        float l = warp_sum(lk * e);
+        if (a.sink) l += expf(sink - mx);
+        if (k < n_splits) w_s[hg * n_splits + k] = e * (gate / l);
     }
     __syncthreads();
     const int nv = wide ? min(vs, a.kv_heads - v0) : 1, W = nv * DV;

@@ -552,36 +552,25 @@ __global__ void __launch_bounds__(128, 4) window_attention_mma_kernel(DlWindowAt
     }
 }
 
-// merge of the page shares: one CTA per (tile, key/value head, position of the tile).  The shares' maxima and sums are
-// gathered into shared memory, every (head, share) weight e^(m_k - m) / l is formed once, then a thread per (head,
-// column) sums the shares.
+// merge of the page shares: one CTA per (tile, key/value head, position of the tile).  Every (head, share) weight
+// e^(m_k - m) / l is formed once, by a warp per head, then a thread per (head, column) sums the shares.
 #define WM_MAX_SPLITS 32
 __global__ void __launch_bounds__(128) window_merge_kernel(DlWindowAttnArgs a, const int* __restrict__ tile_rows, int rq, int n_splits,
                                                            const float* __restrict__ partial) {
-    __shared__ float w_s[WM_ROWS * WM_MAX_SPLITS], l_s[WM_ROWS * WM_MAX_SPLITS];
+    __shared__ float w_s[WM_ROWS * WM_MAX_SPLITS];
     const int tile = blockIdx.x, g = blockIdx.y, r = blockIdx.z, D = a.dim, rep = a.heads / a.kv_heads;
     const int m = tile_rows[(size_t)tile * rq + r];
     if (m < 0) return;
     const float* base = partial + ((size_t)tile * a.kv_heads + g) * n_splits * WM_ROWS * (D + 2);
-    for (int idx = threadIdx.x; idx < rep * n_splits; idx += blockDim.x) {
-        const int hg = idx / n_splits, k = idx - hg * n_splits;
-        const float* p = base + ((size_t)k * WM_ROWS + r * rep + hg) * (D + 2);
-        w_s[idx] = p[D];
-        l_s[idx] = p[D + 1];
-    }
-    __syncthreads();
-    for (int hg = threadIdx.x; hg < rep; hg += blockDim.x) {
-        float mx = -INFINITY, l = 0.f;
-        for (int k = 0; k < n_splits; ++k) mx = fmaxf(mx, w_s[hg * n_splits + k]);
-        for (int k = 0; k < n_splits; ++k) {
-            const float mk = w_s[hg * n_splits + k];
-            const float e = mk == -INFINITY ? 0.f : expf(mk - mx);
-            l += l_s[hg * n_splits + k] * e;
-            w_s[hg * n_splits + k] = e;
-        }
-        if (a.sink) l += expf(a.sink[g * rep + hg] - mx);
-        const float inv = (a.gate ? sigmoid_f(a.gate[(size_t)m * a.ld_gate + g * rep + hg]) : 1.f) / l;
-        for (int k = 0; k < n_splits; ++k) w_s[hg * n_splits + k] *= inv;
+    for (int hg = threadIdx.x >> 5; hg < rep; hg += blockDim.x >> 5) {        // a warp per head, a lane per share
+        const int k = threadIdx.x & 31;
+        const float* p = base + ((size_t)k * WM_ROWS + r * rep + hg) * (D + 2) + D;
+        const float mk = k < n_splits ? p[0] : -INFINITY, lk = k < n_splits ? p[1] : 0.f;
+        const float sink = a.sink ? a.sink[g * rep + hg] : 0.f, gate = a.gate ? sigmoid_f(a.gate[(size_t)m * a.ld_gate + g * rep + hg]) : 1.f;
+        const float mx = warp_max(mk), e = mk == -INFINITY ? 0.f : expf(mk - mx);
+        float l = warp_sum(lk * e);
+        if (a.sink) l += expf(sink - mx);
+        if (k < n_splits) w_s[hg * n_splits + k] = e * (gate / l);
     }
     __syncthreads();
     for (int idx = threadIdx.x; idx < rep * D; idx += blockDim.x) {
