@@ -309,7 +309,7 @@ __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, con
         const int hg = idx / W, c = idx - hg * W, vh = c / DV;
         const float* p = base + (size_t)(r * rep + hg) * (DVP + 2) + vh * DVH + (c - vh * DV);
         float acc = 0.f;                      // a share without pages left zeros and weighs 0: every load can go out at once
-#pragma unroll 8
+#pragma unroll 16
         for (int k = 0; k < n_splits; ++k) acc = fmaf(w_s[hg * n_splits + k], p[(size_t)k * TA_ROWS * (DVP + 2)], acc);
         a.out[(size_t)m * a.ldo + (wide ? (size_t)((g * rep + hg) * a.kv_heads + v0) * DV : (size_t)(g * rep + hg) * DV) + c] = acc;
     }

@@ -577,7 +577,7 @@ __global__ void __launch_bounds__(128) window_merge_kernel(DlWindowAttnArgs a, c
         const int hg = idx / D, c = idx - hg * D;
         const float* p = base + (size_t)(r * rep + hg) * (D + 2) + c;
         float acc = 0.f;                      // a share without pages left zeros and weighs 0: every load can go out at once
-#pragma unroll 8
+#pragma unroll 16
         for (int k = 0; k < n_splits; ++k) acc = fmaf(w_s[hg * n_splits + k], p[(size_t)k * WM_ROWS * (D + 2)], acc);
         a.out[(size_t)m * a.ldo + (size_t)(g * rep + hg) * D + c] = acc;
     }

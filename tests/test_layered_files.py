@@ -276,3 +276,72 @@ def test_vopedra_oracle_mix_gates_state_carry_and_prefix_property():
         w = torch.exp(torch.stack([b[j + 1:, h].sum() + a[j, h] for j in range(T)]))
         num, den = ((w * (kk[:, h] @ q[8, h]))[:, None] * vv[:, h]).sum(0), (w * (kk[:, h] @ q[8, h])).sum().abs()
         assert torch.allclose(o[8, h], num / (torch.clamp(den, min=1.0) + 1e-6 * torch.exp(u[h])), rtol=1e-9, atol=1e-12)
+
+
+def test_silizen_configuration_runs_and_tensor_names(tmp_path):
+    from dllama_b200.models.layered import DESIGNS, example_config_silizen, interpolated_rotary
+    cfg = example_config_silizen()
+    d = str(tmp_path / "d")
+    tensors = write_random_model(d, cfg, seed=1)
+    assert registry.architecture_of(d) == "Silizen" and "Silizen" in registry.ARCHITECTURES
+    c = LayerListConfig.load(d)
+    assert (c.residual, c.streams, c.logit_softcap, c.logit_scale, c.loop_times, c.norm_eps) == ("parallel", 1, 0.0, 0.5, 2, 1e-6)
+    assert c.traits is DESIGNS["Silizen"] and LayerListConfig.from_dict({k: v for k, v in cfg.items() if k != "logit_scale"}).logit_scale == 1.0
+    assert [(l.type, l.weights_of, l.tensors, l.opens) for l in c.layers] == [
+        ("wkv", None, 0, None), ("parallel", None, 1, 0), ("parallel_2", None, 2, None), ("parallel", 1, 1, 1), ("parallel_2", 2, 2, None), ("wkv", None, 3, None)]
+    assert "head" not in tensors and "embed.norm" not in tensors and "l1.norm2" not in tensors and "loop.step" not in tensors
+    assert tensors["loop.in"].shape == (160, 320) and tensors["final.norm.b"].shape == (160,) and tensors["l1.norm1.b"].shape == (160,)
+    assert tensors["l0.mix.mu.w"].shape == (160,) and tensors["l0.mix.u"].shape == (3, 20) and tensors["l0.mix.norm"].shape == (60,)
+    assert tensors["l1.mix.left.q.norm"].shape == (24,) and tensors["l1.mix.left.g"].shape == (6, 160) and "l1.mix.left.out" not in tensors
+    assert tensors["l1.mix.right.a2.b"].shape == (84,) and tensors["l1.mix.right.norm"].shape == (16,)
+    assert tensors["l2.mix.left.k.b"].shape == (96,) and "l2.mix.left.q.norm" not in tensors and tensors["l2.mix.left.out"].shape == (160,)
+    assert tensors["l2.mix.right.v.conv"].shape == (144, 3) and tensors["l2.mix.right.q"].shape == (60, 160) and tensors["l2.mix.right.dt_bias"].shape == (120,)
+    assert "l3.mlp.up" not in tensors
+    # frequencies scaled by wavelength: short ones kept, long ones divided, a blend between
+    f, mag = interpolated_rotary(10000.0, 16, {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 256})
+    g, _ = interpolated_rotary(10000.0, 16, None)
+    turns = 256 * g / (2 * math.pi)
+    assert mag == 1.0 and bool((f[turns > 4] == g[turns > 4]).all()) and torch.allclose(f[turns < 1], g[turns < 1] / 4) and int((turns > 4).sum()) > 0
+    mid = (turns >= 1) & (turns <= 4)
+    assert int(mid.sum()) > 0 and bool(((f[mid] > g[mid] / 4) & (f[mid] < g[mid])).all())
+
+
+def test_silizen_oracle_sink_delta_rule_read_ahead_and_prefix_property():
+    """The oracle itself: appended tokens change nothing before them; the sink is a key of score zero without a value; states carried
+    across a cut equal one walk; a whole write along a unit key replaces what the state held there, and the delta rule over a chunk is
+    the solution of a triangular system; time mixing reads the state ahead of its own write."""
+    import silizen_oracle as S
+    from dllama_b200.models.layered import example_config_silizen
+    cfg = example_config_silizen(width=48, vocab=40, heads=2)
+    t = random_tensors(cfg, seed=2)
+    toks = torch.randint(0, 40, (47,), generator=torch.Generator().manual_seed(3)).tolist()
+    assert torch.allclose(S.model_logits(t, cfg, toks)[:9], S.model_logits(t, cfg, toks[:9]), atol=1e-9)
+    g = torch.Generator().manual_seed(5)
+    rnd = lambda *s: torch.randn(*s, generator=g, dtype=torch.float64)
+    T, H, G, d, dv = 9, 4, 2, 6, 5
+    q, k, v = rnd(T, H, d), rnd(T, G, d), rnd(T, G, dv)
+    o = S.sink_attention_rows(q, k, v, 0.7, softcap=3.0, window=4, slopes=S.distance_slopes(H))
+    for h in range(H):
+        s = 3.0 * torch.tanh(0.7 * (k[5:9, h // 2] @ q[8, h]) / 3.0) - 2.0 ** (-2.0 * (h + 1)) * torch.tensor([3.0, 2.0, 1.0, 0.0], dtype=torch.float64)
+        p = torch.softmax(torch.cat([s, torch.zeros(1, dtype=torch.float64)]), 0)[:4]
+        assert torch.allclose(o[8, h], p @ v[5:9, h // 2], atol=1e-12)
+    q, k, v, f, beta = rnd(T, H, d), S.length_one(rnd(T, H, d)), rnd(T, H, dv), torch.rand(T, H, d, generator=g, dtype=torch.float64), torch.rand(T, H, generator=g, dtype=torch.float64)
+    for rows, extra in ((S.gated_rows, ()), (S.wkv_rows, (rnd(H, d),)), (S.delta_rows, (beta,))):
+        cut = lambda a, b: [x if x.shape[0] == H else x[a:b] for x in extra]
+        whole, end = rows(q, k, v, f, *cut(0, T))
+        first, S1 = rows(q[:4], k[:4], v[:4], f[:4], *cut(0, 4))
+        rest, S2 = rows(q[4:], k[4:], v[4:], f[4:], *cut(4, T), S1)
+        assert torch.allclose(torch.cat([first, rest]), whole, atol=1e-12) and torch.allclose(end, S2, atol=1e-12)
+    same = k[:1].expand(3, H, d)                              # one unit key, written whole three times: the last value stays
+    o, end = S.delta_rows(same, same, v[:3], torch.ones(3, H, d, dtype=torch.float64), torch.ones(3, H, dtype=torch.float64))
+    assert torch.allclose(o[2], v[2], atol=1e-5)
+    o, end = S.delta_rows(q, k, v, f, beta)
+    for h in range(H):                                        # (I + N) u = beta v, N_ij = beta_i k_i . D_ij k_j
+        D = lambda i, j: f[j + 1:i + 1, h].prod(0)
+        N = torch.stack([torch.stack([beta[i, h] * (k[i, h] * D(i, j)) @ k[j, h] if j < i else torch.zeros((), dtype=torch.float64) for j in range(T)]) for i in range(T)])
+        u = torch.linalg.solve(torch.eye(T, dtype=torch.float64) + N, beta[:, h, None] * v[:, h])
+        assert torch.allclose(o[8, h], sum(((q[8, h] * D(8, j)) @ k[j, h]) * u[j] for j in range(T)), atol=1e-10)
+    bonus = rnd(H, d)
+    o, _ = S.wkv_rows(q, k, v, f, bonus)
+    assert torch.allclose(o[0], (q[0] * bonus * k[0]).sum(-1, keepdim=True) * v[0], atol=1e-12)
+    assert torch.allclose(o[1], (q[1] * bonus * k[1]).sum(-1, keepdim=True) * v[1] + (q[1] * k[0]).sum(-1, keepdim=True) * v[0], atol=1e-12)
