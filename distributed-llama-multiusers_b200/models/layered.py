@@ -981,8 +981,12 @@ class WkvMixer:
             self.w0, self.u, self.norm = V(prefix + "w0"), V(prefix + "u").reshape(-1).contiguous(), V(prefix + "norm")
             if tuple(self.mu.shape) != (5, width) or any(t.numel() != H * d for t in (self.w0, self.u, self.norm)):
                 raise ValueError(f"layer {index}: mu, w0, u or norm do not fit {H} heads of {d}")
+            # one image after another: the four products are one grouped launch
+            self.wh = torch.cat(self.w_rkvg.wh) if self.w_rkvg.wh is not None else None
+            if self.wh is not None:
+                self.w_rkvg.wh = None
         else:
-            for n in ("w_rkvg", "w_w1", "w_w2", "w_o", "mu", "w0", "u", "norm", "rank"):
+            for n in ("w_rkvg", "w_w1", "w_w2", "w_o", "mu", "w0", "u", "norm", "rank", "wh"):
                 setattr(self, n, getattr(share, n))
         f32 = dict(dtype=torch.float32, device=eng.device)
         self.state, self.shift_state = torch.zeros(eng.n_slots, H, d, d, **f32), torch.zeros(eng.n_slots, width, **f32)
@@ -993,7 +997,8 @@ class WkvMixer:
 
     def scratch(self) -> Dict[str, int]:
         HD = self.H * self.dim
-        return {"shift": 5 * self.eng.cfg.width, "rkvg": 4 * HD, "w1": self.rank, "az": HD, "ys": HD, "yn": HD}
+        R = self.eng.max_rows
+        return {"shift": 5 * self.eng.cfg.width, "rkvg": (4 * HD * ((R + 7) // 8 * 8) + R - 1) // R, "w1": self.rank, "az": HD, "ys": HD, "yn": HD}
 
     def bind(self, mixers: list):
         pass
@@ -1005,24 +1010,23 @@ class WkvMixer:
         e, L = self.eng, self.eng.L
         H, d, width, R = self.H, self.dim, e.cfg.width, e.max_rows
         HD = H * d
-        rkvg, w1, az, ys, yn = e.buf("rkvg", 4 * HD).view(4, R, HD), e.buf("w1", self.rank), e.buf("az", HD), e.buf("ys", HD), e.buf("yn", HD)
+        rkvg, w1, az, ys, yn = e.stacked("rkvg", 4, HD), e.buf("w1", self.rank), e.buf("az", HD), e.buf("ys", HD), e.buf("yn", HD)
         images = e.shift_images(M)
-        if images is not None:               # every mix straight into the operand image of the product that reads it
-            L.token_shift(e.mamba_batch, M, h, self.mu, self.shift_state, images=(images[0], images[0].numel(), e.ncap))
+        if images is not None:               # every mix straight into its rows of the products' operand image
+            L.token_shift(e.mamba_batch, M, h, self.mu, self.shift_state, images=(images, e.ncap // 8 * 2048, 5 * e.ncap))
         else:
             mix = e.buf("shift", 5 * width).view(5, R, width)
             L.token_shift(e.mamba_batch, M, h, self.mu, self.shift_state, out=mix)
         with e.side(1, M):                   # the decays' low-rank product beside the wide ones; cap 1: tanh
             if images is not None:
-                L.dense_tc(self.w_w1.wh, self.rank, width, images[4], e.ncap, w1, M, epi=L.DENSE_SOFTCAP, param=1.0)
+                L.dense_tc(self.w_w1.wh, self.rank, width, images[4 * (e.ncap // 8 * 2048):], 5 * e.ncap, w1, M, epi=L.DENSE_SOFTCAP, param=1.0)
             else:
                 e.mm(self.w_w1, mix[4], w1, M, epi=L.DENSE_SOFTCAP, param=1.0)
             e.mm(self.w_w2, w1, az, M)
         if images is not None:
-            for s in range(4):
-                L.dense_tc(self.w_rkvg.wh[s], HD, width, images[s], e.ncap, rkvg[s], M)
+            L.dense_tc_grouped(self.wh, self.wh.numel() // 4, 4, e.shift_grp, HD, width, images, 5 * e.ncap, rkvg.view(-1, HD), M)
         else:
-            L.dense_heads(self.w_rkvg.t, mix[0], rkvg[0], M, e.round_x, R * width, R * HD)
+            L.dense_heads(self.w_rkvg.t, mix[0], rkvg[0], M, e.round_x, R * width, e.ncap * HD)
         e.join(1, M)
         L.gated_scan(e.mamba_batch, e.n_seq, rkvg[0], rkvg[2], ys, self.state, H, d, d, k=rkvg[1], f=az, f_bias=self.w0, gate=L.GATE_EXP_EXP,
                      bonus=self.u, **e.gated_chunking(self))
@@ -1437,8 +1441,7 @@ class LayerListEngine:
             self._xh = {k: torch.zeros(n, dtype=torch.uint8, device=dev) for k in ("h", "tmp") + (("h2", "tmp1", "tmp2") if self.cfg.residual == "parallel" else ())}
             self._shift_images = None
             if any(isinstance(mx, WkvMixer) for mx in mixers):
-                n = L.xh_bytes(self.cfg.width, self.ncap)
-                self._shift_images = [t for t in torch.zeros(5, n, dtype=torch.uint8, device=dev)]
+                self._shift_images = torch.zeros(L.xh_bytes(self.cfg.width, 5 * self.ncap), dtype=torch.uint8, device=dev)
         if self.cfg.streams > L.HC_MAX_STREAMS:
             raise ValueError(f"{self.cfg.streams} streams: the kernels keep at most {L.HC_MAX_STREAMS} copies of the residual stream")
         self.x = torch.zeros(R, self.cfg.streams * self.cfg.width, dtype=torch.float32, device=dev)      # row = [streams][width]
@@ -1469,6 +1472,8 @@ class LayerListEngine:
         for rq in sorted({r for mx in mixers if isinstance(mx, WindowAttentionMixer) for r in (mx.tc_rq, mx.tc_rq_small) if r}):
             self._wtile_off[rq] = self._desc_len
             self._desc_len += ((R + rq - 1) // rq + S) * rq
+        # then first row and rows of the four grouped products of time-mixing layers
+        self._shift_off, self._desc_len = self._desc_len, self._desc_len + 8
         self.tile_rows = None
         self.h_desc = torch.zeros(self._desc_len, dtype=torch.int32).pin_memory()
         self.desc = torch.zeros(self._desc_len, dtype=torch.int32, device=dev)
@@ -1479,6 +1484,7 @@ class LayerListEngine:
         self.tile_rows = d[self._tiles_off:self._chunks_off]
         self.chunk_seq = d[self._chunks_off:self._chunks_off + self._max_chunks]
         self.chunk_off = d[self._chunks_off + self._max_chunks:]
+        self.shift_grp = d[self._shift_off:self._shift_off + 8]
         self.mamba_batch = L.mamba_batch(self.pos, self.row_seq, self.seq_start, self.seq_rows, self.seq_slot, self.seq_pos0)
         self.n_seq = 0
         self.block_table = torch.zeros(self.n_slots, self.max_pages, dtype=torch.int32, device=dev)
@@ -1569,7 +1575,8 @@ class LayerListEngine:
         return (self._xh[self._tmp if name == "tmp" else name], self.ncap) if self.tc and M >= TC_MIN_ROWS else None
 
     def shift_images(self, M: int):
-        """The five activation images of a time-mixing layer's mixes, or None where its products read f32 rows."""
+        """The activation image of a time-mixing layer's five mixes (mix s from row s * ncap of 5 * ncap), or None where its products
+        read f32 rows."""
         return self._shift_images if self.tc and M >= TC_MIN_ROWS else None
 
     @contextlib.contextmanager
@@ -1633,6 +1640,10 @@ class LayerListEngine:
         """Scratch `name` as [max_rows][width] (default: the width it was sized for)."""
         w = width or self._widths[name]
         return self._bufs[name][:self.max_rows * w].view(self.max_rows, w)
+
+    def stacked(self, name: str, n: int, width: int) -> torch.Tensor:
+        """Scratch `name` as [n][row capacity of the images][width]."""
+        return self._bufs[name][:n * self.ncap * width].view(n, self.ncap, width)
 
     def weight_bytes(self) -> int:
         n = sum(l.mixer.weight_bytes() for l in self.layers) + sum(f.weight_bytes() for f in {id(l.ff): l.ff for l in self.layers if l.ff}.values())
@@ -1729,6 +1740,8 @@ class LayerListEngine:
                     hd[co + nc], hd[co + self._max_chunks + nc] = n, off
                     nc += 1
             self._n_chunks = nc
+        for k in range(4):
+            hd[self._shift_off + 2 * k], hd[self._shift_off + 2 * k + 1] = k * self.ncap, M
         nl = len(logit_rows)
         hd[5 * R:5 * R + nl] = logit_rows
         if self.pages.dirty:

@@ -120,6 +120,19 @@ def dense_tc(wh: torch.Tensor, N: int, K: int, xh: torch.Tensor, ncap: int, y: t
     lib.count_launch()
 
 
+def dense_tc_grouped(wh: torch.Tensor, group_bytes: int, n_groups: int, grp: torch.Tensor, N: int, K: int, xh: torch.Tensor, ncap: int,
+                     y: torch.Tensor, M: int, epi: int = DENSE_STORE, param: float = 0.0):
+    """One product per group in one launch: rows grp[2 e] .. + grp[2 e + 1] - 1 (int32, on the device; first rows multiples of 8, at most
+    M rows each) of the activation image times the e-th weight image, to the same rows of y."""
+    e = DlEpilogue()
+    e.kind, e.n_dst, e.ld, e.dst_off = EPI_DENSE, 1, y.stride(0), 0
+    e.dst[0] = y.data_ptr()
+    e.dense_op, e.dense_param, e.dense_param2, e.dense_aux, e.dense_aux_ld = epi, param, 0.0, None, 0
+    check_layers(layers_lib().dl_gemm_wh_tc_grouped(wh.data_ptr(), group_bytes, n_groups, grp.data_ptr(), N, _round_up(K, 128), xh.data_ptr(),
+                                                    ncap, M, e, 2, _stream()), "dl_gemm_wh_tc_grouped")
+    lib.count_launch()
+
+
 def rms_norm(x: torch.Tensor, y: torch.Tensor, M: int, dim: int, eps: float, w: Optional[torch.Tensor] = None,
              plus_one: bool = False, groups: int = 1, gate: Optional[torch.Tensor] = None, accumulate: bool = False,
              rows: Optional[torch.Tensor] = None):
@@ -330,7 +343,7 @@ def delta_chunk_floats(M: int, n_seq: int, n_heads: int, dim: int, vdim: int) ->
 def token_shift(batch: DlMambaBatch, M: int, h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, out: Optional[torch.Tensor] = None,
                 images=None):
     """Mix s of row m = h + (h of the row ahead - h) mu[s], mu [mixes][width] f32; to out [mixes][>= M][width] f32, or into images =
-    (first image, bytes from one to the next, ncap).  state [slots][width] f32 carries every slot's last h and is updated."""
+    (first image, bytes from one to the next, row capacity).  state [slots][width] f32 carries every slot's last h and is updated."""
     a = DlShiftArgs()
     a.h, a.ldh, a.mu, a.n_mix, a.width, a.state = h.data_ptr(), h.stride(0), mu.data_ptr(), mu.shape[0], mu.shape[1], state.data_ptr()
     if images is not None:
@@ -718,13 +731,7 @@ class MoeGrouped:
         return self.wh_up.numel() + self.wh_down.numel()
 
     def _gemm(self, wh, group_bytes, N, K, xh, y, M, epi, param=0.0):
-        e = DlEpilogue()
-        e.kind, e.n_dst, e.ld, e.dst_off = EPI_DENSE, 1, y.stride(0), 0
-        e.dst[0] = y.data_ptr()
-        e.dense_op, e.dense_param, e.dense_param2, e.dense_aux, e.dense_aux_ld = epi, param, 0.0, None, 0
-        check_layers(layers_lib().dl_gemm_wh_tc_grouped(wh.data_ptr(), group_bytes, self.E, self.grp.data_ptr(), N, _round_up(K, 128),
-                                                        xh.data_ptr(), self.cap, M, e, 2, _stream()), "dl_gemm_wh_tc_grouped")
-        lib.count_launch()
+        dense_tc_grouped(wh, group_bytes, self.E, self.grp, N, K, xh, self.cap, y, M, epi, param)
 
     def run(self, x: torch.Tensor, M: int, sel: torch.Tensor, wgt: torch.Tensor, y: torch.Tensor):
         """x [M][width] f32, sel / wgt [M][top] -> y [M][width]."""
