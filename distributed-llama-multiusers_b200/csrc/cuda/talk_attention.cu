@@ -31,7 +31,7 @@
 #define TA_PAGE 32
 #define TA_MAX_ROWS 128
 #define TA_MAX_SPLITS 32
-#define TA_MERGE 256            // outputs per CTA of the merge
+#define TA_MERGE 128            // outputs per CTA of the merge
 #define TA_LOG2E 1.4426950408889634f
 #define TA_LN2 0.6931471805599453f
 
@@ -281,7 +281,7 @@ __global__ void __launch_bounds__((NR == 8 || ALLG) ? 256 : 128) talk_attention_
     }
 }
 
-// merge of the page shares: one CTA per (tile, key/value head, position of the tile) and 256 (head, column) outputs.  Every (head,
+// merge of the page shares: one CTA per (tile, key/value head, position of the tile) and TA_MERGE (head, column) outputs.  Every (head,
 // share) weight e^(m_k - m) / l is formed once, by a warp per head, then a thread per (head, column) sums the shares.
 __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, const int* __restrict__ tile_rows, int rq, int n_splits,
                                                          const float* __restrict__ partial, int DVP, int TA_ROWS, int vs) {
@@ -308,9 +308,15 @@ __global__ void __launch_bounds__(128) talk_merge_kernel(DlWindowAttnArgs a, con
     for (int idx = part * TA_MERGE + threadIdx.x; idx < min(rep * W, (part + 1) * TA_MERGE); idx += blockDim.x) {
         const int hg = idx / W, c = idx - hg * W, vh = c / DV;
         const float* p = base + (size_t)(r * rep + hg) * (DVP + 2) + vh * DVH + (c - vh * DV);
-        float acc = 0.f;                      // a share without pages left zeros and weighs 0: every load can go out at once
-#pragma unroll 16
-        for (int k = 0; k < n_splits; ++k) acc = fmaf(w_s[hg * n_splits + k], p[(size_t)k * TA_ROWS * (DVP + 2)], acc);
+        float acc = 0.f;                      // a share without pages left zeros and weighs 0: sixteen shares are in flight at once
+        for (int k0 = 0; k0 < n_splits; k0 += 16) {
+            float v[16];
+#pragma unroll
+            for (int k = 0; k < 16; ++k) v[k] = k0 + k < n_splits ? p[(size_t)(k0 + k) * TA_ROWS * (DVP + 2)] : 0.f;
+#pragma unroll
+            for (int k = 0; k < 16; ++k)
+                if (k0 + k < n_splits) acc = fmaf(w_s[hg * n_splits + k0 + k], v[k], acc);
+        }
         a.out[(size_t)m * a.ldo + (wide ? (size_t)((g * rep + hg) * a.kv_heads + v0) * DV : (size_t)(g * rep + hg) * DV) + c] = acc;
     }
 }

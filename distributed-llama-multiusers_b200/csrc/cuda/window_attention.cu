@@ -576,9 +576,15 @@ __global__ void __launch_bounds__(128) window_merge_kernel(DlWindowAttnArgs a, c
     for (int idx = threadIdx.x; idx < rep * D; idx += blockDim.x) {
         const int hg = idx / D, c = idx - hg * D;
         const float* p = base + (size_t)(r * rep + hg) * (D + 2) + c;
-        float acc = 0.f;                      // a share without pages left zeros and weighs 0: every load can go out at once
-#pragma unroll 16
-        for (int k = 0; k < n_splits; ++k) acc = fmaf(w_s[hg * n_splits + k], p[(size_t)k * WM_ROWS * (D + 2)], acc);
+        float acc = 0.f;                      // a share without pages left zeros and weighs 0: sixteen shares are in flight at once
+        for (int k0 = 0; k0 < n_splits; k0 += 16) {
+            float v[16];
+#pragma unroll
+            for (int k = 0; k < 16; ++k) v[k] = k0 + k < n_splits ? p[(size_t)(k0 + k) * WM_ROWS * (D + 2)] : 0.f;
+#pragma unroll
+            for (int k = 0; k < 16; ++k)
+                if (k0 + k < n_splits) acc = fmaf(w_s[hg * n_splits + k0 + k], v[k], acc);
+        }
         a.out[(size_t)m * a.ldo + (size_t)(g * rep + hg) * D + c] = acc;
     }
 }
