@@ -615,17 +615,17 @@ extern "C" int dl_mlstm_gates(const DlMambaBatch* batch, int n_seq, int longest,
 }
 
 // ------------------------------------------------------------------------------------------------
-// normalised heads: one warp per (row, head); four columns per lane and step (sizes and rows that allow it), up to 512 columns
-// kept in registers between the sum and the scaling
+// normalised heads: one warp per (row, head), half a warp for heads of up to 64 columns; four columns per lane and step (sizes and
+// rows that allow it), up to 512 columns kept in registers between the sum and the scaling
 // ------------------------------------------------------------------------------------------------
 #define HN_WARPS 8
 #define HN_CACHE 4                 // groups of four columns per lane
-template <bool VEC>
+template <bool VEC, int LANES>
 __global__ void __launch_bounds__(HN_WARPS * 32) head_norm_kernel(DlHeadNormArgs a) {
-    const int m = blockIdx.x, lane = threadIdx.x & 31, V = a.vdim;
-    const int h = blockIdx.y * HN_WARPS + (threadIdx.x >> 5);
+    constexpr int NC = LANES == 32 ? HN_CACHE : 1;
+    const int m = blockIdx.x, lane = threadIdx.x & (LANES - 1), V = a.vdim;
+    const int hh = blockIdx.y * (HN_WARPS * 32 / LANES) + threadIdx.x / LANES, h = min(hh, a.n_heads - 1);      // spare lanes repeat the last head
     if (a.xh && blockIdx.y == 0) xh_zero_tail(a.xh, a.ncap, m, a.n_heads * V, threadIdx.x, HN_WARPS * 32);
-    if (h >= a.n_heads) return;
     const float* y = a.y + (size_t)m * a.ld_y + (size_t)h * V;
     const float* w = a.w + (a.w_full ? (size_t)h * V : 0);
     const float* g = a.gate ? a.gate + (size_t)m * a.ld_gate + (size_t)h * V : nullptr;
@@ -633,11 +633,11 @@ __global__ void __launch_bounds__(HN_WARPS * 32) head_norm_kernel(DlHeadNormArgs
     if (a.den) scale = 1.f / (fmaxf(fabsf(a.den[(size_t)m * a.n_heads + h]), a.floor_[(size_t)m * a.n_heads + h]) + 1e-6f);
     if (VEC) {
         const int n4 = V >> 2;
-        float4 v[HN_CACHE], gv[HN_CACHE];
+        float4 v[NC], gv[NC];
         float ss = 0.f;
 #pragma unroll
-        for (int k = 0; k < HN_CACHE; ++k) {
-            const int i = lane + 32 * k;
+        for (int k = 0; k < NC; ++k) {
+            const int i = lane + LANES * k;
             v[k] = gv[k] = make_float4(0.f, 0.f, 0.f, 0.f);
             if (i < n4) {
                 v[k] = reinterpret_cast<const float4*>(y)[i];
@@ -645,14 +645,17 @@ __global__ void __launch_bounds__(HN_WARPS * 32) head_norm_kernel(DlHeadNormArgs
             }
         }
 #pragma unroll
-        for (int k = 0; k < HN_CACHE; ++k) {
+        for (int k = 0; k < NC; ++k) {
             v[k] = make_float4(v[k].x * scale, v[k].y * scale, v[k].z * scale, v[k].w * scale);
             ss = dot4(v[k], v[k], ss);
         }
-        const float inv = 1.f / sqrtf(warp_sum(ss) / (float)V + a.eps);
 #pragma unroll
-        for (int k = 0; k < HN_CACHE; ++k) {
-            const int i = lane + 32 * k;
+        for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if (hh >= a.n_heads) return;
+        const float inv = 1.f / sqrtf(ss / (float)V + a.eps);
+#pragma unroll
+        for (int k = 0; k < NC; ++k) {
+            const int i = lane + LANES * k;
             if (i >= n4) continue;
             const float4 wv = reinterpret_cast<const float4*>(w)[i];
             float4 t = make_float4(v[k].x * inv * wv.x, v[k].y * inv * wv.y, v[k].z * inv * wv.z, v[k].w * inv * wv.w);
@@ -668,6 +671,7 @@ __global__ void __launch_bounds__(HN_WARPS * 32) head_norm_kernel(DlHeadNormArgs
             }
         }
     } else {
+        if (hh >= a.n_heads) return;
         float ss = 0.f;
         for (int i = lane; i < V; i += 32) { const float t = y[i] * scale; ss = fmaf(t, t, ss); }
         const float inv = 1.f / sqrtf(warp_sum(ss) / (float)V + a.eps);
@@ -686,8 +690,9 @@ extern "C" int dl_head_norm(const DlHeadNormArgs* args, void* stream) {
     const auto al = [](const void* p, long long ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
     const bool vec = a.vdim % 4 == 0 && a.vdim <= 128 * HN_CACHE && al(a.y, a.ld_y) && al(a.w, 0) && al(a.gate, a.ld_gate) && al(a.out, a.ld_out);
     const dim3 grid(a.M, (a.n_heads + HN_WARPS - 1) / HN_WARPS);
-    if (vec) head_norm_kernel<true><<<grid, HN_WARPS * 32, 0, (cudaStream_t)stream>>>(a);
-    else head_norm_kernel<false><<<grid, HN_WARPS * 32, 0, (cudaStream_t)stream>>>(a);
+    if (vec && a.vdim <= 64) head_norm_kernel<true, 16><<<dim3(a.M, (a.n_heads + 2 * HN_WARPS - 1) / (2 * HN_WARPS)), HN_WARPS * 32, 0, (cudaStream_t)stream>>>(a);
+    else if (vec) head_norm_kernel<true, 32><<<grid, HN_WARPS * 32, 0, (cudaStream_t)stream>>>(a);
+    else head_norm_kernel<false, 32><<<grid, HN_WARPS * 32, 0, (cudaStream_t)stream>>>(a);
     LAYER_CHECK_LAUNCH("dl_head_norm");
     return 0;
 }
