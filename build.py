@@ -3,7 +3,7 @@
 
   distributed-llama-multiusers_b200/lib/libdllama_b200_cuda.so   nvcc, sm_100a only: the Q40 / f32 Llama kernels
   distributed-llama-multiusers_b200/lib/libdllama_b200_layers.so nvcc, sm_100a only: the kernels of layer-list models
-                                                                 (dense bf16 / f32 weights, latent, windowed, linear and gated linear attention, Mamba-1 / -2)
+                                                                 (dense bf16 / f32 weights, latent, windowed, linear and gated linear attention, the delta rule, Mamba-1 / -2)
   distributed-llama-multiusers_b200/lib/libdllama_b200_host.so   g++, CPU runtime (tokenizer,
                                                                  sampler, codecs, scheduler ...)
 
